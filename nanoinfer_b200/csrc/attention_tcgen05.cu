@@ -94,7 +94,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                             const int* __restrict__ q_start, const int* __restrict__ ctx_lens,
                             const int* __restrict__ block_table, int bt_stride, int page_size, int num_pages,
                             int heads, int kv_heads, float scale, int window, unsigned long long* trace, int trace_cap,
-                            float softcap, int chunk, const float* __restrict__ sinks) {
+                            float softcap, int chunk, const float* __restrict__ sinks, float out_scale) {
     using C = Cfg<HD>;
     constexpr int KEYS = C::KEYS, STAGES = C::STAGES;
     extern __shared__ unsigned char smem_raw[];
@@ -424,7 +424,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             tc_fence_after();
             float l_all = xch[4 * 128 + row] + xch[5 * 128 + row];
             if (FLEX && sinks != nullptr && m_cur != -INFINITY) l_all += ex2(__ldg(sinks + head) * LOG2E - m_cur);   // the sink: no key, no value
-            const float inv = l_all > 0.f ? 1.0f / l_all : 0.f;
+            const float inv = l_all > 0.f ? out_scale / l_all : 0.f;
             __nv_bfloat16* orow = out + ((size_t)(row_begin + tok0 + ti) * heads + head) * HD + half * (HD / 2);
 #pragma unroll
             for (int c = 0; c < HD / 64; ++c) {
@@ -475,7 +475,7 @@ template <int HD, bool FLEX>
 int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, void* out, const int* q_start,
            const int* ctx_lens, const int* block_table, int bt_stride, int page_size, int num_pages, int n_req,
            int max_q_len, int heads, int kv_heads, float scale, int window, float softcap, int chunk, const float* sinks,
-           cudaStream_t stream) {
+           float out_scale, cudaStream_t stream) {
     static bool configured = false;
     if (!configured) {
         NIB_CUDA(cudaFuncSetAttribute(attention_prefill_tc_kernel<HD, FLEX>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg<HD>::SMEM));
@@ -485,7 +485,7 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, 
     dim3 grid(ceil_div(max_q_len, tpt), n_req, kv_heads);
     NIB_CUDA(launch_pdl(attention_prefill_tc_kernel<HD, FLEX>, grid, dim3(THREADS), (size_t)Cfg<HD>::SMEM, stream, mq, mk, mv,
                         (__nv_bfloat16*)out, q_start, ctx_lens, block_table, bt_stride, page_size, num_pages, heads,
-                        kv_heads, scale, window, nib_trace_buffer(), nib_trace_capacity(), softcap, chunk, sinks));
+                        kv_heads, scale, window, nib_trace_buffer(), nib_trace_capacity(), softcap, chunk, sinks, out_scale));
     return 0;
 }
 
@@ -511,12 +511,12 @@ NIB_API int nib_attention_tc_error() {
 }
 
 // Same arguments as nib_attention_prefill_mma plus the number of rows of qkv (m_tokens, for the map's extent), and the
-// options on the scores: softcap (0 = none), chunk (0 = none), sinks [heads] (null = none).
+// options: softcap (0 = none), chunk (0 = none), sinks [heads] (null = none), a factor on the output (32-bit, before it is rounded).
 NIB_API int nib_attention_prefill_tc(const void* qkv, int q_stride, void* out, const int* q_start, const int* ctx_lens,
                                      const int* block_table, int bt_stride, int page_size, const void* k_pages,
                                      const void* v_pages, int num_pages, int n_req, int max_q_len, int m_tokens,
                                      int heads, int kv_heads, int head_dim, float scale, int window, float softcap, int chunk,
-                                     const float* sinks, cudaStream_t stream) {
+                                     const float* sinks, float out_scale, cudaStream_t stream) {
     NIB_REQUIRE(nib_attention_prefill_tc_supported(heads, kv_heads, head_dim, page_size, q_stride),
                 "attention (tcgen05): head_dim %d, %d/%d heads, page size %d are not supported", head_dim, heads, kv_heads, page_size);
     NIB_REQUIRE(n_req >= 0 && max_q_len > 0 && num_pages > 0 && window >= 0 && m_tokens > 0 && chunk >= 0 && softcap >= 0.f && scale > 0.f,
@@ -533,7 +533,7 @@ NIB_API int nib_attention_prefill_tc(const void* qkv, int q_stride, void* out, c
     if (make_map3(&mk, k_pages, head_dim, page_size, planes, head_dim, (long long)page_size * head_dim, page_size, 1)) return 1;
     if (make_map3(&mv, v_pages, head_dim, page_size, planes, head_dim, (long long)page_size * head_dim, page_size, 1)) return 1;
 #define NIB_TC_ATTN(HD, FLEX) launch<HD, FLEX>(mq, mk, mv, out, q_start, ctx_lens, block_table, bt_stride, page_size, num_pages, n_req, max_q_len, \
-                                               heads, kv_heads, scale, window, softcap, chunk, sinks, stream)
+                                               heads, kv_heads, scale, window, softcap, chunk, sinks, out_scale, stream)
     const bool flex = softcap > 0.f || chunk > 0 || sinks != nullptr;
     if (head_dim == 64) return flex ? NIB_TC_ATTN(64, true) : NIB_TC_ATTN(64, false);
     return flex ? NIB_TC_ATTN(128, true) : NIB_TC_ATTN(128, false);

@@ -56,6 +56,25 @@ __device__ __forceinline__ float warp_max(float v) {
     return v;
 }
 
+// Epilogues of the matrix products (the `epi` argument): STORE in the storage type, ADD into floats, F32 floats, SWIGLU
+// silu(gate) * up from two accumulators, QKV see the products; GLU the gated form with constants (NibGlu).
+enum NibEpi : int { EPI_STORE = 0, EPI_ADD = 1, EPI_F32 = 2, EPI_SWIGLU = 3, EPI_QKV = 4, EPI_GLU = 5 };
+__host__ __device__ constexpr bool epi_dual(int epi) { return epi == EPI_SWIGLU || epi == EPI_GLU; }     // two accumulators
+
+// The gated product with constants: g = min(gate, limit), u = clamp(up, -limit, limit), g * sigmoid(alpha * g) * (u + shift).
+struct NibGlu { float alpha, limit, shift; };
+__device__ __forceinline__ float nib_glu_exact(const NibGlu& p, float g, float u) {
+    g = fminf(g, p.limit);
+    u = fminf(fmaxf(u, -p.limit), p.limit);
+    return g / (1.0f + expf(-p.alpha * g)) * (u + p.shift);
+}
+// the fast exponential and division (2 ulp), for results that are rounded to bfloat16
+__device__ __forceinline__ float nib_glu_fast(const NibGlu& p, float g, float u) {
+    g = fminf(g, p.limit);
+    u = fminf(fmaxf(u, -p.limit), p.limit);
+    return __fdividef(g, 1.0f + __expf(-p.alpha * g)) * (u + p.shift);
+}
+
 static inline int ceil_div(long long a, long long b) { return (int)((a + b - 1) / b); }
 
 // Programmatic dependent launch: a kernel launched with launch_pdl may begin while the kernel before it

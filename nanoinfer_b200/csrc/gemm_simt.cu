@@ -8,17 +8,15 @@
 //
 // Epilogues: STORE (T out = acc + bias), ADD (float out += acc + bias: the residual sum),
 // F32 (float out = acc + bias: logits), SWIGLU (two accumulators, W rows n and n + N:
-// T out = silu(gate) * up, silu(g) = g / (1 + exp(-g)), cpp/src/ops.cpp:86-93).
+// T out = silu(gate) * up, silu(g) = g / (1 + exp(-g)), cpp/src/ops.cpp:86-93), GLU (the same with limits and constants).
 #include "common.cuh"
-
-enum { EPI_STORE = 0, EPI_ADD = 1, EPI_F32 = 2, EPI_SWIGLU = 3 };
 
 template <typename T, int EPI>
 __global__ void __launch_bounds__(256)
 gemm_simt_kernel(const T* __restrict__ A, const T* __restrict__ W, const float* __restrict__ bias,
-                 void* __restrict__ out, int M, int N, int K, int lda, int ldo) {
+                 void* __restrict__ out, int M, int N, int K, int lda, int ldo, const NibGlu glu) {
     constexpr int BM = 64, BN = 64, BK = 16, TM = 4, TN = 4;
-    constexpr bool DUAL = (EPI == EPI_SWIGLU);
+    constexpr bool DUAL = epi_dual(EPI);
     __shared__ float As[BK][BM + 1];
     __shared__ float Ws[BK][BN + 1];
     __shared__ float Us[DUAL ? BK : 1][DUAL ? BN + 1 : 1];
@@ -102,7 +100,7 @@ gemm_simt_kernel(const T* __restrict__ A, const T* __restrict__ W, const float* 
                 ((float*)out)[o] = v;
             } else {
                 const float g = v, u = acc2[DUAL ? i : 0][DUAL ? j : 0];
-                Elem<T>::store((T*)out + o, g / (1.0f + expf(-g)) * u);
+                Elem<T>::store((T*)out + o, EPI == EPI_GLU ? nib_glu_exact(glu, g, u) : g / (1.0f + expf(-g)) * u);
             }
         }
     }
@@ -110,14 +108,15 @@ gemm_simt_kernel(const T* __restrict__ A, const T* __restrict__ W, const float* 
 
 template <typename T>
 static int launch_simt(const void* A, const void* W, const float* bias, void* out, int M, int N, int K,
-                       int lda, int ldo, int epi, cudaStream_t stream) {
+                       int lda, int ldo, int epi, const NibGlu& glu, cudaStream_t stream) {
     dim3 grid(ceil_div(N, 64), ceil_div(M, 64));
     dim3 block(256);
     switch (epi) {
-        case EPI_STORE: gemm_simt_kernel<T, EPI_STORE><<<grid, block, 0, stream>>>((const T*)A, (const T*)W, bias, out, M, N, K, lda, ldo); break;
-        case EPI_ADD: gemm_simt_kernel<T, EPI_ADD><<<grid, block, 0, stream>>>((const T*)A, (const T*)W, bias, out, M, N, K, lda, ldo); break;
-        case EPI_F32: gemm_simt_kernel<T, EPI_F32><<<grid, block, 0, stream>>>((const T*)A, (const T*)W, bias, out, M, N, K, lda, ldo); break;
-        case EPI_SWIGLU: gemm_simt_kernel<T, EPI_SWIGLU><<<grid, block, 0, stream>>>((const T*)A, (const T*)W, bias, out, M, N, K, lda, ldo); break;
+        case EPI_STORE: gemm_simt_kernel<T, EPI_STORE><<<grid, block, 0, stream>>>((const T*)A, (const T*)W, bias, out, M, N, K, lda, ldo, glu); break;
+        case EPI_ADD: gemm_simt_kernel<T, EPI_ADD><<<grid, block, 0, stream>>>((const T*)A, (const T*)W, bias, out, M, N, K, lda, ldo, glu); break;
+        case EPI_F32: gemm_simt_kernel<T, EPI_F32><<<grid, block, 0, stream>>>((const T*)A, (const T*)W, bias, out, M, N, K, lda, ldo, glu); break;
+        case EPI_SWIGLU: gemm_simt_kernel<T, EPI_SWIGLU><<<grid, block, 0, stream>>>((const T*)A, (const T*)W, bias, out, M, N, K, lda, ldo, glu); break;
+        case EPI_GLU: gemm_simt_kernel<T, EPI_GLU><<<grid, block, 0, stream>>>((const T*)A, (const T*)W, bias, out, M, N, K, lda, ldo, glu); break;
         default: nib_set_error("gemm: unknown epilogue %d", epi); return 1;
     }
     NIB_LAUNCH_CHECK();
@@ -125,15 +124,17 @@ static int launch_simt(const void* A, const void* W, const float* bias, void* ou
 }
 
 // A [M, K] with row stride lda; W [N, K] (SWIGLU: [2N, K], gate rows then up rows); out [M, N] with
-// row stride ldo. epi: 0 store, 1 add into float, 2 store float, 3 swiglu.
+// row stride ldo. epi: 0 store, 1 add into float, 2 store float, 3 swiglu, 5 the gated form with the constants glu.
 NIB_API int nib_gemm_simt(const void* A, const void* W, const float* bias, void* out, int M, int N, int K,
-                          int lda, int ldo, int epi, int dtype, cudaStream_t stream) {
+                          int lda, int ldo, int epi, int dtype, const NibGlu* glu, cudaStream_t stream) {
     NIB_REQUIRE(M >= 0 && N > 0 && K > 0 && lda >= K && ldo >= N, "gemm: bad sizes M=%d N=%d K=%d lda=%d ldo=%d", M, N, K, lda, ldo);
-    NIB_REQUIRE(epi != EPI_SWIGLU || bias == nullptr, "gemm: the swiglu epilogue takes no bias");
+    NIB_REQUIRE(!epi_dual(epi) || bias == nullptr, "gemm: the gated epilogues take no bias");
+    NIB_REQUIRE(epi != EPI_GLU || glu != nullptr, "gemm: the gated epilogue needs its constants");
+    const NibGlu constants = glu != nullptr ? *glu : NibGlu{};
     if (M == 0) return 0;
     NIB_REQUIRE(ceil_div(M, 64) <= 65535, "gemm: M=%d is too large for one launch", M);
-    if (dtype == NIB_F32) return launch_simt<float>(A, W, bias, out, M, N, K, lda, ldo, epi, stream);
-    if (dtype == NIB_BF16) return launch_simt<__nv_bfloat16>(A, W, bias, out, M, N, K, lda, ldo, epi, stream);
+    if (dtype == NIB_F32) return launch_simt<float>(A, W, bias, out, M, N, K, lda, ldo, epi, constants, stream);
+    if (dtype == NIB_BF16) return launch_simt<__nv_bfloat16>(A, W, bias, out, M, N, K, lda, ldo, epi, constants, stream);
     NIB_REQUIRE(false, "gemm: unknown dtype %d", dtype);
 }
 

@@ -29,7 +29,6 @@
 
 namespace {
 
-enum { EPI_STORE = 0, EPI_ADD = 1, EPI_F32 = 2, EPI_SWIGLU = 3, EPI_QKV = 4 };
 constexpr int WARPS = 8;
 constexpr int MAX_TOKENS = 64;
 
@@ -79,8 +78,8 @@ __global__ void __launch_bounds__(WARPS * 32, 2)      // two CTAs per SM: a proj
 gemm_smallm_kernel(const void* __restrict__ A, const __nv_bfloat16* __restrict__ W, const float* __restrict__ bias,
                    void* __restrict__ out, int tokens, int n_out, int k_dim, int lda, int ldo,
                    const float* __restrict__ gain, float eps, float* __restrict__ scratch, int* __restrict__ counters,
-                   const QkvEpi qe, unsigned long long* trace, int trace_cap) {
-    constexpr bool DUAL = (EPI == EPI_SWIGLU);
+                   const QkvEpi qe, const NibGlu glu, unsigned long long* trace, int trace_cap) {
+    constexpr bool DUAL = epi_dual(EPI);
     constexpr int ACCS = DUAL ? 2 : 1;
     constexpr int GROUPS = WARPS / KSPLIT;
     constexpr int E = NORM ? 5 : 4;                      // accumulator elements per tile, plus the row's sum of squares
@@ -382,6 +381,7 @@ gemm_smallm_kernel(const void* __restrict__ A, const __nv_bfloat16* __restrict__
             else if (EPI == EPI_ADD) ((float*)out)[o] = res[e] + x;
             else if (EPI == EPI_F32) ((float*)out)[o] = x;
             else if (EPI == EPI_SWIGLU) ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(__fdividef(x, 1.0f + __expf(-x)) * (v[ACCS - 1][e] * scale2[e & 1]));
+            else if (EPI == EPI_GLU) ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(nib_glu_fast(glu, x, v[ACCS - 1][e] * scale2[e & 1]));
         }
     };
 
@@ -415,12 +415,12 @@ gemm_smallm_kernel(const void* __restrict__ A, const __nv_bfloat16* __restrict__
 struct Args {
     const void* A; const void* W; const float* bias; void* out; int tokens, N, K, lda, ldo;
     const float* gain; float eps; float* scratch; int* counters; int cross;
-    QkvEpi qe;
+    QkvEpi qe; NibGlu glu;
 };
 
 template <int NT, int KSPLIT, int EPI, bool NORM>
 int launch_one(const Args& a, cudaStream_t stream) {
-    constexpr int ACCS = (EPI == EPI_SWIGLU) ? 2 : 1;
+    constexpr int ACCS = epi_dual(EPI) ? 2 : 1;
     const int groups = ceil_div(a.N, 16);
     dim3 grid(ceil_div(groups, WARPS / KSPLIT), KSPLIT > 1 ? a.cross : 1);
     const size_t smem = KSPLIT > 1 ? (size_t)KSPLIT * ACCS * NT * (NORM ? 5 : 4) * 32 * sizeof(float) : 0;
@@ -431,7 +431,7 @@ int launch_one(const Args& a, cudaStream_t stream) {
     configured = true;
     NIB_CUDA(launch_pdl(gemm_smallm_kernel<NT, KSPLIT, EPI, NORM>, grid, dim3(WARPS * 32), smem, stream,
                         a.A, (const __nv_bfloat16*)a.W, a.bias, a.out, a.tokens, a.N, a.K, a.lda, a.ldo, a.gain, a.eps,
-                        a.scratch, a.counters, a.qe, nib_trace_buffer(), nib_trace_capacity()));
+                        a.scratch, a.counters, a.qe, a.glu, nib_trace_buffer(), nib_trace_capacity()));
     return 0;
 }
 
@@ -442,6 +442,7 @@ int launch_epi(int epi, const Args& a, cudaStream_t stream) {
         case EPI_ADD: return launch_one<NT, KSPLIT, EPI_ADD, NORM>(a, stream);
         case EPI_F32: return launch_one<NT, KSPLIT, EPI_F32, NORM>(a, stream);
         case EPI_SWIGLU: return launch_one<NT, KSPLIT, EPI_SWIGLU, NORM>(a, stream);
+        case EPI_GLU: return launch_one<NT, KSPLIT, EPI_GLU, NORM>(a, stream);
         case EPI_QKV:
             if constexpr (KSPLIT > 1) return launch_one<NT, KSPLIT, EPI_QKV, NORM>(a, stream);
             break;
@@ -486,11 +487,12 @@ NIB_API long long nib_gemm_smallm_scratch_floats(int N, int cross) {
 NIB_API int nib_gemm_smallm(const void* A, const void* W, const float* bias, void* out, int tokens, int N, int K,
                             int lda, int ldo, int epi, const float* gain, float eps, int ksplit, int cross,
                             float* scratch, int* counters, long long scratch_floats, int counter_ints,
-                            cudaStream_t stream) {
+                            const NibGlu* glu, cudaStream_t stream) {
     NIB_REQUIRE(N > 0 && lda >= K && ldo >= N, "gemm (small M): bad sizes tokens=%d N=%d K=%d", tokens, N, K);
     NIB_REQUIRE(nib_gemm_smallm_supported(A, W, tokens, K, lda, gain ? 4 : 2),
                 "gemm (small M): needs 1..64 tokens, K %% 32 == 0 and 16-byte aligned rows (tokens=%d K=%d)", tokens, K);
-    NIB_REQUIRE(epi != EPI_SWIGLU || bias == nullptr, "gemm (small M): the swiglu epilogue takes no bias");
+    NIB_REQUIRE(!epi_dual(epi) || bias == nullptr, "gemm (small M): the gated epilogues take no bias");
+    NIB_REQUIRE(epi != EPI_GLU || glu != nullptr, "gemm (small M): the gated epilogue needs its constants");
     NIB_REQUIRE(gain == nullptr || (((uintptr_t)gain & 15) == 0), "gemm (small M): the gain must be 16-byte aligned");
     const int groups = ceil_div(N, 16), blocks = K / 32;
     if (ksplit == 0) ksplit = (groups < 8 * 148 && blocks >= 8) ? WARPS : 1;   // wide outputs: a warp per row group
@@ -513,7 +515,7 @@ NIB_API int nib_gemm_smallm(const void* A, const void* W, const float* bias, voi
         NIB_REQUIRE(nib_gemm_smallm_scratch_floats(N, cross) <= scratch_floats && groups <= counter_ints,
                     "gemm (small M): workspace too small for N=%d cross=%d", N, cross);
     }
-    Args a{A, W, bias, out, tokens, N, K, lda, ldo, gain, eps, scratch, counters, cross, QkvEpi{}};
+    Args a{A, W, bias, out, tokens, N, K, lda, ldo, gain, eps, scratch, counters, cross, QkvEpi{}, glu != nullptr ? *glu : NibGlu{}};
     if (gain) return launch_tokens<true>(ksplit, epi, a, stream);
     return launch_tokens<false>(ksplit, epi, a, stream);
 }
@@ -546,7 +548,7 @@ NIB_API int nib_gemm_smallm_qkv(const void* A, const void* W, const float* bias,
     NIB_REQUIRE(gain == nullptr || (((uintptr_t)gain & 15) == 0), "gemm (small M, q/k/v): the gain must be 16-byte aligned");
     Args a{A, W, bias, qkv, tokens, N, K, lda, ldq, gain, eps, nullptr, nullptr, 1,
            QkvEpi{heads, kv_heads, head_dim, rot, positions, req_index, cos_t, sin_t, block_table, bt_stride, page_size,
-                  num_pages, (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, writes}};
+                  num_pages, (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, writes}, NibGlu{}};
     if (gain) return launch_tokens<true>(WARPS, EPI_QKV, a, stream);
     return launch_tokens<false>(WARPS, EPI_QKV, a, stream);
 }

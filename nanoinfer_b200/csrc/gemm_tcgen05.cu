@@ -28,7 +28,7 @@
 // stops issuing, waits (bounded) for its own copies in flight, frees its TMEM and returns.
 //
 // Epilogues: STORE bf16 (+bias), ADD into a float tensor (the residual sum), F32 store (logits),
-// SWIGLU (two accumulators from W rows n and n + N: silu(gate) * up). Reference formulas:
+// SWIGLU (two accumulators from W rows n and n + N: silu(gate) * up), GLU (the same with limits and constants). Reference formulas:
 // cpp/src/ops.cpp:42-69 (linear), :86-93 (silu). The reference's tensor-core GEMMs are wmma kernels
 // for sm_89 (cpp/src/cuda/cuda_gemm.cu:484-622).
 #include "tcgen05.cuh"
@@ -39,8 +39,6 @@ using namespace nibp;
 using namespace nibt;
 
 namespace {
-
-enum { EPI_STORE = 0, EPI_ADD = 1, EPI_F32 = 2, EPI_SWIGLU = 3, EPI_QKV = 4 };
 
 constexpr int BLOCK_F = 128;     // output features per CTA (UMMA M)
 constexpr int BLOCK_K = 64;      // elements of K per stage: 128 bytes, one swizzle atom
@@ -71,7 +69,7 @@ __device__ __forceinline__ void red_add_v4(float* p, float a, float b, float c, 
 // 16 consecutive features (first .. first+15) of one token row. v: accumulators (for SWIGLU the gate), u: the up values.
 template <int EPI>
 __device__ __forceinline__ void emit_row16(void* __restrict__ out, const float (&v)[16], const float (&u)[16],
-                                           const float* __restrict__ bias, size_t row_off, int first, int n_out, bool vec_ok) {
+                                           const float* __restrict__ bias, size_t row_off, int first, int n_out, bool vec_ok, const NibGlu& glu) {
     float x[16];
 #pragma unroll
     for (int j = 0; j < 16; ++j) x[j] = v[j];
@@ -93,8 +91,12 @@ __device__ __forceinline__ void emit_row16(void* __restrict__ out, const float (
 #pragma unroll
         for (int j = 0; j < 16; ++j) x[j] = __fdividef(x[j], 1.0f + __expf(-x[j])) * u[j];
     }
+    if (EPI == EPI_GLU) {
+#pragma unroll
+        for (int j = 0; j < 16; ++j) x[j] = nib_glu_fast(glu, x[j], u[j]);
+    }
     if (vec_ok && first + 16 <= n_out) {
-        if (EPI == EPI_STORE || EPI == EPI_SWIGLU) {
+        if (EPI == EPI_STORE || epi_dual(EPI)) {
             uint4 p0, p1;
             __nv_bfloat162* h0 = reinterpret_cast<__nv_bfloat162*>(&p0);
             __nv_bfloat162* h1 = reinterpret_cast<__nv_bfloat162*>(&p1);
@@ -118,7 +120,7 @@ __device__ __forceinline__ void emit_row16(void* __restrict__ out, const float (
     for (int j = 0; j < 16; ++j) {
         if (first + j >= n_out) break;
         const size_t o = row_off + first + j;
-        if (EPI == EPI_STORE || EPI == EPI_SWIGLU) ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(x[j]);
+        if (EPI == EPI_STORE || epi_dual(EPI)) ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(x[j]);
         else if (EPI == EPI_F32) ((float*)out)[o] = x[j];
         else atomicAdd((float*)out + o, x[j]);
     }
@@ -194,7 +196,7 @@ __device__ __forceinline__ void emit_qkv_head(unsigned addr, int f, const float*
 // second accumulator of the swiglu form, b = bias.
 template <int EPI>
 __device__ __forceinline__ void emit16(void* __restrict__ out, const float (&v)[16], const float (&u)[16], float b, int f,
-                                       int first_token, int tokens, int ldo) {
+                                       int first_token, int tokens, int ldo, const NibGlu& glu) {
     if (EPI == EPI_ADD) {
         // The sum into the residual stream is a reduction in memory (red.global.add.f32): nothing is
         // read back, so the epilogue does not wait a memory round trip per batch of tokens. Each element
@@ -213,6 +215,7 @@ __device__ __forceinline__ void emit16(void* __restrict__ out, const float (&v)[
             const float x = v[j] + b;
             if (EPI == EPI_STORE) ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(x);
             else if (EPI == EPI_F32) ((float*)out)[o] = x;
+            else if (EPI == EPI_GLU) ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(nib_glu_fast(glu, x, u[j]));
             else ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(__fdividef(x, 1.0f + __expf(-x)) * u[j]);
         }
     }
@@ -229,10 +232,10 @@ __global__ void __launch_bounds__(THREADS, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_a,
                const float* __restrict__ bias, void* __restrict__ out, int tokens, int n_out, int k_dim, int ldo,
                int splits, int kb_per_split, float* __restrict__ scratch, int* __restrict__ counters, int vec_ok,
-               const QkvRows qe, unsigned long long* trace, int trace_cap) {
-    static_assert(!SWAP || (TOK == BLOCK_F && EPI != EPI_SWIGLU), "the swapped form has tiles of 128 tokens and one accumulator");
+               const QkvRows qe, const NibGlu glu, unsigned long long* trace, int trace_cap) {
+    static_assert(!SWAP || (TOK == BLOCK_F && !epi_dual(EPI)), "the swapped form has tiles of 128 tokens and one accumulator");
     static_assert((EPI == EPI_QKV) == (HD != 0) && (EPI != EPI_QKV || SWAP), "the q/k/v epilogue owns token rows");
-    constexpr bool DUAL = (EPI == EPI_SWIGLU);
+    constexpr bool DUAL = epi_dual(EPI);
     using C = Cfg<TOK, DUAL, HD>;
     extern __shared__ unsigned char smem_raw[];
     unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -424,7 +427,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
 #pragma unroll
                             for (int i = 0; i < 16; ++i) v[i] = __uint_as_float(r[j][i]);
                             if (live && f0 + c + 16 * j < n_out)
-                                emit_row16<EPI>(out, v, v, item_bias, (size_t)t * ldo, f0 + c + 16 * j, n_out, vec_ok != 0);
+                                emit_row16<EPI>(out, v, v, item_bias, (size_t)t * ldo, f0 + c + 16 * j, n_out, vec_ok != 0, glu);
                         }
                     }
                 }
@@ -440,7 +443,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                     float v[16], u[16];
                     tmem_ld16(lane_addr + c, v);
                     if (DUAL) tmem_ld16(lane_addr + TOK + c, u);
-                    if (f < n_out) emit16<EPI>(out, v, u, b, f, t0 + c, tokens, ldo);
+                    if (f < n_out) emit16<EPI>(out, v, u, b, f, t0 + c, tokens, ldo, glu);
                 }
                 // this warp has read its part of the buffer: hand it back to the MMA warp
                 tc_fence_before();
@@ -513,7 +516,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                         }
                     }
                 }
-                if (f < n_out) emit16<EPI>(out, v, u, b, f, t0 + c, tokens, ldo);
+                if (f < n_out) emit16<EPI>(out, v, u, b, f, t0 + c, tokens, ldo, glu);
             }
             }   // !SWAP
         }
@@ -565,8 +568,8 @@ template <int NT, int EPI>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(PAIR_THREADS, 1)
 gemm_pair_kernel(const __grid_constant__ CUtensorMap map_m, const __grid_constant__ CUtensorMap map_n,
                  const float* __restrict__ bias, void* __restrict__ out, int tokens, int n_out, int k_dim, int ldo, int vec_ok,
-                 int splits, int kb_per_split, unsigned long long* trace, int trace_cap) {
-    constexpr bool GU = (EPI == EPI_SWIGLU);                       // the tile's columns: gate rows | up rows of NT/2 features
+                 int splits, int kb_per_split, const NibGlu glu, unsigned long long* trace, int trace_cap) {
+    constexpr bool GU = epi_dual(EPI);                             // the tile's columns: gate rows | up rows of NT/2 features
     constexpr int FEAT = GU ? NT / 2 : NT;                         // output features per tile
     using C = PairCfg<NT>;
     extern __shared__ unsigned char smem_raw[];
@@ -696,7 +699,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_m, const __grid_constan
                 float v[16], u[16];
                 tmem_ld16(lane_addr + c, v);
                 if (GU) tmem_ld16(lane_addr + FEAT + c, u);
-                if (t < tokens) emit_row16<EPI>(out, v, u, item_bias, row_off, f0 + c, n_out, vec_ok != 0);
+                if (t < tokens) emit_row16<EPI>(out, v, u, item_bias, row_off, f0 + c, n_out, vec_ok != 0, glu);
             }
             tc_fence_before();
             __syncwarp();
@@ -760,8 +763,8 @@ int sm_count() {
 
 template <int TOK, int EPI, bool SWAP = false, int HD = 0>
 int launch_tc(const CUtensorMap& mw, const CUtensorMap& ma, const float* bias, void* out, int tokens, int n_out,
-              int k, int ldo, const SplitK& sk, cudaStream_t stream, int vec_ok = 0, const QkvRows& qe = QkvRows{}) {
-    using C = Cfg<TOK, EPI == EPI_SWIGLU, HD>;
+              int k, int ldo, const SplitK& sk, cudaStream_t stream, int vec_ok = 0, const QkvRows& qe = QkvRows{}, const NibGlu& glu = NibGlu{}) {
+    using C = Cfg<TOK, epi_dual(EPI), HD>;
     static bool configured = false;
     if (!configured) {
         NIB_CUDA(cudaFuncSetAttribute(gemm_tc_kernel<TOK, EPI, SWAP, HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM));
@@ -776,27 +779,30 @@ int launch_tc(const CUtensorMap& mw, const CUtensorMap& ma, const float* bias, v
     splits = ceil_div(k_blocks, kb_per_split);               // no split without work
     NIB_REQUIRE(!SWAP || splits == 1 || EPI == EPI_ADD, "gemm (tensor cores): token-row tiles split K only for the sum into the output");
     if (splits > 1 && EPI != EPI_ADD) {
-        const long long need = (long long)tiles * splits * (EPI == EPI_SWIGLU ? 2 : 1) * TOK * BLOCK_F;
+        const long long need = (long long)tiles * splits * (epi_dual(EPI) ? 2 : 1) * TOK * BLOCK_F;
         NIB_REQUIRE(sk.scratch != nullptr && sk.counters != nullptr && need <= sk.scratch_floats && 4LL * tiles <= sk.counter_ints,
                     "gemm (tensor cores): %d splits of %d tiles need %lld floats of scratch and %d counters (have %lld, %lld)",
                     splits, tiles, need, 4 * tiles, sk.scratch_floats, sk.counter_ints);
     }
     const int items = tiles * splits;
     NIB_CUDA(launch_pdl(gemm_tc_kernel<TOK, EPI, SWAP, HD>, dim3(items < sms ? items : sms), dim3(THREADS), (size_t)C::SMEM, stream,
-                        mw, ma, bias, out, tokens, n_out, k, ldo, splits, kb_per_split, sk.scratch, sk.counters, vec_ok, qe,
+                        mw, ma, bias, out, tokens, n_out, k, ldo, splits, kb_per_split, sk.scratch, sk.counters, vec_ok, qe, glu,
                         nib_trace_buffer(), nib_trace_capacity()));
     return 0;
 }
 
 template <int TOK>
 int launch_tc_epi(int epi, const CUtensorMap& mw, const CUtensorMap& ma, const float* bias, void* out, int tokens,
-                  int n_out, int k, int ldo, const SplitK& sk, cudaStream_t stream) {
+                  int n_out, int k, int ldo, const SplitK& sk, const NibGlu& glu, cudaStream_t stream) {
     switch (epi) {
         case EPI_STORE: return launch_tc<TOK, EPI_STORE>(mw, ma, bias, out, tokens, n_out, k, ldo, sk, stream);
         case EPI_ADD: return launch_tc<TOK, EPI_ADD>(mw, ma, bias, out, tokens, n_out, k, ldo, sk, stream);
         case EPI_F32: return launch_tc<TOK, EPI_F32>(mw, ma, bias, out, tokens, n_out, k, ldo, sk, stream);
         case EPI_SWIGLU:
             if constexpr (TOK <= 128) return launch_tc<TOK, EPI_SWIGLU>(mw, ma, bias, out, tokens, n_out, k, ldo, sk, stream);
+            break;
+        case EPI_GLU:
+            if constexpr (TOK <= 128) return launch_tc<TOK, EPI_GLU>(mw, ma, bias, out, tokens, n_out, k, ldo, sk, stream, 0, QkvRows{}, glu);
             break;
     }
     nib_set_error("gemm (tensor cores): unknown epilogue %d", epi);
@@ -805,14 +811,14 @@ int launch_tc_epi(int epi, const CUtensorMap& mw, const CUtensorMap& ma, const f
 
 template <int NT, int EPI>
 int launch_pair(const CUtensorMap& mm, const CUtensorMap& mn, const float* bias, void* out, int tokens, int n_out,
-                int k, int ldo, int vec_ok, int splits, cudaStream_t stream) {
+                int k, int ldo, int vec_ok, int splits, cudaStream_t stream, const NibGlu& glu = NibGlu{}) {
     using C = PairCfg<NT>;
     static bool configured = false;
     if (!configured) {
         NIB_CUDA(cudaFuncSetAttribute(gemm_pair_kernel<NT, EPI>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM));
         configured = true;
     }
-    const int feat = EPI == EPI_SWIGLU ? NT / 2 : NT;
+    const int feat = epi_dual(EPI) ? NT / 2 : NT;
     const int tiles = ceil_div(n_out, feat) * ceil_div(tokens, PAIR_M);
     const int k_blocks = ceil_div(k, BLOCK_K);
     if (EPI != EPI_ADD || splits < 1) splits = 1;
@@ -822,18 +828,19 @@ int launch_pair(const CUtensorMap& mm, const CUtensorMap& mn, const float* bias,
     int ctas = 2 * tiles * splits, most = sm_count() & ~1;
     if (ctas > most) ctas = most;
     NIB_CUDA(launch_pdl(gemm_pair_kernel<NT, EPI>, dim3(ctas), dim3(PAIR_THREADS), (size_t)C::SMEM, stream, mm, mn, bias, out,
-                        tokens, n_out, k, ldo, vec_ok, splits, kb_per_split, nib_trace_buffer(), nib_trace_capacity()));
+                        tokens, n_out, k, ldo, vec_ok, splits, kb_per_split, glu, nib_trace_buffer(), nib_trace_capacity()));
     return 0;
 }
 
 template <int NT>
 int launch_pair_epi(int epi, const CUtensorMap& mm, const CUtensorMap& mn, const float* bias, void* out, int tokens,
-                    int n_out, int k, int ldo, int vec_ok, int splits, cudaStream_t stream) {
+                    int n_out, int k, int ldo, int vec_ok, int splits, const NibGlu& glu, cudaStream_t stream) {
     switch (epi) {
         case EPI_STORE: return launch_pair<NT, EPI_STORE>(mm, mn, bias, out, tokens, n_out, k, ldo, vec_ok, splits, stream);
         case EPI_ADD: return launch_pair<NT, EPI_ADD>(mm, mn, bias, out, tokens, n_out, k, ldo, vec_ok, splits, stream);
         case EPI_F32: return launch_pair<NT, EPI_F32>(mm, mn, bias, out, tokens, n_out, k, ldo, vec_ok, splits, stream);
         case EPI_SWIGLU: return launch_pair<NT, EPI_SWIGLU>(mm, mn, bias, out, tokens, n_out, k, ldo, vec_ok, splits, stream);
+        case EPI_GLU: return launch_pair<NT, EPI_GLU>(mm, mn, bias, out, tokens, n_out, k, ldo, vec_ok, splits, stream, glu);
     }
     nib_set_error("gemm (tensor cores, two SMs per tile): unknown epilogue %d", epi);
     return 1;
@@ -858,23 +865,25 @@ NIB_API int nib_gemm_tc_error() {
 }
 
 // A [tokens, K] bfloat16 with row stride lda; W [N, K] (SWIGLU: [2N, K]); out [tokens, N] with row
-// stride ldo. epi: 0 store bf16, 1 add into float, 2 store float, 3 swiglu. tok_tile: 0 = chosen here.
+// stride ldo. epi: 0 store bf16, 1 add into float, 2 store float, 3 swiglu, 5 the gated form with the constants glu. tok_tile: 0 = chosen here.
 // splits: work items per output tile along K; 0 = chosen here (more than one only when the tiles alone
 // leave SMs idle and the scratch holds the partial sums), 1 = none. scratch/counters: a float buffer and
 // a zeroed int buffer that the kernels of one stream share (the counters are left zeroed).
 NIB_API int nib_gemm_tc_splitk(const void* A, const void* W, const float* bias, void* out, int tokens, int N, int K,
                                int lda, int ldo, int epi, int tok_tile, int splits, float* scratch, int* counters,
-                               long long scratch_floats, long long counter_ints, cudaStream_t stream) {
+                               long long scratch_floats, long long counter_ints, const NibGlu* glu, cudaStream_t stream) {
     NIB_REQUIRE(tokens >= 0 && N > 0 && K > 0 && lda >= K && ldo >= N, "gemm (tensor cores): bad sizes tokens=%d N=%d K=%d", tokens, N, K);
     NIB_REQUIRE(nib_gemm_tc_supported(A, W, K, lda), "gemm (tensor cores): K=%d / lda=%d must be multiples of 8 and bases 16-byte aligned", K, lda);
-    NIB_REQUIRE(epi != EPI_SWIGLU || bias == nullptr, "gemm (tensor cores): the swiglu epilogue takes no bias");
+    NIB_REQUIRE(!epi_dual(epi) || bias == nullptr, "gemm (tensor cores): the gated epilogues take no bias");
+    NIB_REQUIRE(epi != EPI_GLU || glu != nullptr, "gemm (tensor cores): the gated epilogue needs its constants");
+    const NibGlu constants = glu != nullptr ? *glu : NibGlu{};
     NIB_REQUIRE(splits >= 0, "gemm (tensor cores): splits=%d", splits);
     if (tokens == 0) return 0;
     const int f_tiles = ceil_div(N, BLOCK_F);
     if (tok_tile == 0) {
         tok_tile = tokens <= 16 ? 16 : tokens <= 32 ? 32 : tokens <= 64 ? 64 : 128;
         // 256 tokens per tile halves the shared-memory traffic per flop; take it when the grid still fills the GPU
-        if (tokens >= 512 && (long long)f_tiles * ceil_div(tokens, 256) >= 148 && epi != EPI_SWIGLU) tok_tile = 256;
+        if (tokens >= 512 && (long long)f_tiles * ceil_div(tokens, 256) >= 148 && !epi_dual(epi)) tok_tile = 256;
         // 33..64 tokens with few feature tiles (a decode step of 64 requests): two tiles of 32 tokens put twice the
         // SMs on the weights, which are what the step has to stream (measured: 3.4 us a layer at the 0.5B widths).
         // The sum into the output can split K over CTAs instead, which reads large weights once (measured better from
@@ -896,7 +905,7 @@ NIB_API int nib_gemm_tc_splitk(const void* A, const void* W, const float* bias, 
             if (want > k_blocks / 4) want = k_blocks / 4;
             if (epi != EPI_ADD) {
                 // partial sums through the scratch: one warp adds them up, which pays for few tokens only
-                const long long per_split = tiles * (epi == EPI_SWIGLU ? 2 : 1) * tok_tile * BLOCK_F;
+                const long long per_split = tiles * (epi_dual(epi) ? 2 : 1) * tok_tile * BLOCK_F;
                 if (scratch == nullptr || counters == nullptr || tok_tile > 16 || 4 * tiles > counter_ints) want = 1;
                 else if ((long long)want * per_split > scratch_floats) want = (int)(scratch_floats / per_split);
             }
@@ -904,7 +913,7 @@ NIB_API int nib_gemm_tc_splitk(const void* A, const void* W, const float* bias, 
         }
         sk.splits = want;
     }
-    const long long w_rows = (epi == EPI_SWIGLU) ? 2LL * N : N;
+    const long long w_rows = epi_dual(epi) ? 2LL * N : N;
     CUtensorMap mw, ma;
     {
         std::lock_guard<std::mutex> lock(g_map_mutex);
@@ -919,7 +928,7 @@ NIB_API int nib_gemm_tc_splitk(const void* A, const void* W, const float* bias, 
         }
     }
     if (make_map(&ma, A, tokens, K, lda, tok_tile)) return 1;
-    if (tok_tile == BLOCK_F && epi != EPI_SWIGLU && ((uintptr_t)bias & 15) == 0) {
+    if (tok_tile == BLOCK_F && !epi_dual(epi) && ((uintptr_t)bias & 15) == 0) {
         // tiles of 128 tokens: the token-row form (its epilogue writes rows, not columns). It splits K only for the sum.
         int splits_now = sk.splits < 1 ? 1 : sk.splits;
         if (epi == EPI_ADD || splits_now == 1) {
@@ -933,13 +942,13 @@ NIB_API int nib_gemm_tc_splitk(const void* A, const void* W, const float* bias, 
         }
     }
     switch (tok_tile) {
-        case 16: return launch_tc_epi<16>(epi, mw, ma, bias, out, tokens, N, K, ldo, sk, stream);
-        case 32: return launch_tc_epi<32>(epi, mw, ma, bias, out, tokens, N, K, ldo, sk, stream);
-        case 64: return launch_tc_epi<64>(epi, mw, ma, bias, out, tokens, N, K, ldo, sk, stream);
-        case 128: return launch_tc_epi<128>(epi, mw, ma, bias, out, tokens, N, K, ldo, sk, stream);
+        case 16: return launch_tc_epi<16>(epi, mw, ma, bias, out, tokens, N, K, ldo, sk, constants, stream);
+        case 32: return launch_tc_epi<32>(epi, mw, ma, bias, out, tokens, N, K, ldo, sk, constants, stream);
+        case 64: return launch_tc_epi<64>(epi, mw, ma, bias, out, tokens, N, K, ldo, sk, constants, stream);
+        case 128: return launch_tc_epi<128>(epi, mw, ma, bias, out, tokens, N, K, ldo, sk, constants, stream);
         case 256:
-            NIB_REQUIRE(epi != EPI_SWIGLU, "gemm (tensor cores): the swiglu epilogue takes token tiles up to 128 (two accumulators, double buffered)");
-            return launch_tc_epi<256>(epi, mw, ma, bias, out, tokens, N, K, ldo, sk, stream);
+            NIB_REQUIRE(!epi_dual(epi), "gemm (tensor cores): the gated epilogues take token tiles up to 128 (two accumulators, double buffered)");
+            return launch_tc_epi<256>(epi, mw, ma, bias, out, tokens, N, K, ldo, sk, constants, stream);
     }
     NIB_REQUIRE(false, "gemm (tensor cores): token tile %d is not one of 16, 32, 64, 128, 256", tok_tile);
 }
@@ -947,7 +956,7 @@ NIB_API int nib_gemm_tc_splitk(const void* A, const void* W, const float* bias, 
 // The same without split K (no scratch).
 NIB_API int nib_gemm_tc(const void* A, const void* W, const float* bias, void* out, int tokens, int N, int K,
                         int lda, int ldo, int epi, int tok_tile, cudaStream_t stream) {
-    return nib_gemm_tc_splitk(A, W, bias, out, tokens, N, K, lda, ldo, epi, tok_tile, 1, nullptr, nullptr, 0, 0, stream);
+    return nib_gemm_tc_splitk(A, W, bias, out, tokens, N, K, lda, ldo, epi, tok_tile, 1, nullptr, nullptr, 0, 0, nullptr, stream);
 }
 
 // 1 if nib_gemm_tc_qkv takes these sizes: heads of 64 or 128 that are rotated whole (rot == head_dim) or not at all,
@@ -1002,19 +1011,21 @@ NIB_API int nib_gemm_tc_qkv(const void* A, const void* W, const float* bias, voi
 // output features (128 or 256; 0 = 256). splits: work items along K per tile, for the ADD epilogue only
 // (0 = chosen here: enough to give every pair of SMs an item, at least 8 blocks of K each; 1 = none).
 NIB_API int nib_gemm_tc_pair(const void* A, const void* W, const float* bias, void* out, int tokens, int N, int K,
-                             int lda, int ldo, int epi, int n_tile, int splits, cudaStream_t stream) {
+                             int lda, int ldo, int epi, int n_tile, int splits, const NibGlu* glu, cudaStream_t stream) {
     NIB_REQUIRE(tokens >= 0 && N > 0 && K > 0 && lda >= K && ldo >= N, "gemm (two SMs per tile): bad sizes tokens=%d N=%d K=%d", tokens, N, K);
     NIB_REQUIRE(nib_gemm_tc_supported(A, W, K, lda), "gemm (two SMs per tile): K=%d / lda=%d must be multiples of 8 and bases 16-byte aligned", K, lda);
-    NIB_REQUIRE(epi != EPI_SWIGLU || bias == nullptr, "gemm (two SMs per tile): the swiglu epilogue takes no bias");
-    NIB_REQUIRE(epi >= EPI_STORE && epi <= EPI_SWIGLU, "gemm (two SMs per tile): unknown epilogue %d", epi);
+    NIB_REQUIRE(!epi_dual(epi) || bias == nullptr, "gemm (two SMs per tile): the gated epilogues take no bias");
+    NIB_REQUIRE(epi != EPI_GLU || glu != nullptr, "gemm (two SMs per tile): the gated epilogue needs its constants");
+    const NibGlu constants = glu != nullptr ? *glu : NibGlu{};
+    NIB_REQUIRE((epi >= EPI_STORE && epi <= EPI_SWIGLU) || epi == EPI_GLU, "gemm (two SMs per tile): unknown epilogue %d", epi);
     NIB_REQUIRE(((uintptr_t)bias & 15) == 0, "gemm (two SMs per tile): the bias must be 16-byte aligned");
     if (tokens == 0) return 0;
     if (n_tile == 0) n_tile = 256;      // measured: the instruction of 128 columns runs at about half the rate, whatever the grid
     NIB_REQUIRE(n_tile == 128 || n_tile == 256, "gemm (two SMs per tile): feature tile %d is not 128 or 256", n_tile);
     // 16-byte stores and reductions need rows of the output that start on 16 bytes
-    const int elem = (epi == EPI_STORE || epi == EPI_SWIGLU) ? 2 : 4;
+    const int elem = (epi == EPI_STORE || epi_dual(epi)) ? 2 : 4;
     const int vec_ok = (((uintptr_t)out & 15) == 0 && ((long long)ldo * elem) % 16 == 0) ? 1 : 0;
-    const long long w_rows = (epi == EPI_SWIGLU) ? 2LL * N : N;
+    const long long w_rows = epi_dual(epi) ? 2LL * N : N;
     CUtensorMap mm, mn;
     {
         std::lock_guard<std::mutex> lock(g_map_mutex);
@@ -1040,6 +1051,6 @@ NIB_API int nib_gemm_tc_pair(const void* A, const void* W, const float* bias, vo
             if (splits < 1) splits = 1;
         }
     }
-    if (n_tile == 128) return launch_pair_epi<128>(epi, mm, mn, bias, out, tokens, N, K, ldo, vec_ok, splits, stream);
-    return launch_pair_epi<256>(epi, mm, mn, bias, out, tokens, N, K, ldo, vec_ok, splits, stream);
+    if (n_tile == 128) return launch_pair_epi<128>(epi, mm, mn, bias, out, tokens, N, K, ldo, vec_ok, splits, constants, stream);
+    return launch_pair_epi<256>(epi, mm, mn, bias, out, tokens, N, K, ldo, vec_ok, splits, constants, stream);
 }

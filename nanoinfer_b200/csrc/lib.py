@@ -21,7 +21,8 @@ class KernelError(RuntimeError):
 
 
 _DT = {torch.float32: 0, torch.bfloat16: 1}
-_EPI = {"store": 0, "add": 1, "f32": 2, "swiglu": 3}
+_EPI = {"store": 0, "add": 1, "f32": 2, "swiglu": 3, "glu": 5}
+_DUAL = (3, 5)          # the gated epilogues: two accumulators, gate rows and up rows
 _LAYOUT = {"interleaved": 0, "half": 1}     # which elements of a rotated vector make a pair
 
 
@@ -90,7 +91,7 @@ class Kernels:
                      "nib_linear_state_scan", "nib_conv_tokens", "nib_conv_tail", "nib_conv_step", "nib_token_shift", "nib_decay_map", "nib_step_sizes",
                      "nib_attention_prepare", "nib_attention_flex", "nib_attention_flex_mma", "nib_attention_flex_mma_supported",
                      "nib_rmsnorm_add", "nib_moe_route", "nib_moe_max_tiles", "nib_moe_group", "nib_moe_gemm_simt", "nib_moe_combine",
-                     "nib_moe_tc_supported", "nib_moe_tc_error", "nib_moe_gather_rows", "nib_moe_gemm_tc", "nib_moe_step", "nib_moe_step_supported"):
+                     "nib_moe_tc_supported", "nib_moe_tc_error", "nib_moe_gather_rows", "nib_moe_gemm_tc", "nib_moe_step", "nib_moe_step_supported", "nib_moe_identity", "nib_stream_mix", "nib_delta_state_scan", "nib_memory_gates"):
             getattr(self._lib, name).restype = c_int
 
     # ---- plumbing ---------------------------------------------------------------------------
@@ -242,13 +243,13 @@ class Kernels:
             small = m <= 16 and k <= 2048
         elif epi == _EPI["store"]:
             small = m <= 64 and rows <= 6144
-        elif epi == _EPI["swiglu"]:
+        elif epi in _DUAL:
             small = (m <= 8 and weight_bytes <= 64e6) or (m <= 16 and weight_bytes <= 12e6)
         else:
             small = m <= 16 and weight_bytes <= 32e6
         # (inside the gate/up product the norm measured slower, +2 us a layer at the 0.5B widths: 300 CTAs re-read
         # the 32-bit activations; the norm kernel before it costs less)
-        fuse = has_norm and small and epi != _EPI["swiglu"] and (m <= 8 or (m <= 16 and k <= 1024))
+        fuse = has_norm and small and epi not in _DUAL and (m <= 8 or (m <= 16 and k <= 1024))
         return ("smallm" if small else "tc"), fuse
 
     def _use_pair(self, m: int, rows: int, k: int, epi: int) -> bool:
@@ -265,7 +266,7 @@ class Kernels:
         # measured on B200 at the projection sizes of the 0.5B, 1.5B and 7B models, 512..4096 tokens: tiles
         # of 256 tokens x 256 features on two SMs win once there are enough of them to fill the GPU; the
         # fused gate/up form (gate rows in one CTA, up rows in the other) wins from 256 tokens on
-        if epi == _EPI["swiglu"]:
+        if epi in _DUAL:
             return True
         tiles = -(-rows // 256) * -(-m // 256)
         return tiles >= 48
@@ -287,9 +288,9 @@ class Kernels:
         computed it (a computed norm is just a tensor)."""
         return lazy is not None and lazy.resolved is None and lazy.fold.kind == "rms"
 
-    def _gemm(self, a, w, bias32, out, m, n, k, epi):
+    def _gemm(self, a, w, bias32, out, m, n, k, epi, glu=None):
         """bfloat16 goes to the small-M kernel or to the tcgen05 kernel (see ``_route``); shapes neither
-        takes, and 32-bit, run the CUDA-core kernel."""
+        takes, and 32-bit, run the CUDA-core kernel. ``glu``: the constants of the gated epilogue."""
         lazy = a if isinstance(a, LazyNorm) else None
         if lazy is not None and not self._foldable(lazy):
             a, lazy = lazy.resolve(), None
@@ -307,7 +308,7 @@ class Kernels:
                     _ptr(src), _ptr(w), _ptr(bias32), _ptr(out), c_int(m), c_int(n), c_int(k), c_int(src.stride(0)),
                     c_int(out.stride(0)), c_int(epi), _ptr(gain), c_float(lazy.fold.eps if lazy is not None else 0.0),
                     c_int(self.options.smallm_ksplit), c_int(self.options.smallm_cross), _ptr(self._ws_scratch), _ptr(self._ws_counters),
-                    c_longlong(self._ws_scratch.numel()), c_int(self._ws_counters.numel()), self._stream()),
+                    c_longlong(self._ws_scratch.numel()), c_int(self._ws_counters.numel()), glu, self._stream()),
                     "linear (small M)")
                 return
         if lazy is not None:
@@ -316,7 +317,7 @@ class Kernels:
             if self._use_pair(m, w.shape[0], k, epi):
                 self._check(self._lib.nib_gemm_tc_pair(
                     _ptr(a), _ptr(w), _ptr(bias32), _ptr(out), c_int(m), c_int(n), c_int(k), c_int(a.stride(0)),
-                    c_int(out.stride(0)), c_int(epi), c_int(self.options.pair_n_tile), c_int(self.options.tc_splits), self._stream()),
+                    c_int(out.stride(0)), c_int(epi), c_int(self.options.pair_n_tile), c_int(self.options.tc_splits), glu, self._stream()),
                     "linear (tensor cores, two SMs per tile)")
                 return
             self.ensure_workspace(a.device)
@@ -324,18 +325,19 @@ class Kernels:
                 _ptr(a), _ptr(w), _ptr(bias32), _ptr(out), c_int(m), c_int(n), c_int(k), c_int(a.stride(0)),
                 c_int(out.stride(0)), c_int(epi), c_int(self.options.tc_token_tile), c_int(self.options.tc_splits),
                 _ptr(self._ws_scratch), _ptr(self._ws_counters), c_longlong(self._ws_scratch.numel()),
-                c_longlong(self._ws_counters.numel()), self._stream()), "linear (tensor cores)")
+                c_longlong(self._ws_counters.numel()), glu, self._stream()), "linear (tensor cores)")
             return
         self._check(self._lib.nib_gemm_simt(_ptr(a), _ptr(w), _ptr(bias32), _ptr(out), c_int(m), c_int(n), c_int(k),
-                                            c_int(a.stride(0)), c_int(out.stride(0)), c_int(epi), c_int(_DT[a.dtype]),
+                                            c_int(a.stride(0)), c_int(out.stride(0)), c_int(epi), c_int(_DT[a.dtype]), glu,
                                             self._stream()), "linear")
 
     def gemm_tc_error(self) -> int:
         """The error word of the tensor-core GEMM's bounded waits (0 = none); synchronises and clears it."""
         return self._lib.nib_gemm_tc_error()
 
-    def linear_swiglu(self, a, w_gate_up, out):
-        """out[M,I] = silu(a . w[:I]^T) * (a . w[I:]^T)."""
+    def linear_swiglu(self, a, w_gate_up, out, glu=None):
+        """out[M,I] = silu(a . w[:I]^T) * (a . w[I:]^T). With ``glu`` = (alpha, limit, shift): g = min(gate, limit),
+        u = clamp(up, -limit, limit), g * sigmoid(alpha g) * (u + shift)."""
         if not isinstance(a, LazyNorm):
             _need(a, None, "swiglu a")
         _need(w_gate_up, a.dtype, "swiglu w"); _need(out, a.dtype, "swiglu out")
@@ -343,7 +345,7 @@ class Kernels:
         inter = w_gate_up.shape[0] // 2
         if w_gate_up.shape[0] != 2 * inter or w_gate_up.shape[1] != k or tuple(out.shape) != (m, inter):
             raise KernelError("linear_swiglu: shapes do not fit")
-        self._gemm(a, w_gate_up, None, out, m, inter, k, _EPI["swiglu"])
+        self._gemm(a, w_gate_up, None, out, m, inter, k, _EPI["swiglu" if glu is None else "glu"], _glu(glu))
 
     def qkv_project(self, a, w_qkv, bias32, qkv, heads, kv_heads, head_dim, positions, req_index, rotary,
                     block_table, page_size, k_pages, v_pages, writes):
@@ -512,7 +514,7 @@ class Kernels:
                     _ptr(qkv), c_int(qkv.stride(0)), _ptr(out), q_start, lens, table, c_int(bt_stride), c_int(page_size),
                     _ptr(k_pages), _ptr(v_pages), c_int(num_pages), c_int(n_req - n_dec), c_int(max(q_lens[n_dec:])),
                     c_int(m), c_int(heads), c_int(kv_heads), c_int(head_dim), c_float(scale), c_int(window), c_float(0.0), c_int(0), None,
-                    self._stream()), "attention prefill (tcgen05)")
+                    c_float(1.0), self._stream()), "attention prefill (tcgen05)")
             else:
                 self._check(self._lib.nib_attention_prefill_mma(
                     _ptr(qkv), c_int(qkv.stride(0)), _ptr(out), q_start, lens, table, c_int(bt_stride), c_int(page_size),
@@ -691,6 +693,33 @@ class Kernels:
                                               c_int(1 if clear else 0), c_int(_DT[h_out.dtype] if h_out is not None else 0), _ptr(next_gain32),
                                               c_float(next_eps), self._stream()), "rmsnorm_add")
 
+    # ---- several residual streams (pointwise.cu) -----------------------------------------------------------
+    def stream_mix(self, x32, streams, y32=None, mix32=None, out32=None, dst32=None, in32=None, gain32=None, eps=0.0, h_out=None,
+                   sum_out32=None, clear=False):
+        """One pass over the rows between two sublayers of a model with several residual streams. ``x32``: the streams
+        [tokens, streams, width], or one [tokens, width] that they all equal. With ``y32`` (a sublayer's result):
+        z_t = sum_s mix32[s, t] x_s + out32[t] y32, else z = x. z goes to ``dst32`` [tokens, streams, width] (may be x32),
+        sum_s z_s to ``sum_out32``, and rms-norm(sum_s in32[s] z_s) * gain32 to ``h_out``; with ``clear`` y32 is left zeroed."""
+        _need(x32, torch.float32, "stream_mix x")
+        m, width = x32.shape[0], x32.shape[-1]
+        if tuple(x32.shape) not in ((m, width), (m, streams, width)):
+            raise KernelError("stream_mix: x holds one stream or all of them")
+        for t, shape, what in ((y32, (m, width), "y"), (mix32, (streams, streams), "mix"), (out32, (streams,), "out"), (in32, (streams,), "in"),
+                               (dst32, (m, streams, width), "dst"), (gain32, (width,), "gain"), (sum_out32, (m, width), "sum")):
+            if t is not None:
+                _need(t, torch.float32, f"stream_mix {what}")
+                if tuple(t.shape) != shape:
+                    raise KernelError(f"stream_mix: {what} does not fit")
+        if h_out is not None:
+            _need(h_out, None, "stream_mix h")
+            if tuple(h_out.shape) != (m, width):
+                raise KernelError("stream_mix: h does not fit")
+        one = x32.dim() == 2
+        self._check(self._lib.nib_stream_mix(
+            _ptr(x32), c_longlong(width if one else streams * width), c_longlong(0 if one else width), _ptr(y32), _ptr(mix32), _ptr(out32),
+            _ptr(dst32), _ptr(in32), _ptr(gain32), c_float(eps), _ptr(h_out), _ptr(sum_out32), c_int(m), c_int(width), c_int(streams),
+            c_int(1 if clear else 0), c_int(_DT[h_out.dtype] if h_out is not None else 0), self._stream()), "stream_mix")
+
     # ---- routed experts (moe.cu) ---------------------------------------------------------------------------
     def moe_route(self, z32, top, sel_e, sel_w, score="sigmoid", renormalize=False, correction32=None, always=0):
         """From the router logits z32 [tokens, experts]: sel_e [tokens, top] int32 = the experts with the largest logits (the
@@ -762,13 +791,14 @@ class Kernels:
                                            c_int(always), self._stream()), "experts: router, choice and grouping of a short step")
         return plan
 
-    def moe_experts(self, h, sel_e, sel_w, w_gate_up, w_down, out32, plan=None, gated=True, weight_on="input", outputs=None):
+    def moe_experts(self, h, sel_e, sel_w, w_gate_up, w_down, out32, plan=None, gated=True, weight_on="input", outputs=None, glu=None):
         """out32[t] += sum over the token's choices c of W_down,e (silu(W_gate,e x) * (W_up,e x)) with e = sel_e[t, c] and
         x = sel_w[t, c] * h[t]: the weight stands on the expert's input. w_gate_up [experts, 2 ff, hidden] (gate rows, then up
         rows), w_down [experts, hidden, ff]. ``plan``: what ``moe_step`` returned for these choices. Options: ``gated`` False:
         experts W_down relu(W_up x)^2 with w_gate_up [experts, ff, hidden]; ``weight_on`` 'output': x = h[t] and the weight
         multiplies the expert's result; ``outputs``: how many outputs the router has when some of them (from ``experts`` on)
-        are no experts: choices of those add nothing here.
+        are no experts: choices of those add nothing here; ``glu`` = (alpha, limit, shift): the gated form of ``linear_swiglu`` with
+        those constants in place of silu(gate) * up.
 
         On the CUDA cores a token's choices are summed in ascending order; on the tensor cores they are added into the
         token's row by reductions in memory, in no fixed order."""
@@ -784,7 +814,9 @@ class Kernels:
         if m == 0:
             return
         n, dev, dt = m * top, h.device, c_int(_DT[h.dtype])
-        first, w_out = c_int(1 if gated else 2), c_int(1 if weight_on == "output" else 0)
+        if glu is not None and not gated:
+            raise KernelError("moe_experts: the constants of a gated form belong to experts with a gate")
+        first, w_out, glu = c_int((1 if glu is None else 3) if gated else 2), c_int(1 if weight_on == "output" else 0), _glu(glu)
         outputs = experts if outputs is None else outputs
         tc = self._moe_tc(h, w_gate_up, w_down)
         p = plan
@@ -800,20 +832,20 @@ class Kernels:
                                                           c_int(top), self._stream()), "experts: rows in the experts' order")
             self._check(self._lib.nib_moe_gemm_tc(first, _ptr(p.rows), c_int(hidden), c_int(n), _ptr(w_gate_up), c_int(experts), _ptr(act), c_int(ff),
                                                   _ptr(p.tiles), _ptr(p.n_tiles), c_int(p.max_tiles), _ptr(p.src_of), _ptr(sel_w), c_int(top), c_int(ff),
-                                                  c_int(hidden), c_int(0), c_int(p.tile_rows), w_out, self._stream()), "experts: gate, up, activation (tensor cores)")
+                                                  c_int(hidden), c_int(0), c_int(p.tile_rows), w_out, glu, self._stream()), "experts: gate, up, activation (tensor cores)")
             self._check(self._lib.nib_moe_gemm_tc(c_int(0), _ptr(act), c_int(ff), c_int(n), _ptr(w_down), c_int(experts), _ptr(out32), c_int(out32.stride(0)),
                                                   _ptr(p.tiles), _ptr(p.n_tiles), c_int(p.max_tiles), _ptr(p.src_of), _ptr(sel_w), c_int(top), c_int(hidden),
-                                                  c_int(ff), c_int(1 if top == 1 else 2), c_int(p.tile_rows), w_out, self._stream()), "experts: down (tensor cores)")
+                                                  c_int(ff), c_int(1 if top == 1 else 2), c_int(p.tile_rows), w_out, None, self._stream()), "experts: down (tensor cores)")
             return
         scatter = top == 1      # one choice per token: its result goes straight into the token's row
         # (rows of choices that are no experts belong to no tile: they must read as zeros in the sum of a token's choices)
         y = out32 if scatter else (torch.empty if outputs == experts else torch.zeros)((n, hidden), dtype=torch.float32, device=dev)
         self._check(self._lib.nib_moe_gemm_simt(first, _ptr(h), c_int(h.stride(0)), _ptr(w_gate_up), _ptr(act), c_int(ff), _ptr(p.tiles), _ptr(p.n_tiles),
                                                 c_int(p.max_tiles), _ptr(p.src_of), _ptr(sel_w), c_int(top), c_int(ff), c_int(hidden), c_int(0), dt,
-                                                w_out, self._stream()), "experts: gate, up, activation")
+                                                w_out, glu, self._stream()), "experts: gate, up, activation")
         self._check(self._lib.nib_moe_gemm_simt(c_int(0), _ptr(act), c_int(ff), _ptr(w_down), _ptr(y), c_int(y.stride(0)), _ptr(p.tiles), _ptr(p.n_tiles),
                                                 c_int(p.max_tiles), _ptr(p.src_of), _ptr(sel_w), c_int(top), c_int(hidden), c_int(ff), c_int(1 if scatter else 0),
-                                                dt, w_out, self._stream()), "experts: down")
+                                                dt, w_out, None, self._stream()), "experts: down")
         if not scatter:
             self._check(self._lib.nib_moe_combine(_ptr(y), _ptr(p.row_of), _ptr(out32), c_int(m), c_int(hidden), c_int(top), self._stream()),
                         "experts: sum of a token's choices")
@@ -831,15 +863,21 @@ class Kernels:
 
     # ---- gate, norm in groups, skip (pointwise.cu) ---------------------------------------------------------
     def gated_norm(self, o32, out, groups=0, eps=0.0, gain32=None, gate32=None, gate_kind="none", gate_first=False,
-                   skip32=None, skip_coef32=None, out_scale=1.0):
+                   skip32=None, skip_coef32=None, out_scale=1.0, floor32=None, den_eps=0.0):
         """Row by row: y = o32 (+ skip_coef32[head of c] * skip32); times act(gate32) if ``gate_first``; with ``groups`` > 0
         divided by the root mean square of each of ``groups`` equal parts (``eps`` inside the root); times ``gain32`` (a gain
         per channel, or one of a part's size shared by the parts); times act(gate32) if not ``gate_first``; times
-        ``out_scale``. gate_kind: 'none' | 'sigmoid' | 'silu'. ``skip_coef32`` holds one coefficient per head."""
+        ``out_scale``. gate_kind: 'none' | 'sigmoid' | 'silu'. ``skip_coef32`` holds one coefficient per head. With ``floor32``
+        [tokens, groups] every part of o32 is one number wider than a part of ``out``: its last number d is no channel but a
+        divisor, y = o32 / (max(|d|, floor32) + den_eps) comes first."""
         self._rows(o32, torch.float32, "gated_norm o"); self._rows(out, None, "gated_norm out")
-        m, n = o32.shape
-        if tuple(out.shape) != (m, n):
+        m, n = out.shape
+        if tuple(o32.shape) != (m, n if floor32 is None else n + groups):
             raise KernelError("gated_norm: shapes do not fit")
+        if floor32 is not None:
+            self._rows(floor32, torch.float32, "gated_norm floor")
+            if groups <= 0 or tuple(floor32.shape) != (m, groups):
+                raise KernelError("gated_norm: one floor per (token, part)")
         kind = {"none": 0, "sigmoid": 1, "silu": 2}[gate_kind]
         if (kind != 0) != (gate32 is not None) or (skip32 is None) != (skip_coef32 is None):
             raise KernelError("gated_norm: a gate needs its kind, a skip its coefficients")
@@ -861,7 +899,7 @@ class Kernels:
             c_int(1 if gate_first else 0), _ptr(gain32), c_int(0 if gain32 is None else gain32.numel()), _ptr(skip32),
             c_int(0 if skip32 is None else skip32.stride(0)), _ptr(skip_coef32), c_int(0 if skip_coef32 is None else skip_coef32.numel()),
             c_int(groups), c_int(norm), c_float(eps), c_float(out_scale), _ptr(out), c_int(out.stride(0)), c_int(m), c_int(n),
-            c_int(_DT[out.dtype]), self._stream()), "gated_norm")
+            c_int(_DT[out.dtype]), _ptr(floor32), c_int(0 if floor32 is None else floor32.stride(0)), c_float(den_eps), self._stream()), "gated_norm")
 
     # ---- matrix states that decay (linear_state.cu) -------------------------------------------------------
     @staticmethod
@@ -872,19 +910,22 @@ class Kernels:
             raise KernelError(f"{what}: the state does not hold {size} floats from column {off}")
 
     def linear_state_scan(self, q32, k32, v32, w32, state, state_off, ctx, o32, heads, kq_heads, dk, dv, q_scale=1.0,
-                          bonus32=None, v_scale32=None, seg_len=None):
+                          bonus32=None, v_scale32=None, seg_len=None, ones=False):
         """Per request and head, over the step's tokens in order, from and into ``state[slot, state_off:]`` (laid out
         [head, value channel, key channel]): S <- diag(w) S + k (v_scale v)^T, o = S^T (q_scale q); with ``bonus32``
         [heads, dk] instead o = (S_old + diag(bonus) k v^T)^T q before the update. q32, k32: [tokens, kq_heads * dk]
         (head h reads key head h // (heads / kq_heads)); v32, o32: [tokens, heads * dv]; w32: [tokens, heads * dk] (a
-        decay per key channel) or [tokens, heads] (one per head); v_scale32: [tokens, heads].
+        decay per key channel) or [tokens, heads] (one per head); v_scale32: [tokens, heads]. With ``ones`` a head has one
+        value channel more than ``dv``, behind the others, whose value is 1: the state holds heads * (dv + 1) * dk floats and
+        o32 is [tokens, heads * (dv + 1)].
 
         A step in which a request brings 256 tokens or more, and whose walk in order would not fill the GPU, is walked in
         segments of 128 tokens or more side by side (every
         segment from a zero state, the end states chained with the products of the segments' decays, then every segment
         again from its true entry state): the result then depends on the cut by rounding. ``seg_len``: None = that rule,
         0 = never, another multiple of 8 = segments of that length whenever a request brings more."""
-        for t, what, width in ((q32, "q", kq_heads * dk), (k32, "k", kq_heads * dk), (v32, "v", heads * dv), (o32, "o", heads * dv)):
+        extra = 1 if ones else 0
+        for t, what, width in ((q32, "q", kq_heads * dk), (k32, "k", kq_heads * dk), (v32, "v", heads * dv), (o32, "o", heads * (dv + extra))):
             self._rows(t, torch.float32, f"linear_state_scan {what}")
             if tuple(t.shape) != (q32.shape[0], width):
                 raise KernelError(f"linear_state_scan: {what} does not fit")
@@ -900,6 +941,7 @@ class Kernels:
             _need(v_scale32, torch.float32, "linear_state_scan v_scale")
             if tuple(v_scale32.shape) != (q32.shape[0], heads):
                 raise KernelError("linear_state_scan: v_scale does not fit")
+        dv += extra         # from here on the state's value channels
         self._state_row(state, state_off, heads * dv * dk, "linear_state_scan state")
         n_req, longest = ctx.host.num_requests, max(ctx.host.q_lens)
         if seg_len is None:
@@ -921,7 +963,59 @@ class Kernels:
             c_int(w32.stride(0)), c_int(1 if per_channel else 0), _ptr(bonus32), _ptr(v_scale32), _ptr(state), c_longlong(state.stride(0)),
             c_int(state_off), _ptr(ctx.q_start), _ptr(ctx.state_slots), _ptr(o32), c_int(o32.stride(0)), c_int(ctx.host.num_requests),
             c_int(heads), c_int(kq_heads), c_int(dk), c_int(dv), c_float(q_scale), c_int(n_seg), c_int(seg_len if n_seg > 1 else 0), _ptr(scratch),
-            self._stream()), "linear_state_scan")
+            c_int(extra), self._stream()), "linear_state_scan")
+
+    def memory_gates(self, zi32, zf32, bi32, bf32, cap, state, state_off, ctx, decay32, write32, floor32):
+        """Gates of a stabilized matrix memory, per (token, head): i = cap * tanh((zi32 + bi32) / cap), f = log sigmoid(cap *
+        tanh((zf32 + bf32) / cap)), m_t = max(f + m_(t-1), i) from ``state[slot, state_off + head]`` (which becomes the last
+        m); decay32 = exp(f + m_(t-1) - m_t), write32 = exp(i - m_t), floor32 = exp(-m_t), all [tokens, heads]."""
+        for t, what in ((zi32, "i"), (zf32, "f")):
+            self._rows(t, torch.float32, f"memory_gates {what}")
+        m, heads = zi32.shape
+        for t, what in ((decay32, "decay"), (write32, "write"), (floor32, "floor")):
+            _need(t, torch.float32, f"memory_gates {what}")
+        for t in (bi32, bf32):
+            _need(t, torch.float32, "memory_gates bias")
+        if tuple(zf32.shape) != (m, heads) or bi32.numel() != heads or bf32.numel() != heads \
+                or any(tuple(t.shape) != (m, heads) for t in (decay32, write32, floor32)):
+            raise KernelError("memory_gates: shapes do not fit")
+        self._state_row(state, state_off, heads, "memory_gates state")
+        self._check(self._lib.nib_memory_gates(
+            _ptr(zi32), c_int(zi32.stride(0)), _ptr(zf32), c_int(zf32.stride(0)), _ptr(bi32), _ptr(bf32), c_float(cap), _ptr(state),
+            c_longlong(state.stride(0)), c_int(state_off), _ptr(ctx.q_start), _ptr(ctx.state_slots), _ptr(decay32), _ptr(write32), _ptr(floor32),
+            c_int(ctx.host.num_requests), c_int(max(ctx.host.q_lens)), c_int(heads), self._stream()), "memory_gates")
+
+    # ---- the gated delta rule (delta_state.cu) ---------------------------------------------------------------
+    def delta_state_scan(self, q32, k32, v32, z32, b32, state, state_off, ctx, o32, heads, kq_heads, dk, dv, dt_bias32=None, a_log32=None,
+                         q_scale=1.0, unit_eps=1e-6):
+        """Per request and head, over the step's tokens in order, from and into ``state[slot, state_off:]`` (laid out [head,
+        value channel, key channel]), with k and q made unit vectors per head (x / sqrt(sum x^2 + unit_eps), q times
+        ``q_scale``): S <- diag(w) S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q. beta = sigmoid(b32) [tokens, heads];
+        w = exp(-exp(a_log32[head]) * softplus(z32 + dt_bias32)) per (head, key channel), or z32 itself without ``a_log32``.
+        q32, k32: [tokens, kq_heads * dk] (head h reads head h // (heads / kq_heads)); v32, o32: [tokens, heads * dv];
+        z32: [tokens, heads * dk]. Tokens are taken eight at a time; how a request is cut moves the result by rounding."""
+        for t, what, width in ((q32, "q", kq_heads * dk), (k32, "k", kq_heads * dk), (v32, "v", heads * dv), (o32, "o", heads * dv),
+                               (z32, "z", heads * dk), (b32, "beta", heads)):
+            self._rows(t, torch.float32, f"delta_state_scan {what}")
+            if tuple(t.shape) != (q32.shape[0], width):
+                raise KernelError(f"delta_state_scan: {what} does not fit")
+        if (dt_bias32 is None) != (a_log32 is None):
+            raise KernelError("delta_state_scan: step sizes need both their bias and the rates")
+        for t, n in ((dt_bias32, heads * dk), (a_log32, heads)):
+            if t is not None:
+                _need(t, torch.float32, "delta_state_scan decay")
+                if t.numel() != n:
+                    raise KernelError("delta_state_scan: the decays' constants do not fit")
+        self._state_row(state, state_off, heads * dv * dk, "delta_state_scan state")
+        m = q32.shape[0]
+        scratch = torch.empty(m * heads * (4 * dk + 16), dtype=torch.float32, device=q32.device)
+        self.launches += 1
+        self._check(self._lib.nib_delta_state_scan(
+            _ptr(q32), c_int(q32.stride(0)), _ptr(k32), c_int(k32.stride(0)), _ptr(v32), c_int(v32.stride(0)), _ptr(z32), c_int(z32.stride(0)),
+            _ptr(dt_bias32), _ptr(a_log32), _ptr(b32), c_int(b32.stride(0)), _ptr(state), c_longlong(state.stride(0)), c_int(state_off),
+            _ptr(ctx.q_start), _ptr(ctx.state_slots), _ptr(o32), c_int(o32.stride(0)), _ptr(scratch), c_int(m), c_int(ctx.host.num_requests),
+            c_int(max(ctx.host.q_lens)), c_int(heads), c_int(kq_heads), c_int(dk), c_int(dv), c_float(q_scale), c_float(unit_eps),
+            self._stream()), "delta_state_scan")
 
     def conv_tokens(self, x32, w32, bias32, act, state, state_off, ctx, out32, taps):
         """out32[t, c] = act(bias32[c] + sum_j w32[c, j] * x32[t - (taps-1-j), c]) within each request; inputs before the
@@ -1072,7 +1166,7 @@ class Kernels:
             if sinks32.numel() != heads:
                 raise KernelError("attention_flex: one sink per head")
         n_rep = heads // max(1, kv_heads)
-        if q.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and dim == vdim and slopes32 is None and out_scale == 1.0 \
+        if q.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and dim == vdim and slopes32 is None \
                 and max(ctx.host.q_lens) * n_rep > 64 and not self.options.force_general_attention and not self.options.force_mma_prefill \
                 and self._lib.nib_attention_prefill_tc_supported(c_int(heads), c_int(kv_heads), c_int(dim), c_int(page_size), c_int(q.stride(0))) == 1:
             # prompt portions with heads of 64 or 128 (keys and values alike): the tcgen05 kernel's instance with options
@@ -1080,7 +1174,7 @@ class Kernels:
                 _ptr(q), c_int(q.stride(0)), _ptr(out), _ptr(ctx.q_start), _ptr(ctx.ctx_lens), _ptr(block_table), c_int(block_table.stride(0)),
                 c_int(page_size), _ptr(k_pages), _ptr(v_pages), c_int(k_pages.shape[0]), c_int(ctx.host.num_requests), c_int(max(ctx.host.q_lens)),
                 c_int(m), c_int(heads), c_int(kv_heads), c_int(dim), c_float(scale), c_int(window), c_float(softcap), c_int(chunk), _ptr(sinks32),
-                self._stream()), "attention (options, tcgen05)")
+                c_float(out_scale), self._stream()), "attention (options, tcgen05)")
             return
         if q.dtype == torch.bfloat16 and not self.options.force_general_attention and page_size > 0 \
                 and self._lib.nib_attention_flex_mma_supported(c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim), c_int(q.stride(0))) == 1:
@@ -1325,6 +1419,11 @@ class Kernels:
 TIMELINE_KERNELS = {1: "embed", 2: "rmsnorm", 3: "rope_store", 4: "gemm_smallm", 5: "gemm_stream", 6: "gemm_tc",
                     7: "attention_decode", 8: "attention_combine", 9: "argmax", 10: "attention_decode_mma",
                     11: "gemm_pair", 12: "attention_prefill"}
+
+
+def _glu(constants):
+    """(alpha, limit, shift) of the gated epilogue as the kernels read them, None without."""
+    return None if constants is None else (c_float * 3)(*(float(x) for x in constants))
 
 
 def _moe_mode(score: str, renormalize: bool) -> int:

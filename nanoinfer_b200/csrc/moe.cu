@@ -254,14 +254,14 @@ moe_step_kernel(const T* __restrict__ h, int ldh, const T* __restrict__ w_router
     }
 }
 
-// MODE 0: down; 1: gate and up, silu(g) u; 2: up alone, relu(u)^2. w_out: the weight multiplies the down product's result
+// MODE 0: down; 1: gate and up, silu(g) u; 2: up alone, relu(u)^2; 3: gate and up, the gated form with constants. w_out: the weight multiplies the down product's result
 // instead of the first product's input.
 template <typename T, int MODE>
 __global__ void __launch_bounds__(256)
 moe_gemm_simt_kernel(const T* __restrict__ A, int lda, const T* __restrict__ W, void* __restrict__ out, int ldo,
                      const int* __restrict__ tiles, const int* __restrict__ n_tiles, const int* __restrict__ src_of,
-                     const float* __restrict__ sel_w, int top, int N, int K, int scatter, int w_out) {
-    constexpr bool GATE_UP = MODE == 1, FIRST = MODE != 0;
+                     const float* __restrict__ sel_w, int top, int N, int K, int scatter, int w_out, const NibGlu glu) {
+    constexpr bool GATE_UP = MODE == 1 || MODE == 3, FIRST = MODE != 0;
     constexpr int BM = 64, BN = 64, BK = 16, TM = 4, TN = 4;
     pdl_launch_dependents();
     pdl_wait();      // everything this kernel reads may come from the kernel before
@@ -355,7 +355,7 @@ moe_gemm_simt_kernel(const T* __restrict__ A, int lda, const T* __restrict__ W, 
             const size_t o = (size_t)o_row[r] * ldo + n;
             if (GATE_UP) {
                 const float g = acc[i][j] * a_wgt[r], u = acc2[GATE_UP ? i : 0][GATE_UP ? j : 0] * a_wgt[r];
-                Elem<T>::store((T*)out + o, g / (1.0f + expf(-g)) * u);
+                Elem<T>::store((T*)out + o, MODE == 3 ? nib_glu_exact(glu, g, u) : g / (1.0f + expf(-g)) * u);
             } else if (FIRST) {
                 const float u = fmaxf(acc[i][j] * a_wgt[r], 0.f);
                 Elem<T>::store((T*)out + o, u * u);
@@ -442,20 +442,22 @@ NIB_API int nib_moe_step(const void* h, int ldh, const void* w_router, int token
 }
 
 // gate_up 1: A = the tokens' activations [tokens, K] (rows gathered through src_of), W [experts, 2N, K] (gate rows, then
-// up rows), out [entries, N] in the storage type; 2: the same with W [experts, N, K] (no gate) and relu(.)^2. 0: A = [entries, K] in the grouped order, W [experts, N, K], out floats:
+// up rows), out [entries, N] in the storage type; 2: the same with W [experts, N, K] (no gate) and relu(.)^2; 3: like 1 with the gated form of the constants glu. 0: A = [entries, K] in the grouped order, W [experts, N, K], out floats:
 // [entries, N] in the grouped order, or with scatter (one choice per token) added into the token's row of [tokens, N].
 // The tiles must have been made for rows of 64.
 NIB_API int nib_moe_gemm_simt(int gate_up, const void* A, int lda, const void* W, void* out, int ldo, const int* tiles, const int* n_tiles,
                               int max_tiles, const int* src_of, const float* sel_w, int top, int N, int K, int scatter, int dtype,
-                              int w_out, cudaStream_t stream) {
-    NIB_REQUIRE(N > 0 && K > 0 && top > 0 && max_tiles >= 0 && (!scatter || top == 1) && gate_up >= 0 && gate_up <= 2, "moe_gemm: bad sizes");
+                              int w_out, const NibGlu* glu, cudaStream_t stream) {
+    NIB_REQUIRE(N > 0 && K > 0 && top > 0 && max_tiles >= 0 && (!scatter || top == 1) && gate_up >= 0 && gate_up <= 3, "moe_gemm: bad sizes");
+    NIB_REQUIRE(gate_up != 3 || glu != nullptr, "moe_gemm: the gated form needs its constants");
+    const NibGlu constants = glu != nullptr ? *glu : NibGlu{};
     NIB_REQUIRE(dtype == NIB_F32 || dtype == NIB_BF16, "moe_gemm: unknown dtype %d", dtype);
     if (max_tiles == 0) return 0;
     const dim3 grid(ceil_div(N, 64), max_tiles), block(256);
 #define NIB_MG(T, GU) \
-    NIB_CUDA(launch_pdl(moe_gemm_simt_kernel<T, GU>, grid, block, (size_t)0, stream, (const T*)A, lda, (const T*)W, out, ldo, tiles, n_tiles, src_of, sel_w, top, N, K, scatter, w_out))
-    if (dtype == NIB_F32) { if (gate_up == 1) NIB_MG(float, 1); else if (gate_up == 2) NIB_MG(float, 2); else NIB_MG(float, 0); }
-    else { if (gate_up == 1) NIB_MG(__nv_bfloat16, 1); else if (gate_up == 2) NIB_MG(__nv_bfloat16, 2); else NIB_MG(__nv_bfloat16, 0); }
+    NIB_CUDA(launch_pdl(moe_gemm_simt_kernel<T, GU>, grid, block, (size_t)0, stream, (const T*)A, lda, (const T*)W, out, ldo, tiles, n_tiles, src_of, sel_w, top, N, K, scatter, w_out, constants))
+    if (dtype == NIB_F32) { if (gate_up == 1) NIB_MG(float, 1); else if (gate_up == 2) NIB_MG(float, 2); else if (gate_up == 3) NIB_MG(float, 3); else NIB_MG(float, 0); }
+    else { if (gate_up == 1) NIB_MG(__nv_bfloat16, 1); else if (gate_up == 2) NIB_MG(__nv_bfloat16, 2); else if (gate_up == 3) NIB_MG(__nv_bfloat16, 3); else NIB_MG(__nv_bfloat16, 0); }
 #undef NIB_MG
     NIB_LAUNCH_CHECK();
     return 0;

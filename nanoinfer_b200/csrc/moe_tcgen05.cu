@@ -8,6 +8,7 @@
 //             token, else by reductions in memory (the order of a token's choices, and with it the last bit of a sum of
 //             three or more, is not fixed; two addends onto zeros give the same sum in either order).
 //
+// Mode 3: like gate/up, with the gated form of constants (NibGlu) in place of silu(g) u.
 // Experts without a gate (mode 2): act[row] = relu(w u)^2 from one accumulator. With `w_out` the score multiplies the
 // down product's result (in 32-bit, in its epilogue) instead of the first product's accumulators.
 //
@@ -62,8 +63,9 @@ template <int TOK, int MODE>
 __global__ void __launch_bounds__(THREADS, 1)
 moe_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_a, void* __restrict__ out, int ldo,
               const int* __restrict__ tiles, const int* __restrict__ n_tiles, int max_tiles, const int* __restrict__ src_of,
-              const float* __restrict__ sel_w, int top, int n_out, int k_dim, int w_rows, int scatter, int splits, int kb_per_split, int w_out) {
-    constexpr bool GATE_UP = MODE == 1, FIRST = MODE != 0;     // FIRST: the product that reads the tokens' rows and writes activations
+              const float* __restrict__ sel_w, int top, int n_out, int k_dim, int w_rows, int scatter, int splits, int kb_per_split, int w_out,
+              const NibGlu glu) {
+    constexpr bool GATE_UP = MODE == 1 || MODE == 3, FIRST = MODE != 0;     // FIRST: the product that reads the tokens' rows and writes activations
     constexpr bool DUAL = GATE_UP;
     const bool use_w = FIRST != (w_out != 0);                  // whether this product is the one the score multiplies
     // Row tiles of 128: the operands change places, so the ROWS are the instruction's M side (the TMEM lanes) and the 128
@@ -225,7 +227,7 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__
                     for (int j = 0; j < 16; ++j) {
                         if (GATE_UP) {
                             const float g = __uint_as_float(rv[j]) * wg, up = __uint_as_float(ru[j]) * wg;
-                            x[j] = __fdividef(g, 1.0f + __expf(-g)) * up;      // the dense gated product's epilogue has the same forms
+                            x[j] = MODE == 3 ? nib_glu_fast(glu, g, up) : __fdividef(g, 1.0f + __expf(-g)) * up;      // the dense gated product's epilogue has the same forms
                         } else if (FIRST) {
                             const float u = fmaxf(__uint_as_float(rv[j]) * wg, 0.f);
                             x[j] = u * u;
@@ -310,7 +312,7 @@ moe_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__
                         const float wg = s_wgt[quad][c + j];
                         if (GATE_UP) {
                             const float g = v[j] * wg, up = u[j] * wg;
-                            ((__nv_bfloat16*)out)[o] = __float2bfloat16(__fdividef(g, 1.0f + __expf(-g)) * up);
+                            ((__nv_bfloat16*)out)[o] = __float2bfloat16(MODE == 3 ? nib_glu_fast(glu, g, up) : __fdividef(g, 1.0f + __expf(-g)) * up);
                         } else if (FIRST) {
                             const float r = fmaxf(v[j] * wg, 0.f);
                             ((__nv_bfloat16*)out)[o] = __float2bfloat16(r * r);
@@ -392,9 +394,9 @@ int sm_count() {
 template <int TOK, int MODE>
 int launch_moe_tc(const CUtensorMap& mw, const CUtensorMap& ma, void* out, int ldo, const int* tiles, const int* n_tiles, int max_tiles,
                   const int* src_of, const float* sel_w, int top, int N, int K, int w_rows, int scatter, int splits, int w_out,
-                  cudaStream_t stream) {
+                  const NibGlu& glu, cudaStream_t stream) {
     constexpr bool FIRST = MODE != 0;       // the first product, gated or not: its output cannot be split along K
-    using C = Cfg<TOK, MODE == 1>;
+    using C = Cfg<TOK, MODE == 1 || MODE == 3>;
     static bool configured = false;
     if (!configured) {
         NIB_CUDA(cudaFuncSetAttribute(moe_tc_kernel<TOK, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM));
@@ -408,7 +410,7 @@ int launch_moe_tc(const CUtensorMap& mw, const CUtensorMap& ma, void* out, int l
     const long long most = (long long)max_tiles * ceil_div(N, BLOCK_F) * splits;
     const int sms = sm_count();
     NIB_CUDA(launch_pdl(moe_tc_kernel<TOK, MODE>, dim3((unsigned)(most < sms ? most : sms)), dim3(THREADS), (size_t)C::SMEM, stream, mw, ma, out, ldo,
-                        tiles, n_tiles, max_tiles, src_of, sel_w, top, N, K, w_rows, scatter, splits, kb_per_split, w_out));
+                        tiles, n_tiles, max_tiles, src_of, sel_w, top, N, K, w_rows, scatter, splits, kb_per_split, w_out, glu));
     return 0;
 }
 
@@ -445,17 +447,20 @@ NIB_API int nib_moe_gather_rows(const void* src, int lds, void* dst, int ldd, co
 }
 
 // gate_up 1: A = the rows in the grouped order [a_rows, K], W [experts, 2N, K] (gate rows, then up rows), out bfloat16
-// [a_rows, N]; 2: the same with W [experts, N, K] (no gate) and relu(.)^2. 0: A [a_rows, K] in the grouped order, W [experts, N, K], out floats: [a_rows, N] in the grouped order, or
+// [a_rows, N]; 2: the same with W [experts, N, K] (no gate) and relu(.)^2; 3: like 1 with the gated form of the constants glu.
+// 0: A [a_rows, K] in the grouped order, W [experts, N, K], out floats: [a_rows, N] in the grouped order, or
 // with scatter added into the token's row of [tokens, N] (1: plainly, one choice per token; 2: by reductions in memory).
 // The table must have been made for row tiles of `tile_rows` (32 or 128).
 NIB_API int nib_moe_gemm_tc(int gate_up, const void* A, int lda, int a_rows, const void* W, int experts, void* out, int ldo, const int* tiles,
                             const int* n_tiles, int max_tiles, const int* src_of, const float* sel_w, int top, int N, int K, int scatter,
-                            int tile_rows, int w_out, cudaStream_t stream) {
+                            int tile_rows, int w_out, const NibGlu* glu, cudaStream_t stream) {
     NIB_REQUIRE(N > 0 && K > 0 && K % 8 == 0 && lda % 8 == 0 && top > 0 && a_rows >= 0 && experts > 0 && max_tiles >= 0 && scatter >= 0 && scatter <= 2
-                && (scatter != 1 || top == 1) && gate_up >= 0 && gate_up <= 2, "experts (tensor cores): bad sizes");
+                && (scatter != 1 || top == 1) && gate_up >= 0 && gate_up <= 3, "experts (tensor cores): bad sizes");
     NIB_REQUIRE(tile_rows == 32 || tile_rows == 128, "experts (tensor cores): row tiles of 32 or 128, not %d", tile_rows);
+    NIB_REQUIRE(gate_up != 3 || glu != nullptr, "experts (tensor cores): the gated form needs its constants");
+    const NibGlu constants = glu != nullptr ? *glu : NibGlu{};
     if (max_tiles == 0 || a_rows == 0) return 0;
-    const int w_rows = gate_up == 1 ? 2 * N : N;
+    const int w_rows = (gate_up == 1 || gate_up == 3) ? 2 * N : N;
     CUtensorMap mw, ma;
     {
         std::lock_guard<std::mutex> lock(g_expert_map_mutex);
@@ -480,10 +485,10 @@ NIB_API int nib_moe_gemm_tc(int gate_up, const void* A, int lda, int a_rows, con
         if (splits > k_blocks / 4) splits = k_blocks / 4;
         if (splits < 1) splits = 1;
     }
-#define NIB_MT(TOK, GU) launch_moe_tc<TOK, GU>(mw, ma, out, ldo, tiles, n_tiles, max_tiles, src_of, sel_w, top, N, K, w_rows, scatter, splits, w_out, stream)
+#define NIB_MT(TOK, GU) launch_moe_tc<TOK, GU>(mw, ma, out, ldo, tiles, n_tiles, max_tiles, src_of, sel_w, top, N, K, w_rows, scatter, splits, w_out, constants, stream)
     int rc;
-    if (tile_rows == 32) rc = gate_up == 1 ? NIB_MT(32, 1) : (gate_up == 2 ? NIB_MT(32, 2) : NIB_MT(32, 0));
-    else rc = gate_up == 1 ? NIB_MT(128, 1) : (gate_up == 2 ? NIB_MT(128, 2) : NIB_MT(128, 0));
+    if (tile_rows == 32) rc = gate_up == 1 ? NIB_MT(32, 1) : (gate_up == 2 ? NIB_MT(32, 2) : gate_up == 3 ? NIB_MT(32, 3) : NIB_MT(32, 0));
+    else rc = gate_up == 1 ? NIB_MT(128, 1) : (gate_up == 2 ? NIB_MT(128, 2) : gate_up == 3 ? NIB_MT(128, 3) : NIB_MT(128, 0));
 #undef NIB_MT
     if (rc) return rc;
     NIB_LAUNCH_CHECK();

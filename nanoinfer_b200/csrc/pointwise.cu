@@ -397,7 +397,9 @@ NIB_API int nib_depth_mix_norm_pair(float* hist, float* x, const float* coef, in
 
 // ---------------------------------------------------------------------------------- gate, norm in groups, skip
 // For a row o of n floats cut into `groups` equal parts (a warp per (token, part)):
-//     y = o (+ coef[c / (n / n_coef)] * skip)          a skip connection with one coefficient per head
+//     y = o / (max(|den|, floor) + den_eps)             with `floor`: den is the number behind the part's channels in o (the
+//                                                       parts of o then lie width + 1 apart), floor one number per (token, part)
+//     y = y (+ coef[c / (n / n_coef)] * skip)          a skip connection with one coefficient per head
 //     y = y * act(gate)                                 if gate_first
 //     y = y / sqrt(mean_part(y^2) + eps)                if norm
 //     y = y * gain[c % gain_len]                        gain_len = n (a gain per channel) or a part's size (shared)
@@ -414,14 +416,15 @@ __global__ void __launch_bounds__(128)
 gated_norm_kernel(const float* __restrict__ o, int ldo, const float* __restrict__ gate, int ldg, int gate_kind, int gate_first,
                   const float* __restrict__ gain, int gain_len, const float* __restrict__ skip, int lds,
                   const float* __restrict__ coef, int coef_span, int norm, float eps, float out_scale,
-                  T* __restrict__ out, int ld_out, int tokens, int groups, int width) {
+                  T* __restrict__ out, int ld_out, int tokens, int groups, int width, const float* __restrict__ floor_in, int ldf, float den_eps) {
     pdl_launch_dependents();
     pdl_wait();      // everything this kernel reads may come from the kernel before
     const long long w = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
     const int lane = threadIdx.x & 31;
     if (w >= (long long)tokens * groups) return;
-    const int t = (int)(w / groups), c0 = (int)(w % groups) * width;
-    const float* orow = o + (size_t)t * ldo;
+    const int t = (int)(w / groups), part_i = (int)(w % groups), c0 = part_i * width;
+    const float* orow = o + (size_t)t * ldo + (floor_in != nullptr ? part_i : 0);      // (a divisor behind every part)
+    const float den = floor_in != nullptr ? fmaxf(fabsf(orow[c0 + width]), floor_in[(size_t)t * ldf + part_i]) + den_eps : 1.0f;
     const float* grow = gate != nullptr ? gate + (size_t)t * ldg : nullptr;
     const float* srow = skip != nullptr ? skip + (size_t)t * lds : nullptr;
     const bool early = grow != nullptr && gate_kind != 0 && gate_first != 0;
@@ -431,7 +434,7 @@ gated_norm_kernel(const float* __restrict__ o, int ldo, const float* __restrict_
         float ss = 0.f;
         for (int j = lane; j < width; j += 32) {
             const int c = c0 + j;
-            float y = orow[c];
+            float y = floor_in != nullptr ? orow[c] / den : orow[c];
             if (srow != nullptr) y = fmaf(coef[c / coef_span], srow[c], y);
             if (early) y *= gate_act(grow[c], gate_kind);
             ss = fmaf(y, y, ss);
@@ -441,7 +444,7 @@ gated_norm_kernel(const float* __restrict__ o, int ldo, const float* __restrict_
     }
     for (int j = lane; j < width; j += 32) {
         const int c = c0 + j;
-        float y = orow[c];
+        float y = floor_in != nullptr ? orow[c] / den : orow[c];
         if (srow != nullptr) y = fmaf(coef[c / coef_span], srow[c], y);
         if (early) y *= gate_act(grow[c], gate_kind);
         y *= scale;
@@ -458,12 +461,13 @@ __global__ void __launch_bounds__(256)
 gated_norm_block_kernel(const float* __restrict__ o, int ldo, const float* __restrict__ gate, int ldg, int gate_kind, int gate_first,
                         const float* __restrict__ gain, int gain_len, const float* __restrict__ skip, int lds,
                         const float* __restrict__ coef, int coef_span, int norm, float eps, float out_scale,
-                        T* __restrict__ out, int ld_out, int tokens, int groups, int width) {
+                        T* __restrict__ out, int ld_out, int tokens, int groups, int width, const float* __restrict__ floor_in, int ldf, float den_eps) {
     pdl_launch_dependents();
     pdl_wait();      // everything this kernel reads may come from the kernel before
     __shared__ float part[8];
-    const int t = blockIdx.x / groups, c0 = (blockIdx.x % groups) * width;
-    const float* orow = o + (size_t)t * ldo;
+    const int t = blockIdx.x / groups, part_i = blockIdx.x % groups, c0 = part_i * width;
+    const float* orow = o + (size_t)t * ldo + (floor_in != nullptr ? part_i : 0);      // (a divisor behind every part)
+    const float den = floor_in != nullptr ? fmaxf(fabsf(orow[c0 + width]), floor_in[(size_t)t * ldf + part_i]) + den_eps : 1.0f;
     const float* grow = gate != nullptr ? gate + (size_t)t * ldg : nullptr;
     const float* srow = skip != nullptr ? skip + (size_t)t * lds : nullptr;
     const bool early = grow != nullptr && gate_kind != 0 && gate_first != 0;
@@ -473,7 +477,7 @@ gated_norm_block_kernel(const float* __restrict__ o, int ldo, const float* __res
         float ss = 0.f;
         for (int j = threadIdx.x; j < width; j += 256) {
             const int c = c0 + j;
-            float y = orow[c];
+            float y = floor_in != nullptr ? orow[c] / den : orow[c];
             if (srow != nullptr) y = fmaf(coef[c / coef_span], srow[c], y);
             if (early) y *= gate_act(grow[c], gate_kind);
             ss = fmaf(y, y, ss);
@@ -482,7 +486,7 @@ gated_norm_block_kernel(const float* __restrict__ o, int ldo, const float* __res
     }
     for (int j = threadIdx.x; j < width; j += 256) {
         const int c = c0 + j;
-        float y = orow[c];
+        float y = floor_in != nullptr ? orow[c] / den : orow[c];
         if (srow != nullptr) y = fmaf(coef[c / coef_span], srow[c], y);
         if (early) y *= gate_act(grow[c], gate_kind);
         y *= scale;
@@ -494,7 +498,7 @@ gated_norm_block_kernel(const float* __restrict__ o, int ldo, const float* __res
 
 NIB_API int nib_gated_norm(const float* o, int ldo, const float* gate, int ldg, int gate_kind, int gate_first, const float* gain,
                            int gain_len, const float* skip, int lds, const float* coef, int n_coef, int groups, int norm, float eps,
-                           float out_scale, void* out, int ld_out, int tokens, int n, int dtype, cudaStream_t stream) {
+                           float out_scale, void* out, int ld_out, int tokens, int n, int dtype, const float* floor_in, int ldf, float den_eps, cudaStream_t stream) {
     NIB_REQUIRE(tokens >= 0 && n > 0 && groups > 0 && n % groups == 0, "gated_norm: %d channels do not split into %d parts", n, groups);
     NIB_REQUIRE(gain == nullptr || (gain_len > 0 && n % gain_len == 0), "gated_norm: a gain of %d does not tile %d channels", gain_len, n);
     NIB_REQUIRE(skip == nullptr || (coef != nullptr && n_coef > 0 && n % n_coef == 0), "gated_norm: bad skip coefficients");
@@ -503,15 +507,15 @@ NIB_API int nib_gated_norm(const float* o, int ldo, const float* gate, int ldg, 
     const int width = n / groups, span = skip != nullptr ? n / n_coef : 1;
     if (width > 256) {
         const dim3 grid(tokens * groups);
-        if (dtype == NIB_F32) NIB_CUDA(launch_pdl(gated_norm_block_kernel<float>, grid, dim3(256), (size_t)(0), stream, o, ldo, gate, ldg, gate_kind, gate_first, gain, gain_len, skip, lds, coef, span, norm, eps, out_scale, (float*)out, ld_out, tokens, groups, width));
-        else if (dtype == NIB_BF16) NIB_CUDA(launch_pdl(gated_norm_block_kernel<__nv_bfloat16>, grid, dim3(256), (size_t)(0), stream, o, ldo, gate, ldg, gate_kind, gate_first, gain, gain_len, skip, lds, coef, span, norm, eps, out_scale, (__nv_bfloat16*)out, ld_out, tokens, groups, width));
+        if (dtype == NIB_F32) NIB_CUDA(launch_pdl(gated_norm_block_kernel<float>, grid, dim3(256), (size_t)(0), stream, o, ldo, gate, ldg, gate_kind, gate_first, gain, gain_len, skip, lds, coef, span, norm, eps, out_scale, (float*)out, ld_out, tokens, groups, width, floor_in, ldf, den_eps));
+        else if (dtype == NIB_BF16) NIB_CUDA(launch_pdl(gated_norm_block_kernel<__nv_bfloat16>, grid, dim3(256), (size_t)(0), stream, o, ldo, gate, ldg, gate_kind, gate_first, gain, gain_len, skip, lds, coef, span, norm, eps, out_scale, (__nv_bfloat16*)out, ld_out, tokens, groups, width, floor_in, ldf, den_eps));
         else NIB_REQUIRE(false, "gated_norm: unknown dtype %d", dtype);
         NIB_LAUNCH_CHECK();
         return 0;
     }
     const int blocks = ceil_div((long long)tokens * groups, 4);
-    if (dtype == NIB_F32) NIB_CUDA(launch_pdl(gated_norm_kernel<float>, dim3(blocks), dim3(128), (size_t)(0), stream, o, ldo, gate, ldg, gate_kind, gate_first, gain, gain_len, skip, lds, coef, span, norm, eps, out_scale, (float*)out, ld_out, tokens, groups, width));
-    else if (dtype == NIB_BF16) NIB_CUDA(launch_pdl(gated_norm_kernel<__nv_bfloat16>, dim3(blocks), dim3(128), (size_t)(0), stream, o, ldo, gate, ldg, gate_kind, gate_first, gain, gain_len, skip, lds, coef, span, norm, eps, out_scale, (__nv_bfloat16*)out, ld_out, tokens, groups, width));
+    if (dtype == NIB_F32) NIB_CUDA(launch_pdl(gated_norm_kernel<float>, dim3(blocks), dim3(128), (size_t)(0), stream, o, ldo, gate, ldg, gate_kind, gate_first, gain, gain_len, skip, lds, coef, span, norm, eps, out_scale, (float*)out, ld_out, tokens, groups, width, floor_in, ldf, den_eps));
+    else if (dtype == NIB_BF16) NIB_CUDA(launch_pdl(gated_norm_kernel<__nv_bfloat16>, dim3(blocks), dim3(128), (size_t)(0), stream, o, ldo, gate, ldg, gate_kind, gate_first, gain, gain_len, skip, lds, coef, span, norm, eps, out_scale, (__nv_bfloat16*)out, ld_out, tokens, groups, width, floor_in, ldf, den_eps));
     else NIB_REQUIRE(false, "gated_norm: unknown dtype %d", dtype);
     NIB_LAUNCH_CHECK();
     return 0;
@@ -686,4 +690,147 @@ NIB_API int nib_moe_identity(const void* h, int ldh, const int* sel_e, const flo
                             n_real, out, ldo, hidden));
     NIB_LAUNCH_CHECK();
     return 0;
+}
+
+// ---------------------------------------------------------------------------------- several streams around a sublayer
+// A token's residual is `n` streams of `width` floats. Between two sublayers, in one pass over a row (a block per row):
+//     z_t = sum_s mix[s, t] x_s + out[t] y       the streams after the sublayer whose result is y (all from the old ones);
+//     u = sum_s in[s] z_s                         what the next sublayer reads, then h = u / sqrt(mean(u^2) + eps) * gain.
+// Without `y` z = x (the first sublayer); x is read with strides of its own (all streams equal at the start: stream stride
+// 0); `dst` takes z as [row, stream, width] (may be x itself), `sum_out` takes sum_s z_s (may be x of one stream), `h_out` takes h in
+// T; with `clear` y is left zeroed. NS: streams known at compile time, 0: up to SM_MAX. V: elements a load.
+constexpr int SM_MAX = 16;
+
+template <typename T, int NS, int V>
+__global__ void __launch_bounds__(256)
+stream_mix_kernel(const float* x, long long x_row, long long x_stream, float* y, const float* __restrict__ mix, const float* __restrict__ out,
+                  float* dst, const float* __restrict__ in, const float* __restrict__ gain, float eps, T* __restrict__ h_out, float* sum_out,
+                  int width, int n_rt, int clear) {
+    constexpr int N = NS > 0 ? NS : SM_MAX;
+    constexpr int UNROLL = NS > 0 ? NS : 1;     // many streams: plain loops over a thread's own array
+    extern __shared__ __align__(16) float sm_row[];         // u of the row: every thread reads back what it wrote itself
+    __shared__ float s_mix[N * N], s_out[N], s_in[N], part[8];
+    const int n = NS > 0 ? NS : n_rt, tid = threadIdx.x;
+    pdl_launch_dependents();
+    for (int i = tid; i < n * n; i += blockDim.x) s_mix[i] = mix != nullptr ? mix[i] : 0.f;     // weights: no kernel writes them
+    for (int i = tid; i < n; i += blockDim.x) { s_out[i] = out != nullptr ? out[i] : 0.f; s_in[i] = in != nullptr ? in[i] : 0.f; }
+    __syncthreads();
+    pdl_wait();
+    const size_t row = blockIdx.x;
+    const float* xr = x + row * x_row;
+    float* yr = y != nullptr ? y + row * width : nullptr;
+    float ss = 0.f;
+    auto load = [](const float* p, float (&v)[V]) {
+        if constexpr (V == 4) { const float4 a = *reinterpret_cast<const float4*>(p); v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; }
+        else v[0] = *p;
+    };
+    auto store = [](float* p, const float (&v)[V]) {
+        if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+        else *p = v[0];
+    };
+    for (int c = tid * V; c < width; c += blockDim.x * V) {
+        float xv[N][V], yv[V];
+#pragma unroll UNROLL
+        for (int s = 0; s < N; ++s) {
+            if (s >= n) break;
+            load(xr + s * x_stream + c, xv[s]);
+        }
+        if (yr != nullptr) {
+            load(yr + c, yv);
+            if (clear) {
+                const float zero[V] = {};
+                store(yr + c, zero);
+            }
+        }
+        float u[V] = {}, total[V] = {};
+#pragma unroll UNROLL
+        for (int t = 0; t < N; ++t) {
+            if (t >= n) break;
+            float z[V];
+#pragma unroll
+            for (int e = 0; e < V; ++e) {
+                if (yr != nullptr) {
+                    float a = s_out[t] * yv[e];
+#pragma unroll UNROLL
+                    for (int s = 0; s < N; ++s) {
+                        if (s >= n) break;
+                        a = fmaf(s_mix[s * n + t], xv[s][e], a);
+                    }
+                    z[e] = a;
+                } else {
+                    z[e] = xv[t][e];
+                }
+                u[e] = fmaf(s_in[t], z[e], u[e]);
+                total[e] += z[e];
+            }
+            if (dst != nullptr) store(dst + (row * n + t) * width + c, z);
+        }
+        if (sum_out != nullptr) store(sum_out + row * width + c, total);
+        if (h_out != nullptr) {
+            store(sm_row + c, u);
+#pragma unroll
+            for (int e = 0; e < V; ++e) ss = fmaf(u[e], u[e], ss);
+        }
+    }
+    if (h_out == nullptr) return;
+    ss = warp_sum(ss);
+    if ((tid & 31) == 0) part[tid >> 5] = ss;
+    __syncthreads();
+    ss = 0.f;
+    for (int w = 0; w < (int)(blockDim.x >> 5); ++w) ss += part[w];        // the same order in every thread
+    const float scale = 1.0f / sqrtf(ss / (float)width + eps);
+    for (int c = tid * V; c < width; c += blockDim.x * V) {
+        float u[V], g[V];
+        load(sm_row + c, u);
+        load(gain + c, g);
+#pragma unroll
+        for (int e = 0; e < V; ++e) u[e] = u[e] * scale * g[e];
+        T* ho = h_out + row * width + c;
+        if constexpr (V == 4 && sizeof(T) == 2) {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(u[0], u[1]), hi = __floats2bfloat162_rn(u[2], u[3]);
+            uint2 pk;
+            pk.x = *reinterpret_cast<const unsigned*>(&lo);
+            pk.y = *reinterpret_cast<const unsigned*>(&hi);
+            *reinterpret_cast<uint2*>(ho) = pk;
+        } else {
+#pragma unroll
+            for (int e = 0; e < V; ++e) Elem<T>::store(ho + e, u[e]);
+        }
+    }
+}
+
+template <typename T, int NS, int V>
+static int launch_stream_mix(const float* x, long long x_row, long long x_stream, float* y, const float* mix, const float* out, float* dst,
+                             const float* in, const float* gain, float eps, void* h_out, float* sum_out, int rows, int width, int n, int clear,
+                             cudaStream_t stream) {
+    const size_t smem = h_out != nullptr ? (size_t)width * 4 : 0;
+    static size_t configured = 48 * 1024;
+    if (smem > configured) {
+        NIB_CUDA(cudaFuncSetAttribute(stream_mix_kernel<T, NS, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        configured = smem;
+    }
+    const int threads = rows <= 64 && width >= 1024 ? 256 : 128;
+    NIB_CUDA(launch_pdl(stream_mix_kernel<T, NS, V>, dim3(rows), dim3(threads), smem, stream, x, x_row, x_stream, y, mix, out, dst, in, gain, eps,
+                        (T*)h_out, sum_out, width, n, clear));
+    return 0;
+}
+
+NIB_API int nib_stream_mix(const float* x, long long x_row, long long x_stream, float* y, const float* mix, const float* out, float* dst,
+                           const float* in, const float* gain, float eps, void* h_out, float* sum_out, int rows, int width, int n, int clear,
+                           int dtype, cudaStream_t stream) {
+    NIB_REQUIRE(rows >= 0 && width > 0 && width <= 50 * 1024 && n >= 1 && n <= SM_MAX, "stream_mix: rows of up to %d floats, up to %d streams", 50 * 1024, SM_MAX);
+    NIB_REQUIRE(y == nullptr || (mix != nullptr && out != nullptr), "stream_mix: a result needs the matrix and the shares");
+    NIB_REQUIRE(h_out == nullptr || (in != nullptr && gain != nullptr), "stream_mix: a normed sum needs its factors and its gain");
+    NIB_REQUIRE(dtype == NIB_F32 || dtype == NIB_BF16, "stream_mix: unknown dtype %d", dtype);
+    if (rows == 0) return 0;
+    const uintptr_t all = (uintptr_t)x | (uintptr_t)y | (uintptr_t)dst | (uintptr_t)gain | (uintptr_t)h_out | (uintptr_t)sum_out;
+    const bool vec = width % 4 == 0 && (all & 15) == 0 && x_row % 4 == 0 && x_stream % 4 == 0;
+#define NIB_SM3(T, NS, V) return launch_stream_mix<T, NS, V>(x, x_row, x_stream, y, mix, out, dst, in, gain, eps, h_out, sum_out, rows, width, n, clear, stream)
+#define NIB_SM2(T, NS) do { if (vec) NIB_SM3(T, NS, 4); else NIB_SM3(T, NS, 1); } while (0)
+#define NIB_SM(T) do { switch (n) { case 1: NIB_SM2(T, 1); case 2: NIB_SM2(T, 2); case 3: NIB_SM2(T, 3); case 4: NIB_SM2(T, 4); default: NIB_SM3(T, 0, 1); } } while (0)
+    if (dtype == NIB_F32) NIB_SM(float);
+    NIB_SM(__nv_bfloat16);
+#undef NIB_SM
+#undef NIB_SM2
+#undef NIB_SM3
 }

@@ -9,6 +9,9 @@ outputs, the branches read the stream as it is.
 ``sandwich_norm``: ``x += norm_b(mixer(norm_a(x))); x += norm_d(feed_forward(norm_c(x)))``: a norm before and after each
 sublayer.
 
+``multi_stream``: several residual streams; every sublayer reads a norm of a sum of them and its result goes back to all
+(``parts/streams.py``).
+
 ``pre_norm``: ``x += mixer(norm(x)); x += feed_forward(norm(x))`` with a norm of its own before each
 (cpp/src/model.cpp:364-400, nanoinfer/layers.py:328-339). The residual stream ``x`` is 32-bit and
 both sums are made in 32-bit inside the projections that produce the addends.
@@ -21,6 +24,7 @@ import torch
 
 from ..registry import register_arrangement
 from .base import PENDING_STREAM_OP, LayerCache, StepContext, normed_input
+from .streams import StreamSet
 
 
 class PreNormBlock:
@@ -170,7 +174,34 @@ class SandwichNormBlock:
             last.add_normed(y32, x32, 1.0, None, clear=False)
 
 
+class MultiStreamBlock:
+    """Two sublayers around several residual streams (``parts/streams.py``). parts: ``mixer_norm``, ``mixer``,
+    ``mixer_streams`` (the mixer's factors) and optionally ``ffn_norm``, ``ffn``, ``ffn_streams`` (all three or none). The last
+    sublayer's update is left pending, so that blocks of this kind that run one after another (in any order, also the same
+    block again) make one pass over the streams per sublayer."""
+
+    part_names = ("mixer_norm", "mixer", "mixer_streams", "ffn_norm", "ffn", "ffn_streams")
+    resolves_pending = True     # it looks for work left pending on the stream itself
+
+    def __init__(self, parts: Dict[str, object]):
+        self.mixer_norm, self.mixer, self.mixer_streams = parts["mixer_norm"], parts["mixer"], parts["mixer_streams"]
+        self.ffn_norm, self.ffn, self.ffn_streams = parts.get("ffn_norm"), parts.get("ffn"), parts.get("ffn_streams")
+        if len({self.ffn_norm is None, self.ffn is None, self.ffn_streams is None}) != 1:
+            raise ValueError("a feed-forward comes with its norm and its factors on the streams")
+        if self.ffn is not None and self.ffn_streams.streams != self.mixer_streams.streams:
+            raise ValueError("both sublayers work on the same streams")
+        self.part_names = tuple(n for n in MultiStreamBlock.part_names if parts.get(n) is not None)
+
+    def forward(self, x32: torch.Tensor, ctx: StepContext, cache: LayerCache) -> None:
+        streams = StreamSet.of(self.mixer.rt, x32, ctx, self.mixer_streams.streams)
+        self.mixer.forward(streams.enter(self.mixer_streams, self.mixer_norm), streams.y32, ctx, cache)
+        if self.ffn is not None:
+            self.ffn.forward(streams.enter(self.ffn_streams, self.ffn_norm), streams.y32, ctx)
+        ctx.scratch[PENDING_STREAM_OP] = streams
+
+
 register_arrangement("pre_norm", PreNormBlock)
+register_arrangement("multi_stream", MultiStreamBlock)
 register_arrangement("sandwich_norm", SandwichNormBlock)
 register_arrangement("output_norm", OutputNormBlock)
 register_arrangement("parallel", ParallelBlock)

@@ -1,4 +1,6 @@
-"""SwiGLU feed-forward: ``down( silu(gate(h)) * up(h) )``, no biases, added to the residual stream.
+"""SwiGLU feed-forward: ``down( silu(gate(h)) * up(h) )``, no biases, added to the residual stream. With constants
+(``glu`` = (alpha, limit, shift)): ``g = min(gate(h), limit)``, ``u = clamp(up(h), -limit, limit)``,
+``down( g sigmoid(alpha g) (u + shift) )``.
 
 ``silu(g) = g / (1 + exp(-g))`` in 32-bit. Reference: cpp/src/model.cpp:217-223,
 cpp/src/ops.cpp:86-100, nanoinfer/layers.py:243-258.
@@ -15,7 +17,7 @@ from .spec import PartSpec, TensorSpec
 
 
 class SwiGLU(FeedForward):
-    """params: ``hidden``, ``intermediate``. tensors: ``gate_w up_w [intermediate, hidden]``,
+    """params: ``hidden``, ``intermediate``, optionally ``glu`` (alpha, limit, shift). tensors: ``gate_w up_w [intermediate, hidden]``,
     ``down_w [hidden, intermediate]``."""
 
     graph_safe = True   # launches do not depend on which requests are in the batch
@@ -23,9 +25,12 @@ class SwiGLU(FeedForward):
 
     @staticmethod
     def spec(prefix: str, hidden: int, intermediate: int,
-             names=("gate_proj.weight", "up_proj.weight", "down_proj.weight")) -> PartSpec:
+             names=("gate_proj.weight", "up_proj.weight", "down_proj.weight"), glu=None) -> PartSpec:
         """``names``: what the gate, up and down matrices are called behind ``prefix``."""
-        return PartSpec("swiglu", {"hidden": hidden, "intermediate": intermediate}, {
+        params = {"hidden": hidden, "intermediate": intermediate}
+        if glu is not None:
+            params["glu"] = tuple(float(x) for x in glu)
+        return PartSpec("swiglu", params, {
             "gate_w": TensorSpec(f"{prefix}.{names[0]}", (intermediate, hidden)),
             "up_w": TensorSpec(f"{prefix}.{names[1]}", (intermediate, hidden)),
             "down_w": TensorSpec(f"{prefix}.{names[2]}", (hidden, intermediate)),
@@ -35,13 +40,17 @@ class SwiGLU(FeedForward):
         super().__init__(spec, tensors, rt)
         self.hidden = int(spec.params["hidden"])
         self.intermediate = int(spec.params["intermediate"])
+        self.glu = spec.params.get("glu")
         # One fused operand: rows [gate | up].
         self.w_gate_up = rt.matrix(torch.cat([tensors["gate_w"], tensors["up_w"]], dim=0))
         self.w_down = rt.matrix(tensors["down_w"])
 
     def forward(self, h: torch.Tensor, residual32: torch.Tensor, ctx: StepContext) -> None:
         act = torch.empty((h.shape[0], self.intermediate), dtype=self.rt.dtype, device=h.device)
-        self.ops.linear_swiglu(h, self.w_gate_up, act)
+        if self.glu is None:
+            self.ops.linear_swiglu(h, self.w_gate_up, act)
+        else:
+            self.ops.linear_swiglu(h, self.w_gate_up, act, self.glu)
         self.ops.linear(act, self.w_down, None, residual32, "add")
 
 
@@ -94,6 +103,7 @@ class RoutedExperts(FeedForward):
       scores without it;
     * ``renormalize``: the chosen scores are divided by their sum (+ 1e-20);
     * ``weight_on`` "output": the weight multiplies the expert's result, ``sum_e score_e * expert_e(h)``;
+    * ``glu`` (alpha, limit, shift): the gated form of ``SwiGLU`` with those constants in place of ``silu(gate) * up``;
     * ``gated`` False: an expert is ``W_down relu(W_up x)^2`` (tensors ``e<i>_up``, ``e<i>_down``);
     * ``identity`` n: the router has n more outputs behind the experts' that stand for no weights: such a choice adds
       ``weight * h``;
@@ -113,7 +123,8 @@ class RoutedExperts(FeedForward):
 
     @staticmethod
     def spec(prefix: str, hidden: int, ff: int, experts: int, top: int, *, score: str = "sigmoid", correction: bool = False,
-             renormalize: bool = False, weight_on: str = "input", gated: bool = True, identity: int = 0, shared: int = 0) -> PartSpec:
+             renormalize: bool = False, weight_on: str = "input", gated: bool = True, identity: int = 0, shared: int = 0,
+             glu=None) -> PartSpec:
         t = {"router": TensorSpec(f"{prefix}.router", (experts + identity, hidden))}
         if correction:
             t["correction"] = TensorSpec(f"{prefix}.correction", (experts + identity,), "bias")
@@ -128,8 +139,10 @@ class RoutedExperts(FeedForward):
             t["shared_sg"] = TensorSpec(f"{prefix}.shared.sg", (1, hidden))
         params = {"hidden": hidden, "ff": ff, "experts": experts, "top": top}
         options = {"score": score, "correction": bool(correction), "renormalize": bool(renormalize), "weight_on": weight_on,
-                   "gated": bool(gated), "identity": int(identity), "shared": int(shared)}
-        defaults = {"score": "sigmoid", "correction": False, "renormalize": False, "weight_on": "input", "gated": True, "identity": 0, "shared": 0}
+                   "gated": bool(gated), "identity": int(identity), "shared": int(shared),
+                   "glu": None if glu is None else tuple(float(x) for x in glu)}
+        defaults = {"score": "sigmoid", "correction": False, "renormalize": False, "weight_on": "input", "gated": True, "identity": 0, "shared": 0,
+                    "glu": None}
         params.update({k: v for k, v in options.items() if v != defaults[k]})
         return PartSpec("routed_experts", params, t)
 
@@ -141,6 +154,9 @@ class RoutedExperts(FeedForward):
         self.score, self.renormalize = str(p.get("score", "sigmoid")), bool(p.get("renormalize", False))
         self.weight_on, self.gated = str(p.get("weight_on", "input")), bool(p.get("gated", True))
         self.identity, self.shared = int(p.get("identity", 0)), int(p.get("shared", 0))
+        self.glu = p.get("glu")
+        if self.glu is not None and not self.gated:
+            raise ValueError("the constants of a gated form belong to experts with a gate")
         self.outputs = self.experts + self.identity         # what the router chooses among
         if not (1 <= self.top <= self.outputs):
             raise ValueError(f"a token uses {self.top} of {self.outputs} router outputs")
@@ -169,7 +185,7 @@ class RoutedExperts(FeedForward):
         self.w_gate_up = rt.matrix(torch.stack(ups))
         self.w_down = rt.matrix(torch.stack(downs))
         self.plain = self.score == "sigmoid" and not self.renormalize and self.correction is None and self.weight_on == "input" \
-            and self.gated and not self.identity and not self.shared
+            and self.gated and not self.identity and not self.shared and self.glu is None
 
     def forward(self, h, residual32: torch.Tensor, ctx: StepContext) -> None:
         h = as_tensor(h)
@@ -199,8 +215,9 @@ class RoutedExperts(FeedForward):
             z32 = torch.empty((m, self.outputs + extra), dtype=torch.float32, device=dev)
             self.ops.linear(h, self.w_router, None, z32, "f32")
             self.ops.moe_route(z32[:, :self.outputs], self.top, chosen, weight, **options)
+        constants = {} if self.glu is None else {"glu": self.glu}
         self.ops.moe_experts(h, chosen, weight, self.w_gate_up, self.w_down, residual32, plan=plan, gated=self.gated,
-                             weight_on=self.weight_on, outputs=self.outputs + always)
+                             weight_on=self.weight_on, outputs=self.outputs + always, **constants)
         if self.identity:
             self.ops.moe_identity(h, residual32, chosen, weight, self.experts + always)
 

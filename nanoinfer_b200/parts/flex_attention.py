@@ -14,7 +14,8 @@ With ``q = W_q h + b_q`` (likewise k, v), in this order:
   ``(1 - lambda) v + lambda v_first`` with a learned number ``lambda`` each; the blend is what is cached;
 * ``rot`` = (dims, base): the first ``dims`` elements of every q and k head are turned by ``position * base^(-2i/dims)``,
   element i paired with i + dims/2 (``rot_layout`` "half") or 2i with 2i + 1 ("interleaved"); with ``rot_factor`` f
-  every frequency is divided by f (linear position scaling); the angle is formed in 32-bit;
+  every frequency is divided by f (linear position scaling), with ``rot_scaling`` the frequencies are rescaled as
+  ``parts/position.py``: ``scaled_frequencies`` says; the angle is formed in 32-bit;
 * ``unit_norm_after_rot``: every head of q and k is divided by its root mean square AFTER the rotation, no gain;
 * ``values_from_keys``: there is no value projection; a value head is the key head as projected, before norm and
   rotation (``vdim`` = ``dim``);
@@ -36,11 +37,18 @@ import torch
 
 from ..registry import register_part
 from .base import CacheNeed, LayerCache, Mixer, PagedTensor, Runtime, StateNeed, StepContext, as_tensor
+from .position import scaled_frequencies
 from .spec import PartSpec, TensorSpec
 
 
-def rotary_frequencies(dims: int, base: float, factor: float = 1.0) -> torch.Tensor:
-    """``base^(-2i/dims) / factor`` for the ``dims/2`` pairs, computed in 64-bit and rounded to 32-bit once."""
+def rotary_frequencies(dims: int, base: float, factor: float = 1.0, scaling=None) -> torch.Tensor:
+    """``base^(-2i/dims) / factor`` for the ``dims/2`` pairs (or those frequencies rescaled by ``scaling``), computed in 64-bit
+    and rounded to 32-bit once."""
+    if scaling:
+        f, magnitude = scaled_frequencies(dims, base, scaling)
+        if magnitude != 1.0:
+            raise ValueError("a scaling of the frequencies that also scales cos and sin is not an option of this mixer")
+        return (f / float(factor)).to(torch.float32)
     i = torch.arange(dims // 2, dtype=torch.float64)
     return (torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / float(dims)) / float(factor)).to(torch.float32)
 
@@ -48,7 +56,7 @@ def rotary_frequencies(dims: int, base: float, factor: float = 1.0) -> torch.Ten
 class FlexAttention(Mixer):
     """params: ``hidden heads kv_heads dim vdim scale eps`` and the options ``bias`` (q, k, v), ``out_bias``, ``conv``
     (taps), ``qk_norm``, ``rot`` ((dims, base) or None), ``softcap``, ``slope_span``, ``window``, ``chunk``,
-    ``out_gate``, ``out_scale``, ``rot_layout``, ``rot_factor``, ``unit_norm_after_rot``, ``values_from_keys``, ``sink``,
+    ``out_gate``, ``out_scale``, ``rot_layout``, ``rot_factor``, ``rot_scaling``, ``unit_norm_after_rot``, ``values_from_keys``, ``sink``,
     ``v_mix`` (None, "first" or "blend"). tensors: ``q k o``, ``v`` unless the values are the keys, and, by option,
     ``q_b k_b v_b o_b q_conv k_conv v_conv q_norm k_norm g sink vmix``."""
 
@@ -59,7 +67,7 @@ class FlexAttention(Mixer):
     def spec(prefix: str, hidden: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, eps: float, *,
              bias: bool = False, out_bias: bool = False, conv: int = 0, qk_norm: bool = False, rot=None,
              softcap: float = 0.0, slope_span: float = 0.0, window: int = 0, chunk: int = 0, out_gate: bool = False,
-             out_scale: float = 1.0, rot_layout: str = "half", rot_factor: float = 1.0, unit_norm_after_rot: bool = False,
+             out_scale: float = 1.0, rot_layout: str = "half", rot_factor: float = 1.0, rot_scaling=None, unit_norm_after_rot: bool = False,
              values_from_keys: bool = False, sink: bool = False, v_mix=None) -> PartSpec:
         """``qk_norm``: False, True (per head, a gain of the head's size) or "whole"."""
         nq, nk, nv = heads * dim, kv_heads * dim, kv_heads * vdim
@@ -92,7 +100,7 @@ class FlexAttention(Mixer):
                   "slope_span": float(slope_span), "window": int(window), "chunk": int(chunk), "out_gate": out_gate,
                   "out_scale": float(out_scale), "rot_layout": str(rot_layout), "rot_factor": float(rot_factor),
                   "unit_norm_after_rot": bool(unit_norm_after_rot), "values_from_keys": bool(values_from_keys),
-                  "sink": bool(sink), "v_mix": v_mix}
+                  "sink": bool(sink), "v_mix": v_mix, "rot_scaling": dict(rot_scaling) if rot_scaling else None}
         return PartSpec("flex_attention", params, t)
 
     def __init__(self, spec: PartSpec, tensors: Dict[str, torch.Tensor], rt: Runtime):
@@ -140,7 +148,8 @@ class FlexAttention(Mixer):
         self.rot_dims = 0 if rot is None else int(rot[0])
         if self.rot_dims % 2 or self.rot_dims > self.dim:
             raise ValueError(f"rotated width {self.rot_dims} must be even and at most the head size {self.dim}")
-        self.freq = rotary_frequencies(self.rot_dims, float(rot[1]), float(p.get("rot_factor", 1.0))).to(rt.device) if self.rot_dims else None
+        self.freq = rotary_frequencies(self.rot_dims, float(rot[1]), float(p.get("rot_factor", 1.0)),
+                                       p.get("rot_scaling")).to(rt.device) if self.rot_dims else None
         span = float(p.get("slope_span", 0.0))
         self.slopes = None
         if span:

@@ -17,6 +17,12 @@ differ in where q, k, v and the decay come from and in what happens to o:
   last inputs are kept in the state); ``dt = softplus(dt + dt_bias)``; per head the decay is the scalar
   ``exp(-exp(A_log) dt)``, ``k = B`` and ``q = C`` of the head's group, ``v = dt x``; ``y = o + D x``, times ``silu(z)``,
   RMS-normed in ``norm_groups`` equal parts, times a gain, then ``W_o``.
+* ``StabilizedMatrixMemory``: ``q = W_q h / sqrt(dim)``, ``k = W_k h``, ``v = W_v h``; per head a log input gate
+  ``i = cap tanh((W_i h + b_i) / cap)`` and a log forget gate ``f = log sigmoid(cap tanh((W_f h + b_f) / cap))``; with a running
+  maximum ``m_t = max(f + m_(t-1), i)`` (zero at a request's start) the decay is the scalar ``exp(f + m_(t-1) - m_t)`` and
+  ``v`` carries the factor ``exp(i - m_t)``. The sum n of the keys under the same decays and factors is one more value channel
+  (of ones); ``o`` is divided by ``max(|n . q|, exp(-m_t)) + 1e-6``, then by its root mean square per head, times a gain of all
+  heads' size, times ``sigmoid(W_g h)``, then ``W_o``.
 
 Everything that enters the walk is 32-bit: the projections leave the matrix kernels as floats. Each adds
 ``out_scale`` times its result to the residual stream.
@@ -211,6 +217,63 @@ class Mamba2Mixer(Mixer):
         ops.linear(gated, self.w_o, None, residual32, "add")
 
 
+class StabilizedMatrixMemory(Mixer):
+    """params: ``hidden heads dim vdim gate_cap eps out_scale``. tensors: ``q k [heads*dim, hidden]``, ``v g [heads*vdim, hidden]``,
+    ``i f [heads, hidden]``, ``i_b f_b [heads]``, ``norm [heads*vdim]``, ``o [hidden, heads*vdim]``."""
+
+    graph_safe = True   # launches do not depend on which requests are in the batch
+    DEN_EPS = 1e-6
+
+    @staticmethod
+    def spec(prefix: str, hidden: int, heads: int, dim: int, vdim: int, gate_cap: float, eps: float, out_scale: float = 1.0) -> PartSpec:
+        nk, nv = heads * dim, heads * vdim
+        t = {"q": TensorSpec(f"{prefix}.q", (nk, hidden)), "k": TensorSpec(f"{prefix}.k", (nk, hidden)),
+             "v": TensorSpec(f"{prefix}.v", (nv, hidden)), "g": TensorSpec(f"{prefix}.g", (nv, hidden)),
+             "i": TensorSpec(f"{prefix}.i", (heads, hidden)), "i_b": TensorSpec(f"{prefix}.i.b", (heads,), "bias"),
+             "f": TensorSpec(f"{prefix}.f", (heads, hidden)), "f_b": TensorSpec(f"{prefix}.f.b", (heads,), "bias"),
+             "norm": TensorSpec(f"{prefix}.norm", (nv,), "gain"), "o": TensorSpec(f"{prefix}.o", (hidden, nv))}
+        return PartSpec("matrix_memory", {"hidden": hidden, "heads": heads, "dim": dim, "vdim": vdim, "gate_cap": float(gate_cap),
+                                          "eps": float(eps), "out_scale": float(out_scale)}, t)
+
+    def __init__(self, spec: PartSpec, tensors: Dict[str, torch.Tensor], rt: Runtime):
+        super().__init__(spec, tensors, rt)
+        p = spec.params
+        hidden, self.heads, self.dim, self.vdim = int(p["hidden"]), int(p["heads"]), int(p["dim"]), int(p["vdim"])
+        self.cap, self.eps, self.out_scale = float(p["gate_cap"]), float(p["eps"]), float(p.get("out_scale", 1.0))
+        self.nk, self.nv = self.heads * self.dim, self.heads * self.vdim
+        # One product for everything that reads h: rows [q | k | v | g | i | f | zeros up to a multiple of four].
+        n = 2 * self.nk + 2 * self.nv + 2 * self.heads
+        self.width = -(-n // 4) * 4
+        rows = [tensors[x] for x in ("q", "k", "v", "g", "i", "f")] + [torch.zeros((self.width - n, hidden), dtype=tensors["i"].dtype)]
+        self.w_in = rt.matrix(torch.cat(rows, dim=0))
+        self.b_i, self.b_f = rt.vector32(tensors["i_b"]), rt.vector32(tensors["f_b"])
+        self.gain = rt.vector32(tensors["norm"])
+        self.w_o = rt.matrix(tensors["o"])
+        # the state's row: [m of every head, filled up to four | S and n as [head, value channel (n last), key channel]]
+        self.s_off = -(-self.heads // 4) * 4
+
+    def state_need(self) -> StateNeed:
+        return StateNeed((self.s_off + self.heads * (self.vdim + 1) * self.dim,), torch.float32)
+
+    def forward(self, h: torch.Tensor, residual32: torch.Tensor, ctx: StepContext, cache: LayerCache) -> None:
+        h = as_tensor(h)
+        m, dev, ops, nk, nv, heads = h.shape[0], h.device, self.ops, self.nk, self.nv, self.heads
+        p32 = torch.empty((m, self.width), dtype=torch.float32, device=dev)
+        ops.linear(h, self.w_in, None, p32, "f32")
+        gates = 2 * nk + 2 * nv
+        decay, write, floor = torch.empty((3, m, heads), dtype=torch.float32, device=dev).unbind(0)
+        ops.memory_gates(p32[:, gates:gates + heads], p32[:, gates + heads:gates + 2 * heads], self.b_i, self.b_f, self.cap, cache.state, 0, ctx,
+                         decay, write, floor)
+        o32 = torch.empty((m, heads * (self.vdim + 1)), dtype=torch.float32, device=dev)
+        ops.linear_state_scan(p32[:, :nk], p32[:, nk:2 * nk], p32[:, 2 * nk:2 * nk + nv], decay, cache.state, self.s_off, ctx, o32, heads, heads,
+                              self.dim, self.vdim, q_scale=self.dim ** -0.5, v_scale32=write, ones=True)
+        gated = torch.empty((m, nv), dtype=self.rt.dtype, device=dev)
+        ops.gated_norm(o32, gated, groups=heads, eps=self.eps, gain32=self.gain, gate32=p32[:, 2 * nk + nv:gates], gate_kind="sigmoid",
+                       out_scale=self.out_scale, floor32=floor, den_eps=self.DEN_EPS)
+        ops.linear(gated, self.w_o, None, residual32, "add")
+
+
 register_part("gated_linear_attention", GatedLinearAttention)
+register_part("matrix_memory", StabilizedMatrixMemory)
 register_part("time_mix", ShiftedTimeMix)
 register_part("mamba2", Mamba2Mixer)

@@ -66,7 +66,10 @@ register_part("no_position", NoPositionEncoding)
 def scaled_frequencies(dims: int, base: float, scaling=None):
     """Frequencies of the ``dims/2`` rotated pairs, ``f_i = base^(-2i/dims)``, optionally rescaled the YaRN way, and
     the factor on cos and sin. ``scaling`` = {factor} alone: every frequency is divided by ``factor`` (linear scaling of
-    the positions), cos and sin as they are. ``scaling`` = {factor, original, fast, slow}: a pair that turns more than ``fast``
+    the positions), cos and sin as they are. ``scaling`` = {factor, original, low, high}: by the wavelength ``l = 2 pi / f``:
+    a pair with ``l < original / high`` keeps its frequency, one with ``l > original / low`` has it divided by ``factor``, and
+    between the two, with ``s = (original / l - low) / (high - low)``, it is ``(1 - s) f / factor + s f``; cos and sin as they
+    are. ``scaling`` = {factor, original, fast, slow}: a pair that turns more than ``fast``
     times within ``original`` positions keeps its frequency, one that turns fewer than ``slow`` times has it divided
     by ``factor``, linearly blended in between over the pair index: with
     ``turn_dim(t) = dims * ln(original / (2 pi t)) / (2 ln base)``, ``lo = max(floor(turn_dim(fast)), 0)``,
@@ -81,6 +84,12 @@ def scaled_frequencies(dims: int, base: float, scaling=None):
     if "original" not in scaling:
         return f / float(scaling["factor"]), 1.0
     factor, original = float(scaling["factor"]), float(scaling["original"])
+    if "low" in scaling:
+        low, high = float(scaling["low"]), float(scaling["high"])
+        wavelength = 2.0 * math.pi / f
+        share = (original / wavelength - low) / (high - low) if high != low else torch.zeros_like(f)
+        blended = (1.0 - share) * f / factor + share * f
+        return torch.where(wavelength > original / low, f / factor, torch.where(wavelength < original / high, f, blended)), 1.0
 
     def turn_dim(turns: float) -> float:
         return dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(float(base)))

@@ -2,7 +2,8 @@
 configuration and a seed.
 
 Distributions: N(0, 0.02) for matrices, embeddings and biases, 1 + N(0, 0.1) for norm gains, N(0, 1) for "unit"
-tensors (logits of decays, coefficients of an activation), (1 + N(0, 0.3)) / n for the n weights of an average ("mix").
+tensors (logits of decays, coefficients of an activation), (1 + N(0, 0.3)) / n for the n weights of an average ("mix"), the identity plus
+N(0, 0.1) for a square matrix that mixes streams ("near_identity").
 Each tensor has a generator of its own, seeded from (seed, tensor name), so a tensor's values do
 not depend on which other tensors exist or in which order they are made. The reference has no
 such mode in its C++ engine; its oracle tests build ``Model(cfg)`` with framework-default
@@ -35,6 +36,8 @@ def random_tensor(ts: TensorSpec, seed: int, dtype: torch.dtype) -> torch.Tensor
         x = 1.0 + 0.1 * x
     elif ts.init == "mix":      # weights of an average: each near 1/n
         x = (1.0 + 0.3 * x) / max(1, x.numel())
+    elif ts.init == "near_identity":
+        x = torch.eye(ts.shape[0]) + 0.1 * x
     elif ts.init == "mix01":    # blend factors between two inputs: uniform in 0..1
         x = torch.rand(ts.shape, generator=g, dtype=torch.float32)
     elif ts.init in _STD:

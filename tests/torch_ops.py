@@ -34,12 +34,21 @@ class TorchOps:
         else:
             raise ValueError(mode)
 
-    def linear_swiglu(self, a, w_gate_up, out):
+    @staticmethod
+    def _glu(g, u, constants):
+        """g sigmoid(alpha g) (u + shift) with g cut off above and u on both sides."""
+        if constants is None:
+            return g / (1.0 + torch.exp(-g)) * u
+        alpha, limit, shift = constants
+        g, u = torch.clamp(g, max=limit), torch.clamp(u, -limit, limit)
+        return g / (1.0 + torch.exp(-alpha * g)) * (u + shift)
+
+    def linear_swiglu(self, a, w_gate_up, out, glu=None):
         a = as_tensor(a)
         inter = w_gate_up.shape[0] // 2
         g = a.double() @ w_gate_up[:inter].double().t()
         u = a.double() @ w_gate_up[inter:].double().t()
-        out.copy_((g / (1.0 + torch.exp(-g)) * u).to(out.dtype))
+        out.copy_(self._glu(g, u, glu).to(out.dtype))
 
     def qkv_project(self, a, w_qkv, bias32, qkv, heads, kv_heads, head_dim, positions, req_index, rotary,
                     block_table, page_size, k_pages, v_pages, writes):
@@ -210,9 +219,13 @@ class TorchOps:
 
     # ---- gate, norm in groups, skip (pointwise.cu) ---------------------------------------------------
     def gated_norm(self, o32, out, groups=0, eps=0.0, gain32=None, gate32=None, gate_kind="none", gate_first=False,
-                   skip32=None, skip_coef32=None, out_scale=1.0):
-        m, n = o32.shape
+                   skip32=None, skip_coef32=None, out_scale=1.0, floor32=None, den_eps=0.0):
+        m, n = out.shape
         y = o32.double()
+        if floor32 is not None:
+            y = y.view(m, groups, n // groups + 1)
+            den = torch.maximum(y[..., -1:].abs(), floor32.double()[..., None]) + den_eps
+            y = (y[..., :-1] / den).reshape(m, n)
         if skip32 is not None:
             y = y + skip32.double() * skip_coef32.double().repeat_interleave(n // skip_coef32.numel())
         act = {"sigmoid": torch.sigmoid, "silu": lambda z: z * torch.sigmoid(z)}.get(gate_kind)
@@ -287,7 +300,10 @@ class TorchOps:
         decay_out.copy_(torch.exp(-torch.exp(a_log32.double()) * dt_out.double()).to(torch.float32))
 
     def linear_state_scan(self, q32, k32, v32, w32, state, state_off, ctx, o32, heads, kq_heads, dk, dv, q_scale=1.0,
-                          bonus32=None, v_scale32=None, seg_len=None):
+                          bonus32=None, v_scale32=None, seg_len=None, ones=False):
+        if ones:
+            v32 = torch.cat([v32.reshape(-1, heads, dv), torch.ones(v32.shape[0], heads, 1)], -1).reshape(v32.shape[0], -1)
+            dv += 1
         start = 0
         rep = heads // kq_heads
         per_channel = w32.shape[1] == heads * dk
@@ -309,6 +325,41 @@ class TorchOps:
                     s = w[:, :, None] * s + kv
                     o = torch.einsum("hkv,hk->hv", s, q)
                 o32[t] = o.reshape(-1).to(torch.float32)
+            flat.copy_(s.transpose(1, 2).reshape(-1).to(torch.float32))
+            start += q_len
+
+    def memory_gates(self, zi32, zf32, bi32, bf32, cap, state, state_off, ctx, decay32, write32, floor32):
+        i = cap * torch.tanh((zi32.double() + bi32.double()) / cap)
+        f = torch.nn.functional.logsigmoid(cap * torch.tanh((zf32.double() + bf32.double()) / cap))
+        start, heads = 0, zi32.shape[1]
+        for q_len, slot in zip(ctx.host.q_lens, ctx.host.slots):
+            m = state[slot, state_off:state_off + heads].double()
+            for t in range(start, start + q_len):
+                new = torch.maximum(f[t] + m, i[t]).to(torch.float32).double()
+                decay32[t], write32[t], floor32[t] = torch.exp(f[t] + m - new), torch.exp(i[t] - new), torch.exp(-new)
+                m = new
+            state[slot, state_off:state_off + heads] = m.to(torch.float32)
+            start += q_len
+
+    def delta_state_scan(self, q32, k32, v32, z32, b32, state, state_off, ctx, o32, heads, kq_heads, dk, dv, dt_bias32=None, a_log32=None,
+                         q_scale=1.0, unit_eps=1e-6):
+        m, rep = q32.shape[0], heads // kq_heads
+        unit = lambda x: (x / torch.sqrt(x.pow(2).sum(-1, keepdim=True) + unit_eps)).repeat_interleave(rep, 1)
+        q, k = unit(q32.double().reshape(m, kq_heads, dk)) * q_scale, unit(k32.double().reshape(m, kq_heads, dk))
+        v, w = v32.double().reshape(m, heads, dv), z32.double()
+        if a_log32 is not None:
+            step = torch.nn.functional.softplus(w + dt_bias32.double(), threshold=1e9).view(m, heads, dk)
+            w = torch.exp(-torch.exp(a_log32.double())[None, :, None] * step)
+        w, beta = w.reshape(m, heads, dk), torch.sigmoid(b32.double())
+        start = 0
+        for q_len, slot in zip(ctx.host.q_lens, ctx.host.slots):
+            flat = state[slot, state_off:state_off + heads * dv * dk]
+            s = flat.double().view(heads, dv, dk).transpose(1, 2).clone()
+            for t in range(start, start + q_len):
+                s = w[t][:, :, None] * s
+                u = beta[t][:, None] * (v[t] - torch.einsum("hkv,hk->hv", s, k[t]))
+                s = s + k[t][:, :, None] * u[:, None, :]
+                o32[t] = torch.einsum("hkv,hk->hv", s, q[t]).reshape(-1).to(torch.float32)
             flat.copy_(s.transpose(1, 2).reshape(-1).to(torch.float32))
             start += q_len
 
@@ -429,6 +480,26 @@ class TorchOps:
             v = v * torch.sigmoid(gate32.double())
         out.copy_(v.to(out.dtype))
 
+    # ---- several residual streams (pointwise.cu) ---------------------------------------------------------------
+    def stream_mix(self, x32, streams, y32=None, mix32=None, out32=None, dst32=None, in32=None, gain32=None, eps=0.0, h_out=None,
+                   sum_out32=None, clear=False):
+        x = x32.double()
+        if x.dim() == 2:
+            x = x[:, None, :].expand(-1, streams, -1)
+        z = x
+        if y32 is not None:
+            z = torch.einsum("rsw,st->rtw", x, mix32.double()) + out32.double()[None, :, None] * y32.double()[:, None, :]
+        z = z.to(torch.float32).double()
+        if h_out is not None:
+            u = torch.einsum("rsw,s->rw", z, in32.double())
+            h_out.copy_((u / torch.sqrt(u.pow(2).mean(-1, keepdim=True) + eps) * gain32.double()).to(h_out.dtype))
+        if dst32 is not None:
+            dst32.copy_(z.to(torch.float32))
+        if sum_out32 is not None:
+            sum_out32.copy_(z.sum(1).to(torch.float32))
+        if clear and y32 is not None:
+            y32.zero_()
+
     # ---- the norm on a branch's output, and routed experts (pointwise.cu, moe.cu) -----------------------------
     def rmsnorm_add(self, y32, gain32, eps, mult, x32, h_out=None, clear=False, next_gain32=None, next_eps=0.0):
         y = y32.double()
@@ -466,7 +537,7 @@ class TorchOps:
         sel_e.copy_(order.to(torch.int32))
         sel_w.copy_(w.to(torch.float32))
 
-    def moe_experts(self, h, sel_e, sel_w, w_gate_up, w_down, out32, plan=None, gated=True, weight_on="input", outputs=None):
+    def moe_experts(self, h, sel_e, sel_w, w_gate_up, w_down, out32, plan=None, gated=True, weight_on="input", outputs=None, glu=None):
         ff = w_down.shape[2]
         acc = out32.double()
         for t in range(h.shape[0]):
@@ -478,7 +549,7 @@ class TorchOps:
                 if gated:
                     g = (w_gate_up[e, :ff].double() @ h[t].double()) * w_in
                     u = (w_gate_up[e, ff:].double() @ h[t].double()) * w_in
-                    act = (g / (1.0 + torch.exp(-g)) * u).to(h.dtype).double()
+                    act = self._glu(g, u, glu).to(h.dtype).double()
                 else:
                     act = (torch.relu((w_gate_up[e].double() @ h[t].double()) * w_in) ** 2).to(h.dtype).double()
                 acc[t] += w_res * (w_down[e].double() @ act)
