@@ -590,8 +590,36 @@ def dusilorn_configs(size: dict):
     return dus, design_configs(dict(DESIGN_SIZES["1k"], **{k: size[k] for k in ("width", "heads", "head_dim", "ff_swiglu", "vocab", "layers")}))[1]
 
 
+# A Pilonex stack at the same widths, two residual streams: six layers of which the first two run twice (eight layer runs, as many
+# as the Qwen2 decoder has layers): windowed attention with the Qwen2 decoder's head counts and head size beside a gated
+# delta rule, and matrix memories. Feed-forwards of the clamped gated form by turns dense, as wide as the Qwen2 decoder's,
+# and mixtures of 8 experts of which a token uses 2, each half as wide.
+PILONEX_SIZES = {
+    "1k": {"width": 1024, "heads": 16, "head_dim": 64, "ff_swiglu": 2816, "delta_heads": 8, "rank": 64, "memory_heads": 8, "experts": 8, "top": 2,
+           "window": 1024, "streams": 2, "vocab": 32000, "layers": 8},
+    "2k": {"width": 2048, "heads": 16, "head_dim": 128, "ff_swiglu": 5632, "delta_heads": 8, "rank": 64, "memory_heads": 8, "experts": 8, "top": 2,
+           "window": 1024, "streams": 2, "vocab": 32000, "layers": 8},
+}
+
+
+def pilonex_configs(size: dict):
+    h, d, n = size["heads"], size["head_dim"], size["delta_heads"]
+    dense = {"kind": "dense", "ff": size["ff_swiglu"], "limit": 7.0}
+    routed = {"kind": "moe", "expert": {"ff": size["ff_swiglu"] // size["top"], "limit": 7.0}, "router": {"experts": size["experts"], "top": size["top"]}}
+    pair = {"left": {"heads": h, "kv_heads": 2, "dim": d, "vdim": d, "scale": d ** -0.5, "mask": {"size": size["window"]},
+                     "rot": {"dims": d, "base": 500000.0, "scaling": {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 4096}}},
+            "right": {"heads": n, "kv_heads": n, "dim": d, "vdim": d, "conv": 4, "decay_rank": size["rank"], "gate_rank": size["rank"]},
+            "left_scale": 1.0, "right_scale": 0.75}
+    memory = {"heads": size["memory_heads"], "dim": d, "vdim": size["width"] // size["memory_heads"], "gate_cap": 15.0}
+    order = [("parallel", dense), ("parallel", routed), ("mlstm", dense), ("parallel", routed), ("mlstm", dense), ("parallel", routed)]
+    layers = [{"type": t, "mixer": pair if t == "parallel" else memory, "mlp": mlp} for t, mlp in order]
+    pil = {"architecture": "Pilonex", "vocab": size["vocab"], "width": size["width"], "norm": {"eps": 1e-5}, "streams": size["streams"],
+           "loop": {"start": 0, "stop": 2, "times": 2}, "layers": layers}
+    return pil, design_configs(dict(DESIGN_SIZES["1k"], **{k: size[k] for k in ("width", "heads", "head_dim", "ff_swiglu", "vocab", "layers")}))[1]
+
+
 def run_design(args) -> dict:
-    """Prefill and decode throughput of a design (Nezalorn, Vafozen, Darotar, Dusilorn) beside the Qwen2 decoder at equal size (random
+    """Prefill and decode throughput of a design (Nezalorn, Vafozen, Darotar, Dusilorn, Pilonex) beside the Qwen2 decoder at equal size (random
     weights, bfloat16, device-timed with CUDA events), and where one eager step's time goes, launch kind by launch kind."""
     import numpy as np
     import torch
@@ -604,7 +632,8 @@ def run_design(args) -> dict:
     steps, warmup = min(args.steps, 64), max(3, args.warmup)
     design = args.design
     sizes, configs = {"nezalorn": (DESIGN_SIZES, design_configs), "vafozen": (VAFOZEN_SIZES, vafozen_configs),
-                      "darotar": (DAROTAR_SIZES, darotar_configs), "dusilorn": (DUSILORN_SIZES, dusilorn_configs)}[design]
+                      "darotar": (DAROTAR_SIZES, darotar_configs), "dusilorn": (DUSILORN_SIZES, dusilorn_configs),
+                      "pilonex": (PILONEX_SIZES, pilonex_configs)}[design]
     out = {"impl": "ours", "design": design, "dtype": "bf16", "data": "synthetic: seeded random weights and random token ids",
            "peaks": {"hbm_gbs": pk["hbm_gbs"], "bf16_tflops": pk["bf16_tflops"], "source": pk["source"]},
            "config": {"prefill_tokens": t_pre, "decode_batch": batch, "decode_context": ctx, "page_size": 16}, "sizes": {}}
@@ -836,7 +865,7 @@ def main() -> int:
                     help="add a 'kernels' block: where the time of a decode step and of a prompt portion goes, kernel kind by "
                          "kind, with bytes or FLOPs and the fraction of the measured peak")
     ap.add_argument("--shape", default="0.5b", choices=sorted(SHAPES), help="layer sizes: the family's 0.5B (default), 1.5B or 7B")
-    ap.add_argument("--design", default=None, choices=["nezalorn", "vafozen", "darotar", "dusilorn"],
+    ap.add_argument("--design", default=None, choices=["nezalorn", "vafozen", "darotar", "dusilorn", "pilonex"],
                     help="instead of the headline workload: prefill and decode throughput of this design beside the Qwen2 "
                          "decoder at equal size (--design-sizes, --prefill-tokens, --batch, --context up to 2048, --breakdown)")
     ap.add_argument("--design-sizes", default="", help="comma-separated names of DESIGN_SIZES (default: all)")

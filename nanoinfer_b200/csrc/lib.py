@@ -91,8 +91,9 @@ class Kernels:
                      "nib_linear_state_scan", "nib_conv_tokens", "nib_conv_tail", "nib_conv_step", "nib_token_shift", "nib_decay_map", "nib_step_sizes",
                      "nib_attention_prepare", "nib_attention_flex", "nib_attention_flex_mma", "nib_attention_flex_mma_supported",
                      "nib_rmsnorm_add", "nib_moe_route", "nib_moe_max_tiles", "nib_moe_group", "nib_moe_gemm_simt", "nib_moe_combine",
-                     "nib_moe_tc_supported", "nib_moe_tc_error", "nib_moe_gather_rows", "nib_moe_gemm_tc", "nib_moe_step", "nib_moe_step_supported", "nib_moe_identity", "nib_stream_mix", "nib_delta_state_scan", "nib_memory_gates"):
+                     "nib_moe_tc_supported", "nib_moe_tc_error", "nib_moe_gather_rows", "nib_moe_gemm_tc", "nib_moe_step", "nib_moe_step_supported", "nib_moe_identity", "nib_stream_mix", "nib_grouped_state_scan", "nib_grouped_state_error", "nib_memory_gates"):
             getattr(self._lib, name).restype = c_int
+        self._lib.nib_grouped_state_scratch.restype = c_longlong
 
     # ---- plumbing ---------------------------------------------------------------------------
     def _check(self, rc: int, what: str) -> None:
@@ -545,6 +546,7 @@ class Kernels:
             ("tcgen05 prefill attention (attention_tcgen05.cu)", self.attention_tc_error(), _ATTN_TC_ROLES),
             ("TMA decode attention (attention_decode_tma.cu)", self.attention_decode_tma_error(), _DECODE_TMA_ROLES),
             ("routed experts on the tensor cores (moe_tcgen05.cu)", self._lib.nib_moe_tc_error(), _GEMM_TC_ROLES),
+            ("walk over matrix states (grouped_state.cu)", self._lib.nib_grouped_state_error(), {1: "walking warp: a group never arrived", 2: "sending warp: a buffer was never freed"}),
         ])
 
     def decode_splits(self, n_tokens: int, kv_heads: int, max_ctx: int, window: int, tma: bool = False,
@@ -910,22 +912,19 @@ class Kernels:
             raise KernelError(f"{what}: the state does not hold {size} floats from column {off}")
 
     def linear_state_scan(self, q32, k32, v32, w32, state, state_off, ctx, o32, heads, kq_heads, dk, dv, q_scale=1.0,
-                          bonus32=None, v_scale32=None, seg_len=None, ones=False):
+                          bonus32=None, v_scale32=None, seg_len=None):
         """Per request and head, over the step's tokens in order, from and into ``state[slot, state_off:]`` (laid out
         [head, value channel, key channel]): S <- diag(w) S + k (v_scale v)^T, o = S^T (q_scale q); with ``bonus32``
         [heads, dk] instead o = (S_old + diag(bonus) k v^T)^T q before the update. q32, k32: [tokens, kq_heads * dk]
         (head h reads key head h // (heads / kq_heads)); v32, o32: [tokens, heads * dv]; w32: [tokens, heads * dk] (a
-        decay per key channel) or [tokens, heads] (one per head); v_scale32: [tokens, heads]. With ``ones`` a head has one
-        value channel more than ``dv``, behind the others, whose value is 1: the state holds heads * (dv + 1) * dk floats and
-        o32 is [tokens, heads * (dv + 1)].
+        decay per key channel) or [tokens, heads] (one per head); v_scale32: [tokens, heads].
 
         A step in which a request brings 256 tokens or more, and whose walk in order would not fill the GPU, is walked in
         segments of 128 tokens or more side by side (every
         segment from a zero state, the end states chained with the products of the segments' decays, then every segment
         again from its true entry state): the result then depends on the cut by rounding. ``seg_len``: None = that rule,
         0 = never, another multiple of 8 = segments of that length whenever a request brings more."""
-        extra = 1 if ones else 0
-        for t, what, width in ((q32, "q", kq_heads * dk), (k32, "k", kq_heads * dk), (v32, "v", heads * dv), (o32, "o", heads * (dv + extra))):
+        for t, what, width in ((q32, "q", kq_heads * dk), (k32, "k", kq_heads * dk), (v32, "v", heads * dv), (o32, "o", heads * dv)):
             self._rows(t, torch.float32, f"linear_state_scan {what}")
             if tuple(t.shape) != (q32.shape[0], width):
                 raise KernelError(f"linear_state_scan: {what} does not fit")
@@ -941,7 +940,6 @@ class Kernels:
             _need(v_scale32, torch.float32, "linear_state_scan v_scale")
             if tuple(v_scale32.shape) != (q32.shape[0], heads):
                 raise KernelError("linear_state_scan: v_scale does not fit")
-        dv += extra         # from here on the state's value channels
         self._state_row(state, state_off, heads * dv * dk, "linear_state_scan state")
         n_req, longest = ctx.host.num_requests, max(ctx.host.q_lens)
         if seg_len is None:
@@ -963,7 +961,7 @@ class Kernels:
             c_int(w32.stride(0)), c_int(1 if per_channel else 0), _ptr(bonus32), _ptr(v_scale32), _ptr(state), c_longlong(state.stride(0)),
             c_int(state_off), _ptr(ctx.q_start), _ptr(ctx.state_slots), _ptr(o32), c_int(o32.stride(0)), c_int(ctx.host.num_requests),
             c_int(heads), c_int(kq_heads), c_int(dk), c_int(dv), c_float(q_scale), c_int(n_seg), c_int(seg_len if n_seg > 1 else 0), _ptr(scratch),
-            c_int(extra), self._stream()), "linear_state_scan")
+            self._stream()), "linear_state_scan")
 
     def memory_gates(self, zi32, zf32, bi32, bf32, cap, state, state_off, ctx, decay32, write32, floor32):
         """Gates of a stabilized matrix memory, per (token, head): i = cap * tanh((zi32 + bi32) / cap), f = log sigmoid(cap *
@@ -985,37 +983,52 @@ class Kernels:
             c_longlong(state.stride(0)), c_int(state_off), _ptr(ctx.q_start), _ptr(ctx.state_slots), _ptr(decay32), _ptr(write32), _ptr(floor32),
             c_int(ctx.host.num_requests), c_int(max(ctx.host.q_lens)), c_int(heads), self._stream()), "memory_gates")
 
-    # ---- the gated delta rule (delta_state.cu) ---------------------------------------------------------------
-    def delta_state_scan(self, q32, k32, v32, z32, b32, state, state_off, ctx, o32, heads, kq_heads, dk, dv, dt_bias32=None, a_log32=None,
-                         q_scale=1.0, unit_eps=1e-6):
-        """Per request and head, over the step's tokens in order, from and into ``state[slot, state_off:]`` (laid out [head,
-        value channel, key channel]), with k and q made unit vectors per head (x / sqrt(sum x^2 + unit_eps), q times
-        ``q_scale``): S <- diag(w) S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q. beta = sigmoid(b32) [tokens, heads];
-        w = exp(-exp(a_log32[head]) * softplus(z32 + dt_bias32)) per (head, key channel), or z32 itself without ``a_log32``.
-        q32, k32: [tokens, kq_heads * dk] (head h reads head h // (heads / kq_heads)); v32, o32: [tokens, heads * dv];
-        z32: [tokens, heads * dk]. Tokens are taken eight at a time; how a request is cut moves the result by rounding."""
-        for t, what, width in ((q32, "q", kq_heads * dk), (k32, "k", kq_heads * dk), (v32, "v", heads * dv), (o32, "o", heads * dv),
-                               (z32, "z", heads * dk), (b32, "beta", heads)):
-            self._rows(t, torch.float32, f"delta_state_scan {what}")
-            if tuple(t.shape) != (q32.shape[0], width):
-                raise KernelError(f"delta_state_scan: {what} does not fit")
-        if (dt_bias32 is None) != (a_log32 is None):
-            raise KernelError("delta_state_scan: step sizes need both their bias and the rates")
-        for t, n in ((dt_bias32, heads * dk), (a_log32, heads)):
-            if t is not None:
-                _need(t, torch.float32, "delta_state_scan decay")
-                if t.numel() != n:
-                    raise KernelError("delta_state_scan: the decays' constants do not fit")
-        self._state_row(state, state_off, heads * dv * dk, "delta_state_scan state")
+    # ---- walks over matrix states, eight tokens at a time (grouped_state.cu) -----------------------------------
+    def grouped_state_scan(self, q32, k32, v32, z32, state, state_off, ctx, o32, heads, kq_heads, dk, dv, beta32=None, rate32=None,
+                           dt_bias32=None, q_scale=1.0, unit_eps=None, k_scale32=None, ones=False):
+        """Per request and head, over the step's tokens in order, from and into ``state[slot, state_off:]`` (laid out [head, value
+        channel, key channel]). With ``beta32`` [tokens, heads] (logits, beta = sigmoid) the delta rule: S <- diag(w) S,
+        u = beta (v - S^T k), S <- S + k u^T, o = S^T q; without it S <- diag(w) S + k v^T, o = S^T q. q32, k32: [tokens, kq_heads * dk]
+        (head h reads head h // (heads / kq_heads)); v32, o32: [tokens, heads * dv]. z32: [tokens, heads * dk], the decays w, or with
+        ``rate32`` [heads] and ``dt_bias32`` [heads * dk] the logits of step sizes, w = exp(-rate32 * softplus(z32 + dt_bias32)); or
+        [tokens, heads], one decay per head. ``unit_eps``: q and k become unit vectors per head (x / sqrt(sum x^2 + unit_eps));
+        queries are then multiplied by ``q_scale``, keys by ``k_scale32`` [tokens, heads]. With ``ones`` a head has one value channel
+        more, behind the others, whose value is 1: the state holds heads * (dv + 1) * dk floats, o32 is [tokens, heads * (dv + 1)].
+        How a request is cut moves the result by rounding."""
+        extra = 1 if ones else 0
         m = q32.shape[0]
-        scratch = torch.empty(m * heads * (4 * dk + 16), dtype=torch.float32, device=q32.device)
+        for t, what, width in ((q32, "q", kq_heads * dk), (k32, "k", kq_heads * dk), (v32, "v", heads * dv), (o32, "o", heads * (dv + extra))):
+            self._rows(t, torch.float32, f"grouped_state_scan {what}")
+            if tuple(t.shape) != (m, width):
+                raise KernelError(f"grouped_state_scan: {what} does not fit")
+        self._rows(z32, torch.float32, "grouped_state_scan decay")
+        if (rate32 is None) != (dt_bias32 is None):
+            raise KernelError("grouped_state_scan: step sizes need both their bias and the rates")
+        kind = 0 if rate32 is not None else (1 if z32.shape[1] == heads * dk else 2)
+        if tuple(z32.shape) != (m, heads if kind == 2 else heads * dk):
+            raise KernelError("grouped_state_scan: the decay is neither per key channel nor per head")
+        for t, n, what in ((dt_bias32, heads * dk, "bias"), (rate32, heads, "rates")):
+            if t is not None:
+                _need(t, torch.float32, f"grouped_state_scan {what}")
+                if t.numel() != n:
+                    raise KernelError(f"grouped_state_scan: the decays' {what} do not fit")
+        for t, what in ((beta32, "beta"), (k_scale32, "k_scale")):
+            if t is not None:
+                self._rows(t, torch.float32, f"grouped_state_scan {what}")
+                if tuple(t.shape) != (m, heads):
+                    raise KernelError(f"grouped_state_scan: {what} does not fit")
+        if k_scale32 is not None and not k_scale32.is_contiguous():
+            raise KernelError("grouped_state_scan: k_scale must be contiguous")
+        self._state_row(state, state_off, heads * (dv + extra) * dk, "grouped_state_scan state")
+        floats = self._lib.nib_grouped_state_scratch(c_longlong(m), c_int(ctx.host.num_requests), c_int(heads), c_int(dk), c_int(0 if beta32 is None else 1))
+        scratch = torch.empty(floats, dtype=torch.float32, device=q32.device)
         self.launches += 1
-        self._check(self._lib.nib_delta_state_scan(
+        self._check(self._lib.nib_grouped_state_scan(
             _ptr(q32), c_int(q32.stride(0)), _ptr(k32), c_int(k32.stride(0)), _ptr(v32), c_int(v32.stride(0)), _ptr(z32), c_int(z32.stride(0)),
-            _ptr(dt_bias32), _ptr(a_log32), _ptr(b32), c_int(b32.stride(0)), _ptr(state), c_longlong(state.stride(0)), c_int(state_off),
-            _ptr(ctx.q_start), _ptr(ctx.state_slots), _ptr(o32), c_int(o32.stride(0)), _ptr(scratch), c_int(m), c_int(ctx.host.num_requests),
-            c_int(max(ctx.host.q_lens)), c_int(heads), c_int(kq_heads), c_int(dk), c_int(dv), c_float(q_scale), c_float(unit_eps),
-            self._stream()), "delta_state_scan")
+            c_int(kind), _ptr(dt_bias32), _ptr(rate32), _ptr(beta32), c_int(0 if beta32 is None else beta32.stride(0)), _ptr(k_scale32), _ptr(state),
+            c_longlong(state.stride(0)), c_int(state_off), _ptr(ctx.q_start), _ptr(ctx.state_slots), _ptr(o32), c_int(o32.stride(0)), _ptr(scratch),
+            c_int(m), c_int(ctx.host.num_requests), c_int(max(ctx.host.q_lens)), c_int(heads), c_int(kq_heads), c_int(dk), c_int(dv), c_int(extra),
+            c_float(q_scale), c_float(-1.0 if unit_eps is None else unit_eps), self._stream()), "grouped_state_scan")
 
     def conv_tokens(self, x32, w32, bias32, act, state, state_off, ctx, out32, taps):
         """out32[t, c] = act(bias32[c] + sum_j w32[c, j] * x32[t - (taps-1-j), c]) within each request; inputs before the

@@ -9,11 +9,9 @@
 //    update (o_t = S_t^T q_t) or, with a bonus u, before it (o_t = (S_(t-1) + diag(u) k_t v_t^T)^T q_t). The decay is a
 //    vector per key channel or one number per head; q and k may be shared by groups of heads; v may carry a factor per
 //    (token, head). Gated linear attention, a time mix with bonus and a state-space mixer with scalar decays are this
-//    walk with different inputs. With `ones` a head has one more value channel whose value is 1 (times the factor): the
-//    sum of the keys under the same decays, which a normalizer reads.
+//    walk with different inputs.
 //  * conv_tokens / conv_tail: a short causal convolution per channel whose last taps-1 inputs are kept in the state.
 //  * token_shift: blends of every token with the token before it (the request's last token is kept in the state).
-//  * memory_gates: decay, factor on the values and floor of the normalizer of a matrix memory with exponential gates.
 //  * decay_map, step_sizes: the decays, rounded to 32 bits once from 64-bit exponentials (a decay is raised to hundreds
 //    of powers along a sequence).
 #include "common.cuh"
@@ -66,8 +64,7 @@ linear_state_scan_kernel(const float* __restrict__ q, int ldq, const float* __re
                          const float* __restrict__ v_scale, float* __restrict__ state, long long state_ld, int state_off,
                          const int* __restrict__ q_start, const int* __restrict__ slots, float* __restrict__ o, int ldo,
                          int heads, int kq_heads, int dk, int dv, float q_scale, int n_seg, int seg_len,
-                         float* __restrict__ seg_state, float* __restrict__ seg_decay, int vec, int ones) {
-    // dv counts the value channels of the state and of the output, the column of ones among them; v has dv - ones a head
+                         float* __restrict__ seg_state, float* __restrict__ seg_decay, int vec) {
     using L = LsLayout<C, PER_CHANNEL>;
     constexpr int DKP = L::DKP, TB = L::TB, STAGES = L::STAGES;
     extern __shared__ __align__(16) float ls_smem[];
@@ -125,10 +122,8 @@ linear_state_scan_kernel(const float* __restrict__ q, int ldq, const float* __re
         }
         for (int e = threadIdx.x; e < TB * LS_COLS; e += LS_THREADS) {
             const int tt = e / LS_COLS, cc = e % LS_COLS, jj = blockIdx.x * LS_COLS + cc;
-            const int dvv = dv - ones;
-            const bool ok = tt < nt && jj < dvv;
-            if (ones && jj == dvv) v_s(buf, tt)[cc] = 1.0f;     // (with a key of zeros beyond the chunk it adds nothing)
-            else ls_cp_async_4(v_s(buf, tt) + cc, v + (size_t)(base + (ok ? tt : 0)) * ldv + (size_t)h * dvv + (ok ? jj : 0), ok);
+            const bool ok = tt < nt && jj < dv;
+            ls_cp_async_4(v_s(buf, tt) + cc, v + (size_t)(base + (ok ? tt : 0)) * ldv + (size_t)h * dv + (ok ? jj : 0), ok);
         }
         if (threadIdx.x < TB) {
             const int tt = threadIdx.x;
@@ -266,16 +261,14 @@ NIB_API long long nib_linear_state_scan_scratch(int n_req, int n_seg, int heads,
 
 // n_seg <= 1: every request's tokens in order, one block per (request, head, 16 value columns). n_seg > 1 (long
 // prompts): segments of seg_len tokens side by side (see the kernel); scratch holds nib_linear_state_scan_scratch floats.
-// ones 1: dv counts one more value channel than v has, whose value is 1 (state and output are dv wide per head).
 NIB_API int nib_linear_state_scan(const float* q, int ldq, const float* k, int ldk, const float* v, int ldv, const float* w, int ldw,
                                   int w_per_channel, const float* bonus, const float* v_scale, float* state, long long state_ld,
                                   int state_off, const int* q_start, const int* slots, float* o, int ldo, int n_req, int heads,
                                   int kq_heads, int dk, int dv, float q_scale, int n_seg, int seg_len, float* scratch,
-                                  int ones, cudaStream_t stream) {
+                                  cudaStream_t stream) {
     NIB_REQUIRE(heads > 0 && kq_heads > 0 && heads % kq_heads == 0, "linear_state_scan: %d heads do not share %d key heads", heads, kq_heads);
     NIB_REQUIRE(dk > 0 && dk <= 256 && dv > 0, "linear_state_scan: key size %d is outside 1..256", dk);
     NIB_REQUIRE(n_seg <= 1 || (scratch != nullptr && seg_len > 0 && seg_len % 8 == 0), "linear_state_scan: segments need scratch and a length that is a multiple of 8");
-    NIB_REQUIRE(ones == 0 || (ones == 1 && dv > 1), "linear_state_scan: a column of ones stands beside value channels");
     if (n_req <= 0) return 0;
     const bool cut = n_seg > 1;
     auto aligned = [](const void* p, int ld) { return ((uintptr_t)p & 15) == 0 && ld % 4 == 0; };
@@ -294,7 +287,7 @@ NIB_API int nib_linear_state_scan(const float* q, int ldq, const float* k, int l
         const dim3 grid(ceil_div(dv, LS_COLS), heads, n_req * (MODE == 0 ? 1 : n_seg));                                             \
         linear_state_scan_kernel<C, PC, B, MODE><<<grid, block, LsLayout<C, PC>::BYTES, stream>>>(                                  \
             q, ldq, k, ldk, v, ldv, w, ldw, bonus, v_scale, state, state_ld, state_off, q_start, slots, o, ldo, heads, kq_heads,    \
-            dk, dv, q_scale, n_seg, seg_len, seg_state, seg_decay, vec, ones);                                                          \
+            dk, dv, q_scale, n_seg, seg_len, seg_state, seg_decay, vec);                                                            \
         NIB_LAUNCH_CHECK();                                                                                                         \
     } while (0)
 #define NIB_LS_LAUNCH3(C, PC, B)                                                                                                    \
@@ -539,79 +532,6 @@ NIB_API int nib_step_sizes(const float* raw, int ld, const float* bias, const fl
     NIB_REQUIRE(tokens >= 0 && heads > 0, "step_sizes: bad sizes");
     if (tokens == 0) return 0;
     NIB_CUDA(launch_pdl(step_sizes_kernel, dim3(ceil_div((long long)tokens * heads, 256)), dim3(256), (size_t)0, stream, raw, ld, bias, a_log, dt, decay, tokens, heads));
-    NIB_LAUNCH_CHECK();
-    return 0;
-}
-
-// ---------------------------------------------------------------------------------- gates of a stabilized matrix memory
-// Per (token, head): the log input gate i = cap * tanh((zi + bi) / cap), the log forget gate f = log sigmoid(cap * tanh((zf +
-// bf) / cap)), and the running maximum m_t = max(f + m_(t-1), i), which starts at the state's number (zero at a request's
-// start) and is kept there. Out: decay = exp(f + m_(t-1) - m_t), write = exp(i - m_t), floor = exp(-m_t). A block per
-// (request, head), a thread per token: the maxima are a scan over the maps m -> max(m + f, a) (composed in warps, then across
-// the block's warps), in 64-bit; m_t is rounded to 32 bits before anything is formed from it, so that the numbers a state was
-// scaled with are exactly those the next step finds.
-__device__ __forceinline__ double mg_shfl_up(double x, int o) { return __shfl_up_sync(0xffffffffu, x, o); }
-
-__global__ void __launch_bounds__(1024)
-memory_gates_kernel(const float* __restrict__ zi, int ldi, const float* __restrict__ zf, int ldf, const float* __restrict__ bi,
-                    const float* __restrict__ bf, float cap, float* __restrict__ state, long long state_ld, int state_off,
-                    const int* __restrict__ q_start, const int* __restrict__ slots, float* __restrict__ decay, float* __restrict__ write,
-                    float* __restrict__ floor_out, int heads) {
-    __shared__ double s_f[32], s_a[32];
-    __shared__ float s_m[32];
-    pdl_launch_dependents();
-    pdl_wait();      // everything this kernel reads may come from the kernel before
-    const int h = blockIdx.x, req = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
-    const int row0 = q_start[req], row1 = q_start[req + 1];
-    if (row0 >= row1) return;
-    float* st = state + (long long)slots[req] * state_ld + state_off + h;
-    float m_in = *st;
-    const double c = (double)cap;
-    for (int base = row0; base < row1; base += blockDim.x) {
-        const int t = base + threadIdx.x;
-        const bool live = t < row1;
-        double i = 0.0, f = 0.0;
-        if (live) {
-            i = c * tanh(((double)zi[(size_t)t * ldi + h] + (double)bi[h]) / c);
-            const double x = c * tanh(((double)zf[(size_t)t * ldf + h] + (double)bf[h]) / c);
-            f = x >= 0.0 ? -log1p(exp(-x)) : x - log1p(exp(x));
-        }
-        // the maps of this warp's tokens, composed: m -> max(m + F, A)
-        double F = f, A = live ? i : -INFINITY;
-#pragma unroll
-        for (int o = 1; o < 32; o <<= 1) {
-            const double pF = mg_shfl_up(F, o), pA = mg_shfl_up(A, o);
-            if (lane >= o) { A = fmax(pA + F, A); F += pF; }
-        }
-        if (lane == 31) { s_f[warp] = F; s_a[warp] = A; }
-        __syncthreads();
-        double m0 = (double)m_in;
-        for (int w = 0; w < warp; ++w) m0 = fmax(m0 + s_f[w], s_a[w]);
-        const float m = (float)fmax(m0 + F, A);
-        float before = __shfl_up_sync(0xffffffffu, m, 1);
-        if (lane == 31) s_m[warp] = m;
-        __syncthreads();
-        if (lane == 0) before = warp == 0 ? m_in : s_m[warp - 1];
-        if (live) {
-            const size_t at = (size_t)t * heads + h;
-            decay[at] = (float)exp(f + (double)before - (double)m);
-            write[at] = (float)exp(i - (double)m);
-            floor_out[at] = (float)exp(-(double)m);
-            if (t == row1 - 1) *st = m;
-        }
-        m_in = s_m[warps - 1];      // (a block that goes on is full: its last thread holds a token)
-        __syncthreads();
-    }
-}
-
-NIB_API int nib_memory_gates(const float* zi, int ldi, const float* zf, int ldf, const float* bi, const float* bf, float cap, float* state,
-                             long long state_ld, int state_off, const int* q_start, const int* slots, float* decay, float* write,
-                             float* floor_out, int n_req, int longest, int heads, cudaStream_t stream) {
-    NIB_REQUIRE(n_req >= 0 && n_req <= 65535 && heads > 0 && cap > 0.f && bi != nullptr && bf != nullptr, "memory_gates: bad sizes");
-    if (n_req == 0 || longest <= 0) return 0;
-    const int threads = longest >= 1024 ? 1024 : ((longest + 31) / 32) * 32;
-    NIB_CUDA(launch_pdl(memory_gates_kernel, dim3(heads, n_req), dim3(threads), (size_t)0, stream, zi, ldi, zf, ldf, bi, bf, cap, state, state_ld,
-                        state_off, q_start, slots, decay, write, floor_out, heads));
     NIB_LAUNCH_CHECK();
     return 0;
 }

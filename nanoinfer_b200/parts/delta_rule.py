@@ -137,7 +137,7 @@ class GatedDeltaRule(Mixer):
         w2[self.nk:, ra:ra + rg] = tensors["g2"]
         self.w_2 = rt.matrix(w2)
         self.conv_w = rt.vector32(torch.cat([tensors[n + "_conv"] for n in ("q", "k", "v")], dim=0))
-        self.a_log, self.dt_bias = rt.vector32(tensors["A_log"]), rt.vector32(tensors["dt_bias"])
+        self.rate, self.dt_bias = rt.vector32(torch.exp(tensors["A_log"].double()).to(torch.float32)), rt.vector32(tensors["dt_bias"])
         self.gain = rt.vector32(tensors["norm"])
         self.w_o = rt.matrix(tensors["o"])
         self.conv_state = (self.taps - 1) * self.n_conv
@@ -158,9 +158,9 @@ class GatedDeltaRule(Mixer):
         zg = torch.empty((m, nk + nv), dtype=torch.float32, device=dev)
         ops.linear(inner, self.w_2, None, zg, "f32")
         o32 = torch.empty((m, nv), dtype=torch.float32, device=dev)
-        ops.delta_state_scan(qkv[:, :nq], qkv[:, nq:2 * nq], qkv[:, 2 * nq:], zg[:, :nk], p32[:, self.b_col:self.b_col + self.heads], cache.state,
-                             self.conv_state, ctx, o32, self.heads, self.kv_heads, self.dim, self.vdim, dt_bias32=self.dt_bias,
-                             a_log32=self.a_log, q_scale=self.dim ** -0.5, unit_eps=self.UNIT_EPS)
+        ops.grouped_state_scan(qkv[:, :nq], qkv[:, nq:2 * nq], qkv[:, 2 * nq:], zg[:, :nk], cache.state, self.conv_state, ctx, o32, self.heads,
+                               self.kv_heads, self.dim, self.vdim, beta32=p32[:, self.b_col:self.b_col + self.heads], rate32=self.rate,
+                               dt_bias32=self.dt_bias, q_scale=self.dim ** -0.5, unit_eps=self.UNIT_EPS)
         gated = torch.empty((m, nv), dtype=self.rt.dtype, device=dev)
         ops.gated_norm(o32, gated, groups=self.heads, eps=self.eps, gain32=self.gain, gate32=zg[:, nk:], gate_kind="sigmoid",
                        out_scale=self.out_scale)

@@ -3,8 +3,8 @@
     S_t = diag(w_t) S_(t-1) + k_t v_t^T          (S: key channel x value channel, 32-bit, zero at a request's start)
 
 read either after the update (``o_t = S_t^T q_t``) or before it with a bonus for the current token
-(``o_t = (S_(t-1) + diag(u) k_t v_t^T)^T q_t``). One kernel walks all of them (``ops.linear_state_scan``); the classes
-differ in where q, k, v and the decay come from and in what happens to o:
+(``o_t = (S_(t-1) + diag(u) k_t v_t^T)^T q_t``). A kernel of the library walks each of them (``ops.linear_state_scan``, token
+by token; ``ops.grouped_state_scan``, eight tokens at a time); the classes differ in where q, k, v and the decay come from and in what happens to o:
 
 * ``GatedLinearAttention``: ``q = W_q h / sqrt(dim)``, ``k = W_k h``, ``v = W_v h``, decay per key channel
   ``sigmoid(W_a2 W_a1 h + b)^(1/tau)``; o is RMS-normed per head (gain of ``vdim``, shared by the heads), times
@@ -20,7 +20,7 @@ differ in where q, k, v and the decay come from and in what happens to o:
 * ``StabilizedMatrixMemory``: ``q = W_q h / sqrt(dim)``, ``k = W_k h``, ``v = W_v h``; per head a log input gate
   ``i = cap tanh((W_i h + b_i) / cap)`` and a log forget gate ``f = log sigmoid(cap tanh((W_f h + b_f) / cap))``; with a running
   maximum ``m_t = max(f + m_(t-1), i)`` (zero at a request's start) the decay is the scalar ``exp(f + m_(t-1) - m_t)`` and
-  ``v`` carries the factor ``exp(i - m_t)``. The sum n of the keys under the same decays and factors is one more value channel
+  ``k`` carries the factor ``exp(i - m_t)``. The sum n of the keys under the same decays and factors is one more value channel
   (of ones); ``o`` is divided by ``max(|n . q|, exp(-m_t)) + 1e-6``, then by its root mean square per head, times a gain of all
   heads' size, times ``sigmoid(W_g h)``, then ``W_o``.
 
@@ -265,8 +265,8 @@ class StabilizedMatrixMemory(Mixer):
         ops.memory_gates(p32[:, gates:gates + heads], p32[:, gates + heads:gates + 2 * heads], self.b_i, self.b_f, self.cap, cache.state, 0, ctx,
                          decay, write, floor)
         o32 = torch.empty((m, heads * (self.vdim + 1)), dtype=torch.float32, device=dev)
-        ops.linear_state_scan(p32[:, :nk], p32[:, nk:2 * nk], p32[:, 2 * nk:2 * nk + nv], decay, cache.state, self.s_off, ctx, o32, heads, heads,
-                              self.dim, self.vdim, q_scale=self.dim ** -0.5, v_scale32=write, ones=True)
+        ops.grouped_state_scan(p32[:, :nk], p32[:, nk:2 * nk], p32[:, 2 * nk:2 * nk + nv], decay, cache.state, self.s_off, ctx, o32, heads, heads,
+                               self.dim, self.vdim, q_scale=self.dim ** -0.5, k_scale32=write, ones=True)
         gated = torch.empty((m, nv), dtype=self.rt.dtype, device=dev)
         ops.gated_norm(o32, gated, groups=heads, eps=self.eps, gain32=self.gain, gate32=p32[:, 2 * nk + nv:gates], gate_kind="sigmoid",
                        out_scale=self.out_scale, floor32=floor, den_eps=self.DEN_EPS)

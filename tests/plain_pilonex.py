@@ -86,7 +86,7 @@ def window_attention(m, w, p, h, eps):
     k = unit_rms((h @ w[p + ".k"].t()).view(t_len, groups, dim), eps) * w[p + ".k.norm"]
     q, k = kept(rotate_half_pairs(q, m["rot"])), kept(rotate_half_pairs(k, m["rot"]))
     v = kept(h @ w[p + ".v"].t()).view(t_len, groups, vdim)
-    mask = mask_window(t_len, int(m["mask"]["size"]))
+    mask = mask_window(t_len, int(m["mask"]["size"]) if m.get("mask") else t_len)
     out = torch.zeros(t_len, heads, vdim, dtype=F)
     for n in range(heads):
         g = n // (heads // groups)

@@ -111,3 +111,19 @@ def test_the_fifth_designs_bench_sizes_are_configurations_the_registry_takes():
         mlp = dus["layers"][1]["mlp"]
         assert 2 * (mlp["router"]["top"] * mlp["expert"]["ff"] + mlp["shared"]["ff"]) == 3 * size["ff_swiglu"]
         assert dus["layers"][0]["mlp"]["kind"] == "dense" and plan.layers[1].parts["mixer"].params["v_mix"] == "blend"
+
+
+def test_the_sixth_designs_bench_sizes_are_configurations_the_registry_takes():
+    """``--design pilonex``: both models of a size are valid configurations of equal width and vocabulary, with as many layer
+    runs (two layers run twice) as the dense decoder has layers; a token passes through as many feed-forward parameters."""
+    from nanoinfer_b200.registry import config_from_json_dict, plan_for
+    for size in bench.PILONEX_SIZES.values():
+        pil, dense = bench.pilonex_configs(size)
+        plan, dense_plan = plan_for(config_from_json_dict(pil)), plan_for(config_from_json_dict(dense))
+        assert len(plan.schedule) == len(dense_plan.layers) == size["layers"] and len(plan.layers) == size["layers"] - 2
+        assert [e.layer for e in plan.schedule] == [0, 1, 0, 1, 2, 3, 4, 5]
+        assert plan.hidden_size == dense_plan.hidden_size == size["width"] and plan.vocab_size == dense_plan.vocab_size
+        kinds = [layer["type"] for layer in pil["layers"]]
+        assert kinds.count("parallel") == 4 and kinds.count("mlstm") == 2
+        moe = pil["layers"][1]["mlp"]
+        assert moe["router"]["top"] * moe["expert"]["ff"] == size["ff_swiglu"] == pil["layers"][0]["mlp"]["ff"]

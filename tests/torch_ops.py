@@ -300,10 +300,7 @@ class TorchOps:
         decay_out.copy_(torch.exp(-torch.exp(a_log32.double()) * dt_out.double()).to(torch.float32))
 
     def linear_state_scan(self, q32, k32, v32, w32, state, state_off, ctx, o32, heads, kq_heads, dk, dv, q_scale=1.0,
-                          bonus32=None, v_scale32=None, seg_len=None, ones=False):
-        if ones:
-            v32 = torch.cat([v32.reshape(-1, heads, dv), torch.ones(v32.shape[0], heads, 1)], -1).reshape(v32.shape[0], -1)
-            dv += 1
+                          bonus32=None, v_scale32=None, seg_len=None):
         start = 0
         rep = heads // kq_heads
         per_channel = w32.shape[1] == heads * dk
@@ -341,23 +338,31 @@ class TorchOps:
             state[slot, state_off:state_off + heads] = m.to(torch.float32)
             start += q_len
 
-    def delta_state_scan(self, q32, k32, v32, z32, b32, state, state_off, ctx, o32, heads, kq_heads, dk, dv, dt_bias32=None, a_log32=None,
-                         q_scale=1.0, unit_eps=1e-6):
+    def grouped_state_scan(self, q32, k32, v32, z32, state, state_off, ctx, o32, heads, kq_heads, dk, dv, beta32=None, rate32=None,
+                           dt_bias32=None, q_scale=1.0, unit_eps=None, k_scale32=None, ones=False):
         m, rep = q32.shape[0], heads // kq_heads
-        unit = lambda x: (x / torch.sqrt(x.pow(2).sum(-1, keepdim=True) + unit_eps)).repeat_interleave(rep, 1)
-        q, k = unit(q32.double().reshape(m, kq_heads, dk)) * q_scale, unit(k32.double().reshape(m, kq_heads, dk))
+        q, k = q32.double().reshape(m, kq_heads, dk), k32.double().reshape(m, kq_heads, dk)
+        if unit_eps is not None:
+            q, k = (x / torch.sqrt(x.pow(2).sum(-1, keepdim=True) + unit_eps) for x in (q, k))
+        q, k = q.repeat_interleave(rep, 1) * q_scale, k.repeat_interleave(rep, 1)
+        if k_scale32 is not None:
+            k = k * k_scale32.double()[..., None]
         v, w = v32.double().reshape(m, heads, dv), z32.double()
-        if a_log32 is not None:
+        if ones:
+            v, dv = torch.cat([v, torch.ones(m, heads, 1, dtype=torch.float64)], -1), dv + 1
+        if rate32 is not None:
             step = torch.nn.functional.softplus(w + dt_bias32.double(), threshold=1e9).view(m, heads, dk)
-            w = torch.exp(-torch.exp(a_log32.double())[None, :, None] * step)
-        w, beta = w.reshape(m, heads, dk), torch.sigmoid(b32.double())
+            w = torch.exp(-rate32.double()[None, :, None] * step)
+        w = w.reshape(m, heads, dk) if w.numel() == m * heads * dk else w.reshape(m, heads, 1).expand(m, heads, dk)
         start = 0
         for q_len, slot in zip(ctx.host.q_lens, ctx.host.slots):
             flat = state[slot, state_off:state_off + heads * dv * dk]
             s = flat.double().view(heads, dv, dk).transpose(1, 2).clone()
             for t in range(start, start + q_len):
                 s = w[t][:, :, None] * s
-                u = beta[t][:, None] * (v[t] - torch.einsum("hkv,hk->hv", s, k[t]))
+                u = v[t]
+                if beta32 is not None:
+                    u = torch.sigmoid(beta32[t].double())[:, None] * (u - torch.einsum("hkv,hk->hv", s, k[t]))
                 s = s + k[t][:, :, None] * u[:, None, :]
                 o32[t] = torch.einsum("hkv,hk->hv", s, q[t]).reshape(-1).to(torch.float32)
             flat.copy_(s.transpose(1, 2).reshape(-1).to(torch.float32))
