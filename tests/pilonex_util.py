@@ -170,6 +170,21 @@ def plain_logits(folder, ids, stored_as=None):
         return plain.logits(cfg, w, list(ids))
 
 
+def assert_within_32_bit(folder, ids, got, ref, what=""):
+    """``got`` (an engine in 32-bit) against ``ref`` (the plain implementation in float64): the common 32-bit tolerance, or three
+    times what the plain implementation in 32-bit is off by where this model's own arithmetic is worse conditioned."""
+    import plain_pilonex as plain
+    from gpu_util import F32_REL
+    cfg, w = read_model(folder)
+    with plain.computed_in(torch.float32):
+        own = plain.logits(cfg, w, list(ids))
+    got = got.detach().double().cpu()
+    assert got.shape == ref.shape and torch.isfinite(got).all(), (what, got.shape, ref.shape)
+    bound = max(F32_REL * max(1.0, ref.abs().max().item()), 3.0 * (own.double()[:ref.shape[0]] - ref).abs().max().item())
+    err = (got - ref).abs().max().item()
+    assert err <= bound < 0.01 * ref.abs().max().item(), f"{what}: max err {err:.3e}, bound {bound:.3e}"
+
+
 def random_config(rng, small=True):
     """A configuration with random layer order, sizes and constants. ``small``: odd sizes, ones, sizes no kernel's fast path
     takes; else sizes of a small real model."""

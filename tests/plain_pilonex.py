@@ -4,6 +4,9 @@ the tests compare the engine with it.
 A model is ``(config dict, {tensor name: tensor})``. ``logits(cfg, w, ids)`` returns ``[len(ids), vocab]``;
 ``forward(cfg, w, ids)`` also returns the sum of the streams after every layer run (a looped layer counts every time).
 
+Computed in float64; ``with computed_in(torch.float32):`` the same statements in 32-bit, whose distance to the 64-bit result is what
+32-bit arithmetic alone does to a model (a head of one channel, normed, turns a small number into a sign).
+
 With a storage type set (``with stored_as(torch.bfloat16):``) every tensor that an engine keeps in that type between two
 operations is rounded to it; the distance to the unrounded result is what rounding alone does to the model's logits.
 """
@@ -26,6 +29,19 @@ class stored_as:
     def __exit__(self, *exc):
         global _STORED
         _STORED = self.before
+
+
+class computed_in:
+    def __init__(self, dtype):
+        self.dtype = dtype
+
+    def __enter__(self):
+        global F
+        self.before, F = F, self.dtype
+
+    def __exit__(self, *exc):
+        global F
+        F = self.before
 
 
 def kept(x):
