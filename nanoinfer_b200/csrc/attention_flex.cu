@@ -163,7 +163,9 @@ attention_prepare_kernel(const float* __restrict__ qkv, int ld, T* __restrict__ 
 // ---- the same for bfloat16 storage, eight elements a thread --------------------------------------------------------------
 // A block per token; a work item is eight consecutive elements of a head (two 16-byte loads of floats, one 16-byte store of
 // bfloat16), or, inside the rotated part of a q or k head, the eight elements at c and their mates at c + rot/2 together,
-// so that an angle's sine and cosine are formed once a pair. Takes: no norm or the norm over the whole projection, pairs
+// so that an angle's sine and cosine are formed once a pair. Takes: no norm, the norm over the whole projection, or the norm of
+// every head where a head is 16, 32, 64 or 128 wide (the sums of squares of all heads first, a quarter of a head's width in lanes
+// each), pairs
 // (i, i + rot/2) with rot a multiple of 16, head sizes in multiples of 8, values of their own (blended or not). The token's
 // page and slot are looked up once. Same arithmetic per element as the kernel above.
 __device__ __forceinline__ void load8(const float* p, float (&x)[8]) {
@@ -186,7 +188,8 @@ attention_prepare_vec_kernel(const float* __restrict__ qkv, int ld, __nv_bfloat1
                              const int* __restrict__ positions, const int* __restrict__ req_index, const int* __restrict__ block_table,
                              int bt_stride, int page_size, __nv_bfloat16* __restrict__ k_pages, __nv_bfloat16* __restrict__ v_pages, int num_pages,
                              int heads, int kv_heads, int dk, int dv, int writes, const float* __restrict__ v_first, int ld_first,
-                             const float* __restrict__ vmix) {
+                             const float* __restrict__ vmix, int per_head_norm) {
+    extern __shared__ float head_norm[];        // 1 / rms of every q, then every k head (norm of every head only)
     pdl_launch_dependents();
     pdl_wait();      // everything this kernel reads may come from the kernel before
     __shared__ float red[2][4];
@@ -194,7 +197,16 @@ attention_prepare_vec_kernel(const float* __restrict__ qkv, int ld, __nv_bfloat1
     const float* row = qkv + (size_t)t * ld;
     const int nq = heads * dk, nk = kv_heads * dk;
     float whole_q = 1.0f, whole_k = 1.0f;
-    if (q_gain != nullptr) {        // the norm over the whole projection: one sum of squares for q, one for k
+    if (q_gain != nullptr && per_head_norm) {
+        const int lanes = dk / 4;
+        for (int c = tid * 4; c < (((nq + nk) + 127) & ~127); c += 128 * 4) {      // whole warps take part in the exchanges
+            const float4 v = c < nq + nk ? *reinterpret_cast<const float4*>(row + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+            float ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w)));
+            for (int m = lanes >> 1; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+            if (c < nq + nk && c % dk == 0) head_norm[c / dk] = 1.0f / sqrtf(ss / (float)dk + eps);
+        }
+        __syncthreads();
+    } else if (q_gain != nullptr) {        // the norm over the whole projection: one sum of squares for q, one for k
         float sq = 0.f, sk = 0.f;
         for (int c = tid * 4; c < nq; c += 128 * 4) {
             const float4 v = *reinterpret_cast<const float4*>(row + c);
@@ -244,7 +256,8 @@ attention_prepare_vec_kernel(const float* __restrict__ qkv, int ld, __nv_bfloat1
         if (!is_q && slot < 0) continue;
         const float* src = row + (size_t)hq * dk;                // q heads and k heads lie one behind the other
         const float* gain = is_q ? q_gain : k_gain;
-        const float norm = is_q ? whole_q : whole_k;
+        const float norm = per_head_norm && gain != nullptr ? head_norm[hq] : (is_q ? whole_q : whole_k);
+        const int gain_at = per_head_norm ? 0 : head * dk;      // a head's gain is shared by the heads
         __nv_bfloat16* dst = is_q ? q_out + (size_t)t * nq + (size_t)head * dk
                                   : k_pages + ((size_t)slot + (size_t)head * page_size) * dk;
         if (w < half / 8) {                                     // eight rotated pairs: elements c.. and c + rot/2..
@@ -254,8 +267,8 @@ attention_prepare_vec_kernel(const float* __restrict__ qkv, int ld, __nv_bfloat1
             load8(src + c + half, b);
             if (gain != nullptr) {
                 float ga[8], gb[8];
-                load8(gain + (size_t)head * dk + c, ga);
-                load8(gain + (size_t)head * dk + c + half, gb);
+                load8(gain + gain_at + c, ga);
+                load8(gain + gain_at + c + half, gb);
 #pragma unroll
                 for (int e = 0; e < 8; ++e) { a[e] = a[e] * norm * ga[e]; b[e] = b[e] * norm * gb[e]; }
             }
@@ -277,7 +290,7 @@ attention_prepare_vec_kernel(const float* __restrict__ qkv, int ld, __nv_bfloat1
             load8(src + c, a);
             if (gain != nullptr) {
                 float ga[8];
-                load8(gain + (size_t)head * dk + c, ga);
+                load8(gain + gain_at + c, ga);
 #pragma unroll
                 for (int e = 0; e < 8; ++e) a[e] = a[e] * norm * ga[e];
             }
@@ -305,11 +318,12 @@ NIB_API int nib_attention_prepare(const float* qkv, int ld, void* q_out, const f
     const bool aligned16 = ((uintptr_t)qkv % 16 == 0) && ld % 4 == 0 && (uintptr_t)q_out % 16 == 0 && (!writes || ((uintptr_t)k_pages % 16 == 0 && (uintptr_t)v_pages % 16 == 0))
         && (q_gain == nullptr || ((uintptr_t)q_gain % 16 == 0 && (uintptr_t)k_gain % 16 == 0)) && (rot == 0 || (uintptr_t)freq % 16 == 0)
         && (v_first == nullptr || ((uintptr_t)v_first % 16 == 0 && ld_first % 4 == 0));
+    const bool head_norm = q_gain != nullptr && !(flags & FXP_NORM_WHOLE) && (dk == 16 || dk == 32 || dk == 64 || dk == 128);
     if (dtype == NIB_BF16 && tokens >= 256 && aligned16 && dk % 8 == 0 && dv % 8 == 0 && rot % 16 == 0 && (flags & ~FXP_NORM_WHOLE) == 0
-        && ((q_gain != nullptr) == ((flags & FXP_NORM_WHOLE) != 0))) {
-        NIB_CUDA(launch_pdl(attention_prepare_vec_kernel, dim3(tokens), dim3(128), (size_t)0, stream, qkv, ld, (__nv_bfloat16*)q_out, q_gain, k_gain, eps, freq,
+        && (q_gain == nullptr || (flags & FXP_NORM_WHOLE) || (head_norm && (heads + kv_heads) <= 8192))) {
+        NIB_CUDA(launch_pdl(attention_prepare_vec_kernel, dim3(tokens), dim3(128), head_norm ? (size_t)(heads + kv_heads) * 4 : (size_t)0, stream, qkv, ld, (__nv_bfloat16*)q_out, q_gain, k_gain, eps, freq,
                             rot, positions, req_index, block_table, bt_stride, page_size, (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, num_pages, heads,
-                            kv_heads, dk, dv, writes, v_first, ld_first, vmix));
+                            kv_heads, dk, dv, writes, v_first, ld_first, vmix, head_norm ? 1 : 0));
         NIB_LAUNCH_CHECK();
         return 0;
     }

@@ -372,7 +372,7 @@ group_walk_kernel(const float* __restrict__ work, const float* __restrict__ v, i
 #pragma unroll
             for (int i = 0; i < C; ++i) S[i] = fmaf(ks[t][i], x[t], S[i]);
         const float out = val + row_times(d0, d1, x);
-        if (writer && base + token < row1 && live) o[(size_t)(base + token) * ldo + (size_t)h * cols + j] = out;
+        if (writer && base + token < row1 && live) o[(size_t)(base + token) * ldo + (is_one ? (size_t)heads * dv + h : (size_t)h * dv + j)] = out;
     }
     pdl_launch_dependents();        // only now: blocks of the next kernel that became resident earlier would sit beside a long walk
     if (live) {
@@ -429,7 +429,7 @@ NIB_API int nib_grouped_state_error() {
 }
 
 // b [tokens, heads] (logits of beta): the delta rule; null: the plain rule. q, k: [tokens, kq_heads * dk]; z: [tokens, heads * dk] or
-// [tokens, heads] (GS_HEAD); v: [tokens, heads * dv], o: [tokens, heads * (dv + ones)]; all floats with row strides. unit_eps >= 0:
+// [tokens, heads] (GS_HEAD); v: [tokens, heads * dv], o: [tokens, heads * dv], with ones another heads columns behind them; all floats with row strides. unit_eps >= 0:
 // q and k are made unit vectors here (x / sqrt(sum x^2 + unit_eps)); queries times q_scale; k_scale [tokens, heads] or null: a factor
 // on the keys. ones 1: the state has one more value channel whose value is 1. longest: the most tokens a request brings.
 NIB_API int nib_grouped_state_scan(const float* q, int ldq, const float* k, int ldk, const float* v, int ldv, const float* z, int ldz, int z_kind,

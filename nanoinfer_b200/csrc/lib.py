@@ -870,8 +870,8 @@ class Kernels:
         divided by the root mean square of each of ``groups`` equal parts (``eps`` inside the root); times ``gain32`` (a gain
         per channel, or one of a part's size shared by the parts); times act(gate32) if not ``gate_first``; times
         ``out_scale``. gate_kind: 'none' | 'sigmoid' | 'silu'. ``skip_coef32`` holds one coefficient per head. With ``floor32``
-        [tokens, groups] every part of o32 is one number wider than a part of ``out``: its last number d is no channel but a
-        divisor, y = o32 / (max(|d|, floor32) + den_eps) comes first."""
+        [tokens, groups] the rows of o32 hold ``groups`` more numbers d behind the channels, a divisor per part:
+        y = o32 / (max(|d|, floor32) + den_eps) comes first."""
         self._rows(o32, torch.float32, "gated_norm o"); self._rows(out, None, "gated_norm out")
         m, n = out.shape
         if tuple(o32.shape) != (m, n if floor32 is None else n + groups):
@@ -993,8 +993,8 @@ class Kernels:
         ``rate32`` [heads] and ``dt_bias32`` [heads * dk] the logits of step sizes, w = exp(-rate32 * softplus(z32 + dt_bias32)); or
         [tokens, heads], one decay per head. ``unit_eps``: q and k become unit vectors per head (x / sqrt(sum x^2 + unit_eps));
         queries are then multiplied by ``q_scale``, keys by ``k_scale32`` [tokens, heads]. With ``ones`` a head has one value channel
-        more, behind the others, whose value is 1: the state holds heads * (dv + 1) * dk floats, o32 is [tokens, heads * (dv + 1)].
-        How a request is cut moves the result by rounding."""
+        more, behind the others, whose value is 1: the state holds heads * (dv + 1) * dk floats, o32 is [tokens, heads * dv + heads], that
+        channel's outputs of all heads behind the others. How a request is cut moves the result by rounding."""
         extra = 1 if ones else 0
         m = q32.shape[0]
         for t, what, width in ((q32, "q", kq_heads * dk), (k32, "k", kq_heads * dk), (v32, "v", heads * dv), (o32, "o", heads * (dv + extra))):

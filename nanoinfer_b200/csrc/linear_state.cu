@@ -346,6 +346,63 @@ conv_tokens_kernel(const float* __restrict__ x, int ldx, const float* __restrict
     y[(size_t)t * ldy + c] = acc;
 }
 
+// The same, four channels and eight consecutive tokens a thread: the inputs of a token's window slide through registers, so
+// every input is read once a thread. Up to CONV_VEC_TAPS taps; the same arithmetic per output (taps in ascending order from the
+// bias).
+constexpr int CONV_VEC_TAPS = 8, CONV_VEC_TOKENS = 8;
+
+template <int TAPS>
+__global__ void __launch_bounds__(128)
+conv_tokens_vec_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ w, const float* __restrict__ bias, int act,
+                       const float* __restrict__ state, long long state_ld, int state_off, const int* __restrict__ q_start,
+                       const int* __restrict__ req_index, const int* __restrict__ slots, float* __restrict__ y, int ldy,
+                       int tokens, int width) {
+    pdl_launch_dependents();
+    const int c = (blockIdx.y * 128 + threadIdx.x) * 4, t0 = blockIdx.x * CONV_VEC_TOKENS, t1 = min(tokens, t0 + CONV_VEC_TOKENS);
+    if (c >= width) return;
+    float wt[4][TAPS], b[4];        // weights: no kernel writes them
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+        b[e] = bias != nullptr ? bias[c + e] : 0.f;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) wt[e][j] = w[(size_t)(c + e) * TAPS + j];
+    }
+    pdl_wait();      // everything else this kernel reads may come from the kernel before
+    float4 win[TAPS > 1 ? TAPS - 1 : 1];
+    int request = -1;
+    for (int t = t0; t < t1; ++t) {
+        const int r = req_index[t];
+        if (r != request) {     // the first token of the thread, or of a request: its window from the rows before it, or from the history
+            request = r;
+            const int first = q_start[r], i = t - first;
+            const float* hist = TAPS > 1 ? state + (long long)slots[r] * state_ld + state_off : nullptr;
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; ++j) {
+                const int s = i - (TAPS - 1) + j;
+                const float* from = s >= 0 ? x + (size_t)(first + s) * ldx + c : hist + (size_t)(TAPS - 1 + s) * width + c;
+                if (s >= 0) win[j] = *reinterpret_cast<const float4*>(from);
+                else win[j] = make_float4(from[0], from[1], from[2], from[3]);
+            }
+        }
+        const float4 u = *reinterpret_cast<const float4*>(x + (size_t)t * ldx + c);
+        float acc[4] = {b[0], b[1], b[2], b[3]};
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) {
+            const float4 v = j < TAPS - 1 ? win[TAPS > 1 ? (j < TAPS - 1 ? j : 0) : 0] : u;
+            acc[0] = fmaf(wt[0][j], v.x, acc[0]); acc[1] = fmaf(wt[1][j], v.y, acc[1]);
+            acc[2] = fmaf(wt[2][j], v.z, acc[2]); acc[3] = fmaf(wt[3][j], v.w, acc[3]);
+        }
+        if (act == 1) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) acc[e] = acc[e] / (1.0f + expf(-acc[e]));
+        }
+        *reinterpret_cast<float4*>(y + (size_t)t * ldy + c) = make_float4(acc[0], acc[1], acc[2], acc[3]);
+#pragma unroll
+        for (int j = 0; j < TAPS - 2; ++j) win[j] = win[j + 1];
+        if (TAPS > 1) win[TAPS > 1 ? TAPS - 2 : 0] = u;
+    }
+}
+
 // The history rows become the request's last taps-1 inputs (old rows move up when the step brought fewer). One thread
 // per (request, channel); row i is written after rows >= i were read, so the move is safe in place.
 __global__ void __launch_bounds__(256)
@@ -369,6 +426,16 @@ NIB_API int nib_conv_tokens(const float* x, int ldx, const float* w, const float
                             int width, int taps, cudaStream_t stream) {
     NIB_REQUIRE(tokens >= 0 && width > 0 && taps >= 1 && (taps == 1 || state != nullptr), "conv_tokens: bad sizes or no state for %d taps", taps);
     if (tokens == 0) return 0;
+    if (taps <= CONV_VEC_TAPS && width % 4 == 0 && ldx % 4 == 0 && ldy % 4 == 0 && (((uintptr_t)x | (uintptr_t)y) & 15) == 0) {
+        const dim3 grid(ceil_div(tokens, CONV_VEC_TOKENS), ceil_div(width, 512));
+#define NIB_CV(TAPS) \
+    case TAPS: NIB_CUDA(launch_pdl(conv_tokens_vec_kernel<TAPS>, grid, dim3(128), (size_t)0, stream, x, ldx, w, bias, act, state, state_ld, state_off, \
+                                   q_start, req_index, slots, y, ldy, tokens, width)); break;
+        switch (taps) { NIB_CV(1) NIB_CV(2) NIB_CV(3) NIB_CV(4) NIB_CV(5) NIB_CV(6) NIB_CV(7) NIB_CV(8) }
+#undef NIB_CV
+        NIB_LAUNCH_CHECK();
+        return 0;
+    }
     NIB_CUDA(launch_pdl(conv_tokens_kernel, dim3(ceil_div((long long)tokens * width, 256)), dim3(256), (size_t)0, stream, x, ldx, w, bias, act,
                         state, state_ld, state_off, q_start, req_index, slots, y, ldy, tokens, width, taps));
     NIB_LAUNCH_CHECK();

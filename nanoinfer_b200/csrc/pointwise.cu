@@ -397,8 +397,8 @@ NIB_API int nib_depth_mix_norm_pair(float* hist, float* x, const float* coef, in
 
 // ---------------------------------------------------------------------------------- gate, norm in groups, skip
 // For a row o of n floats cut into `groups` equal parts (a warp per (token, part)):
-//     y = o / (max(|den|, floor) + den_eps)             with `floor`: den is the number behind the part's channels in o (the
-//                                                       parts of o then lie width + 1 apart), floor one number per (token, part)
+//     y = o / (max(|den|, floor) + den_eps)             with `floor`: den is the part's number behind ALL channels
+//                                                       of the row of o, floor one number per (token, part)
 //     y = y (+ coef[c / (n / n_coef)] * skip)          a skip connection with one coefficient per head
 //     y = y * act(gate)                                 if gate_first
 //     y = y / sqrt(mean_part(y^2) + eps)                if norm
@@ -423,8 +423,8 @@ gated_norm_kernel(const float* __restrict__ o, int ldo, const float* __restrict_
     const int lane = threadIdx.x & 31;
     if (w >= (long long)tokens * groups) return;
     const int t = (int)(w / groups), part_i = (int)(w % groups), c0 = part_i * width;
-    const float* orow = o + (size_t)t * ldo + (floor_in != nullptr ? part_i : 0);      // (a divisor behind every part)
-    const float den = floor_in != nullptr ? fmaxf(fabsf(orow[c0 + width]), floor_in[(size_t)t * ldf + part_i]) + den_eps : 1.0f;
+    const float* orow = o + (size_t)t * ldo;
+    const float den = floor_in != nullptr ? fmaxf(fabsf(orow[groups * width + part_i]), floor_in[(size_t)t * ldf + part_i]) + den_eps : 1.0f;
     const float* grow = gate != nullptr ? gate + (size_t)t * ldg : nullptr;
     const float* srow = skip != nullptr ? skip + (size_t)t * lds : nullptr;
     const bool early = grow != nullptr && gate_kind != 0 && gate_first != 0;
@@ -466,8 +466,8 @@ gated_norm_block_kernel(const float* __restrict__ o, int ldo, const float* __res
     pdl_wait();      // everything this kernel reads may come from the kernel before
     __shared__ float part[8];
     const int t = blockIdx.x / groups, part_i = blockIdx.x % groups, c0 = part_i * width;
-    const float* orow = o + (size_t)t * ldo + (floor_in != nullptr ? part_i : 0);      // (a divisor behind every part)
-    const float den = floor_in != nullptr ? fmaxf(fabsf(orow[c0 + width]), floor_in[(size_t)t * ldf + part_i]) + den_eps : 1.0f;
+    const float* orow = o + (size_t)t * ldo;
+    const float den = floor_in != nullptr ? fmaxf(fabsf(orow[groups * width + part_i]), floor_in[(size_t)t * ldf + part_i]) + den_eps : 1.0f;
     const float* grow = gate != nullptr ? gate + (size_t)t * ldg : nullptr;
     const float* srow = skip != nullptr ? skip + (size_t)t * lds : nullptr;
     const bool early = grow != nullptr && gate_kind != 0 && gate_first != 0;
@@ -496,6 +496,49 @@ gated_norm_block_kernel(const float* __restrict__ o, int ldo, const float* __res
     }
 }
 
+// The same for parts of 16, 32, 64 or 128 channels without a skip and with the gate (if any) behind the norm: LPP = width / 4
+// lanes a part, four channels a lane, held in registers between the sum of squares and the result.
+template <typename T, int LPP>
+__global__ void __launch_bounds__(128)
+gated_norm_vec_kernel(const float* __restrict__ o, int ldo, const float* __restrict__ gate, int ldg, int gate_kind, const float* __restrict__ gain,
+                      int gain_len, float eps, float out_scale, T* __restrict__ out, int ld_out, int tokens, int groups,
+                      const float* __restrict__ floor_in, int ldf, float den_eps) {
+    constexpr int WIDTH = 4 * LPP;
+    pdl_launch_dependents();
+    pdl_wait();      // everything this kernel reads may come from the kernel before
+    const long long p = ((long long)blockIdx.x * 128 + threadIdx.x) / LPP;
+    const int sub = threadIdx.x % LPP;
+    const bool live = p < (long long)tokens * groups;
+    const int t = live ? (int)(p / groups) : 0, part_i = live ? (int)(p % groups) : 0, c = part_i * WIDTH + sub * 4;
+    float4 y = *reinterpret_cast<const float4*>(o + (size_t)t * ldo + c);
+    float4 gv = make_float4(0.f, 0.f, 0.f, 0.f), ga = make_float4(1.f, 1.f, 1.f, 1.f);
+    if (gate != nullptr) gv = *reinterpret_cast<const float4*>(gate + (size_t)t * ldg + c);
+    if (gain != nullptr) ga = __ldg(reinterpret_cast<const float4*>(gain + c % gain_len));
+    if (floor_in != nullptr) {
+        const float den = fmaxf(fabsf(o[(size_t)t * ldo + groups * WIDTH + part_i]), floor_in[(size_t)t * ldf + part_i]) + den_eps;
+        y.x /= den; y.y /= den; y.z /= den; y.w /= den;
+    }
+    float ss = fmaf(y.x, y.x, fmaf(y.y, y.y, fmaf(y.z, y.z, y.w * y.w)));
+#pragma unroll
+    for (int m = LPP / 2; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+    const float scale = 1.0f / sqrtf(ss / (float)WIDTH + eps);
+    float v[4] = {y.x * scale * ga.x, y.y * scale * ga.y, y.z * scale * ga.z, y.w * scale * ga.w};
+    if (gate != nullptr && gate_kind != 0) {
+        v[0] *= gate_act(gv.x, gate_kind); v[1] *= gate_act(gv.y, gate_kind); v[2] *= gate_act(gv.z, gate_kind); v[3] *= gate_act(gv.w, gate_kind);
+    }
+    if (!live) return;
+    T* to = out + (size_t)t * ld_out + c;
+    if constexpr (sizeof(T) == 4) {
+        *reinterpret_cast<float4*>(to) = make_float4(v[0] * out_scale, v[1] * out_scale, v[2] * out_scale, v[3] * out_scale);
+    } else {
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0] * out_scale, v[1] * out_scale), hi = __floats2bfloat162_rn(v[2] * out_scale, v[3] * out_scale);
+        uint2 pk;
+        pk.x = *reinterpret_cast<const unsigned*>(&lo);
+        pk.y = *reinterpret_cast<const unsigned*>(&hi);
+        *reinterpret_cast<uint2*>(to) = pk;
+    }
+}
+
 NIB_API int nib_gated_norm(const float* o, int ldo, const float* gate, int ldg, int gate_kind, int gate_first, const float* gain,
                            int gain_len, const float* skip, int lds, const float* coef, int n_coef, int groups, int norm, float eps,
                            float out_scale, void* out, int ld_out, int tokens, int n, int dtype, const float* floor_in, int ldf, float den_eps, cudaStream_t stream) {
@@ -505,6 +548,20 @@ NIB_API int nib_gated_norm(const float* o, int ldo, const float* gate, int ldg, 
     NIB_REQUIRE(gate_kind >= 0 && gate_kind <= 2, "gated_norm: unknown gate kind %d", gate_kind);
     if (tokens == 0) return 0;
     const int width = n / groups, span = skip != nullptr ? n / n_coef : 1;
+    const bool rows16 = (((uintptr_t)o | (uintptr_t)gate | (uintptr_t)gain | (uintptr_t)out) & 15) == 0 && ldo % 4 == 0 && ldg % 4 == 0
+        && (ld_out * (dtype == NIB_F32 ? 4 : 2)) % 8 == 0 && (gain == nullptr || gain_len % 4 == 0);
+    if (norm && skip == nullptr && (gate == nullptr || !gate_first) && rows16 && (width == 16 || width == 32 || width == 64 || width == 128)
+        && (dtype == NIB_F32 || dtype == NIB_BF16)) {
+        const dim3 grid(ceil_div((long long)tokens * groups * (width / 4), 128));
+#define NIB_GV(T, LPP) NIB_CUDA(launch_pdl(gated_norm_vec_kernel<T, LPP>, grid, dim3(128), (size_t)0, stream, o, ldo, gate, ldg, gate_kind, gain, gain_len, eps, \
+                                           out_scale, (T*)out, ld_out, tokens, groups, floor_in, ldf, den_eps))
+#define NIB_GW(T) do { if (width == 16) NIB_GV(T, 4); else if (width == 32) NIB_GV(T, 8); else if (width == 64) NIB_GV(T, 16); else NIB_GV(T, 32); } while (0)
+        if (dtype == NIB_F32) NIB_GW(float); else NIB_GW(__nv_bfloat16);
+#undef NIB_GW
+#undef NIB_GV
+        NIB_LAUNCH_CHECK();
+        return 0;
+    }
     if (width > 256) {
         const dim3 grid(tokens * groups);
         if (dtype == NIB_F32) NIB_CUDA(launch_pdl(gated_norm_block_kernel<float>, grid, dim3(256), (size_t)(0), stream, o, ldo, gate, ldg, gate_kind, gate_first, gain, gain_len, skip, lds, coef, span, norm, eps, out_scale, (float*)out, ld_out, tokens, groups, width, floor_in, ldf, den_eps));
@@ -698,10 +755,12 @@ NIB_API int nib_moe_identity(const void* h, int ldh, const int* sel_e, const flo
 //     u = sum_s in[s] z_s                         what the next sublayer reads, then h = u / sqrt(mean(u^2) + eps) * gain.
 // Without `y` z = x (the first sublayer); x is read with strides of its own (all streams equal at the start: stream stride
 // 0); `dst` takes z as [row, stream, width] (may be x itself), `sum_out` takes sum_s z_s (may be x of one stream), `h_out` takes h in
-// T; with `clear` y is left zeroed. NS: streams known at compile time, 0: up to SM_MAX. V: elements a load.
+// T; with `clear` y is left zeroed. NS: streams known at compile time (their factors then sit in registers), 0: up to SM_MAX.
+// V: elements a load. IT: how many times a thread comes round in a row, its part of u then stays in registers; 0: any, u in
+// shared memory.
 constexpr int SM_MAX = 16;
 
-template <typename T, int NS, int V>
+template <typename T, int NS, int V, int IT>
 __global__ void __launch_bounds__(256)
 stream_mix_kernel(const float* x, long long x_row, long long x_stream, float* y, const float* __restrict__ mix, const float* __restrict__ out,
                   float* dst, const float* __restrict__ in, const float* __restrict__ gain, float eps, T* __restrict__ h_out, float* sum_out,
@@ -709,17 +768,21 @@ stream_mix_kernel(const float* x, long long x_row, long long x_stream, float* y,
     constexpr int N = NS > 0 ? NS : SM_MAX;
     constexpr int UNROLL = NS > 0 ? NS : 1;     // many streams: plain loops over a thread's own array
     extern __shared__ __align__(16) float sm_row[];         // u of the row: every thread reads back what it wrote itself
-    __shared__ float s_mix[N * N], s_out[N], s_in[N], part[8];
+    __shared__ float part[8];
     const int n = NS > 0 ? NS : n_rt, tid = threadIdx.x;
     pdl_launch_dependents();
-    for (int i = tid; i < n * n; i += blockDim.x) s_mix[i] = mix != nullptr ? mix[i] : 0.f;     // weights: no kernel writes them
-    for (int i = tid; i < n; i += blockDim.x) { s_out[i] = out != nullptr ? out[i] : 0.f; s_in[i] = in != nullptr ? in[i] : 0.f; }
-    __syncthreads();
-    pdl_wait();
-    const size_t row = blockIdx.x;
-    const float* xr = x + row * x_row;
-    float* yr = y != nullptr ? y + row * width : nullptr;
-    float ss = 0.f;
+    float f_mix[N * N], f_out[N], f_in[N];      // weights: no kernel writes them
+#pragma unroll UNROLL
+    for (int s = 0; s < N; ++s) {
+        if (s >= n) break;
+        f_out[s] = out != nullptr ? __ldg(out + s) : 0.f;
+        f_in[s] = in != nullptr ? __ldg(in + s) : 0.f;
+#pragma unroll UNROLL
+        for (int t = 0; t < N; ++t) {
+            if (t >= n) break;
+            f_mix[s * N + t] = mix != nullptr ? __ldg(mix + s * n + t) : 0.f;
+        }
+    }
     auto load = [](const float* p, float (&v)[V]) {
         if constexpr (V == 4) { const float4 a = *reinterpret_cast<const float4*>(p); v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; }
         else v[0] = *p;
@@ -728,8 +791,20 @@ stream_mix_kernel(const float* x, long long x_row, long long x_stream, float* y,
         if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
         else *p = v[0];
     };
-    for (int c = tid * V; c < width; c += blockDim.x * V) {
-        float xv[N][V], yv[V];
+    const int stride = blockDim.x * V;
+    float held[IT > 0 ? IT : 1][V], g[IT > 0 ? IT : 1][V];
+    if constexpr (IT > 0) {
+#pragma unroll
+        for (int i = 0; i < IT; ++i)
+            if (h_out != nullptr && tid * V + i * stride < width) load(gain + tid * V + i * stride, g[i]);
+    }
+    pdl_wait();
+    const size_t row = blockIdx.x;
+    const float* xr = x + row * x_row;
+    float* yr = y != nullptr ? y + row * width : nullptr;
+    float ss = 0.f;
+    auto one = [&](int c, float (&u)[V]) {
+        float xv[N][V], yv[V], total[V] = {};
 #pragma unroll UNROLL
         for (int s = 0; s < N; ++s) {
             if (s >= n) break;
@@ -742,7 +817,8 @@ stream_mix_kernel(const float* x, long long x_row, long long x_stream, float* y,
                 store(yr + c, zero);
             }
         }
-        float u[V] = {}, total[V] = {};
+#pragma unroll
+        for (int e = 0; e < V; ++e) u[e] = 0.f;
 #pragma unroll UNROLL
         for (int t = 0; t < N; ++t) {
             if (t >= n) break;
@@ -750,26 +826,34 @@ stream_mix_kernel(const float* x, long long x_row, long long x_stream, float* y,
 #pragma unroll
             for (int e = 0; e < V; ++e) {
                 if (yr != nullptr) {
-                    float a = s_out[t] * yv[e];
+                    float a = f_out[t] * yv[e];
 #pragma unroll UNROLL
                     for (int s = 0; s < N; ++s) {
                         if (s >= n) break;
-                        a = fmaf(s_mix[s * n + t], xv[s][e], a);
+                        a = fmaf(f_mix[s * N + t], xv[s][e], a);
                     }
                     z[e] = a;
                 } else {
                     z[e] = xv[t][e];
                 }
-                u[e] = fmaf(s_in[t], z[e], u[e]);
+                u[e] = fmaf(f_in[t], z[e], u[e]);
                 total[e] += z[e];
             }
             if (dst != nullptr) store(dst + (row * n + t) * width + c, z);
         }
         if (sum_out != nullptr) store(sum_out + row * width + c, total);
-        if (h_out != nullptr) {
-            store(sm_row + c, u);
 #pragma unroll
-            for (int e = 0; e < V; ++e) ss = fmaf(u[e], u[e], ss);
+        for (int e = 0; e < V; ++e) ss = fmaf(u[e], u[e], ss);
+    };
+    if constexpr (IT > 0) {
+#pragma unroll
+        for (int i = 0; i < IT; ++i)
+            if (tid * V + i * stride < width) one(tid * V + i * stride, held[i]);
+    } else {
+        for (int c = tid * V; c < width; c += stride) {
+            float u[V];
+            one(c, u);
+            if (h_out != nullptr) store(sm_row + c, u);
         }
     }
     if (h_out == nullptr) return;
@@ -779,38 +863,47 @@ stream_mix_kernel(const float* x, long long x_row, long long x_stream, float* y,
     ss = 0.f;
     for (int w = 0; w < (int)(blockDim.x >> 5); ++w) ss += part[w];        // the same order in every thread
     const float scale = 1.0f / sqrtf(ss / (float)width + eps);
-    for (int c = tid * V; c < width; c += blockDim.x * V) {
-        float u[V], g[V];
-        load(sm_row + c, u);
-        load(gain + c, g);
-#pragma unroll
-        for (int e = 0; e < V; ++e) u[e] = u[e] * scale * g[e];
+    auto emit = [&](int c, const float (&u)[V], const float (&gv)[V]) {
         T* ho = h_out + row * width + c;
         if constexpr (V == 4 && sizeof(T) == 2) {
-            const __nv_bfloat162 lo = __floats2bfloat162_rn(u[0], u[1]), hi = __floats2bfloat162_rn(u[2], u[3]);
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(u[0] * scale * gv[0], u[1] * scale * gv[1]);
+            const __nv_bfloat162 hi = __floats2bfloat162_rn(u[2] * scale * gv[2], u[3] * scale * gv[3]);
             uint2 pk;
             pk.x = *reinterpret_cast<const unsigned*>(&lo);
             pk.y = *reinterpret_cast<const unsigned*>(&hi);
             *reinterpret_cast<uint2*>(ho) = pk;
         } else {
 #pragma unroll
-            for (int e = 0; e < V; ++e) Elem<T>::store(ho + e, u[e]);
+            for (int e = 0; e < V; ++e) Elem<T>::store(ho + e, u[e] * scale * gv[e]);
+        }
+    };
+    if constexpr (IT > 0) {
+#pragma unroll
+        for (int i = 0; i < IT; ++i)
+            if (tid * V + i * stride < width) emit(tid * V + i * stride, held[i], g[i]);
+    } else {
+        for (int c = tid * V; c < width; c += stride) {
+            float u[V], gv[V];
+            load(sm_row + c, u);
+            load(gain + c, gv);
+            emit(c, u, gv);
         }
     }
 }
 
-template <typename T, int NS, int V>
+template <typename T, int NS, int V, int IT>
 static int launch_stream_mix(const float* x, long long x_row, long long x_stream, float* y, const float* mix, const float* out, float* dst,
                              const float* in, const float* gain, float eps, void* h_out, float* sum_out, int rows, int width, int n, int clear,
                              cudaStream_t stream) {
-    const size_t smem = h_out != nullptr ? (size_t)width * 4 : 0;
+    const size_t smem = h_out != nullptr && IT == 0 ? (size_t)width * 4 : 0;
     static size_t configured = 48 * 1024;
     if (smem > configured) {
-        NIB_CUDA(cudaFuncSetAttribute(stream_mix_kernel<T, NS, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        NIB_CUDA(cudaFuncSetAttribute(stream_mix_kernel<T, NS, V, IT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         configured = smem;
     }
-    const int threads = rows <= 64 && width >= 1024 ? 256 : 128;
-    NIB_CUDA(launch_pdl(stream_mix_kernel<T, NS, V>, dim3(rows), dim3(threads), smem, stream, x, x_row, x_stream, y, mix, out, dst, in, gain, eps,
+    // enough threads for a row in IT turns, whole warps
+    const int threads = IT > 0 ? ((ceil_div(width, V * IT) + 31) / 32) * 32 : 256;
+    NIB_CUDA(launch_pdl(stream_mix_kernel<T, NS, V, IT>, dim3(rows), dim3(threads), smem, stream, x, x_row, x_stream, y, mix, out, dst, in, gain, eps,
                         (T*)h_out, sum_out, width, n, clear));
     return 0;
 }
@@ -825,9 +918,9 @@ NIB_API int nib_stream_mix(const float* x, long long x_row, long long x_stream, 
     if (rows == 0) return 0;
     const uintptr_t all = (uintptr_t)x | (uintptr_t)y | (uintptr_t)dst | (uintptr_t)gain | (uintptr_t)h_out | (uintptr_t)sum_out;
     const bool vec = width % 4 == 0 && (all & 15) == 0 && x_row % 4 == 0 && x_stream % 4 == 0;
-#define NIB_SM3(T, NS, V) return launch_stream_mix<T, NS, V>(x, x_row, x_stream, y, mix, out, dst, in, gain, eps, h_out, sum_out, rows, width, n, clear, stream)
-#define NIB_SM2(T, NS) do { if (vec) NIB_SM3(T, NS, 4); else NIB_SM3(T, NS, 1); } while (0)
-#define NIB_SM(T) do { switch (n) { case 1: NIB_SM2(T, 1); case 2: NIB_SM2(T, 2); case 3: NIB_SM2(T, 3); case 4: NIB_SM2(T, 4); default: NIB_SM3(T, 0, 1); } } while (0)
+#define NIB_SM3(T, NS, V, IT) return launch_stream_mix<T, NS, V, IT>(x, x_row, x_stream, y, mix, out, dst, in, gain, eps, h_out, sum_out, rows, width, n, clear, stream)
+#define NIB_SM2(T, NS) do { if (!vec) NIB_SM3(T, NS, 1, 0); if (width <= 1024) NIB_SM3(T, NS, 4, 1); if (width <= 2048) NIB_SM3(T, NS, 4, 2); NIB_SM3(T, NS, 4, 0); } while (0)
+#define NIB_SM(T) do { switch (n) { case 1: NIB_SM2(T, 1); case 2: NIB_SM2(T, 2); case 3: NIB_SM2(T, 3); case 4: NIB_SM2(T, 4); default: NIB_SM3(T, 0, 1, 0); } } while (0)
     if (dtype == NIB_F32) NIB_SM(float);
     NIB_SM(__nv_bfloat16);
 #undef NIB_SM

@@ -133,11 +133,11 @@ def test_gates_keep_a_running_maximum_across_steps(ops, heads, cap):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("m,heads,d", [(5, 3, 20), (3, 2, 300), (40, 1, 7)])
+@pytest.mark.parametrize("m,heads,d", [(5, 3, 20), (3, 2, 300), (40, 1, 7), (9, 4, 64), (33, 2, 128), (7, 5, 16)])
 def test_norm_of_a_part_behind_its_divisor(ops, dtype, m, heads, d):
-    """The number behind a part divides it (its size, or the floor where that is larger, plus a small constant)."""
+    """A part's number behind the channels divides it (its size, or the floor where that is larger, plus a small constant)."""
     o, gate = rnd(m, heads * (d + 1), seed=1), rnd(m, heads * d, seed=2)
-    o[:, d] = 1e-7
+    o[:, heads * d] = 1e-7
     floor = torch.rand(m, heads, generator=torch.Generator().manual_seed(3)).to(DEV) * 1.5
     kw = dict(groups=heads, eps=1e-5, gain32=rnd(heads * d, seed=4), gate32=gate, gate_kind="sigmoid", out_scale=0.7, floor32=floor, den_eps=1e-6)
     out, ref = torch.empty(m, heads * d, dtype=dtype, device=DEV), torch.empty(m, heads * d, dtype=torch.float64)

@@ -223,9 +223,8 @@ class TorchOps:
         m, n = out.shape
         y = o32.double()
         if floor32 is not None:
-            y = y.view(m, groups, n // groups + 1)
-            den = torch.maximum(y[..., -1:].abs(), floor32.double()[..., None]) + den_eps
-            y = (y[..., :-1] / den).reshape(m, n)
+            den = torch.maximum(y[:, n:].abs(), floor32.double()) + den_eps
+            y = (y[:, :n].view(m, groups, n // groups) / den[..., None]).reshape(m, n)
         if skip32 is not None:
             y = y + skip32.double() * skip_coef32.double().repeat_interleave(n // skip_coef32.numel())
         act = {"sigmoid": torch.sigmoid, "silu": lambda z: z * torch.sigmoid(z)}.get(gate_kind)
@@ -364,7 +363,8 @@ class TorchOps:
                 if beta32 is not None:
                     u = torch.sigmoid(beta32[t].double())[:, None] * (u - torch.einsum("hkv,hk->hv", s, k[t]))
                 s = s + k[t][:, :, None] * u[:, None, :]
-                o32[t] = torch.einsum("hkv,hk->hv", s, q[t]).reshape(-1).to(torch.float32)
+                o = torch.einsum("hkv,hk->hv", s, q[t])
+                o32[t] = (torch.cat([o[:, :-1].reshape(-1), o[:, -1]]) if ones else o.reshape(-1)).to(torch.float32)
             flat.copy_(s.transpose(1, 2).reshape(-1).to(torch.float32))
             start += q_len
 
