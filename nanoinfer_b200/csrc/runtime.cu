@@ -33,7 +33,19 @@ NIB_API int nib_sm_count() {
 
 // Programmatic dependent launch of the decode kernels: on unless switched off (nib_set_pdl(0)).
 static int g_pdl = 1;
-bool nib_pdl_enabled() { return g_pdl != 0; }
+static thread_local bool g_pdl_skip = false;     // the next launch is a plain one
+
+bool nib_pdl_enabled() {
+    const bool skip = g_pdl_skip;
+    g_pdl_skip = false;
+    return g_pdl != 0 && !skip;
+}
+
+// The next launch of this thread gets no programmatic dependency: what it depends on lies in two streams.
+NIB_API int nib_pdl_skip_next() {
+    g_pdl_skip = true;
+    return 0;
+}
 NIB_API void nib_set_pdl(int on) { g_pdl = on; }
 
 // cuTensorMapEncodeTiled, looked up once through the runtime; nullptr if this driver does not offer it.

@@ -248,6 +248,30 @@ class Mixer(Part):
         raise NotImplementedError
 
 
+class ProjectedMixer(Mixer):
+    """A mixer of the form product -> mix -> product: one product of everything that reads the normed input (``take_input``),
+    ``mix`` from its 32-bit rows to the rows that enter the output product, and that product (``w_o``, ``b_o``), added to the
+    stream. A pair of such mixers can make one input product for both (``joint_input``)."""
+
+    b_o: Optional[torch.Tensor] = None
+
+    def take_input(self, rows: torch.Tensor, bias: Optional[torch.Tensor], joint: bool) -> None:
+        """The input product's matrix as stored and its bias; with ``joint`` both stay where they are for the pair to join."""
+        self.in_width = rows.shape[0]
+        self.in_rows, self.in_bias = (rows, bias) if joint else (None, None)
+        self.w_in = None if joint else self.rt.matrix(rows)
+        self.b_in = self.rt.vector32(bias) if bias is not None and not joint else None
+
+    def mix(self, p32: torch.Tensor, ctx: StepContext, cache: LayerCache) -> torch.Tensor:
+        raise NotImplementedError
+
+    def forward(self, h: torch.Tensor, residual32: torch.Tensor, ctx: StepContext, cache: LayerCache) -> None:
+        h = as_tensor(h)
+        p32 = torch.empty((h.shape[0], self.in_width), dtype=torch.float32, device=h.device)
+        self.ops.linear(h, self.w_in, self.b_in, p32, "f32")
+        self.ops.linear(self.mix(p32, ctx, cache), self.w_o, self.b_o, residual32, "add")
+
+
 class FeedForward(Part):
     def forward(self, h: torch.Tensor, residual32: torch.Tensor, ctx: StepContext) -> None:
         raise NotImplementedError

@@ -29,7 +29,7 @@ from typing import Dict
 import torch
 
 from ..registry import register_part
-from .base import LayerCache, Mixer, Runtime, StateNeed, StepContext, as_tensor
+from .base import LayerCache, Mixer, ProjectedMixer, Runtime, StateNeed, StepContext
 from .spec import PartSpec, TensorSpec
 
 
@@ -87,8 +87,9 @@ class GeneralizedDeltaRule(Mixer):
         ops.linear(gated, self.w_o, None, residual32, "add")
 
 
-class GatedDeltaRule(Mixer):
-    """params: ``hidden heads kv_heads dim vdim conv decay_rank gate_rank eps out_scale``. tensors: ``q k [kv_heads*dim, hidden]``,
+class GatedDeltaRule(ProjectedMixer):
+    """params: ``hidden heads kv_heads dim vdim conv decay_rank gate_rank eps out_scale``, optionally ``joint_input``.
+    tensors: ``q k [kv_heads*dim, hidden]``,
     ``v [heads*vdim, hidden]``, ``q_conv k_conv v_conv [channels, conv]`` (last column = the current token), ``b [heads, hidden]``,
     ``a1 [decay_rank, hidden]``, ``a2 [heads*dim, decay_rank]``, ``A_log [heads]``, ``dt_bias [heads*dim]``, ``g1 [gate_rank, hidden]``,
     ``g2 [heads*vdim, gate_rank]``, ``norm [vdim]``, ``o [hidden, heads*vdim]``."""
@@ -129,8 +130,8 @@ class GatedDeltaRule(Mixer):
         fill = lambda n: torch.zeros((n, self.hidden), dtype=tensors["b"].dtype)
         self.b_col = self.n_conv + self.inner
         rows = [tensors[x] for x in ("q", "k", "v", "a1", "g1")] + [fill(self.inner - ra - rg), tensors["b"]]
-        self.width = -(-(self.b_col + self.heads) // 4) * 4
-        self.w_in = rt.matrix(torch.cat(rows + [fill(self.width - self.b_col - self.heads)], dim=0))
+        width = -(-(self.b_col + self.heads) // 4) * 4
+        self.take_input(torch.cat(rows + [fill(width - self.b_col - self.heads)], dim=0), None, bool(p.get("joint_input")))
         # One product for both second layers: [a2 | 0 ; 0 | g2].
         w2 = torch.zeros((self.nk + self.nv, self.inner), dtype=tensors["a2"].dtype)
         w2[:self.nk, :ra] = tensors["a2"]
@@ -146,11 +147,8 @@ class GatedDeltaRule(Mixer):
         # [the convolution's last taps-1 inputs | S as [head, value channel, key channel]]
         return StateNeed((self.conv_state + self.heads * self.vdim * self.dim,), torch.float32)
 
-    def forward(self, h: torch.Tensor, residual32: torch.Tensor, ctx: StepContext, cache: LayerCache) -> None:
-        h = as_tensor(h)
-        m, dev, ops, nq, nk, nv = h.shape[0], h.device, self.ops, self.nq, self.nk, self.nv
-        p32 = torch.empty((m, self.width), dtype=torch.float32, device=dev)
-        ops.linear(h, self.w_in, None, p32, "f32")
+    def mix(self, p32: torch.Tensor, ctx: StepContext, cache: LayerCache) -> torch.Tensor:
+        m, dev, ops, nq, nk, nv = p32.shape[0], p32.device, self.ops, self.nq, self.nk, self.nv
         qkv = torch.empty((m, self.n_conv), dtype=torch.float32, device=dev)
         ops.conv_step(p32[:, :self.n_conv], self.conv_w, None, "silu", cache.state, 0, ctx, qkv, self.taps)
         inner = torch.empty((m, self.inner), dtype=self.rt.dtype, device=dev)
@@ -164,7 +162,7 @@ class GatedDeltaRule(Mixer):
         gated = torch.empty((m, nv), dtype=self.rt.dtype, device=dev)
         ops.gated_norm(o32, gated, groups=self.heads, eps=self.eps, gain32=self.gain, gate32=zg[:, nk:], gate_kind="sigmoid",
                        out_scale=self.out_scale)
-        ops.linear(gated, self.w_o, None, residual32, "add")
+        return gated
 
 
 register_part("general_delta", GeneralizedDeltaRule)

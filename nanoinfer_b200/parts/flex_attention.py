@@ -36,7 +36,7 @@ from typing import Dict, Optional
 import torch
 
 from ..registry import register_part
-from .base import CacheNeed, LayerCache, Mixer, PagedTensor, Runtime, StateNeed, StepContext, as_tensor
+from .base import CacheNeed, LayerCache, PagedTensor, ProjectedMixer, Runtime, StateNeed, StepContext
 from .position import scaled_frequencies
 from .spec import PartSpec, TensorSpec
 
@@ -53,11 +53,11 @@ def rotary_frequencies(dims: int, base: float, factor: float = 1.0, scaling=None
     return (torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / float(dims)) / float(factor)).to(torch.float32)
 
 
-class FlexAttention(Mixer):
+class FlexAttention(ProjectedMixer):
     """params: ``hidden heads kv_heads dim vdim scale eps`` and the options ``bias`` (q, k, v), ``out_bias``, ``conv``
     (taps), ``qk_norm``, ``rot`` ((dims, base) or None), ``softcap``, ``slope_span``, ``window``, ``chunk``,
     ``out_gate``, ``out_scale``, ``rot_layout``, ``rot_factor``, ``rot_scaling``, ``unit_norm_after_rot``, ``values_from_keys``, ``sink``,
-    ``v_mix`` (None, "first" or "blend"). tensors: ``q k o``, ``v`` unless the values are the keys, and, by option,
+    ``v_mix`` (None, "first" or "blend"), ``joint_input`` (the input product is made by a pair for both of its halves). tensors: ``q k o``, ``v`` unless the values are the keys, and, by option,
     ``q_b k_b v_b o_b q_conv k_conv v_conv q_norm k_norm g sink vmix``."""
 
     graph_safe = True   # launches do not depend on which requests are in the batch
@@ -129,12 +129,11 @@ class FlexAttention(Mixer):
         # One product for everything that reads h: rows [q | k | v | gate]; the gate has no bias.
         named = ("q", "k") if self.values_from_keys else ("q", "k", "v")
         rows = [tensors[n] for n in named] + ([tensors["g"]] if self.out_gate else [])
-        self.w_in = rt.matrix(torch.cat(rows, dim=0))
-        self.b_in = None
+        b = None
         if p.get("bias"):
             b = torch.zeros(self.n_qkv + self.n_gate, dtype=torch.float32)
             b[:self.n_qkv] = torch.cat([tensors[n + "_b"] for n in named]).to(torch.float32)
-            self.b_in = rt.vector32(b)
+        self.take_input(torch.cat(rows, dim=0), b, bool(p.get("joint_input")))
         self.conv_w = rt.vector32(torch.cat([tensors[n + "_conv"] for n in named], dim=0)) if self.taps else None
         self.q_gain = rt.vector32(tensors["q_norm"]) if p.get("qk_norm") else None
         self.k_gain = rt.vector32(tensors["k_norm"]) if p.get("qk_norm") else None
@@ -168,11 +167,8 @@ class FlexAttention(Mixer):
     def state_need(self) -> Optional[StateNeed]:
         return StateNeed(((self.taps - 1) * self.n_qkv,), torch.float32) if self.taps > 1 else None
 
-    def forward(self, h: torch.Tensor, residual32: torch.Tensor, ctx: StepContext, cache: LayerCache) -> None:
-        h = as_tensor(h)
-        m, dev, ops = h.shape[0], h.device, self.ops
-        p32 = torch.empty((m, self.n_qkv + self.n_gate), dtype=torch.float32, device=dev)
-        ops.linear(h, self.w_in, self.b_in, p32, "f32")
+    def mix(self, p32: torch.Tensor, ctx: StepContext, cache: LayerCache) -> torch.Tensor:
+        m, dev, ops = p32.shape[0], p32.device, self.ops
         qkv32 = p32[:, :self.n_qkv]
         if self.taps:
             conv32 = torch.empty((m, self.n_qkv), dtype=torch.float32, device=dev)
@@ -200,7 +196,7 @@ class FlexAttention(Mixer):
             a = torch.empty((m, self.heads * self.vdim), dtype=self.rt.dtype, device=dev)
             ops.gated_norm(attn, a, gate32=p32[:, self.n_qkv:], gate_kind="sigmoid", out_scale=self.out_scale)
             attn = a
-        ops.linear(attn, self.w_o, self.b_o, residual32, "add")
+        return attn
 
 
 register_part("flex_attention", FlexAttention)
