@@ -20,7 +20,8 @@
 //  * group_prepare: a warp per (group, head): unit keys and queries, decays, beta, the vectors W_t k_t, W_t q_t, W_(s,n] k_s,
 //    W_n, and the matrices A and D; parallel over the whole step.
 //    What the walk reads of a (group, head) lies in ONE block of the scratch.
-//  * group_walk: a warp per value channel of a head of a request, its key channels in the lanes' registers; the warps of a block
+//  * group_walk: a warp per one or two value channels of a head of a request, their key channels in the lanes' registers (two
+//    channels read a staged vector once: where the walk is bound by shared memory, not by its chain); the warps of a block
 //    share a group's block, which a warp of its own brings into shared memory (one bulk copy) several groups ahead. Per group: dot products with S_0 for the eight tokens, their sums over the lanes together (each
 //    exchange halves what a lane holds), 8 x 8 products with the matrices, one update of S.
 // Groups start at the step's first token of a request: a result depends on how the request was cut by rounding only.
@@ -36,7 +37,8 @@ __device__ int g_group_walk_error = 0;      // 0, or (role << 16 | blockIdx.x) o
 // A (group, head)'s block, in floats: W_t q_t, W_(t,n] k_t and (delta) W_t k_t for the eight tokens (rows of DKP floats, channels
 // beyond dk and tokens that do not exist zero), W_n, D and (delta) A.
 template <int C, bool DELTA> struct GsLayout {
-    static constexpr int WARPS = C <= 2 ? 4 : 8;        // value channels per block of threads
+    static constexpr int NC = C >= 8 || (DELTA && C < 4) ? 1 : 2;           // value channels per warp
+    static constexpr int WARPS = 4, COLS = WARPS * NC;         // walking warps, value channels per block of threads
     static constexpr int DKP = 32 * C, VECS = DELTA ? 3 : 2;
     static constexpr int Q0 = 0, S0 = GS_T * DKP, K0 = 2 * GS_T * DKP, W0 = VECS * GS_T * DKP, D0 = W0 + DKP, A0 = D0 + GS_T * GS_T,
                          SIZE = A0 + (DELTA ? GS_T * GS_T : 0);
@@ -200,14 +202,13 @@ group_walk_kernel(const float* __restrict__ work, const float* __restrict__ v, i
                   const int* __restrict__ q_start, const int* __restrict__ slots, float* __restrict__ o, int ldo, int heads, int dk, int dv,
                   int ones) {
     using L = GsLayout<C, DELTA>;
-    constexpr int DKP = L::DKP, STAGES = L::STAGES, WARPS = L::WARPS;
+    constexpr int DKP = L::DKP, STAGES = L::STAGES, WARPS = L::WARPS, NC = L::NC, COLS = L::COLS;
     extern __shared__ __align__(16) float gs_smem[];
     __shared__ unsigned long long full[STAGES], empty[STAGES];
-    __shared__ float s_v[STAGES][GS_T * WARPS];
+    __shared__ __align__(16) float s_v[STAGES][COLS * GS_T];      // a channel's eight values lie together
     __shared__ volatile int s_failed;
     const int req = blockIdx.z, h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int cols = dv + ones, j = blockIdx.x * WARPS + warp;      // value channels of the state, a column of ones behind the others
-    const bool live = j < cols;
+    const int cols = dv + ones, j0 = blockIdx.x * COLS + warp * NC;      // value channels of the state, a column of ones behind the others
     const int row0 = q_start[req], row1 = q_start[req + 1];
     const int groups = (row1 - row0 + GS_T - 1) / GS_T;
     if (threadIdx.x == 0) {
@@ -235,8 +236,8 @@ group_walk_kernel(const float* __restrict__ work, const float* __restrict__ v, i
                 bulk_copy_g2s(gs_smem + st * L::SIZE, src + (size_t)g * heads * L::SIZE, L::SIZE * 4, &full[st]);
             }
 #pragma unroll
-            for (int e = lane; e < GS_T * WARPS; e += 32) {     // the values of the block's channels (a column of ones has none)
-                const int t = g * GS_T + e / WARPS, jj = blockIdx.x * WARPS + e % WARPS;
+            for (int e = lane; e < GS_T * COLS; e += 32) {     // the values of the block's channels (a column of ones has none)
+                const int t = g * GS_T + e % GS_T, jj = blockIdx.x * COLS + e / GS_T;
                 const bool there = t < row1 - row0 && jj < dv;
                 const float* from = v + (size_t)(row0 + (there ? t : 0)) * ldv + (size_t)h * dv + (there ? jj : 0);
                 const int n = there ? 4 : 0;        // 0 source bytes: the destination is zero-filled
@@ -251,12 +252,14 @@ group_walk_kernel(const float* __restrict__ work, const float* __restrict__ v, i
         asm volatile("cp.async.wait_all;\n" ::: "memory");
         return;
     }
-    float* srow = state + (long long)slots[req] * state_ld + state_off + ((long long)h * cols + (live ? j : 0)) * dk;
+    float* head_state = state + (long long)slots[req] * state_ld + state_off + (long long)h * cols * dk;
     // lane l owns the channels l * C .. + C - 1 (C = 8: l * 4 .. + 3 of both halves): a warp's load of a vector is contiguous
     auto channel = [&](int i) { return C == 8 ? (i >> 2) * 128 + lane * 4 + (i & 3) : lane * C + i; };
-    float S[C];
+    float S[NC][C];
 #pragma unroll
-    for (int i = 0; i < C; ++i) S[i] = (live && channel(i) < dk) ? srow[channel(i)] : 0.f;
+    for (int n = 0; n < NC; ++n)
+#pragma unroll
+        for (int i = 0; i < C; ++i) S[n][i] = (j0 + n < cols && channel(i) < dk) ? head_state[(long long)(j0 + n) * dk + channel(i)] : 0.f;
     auto take = [&](const float* row, float (&x)[C]) {
         if constexpr (C == 1) x[0] = row[lane];
         else if constexpr (C == 2) { const float2 a = *reinterpret_cast<const float2*>(row + lane * 2); x[0] = a.x; x[1] = a.y; }
@@ -273,8 +276,8 @@ group_walk_kernel(const float* __restrict__ work, const float* __restrict__ v, i
         const float s2 = fmaf(b.y, x[5], b.x * x[4]), s3 = fmaf(b.w, x[7], b.z * x[6]);
         return (s0 + s1) + (s2 + s3);
     };
-    // Sums over the lanes of N values a lane (8 or 16), each exchange halving what a lane holds. A lane ends with the value
-    // whose index its upper bits spell: 16 values: lane >> 1; 8 values: lane >> 2.
+    // Sums over the lanes of N values a lane (8, 16 or 32), each exchange halving what a lane holds. A lane ends with value
+    // lane / (32 / N).
     auto sums = [&](auto& p, auto count) {
         constexpr int N = decltype(count)::value;
 #pragma unroll
@@ -310,9 +313,11 @@ group_walk_kernel(const float* __restrict__ work, const float* __restrict__ v, i
         }
         return ok;
     };
-    const bool is_one = ones != 0 && j == dv;       // the column of ones
-    const int token = DELTA ? (lane >> 1) & (GS_T - 1) : lane >> 2;     // whose sum this lane ends with
-    const bool writer = DELTA ? lane >= 16 && (lane & 1) == 0 : (lane & 3) == 0;
+    constexpr int N = (DELTA ? 2 : 1) * NC * GS_T, EACH = 32 / N;      // sums per group: (DELTA: both dot products) x channels x tokens
+    const int token = (lane / EACH) % GS_T, mine_n = (lane / EACH) / GS_T % NC;        // whose sum this lane ends with
+    const bool writer = lane % EACH == 0 && (!DELTA || lane >= 16) && j0 + mine_n < cols;
+    const int my_col = warp * NC + mine_n, my_j = j0 + mine_n;
+    const bool my_one = ones != 0 && my_j == dv;        // the column of ones
     bool ok = true;
     if (groups > 0) {
         ok = arrived(0);
@@ -322,19 +327,21 @@ group_walk_kernel(const float* __restrict__ work, const float* __restrict__ v, i
         const int base = row0 + g * GS_T;
         const float* st = gs_smem + (g % STAGES) * L::SIZE;
         const float* vs = s_v[g % STAGES];
-        float p[DELTA ? 2 * GS_T : GS_T];
+        float p[N];
 #pragma unroll
-        for (int t = 0; t < GS_T; ++t) {
-            float pa = 0.f, pb = 0.f;
+        for (int n = 0; n < NC; ++n)
 #pragma unroll
-            for (int i = 0; i < C; ++i) {
-                if constexpr (DELTA) pa = fmaf(kd[DELTA ? t : 0][i], S[i], pa);
-                pb = fmaf(qd[t][i], S[i], pb);
+            for (int t = 0; t < GS_T; ++t) {
+                float pa = 0.f, pb = 0.f;
+#pragma unroll
+                for (int i = 0; i < C; ++i) {
+                    if constexpr (DELTA) pa = fmaf(kd[DELTA ? t : 0][i], S[n][i], pa);
+                    pb = fmaf(qd[t][i], S[n][i], pb);
+                }
+                if constexpr (DELTA) p[n * GS_T + t] = pa;
+                p[(DELTA ? NC * GS_T : 0) + n * GS_T + t] = pb;
             }
-            if constexpr (DELTA) p[t] = pa;
-            p[(DELTA ? GS_T : 0) + t] = pb;
-        }
-        float ks[GS_T][C], wn[C], x[GS_T];
+        float ks[GS_T][C], wn[C], x[NC][GS_T];      // x: u of the group's tokens, known to every lane
 #pragma unroll
         for (int t = 0; t < GS_T; ++t) take(st + L::S0 + t * DKP, ks[t]);
         take(st + L::W0, wn);
@@ -344,42 +351,63 @@ group_walk_kernel(const float* __restrict__ work, const float* __restrict__ v, i
         if constexpr (DELTA) {
             a0 = *reinterpret_cast<const float4*>(st + L::A0 + token * GS_T);
             a1 = *reinterpret_cast<const float4*>(st + L::A0 + token * GS_T + 4);
-            mine = is_one ? 1.0f : vs[token * WARPS + warp];
+            mine = my_one ? 1.0f : vs[my_col * GS_T + token];
         } else {
 #pragma unroll
-            for (int t = 0; t < GS_T; ++t) x[t] = is_one ? 1.0f : vs[t * WARPS + warp];
+            for (int n = 0; n < NC; ++n) {
+                const float4 va = *reinterpret_cast<const float4*>(vs + (warp * NC + n) * GS_T), vb = *reinterpret_cast<const float4*>(vs + (warp * NC + n) * GS_T + 4);
+                const bool one = ones != 0 && j0 + n == dv;
+                x[n][0] = one ? 1.f : va.x; x[n][1] = one ? 1.f : va.y; x[n][2] = one ? 1.f : va.z; x[n][3] = one ? 1.f : va.w;
+                x[n][4] = one ? 1.f : vb.x; x[n][5] = one ? 1.f : vb.y; x[n][6] = one ? 1.f : vb.z; x[n][7] = one ? 1.f : vb.w;
+            }
         }
 #pragma unroll
-        for (int i = 0; i < C; ++i) S[i] *= wn[i];
-        // DELTA: lanes 0..15 end with (W k)^T S_0 of token lane >> 1, lanes 16..31 with (W q)^T S_0 of theirs
-        const float val = sums(p, std::integral_constant<int, DELTA ? 2 * GS_T : GS_T>{});
+        for (int n = 0; n < NC; ++n)
+#pragma unroll
+            for (int i = 0; i < C; ++i) S[n][i] *= wn[i];
+        // DELTA: the lower half of the lanes ends with (W k)^T S_0 of their channel and token, the upper half with (W q)^T S_0
+        const float val = sums(p, std::integral_constant<int, N>{});
         __syncwarp();
         if (lane == 0) mbar_arrive(&empty[g % STAGES]);     // this warp has read what it needs of the group
         if (g + 1 < groups) {
             ok = arrived(g + 1);
             fetch(gs_smem + ((g + 1) % STAGES) * L::SIZE);
         }
+        auto of_mine = [&](float (&y)[GS_T]) {      // x of this lane's channel
+#pragma unroll
+            for (int t = 0; t < GS_T; ++t) y[t] = NC == 2 && mine_n != 0 ? x[NC - 1][t] : x[0][t];
+        };
+        float y[GS_T];
         if constexpr (DELTA) {
             mine -= val;
 #pragma unroll
-            for (int t = 0; t < GS_T; ++t) x[t] = __shfl_sync(0xffffffffu, mine, 2 * t);
-            const float um = row_times(a0, a1, x);
+            for (int n = 0; n < NC; ++n)
 #pragma unroll
-            for (int t = 0; t < GS_T; ++t) x[t] = __shfl_sync(0xffffffffu, um, 2 * t);
+                for (int t = 0; t < GS_T; ++t) x[n][t] = __shfl_sync(0xffffffffu, mine, (n * GS_T + t) * EACH);
+            of_mine(y);
+            const float um = row_times(a0, a1, y);
+#pragma unroll
+            for (int n = 0; n < NC; ++n)
+#pragma unroll
+                for (int t = 0; t < GS_T; ++t) x[n][t] = __shfl_sync(0xffffffffu, um, (n * GS_T + t) * EACH);
         }
 #pragma unroll
         for (int t = 0; t < GS_T; ++t)
 #pragma unroll
-            for (int i = 0; i < C; ++i) S[i] = fmaf(ks[t][i], x[t], S[i]);
-        const float out = val + row_times(d0, d1, x);
-        if (writer && base + token < row1 && live) o[(size_t)(base + token) * ldo + (is_one ? (size_t)heads * dv + h : (size_t)h * dv + j)] = out;
+            for (int n = 0; n < NC; ++n)
+#pragma unroll
+                for (int i = 0; i < C; ++i) S[n][i] = fmaf(ks[t][i], x[n][t], S[n][i]);
+        of_mine(y);
+        const float out = val + row_times(d0, d1, y);
+        if (writer && base + token < row1)
+            o[(size_t)(base + token) * ldo + (my_one ? (size_t)heads * dv + h : (size_t)h * dv + my_j)] = out;
     }
     pdl_launch_dependents();        // only now: blocks of the next kernel that became resident earlier would sit beside a long walk
-    if (live) {
+#pragma unroll
+    for (int n = 0; n < NC; ++n)
 #pragma unroll
         for (int i = 0; i < C; ++i)
-            if (channel(i) < dk) srow[channel(i)] = S[i];
-    }
+            if (j0 + n < cols && channel(i) < dk) head_state[(long long)(j0 + n) * dk + channel(i)] = S[n][i];
 }
 
 namespace {
@@ -399,7 +427,7 @@ int launch_group(const float* q, int ldq, const float* k, int ldk, const float* 
     NIB_CUDA(launch_pdl(group_prepare_kernel<CPL, DELTA>, pgrid, dim3(128), (size_t)0, stream, q, ldq, k, ldk, z, ldz, z_kind, dt_bias, rate, b, ldb,
                         k_scale, q_start, work, heads, kq_heads, dk, q_scale, unit_eps));
     NIB_LAUNCH_CHECK();
-    const dim3 grid(ceil_div(dv + ones, L::WARPS), heads, n_req);
+    const dim3 grid(ceil_div(dv + ones, L::COLS), heads, n_req);
     if (longest <= 64) {
         NIB_CUDA(launch_pdl(group_walk_kernel<CPL, DELTA>, grid, dim3(L::WARPS * 32 + 32), (size_t)L::BYTES, stream, work, v, ldv, state, state_ld, state_off,
                             q_start, slots, o, ldo, heads, dk, dv, ones));

@@ -496,46 +496,56 @@ gated_norm_block_kernel(const float* __restrict__ o, int ldo, const float* __res
     }
 }
 
-// The same for parts of 16, 32, 64 or 128 channels without a skip and with the gate (if any) behind the norm: LPP = width / 4
-// lanes a part, four channels a lane, held in registers between the sum of squares and the result.
-template <typename T, int LPP>
+// The same for parts of 16, 32, 64, 128 or 256 channels without a skip and with the gate (if any) behind the norm: LPP lanes a
+// part, NV times four channels a lane, held in registers between the sum of squares and the result.
+template <typename T, int LPP, int NV>
 __global__ void __launch_bounds__(128)
 gated_norm_vec_kernel(const float* __restrict__ o, int ldo, const float* __restrict__ gate, int ldg, int gate_kind, const float* __restrict__ gain,
                       int gain_len, float eps, float out_scale, T* __restrict__ out, int ld_out, int tokens, int groups,
                       const float* __restrict__ floor_in, int ldf, float den_eps) {
-    constexpr int WIDTH = 4 * LPP;
+    constexpr int WIDTH = 4 * LPP * NV;
     pdl_launch_dependents();
     pdl_wait();      // everything this kernel reads may come from the kernel before
     const long long p = ((long long)blockIdx.x * 128 + threadIdx.x) / LPP;
     const int sub = threadIdx.x % LPP;
     const bool live = p < (long long)tokens * groups;
-    const int t = live ? (int)(p / groups) : 0, part_i = live ? (int)(p % groups) : 0, c = part_i * WIDTH + sub * 4;
-    float4 y = *reinterpret_cast<const float4*>(o + (size_t)t * ldo + c);
-    float4 gv = make_float4(0.f, 0.f, 0.f, 0.f), ga = make_float4(1.f, 1.f, 1.f, 1.f);
-    if (gate != nullptr) gv = *reinterpret_cast<const float4*>(gate + (size_t)t * ldg + c);
-    if (gain != nullptr) ga = __ldg(reinterpret_cast<const float4*>(gain + c % gain_len));
-    if (floor_in != nullptr) {
-        const float den = fmaxf(fabsf(o[(size_t)t * ldo + groups * WIDTH + part_i]), floor_in[(size_t)t * ldf + part_i]) + den_eps;
-        y.x /= den; y.y /= den; y.z /= den; y.w /= den;
+    const int t = live ? (int)(p / groups) : 0, part_i = live ? (int)(p % groups) : 0, c0 = part_i * WIDTH + sub * 4;
+    float4 y[NV], gv[NV], ga[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = c0 + i * 4 * LPP;
+        y[i] = *reinterpret_cast<const float4*>(o + (size_t)t * ldo + c);
+        gv[i] = gate != nullptr ? *reinterpret_cast<const float4*>(gate + (size_t)t * ldg + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        ga[i] = gain != nullptr ? __ldg(reinterpret_cast<const float4*>(gain + c % gain_len)) : make_float4(1.f, 1.f, 1.f, 1.f);
     }
-    float ss = fmaf(y.x, y.x, fmaf(y.y, y.y, fmaf(y.z, y.z, y.w * y.w)));
+    float ss = 0.f, den = 1.f;
+    if (floor_in != nullptr) den = fmaxf(fabsf(o[(size_t)t * ldo + groups * WIDTH + part_i]), floor_in[(size_t)t * ldf + part_i]) + den_eps;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        if (floor_in != nullptr) { y[i].x /= den; y[i].y /= den; y[i].z /= den; y[i].w /= den; }
+        ss = fmaf(y[i].x, y[i].x, fmaf(y[i].y, y[i].y, fmaf(y[i].z, y[i].z, fmaf(y[i].w, y[i].w, ss))));
+    }
 #pragma unroll
     for (int m = LPP / 2; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
-    const float scale = 1.0f / sqrtf(ss / (float)WIDTH + eps);
-    float v[4] = {y.x * scale * ga.x, y.y * scale * ga.y, y.z * scale * ga.z, y.w * scale * ga.w};
-    if (gate != nullptr && gate_kind != 0) {
-        v[0] *= gate_act(gv.x, gate_kind); v[1] *= gate_act(gv.y, gate_kind); v[2] *= gate_act(gv.z, gate_kind); v[3] *= gate_act(gv.w, gate_kind);
-    }
     if (!live) return;
-    T* to = out + (size_t)t * ld_out + c;
-    if constexpr (sizeof(T) == 4) {
-        *reinterpret_cast<float4*>(to) = make_float4(v[0] * out_scale, v[1] * out_scale, v[2] * out_scale, v[3] * out_scale);
-    } else {
-        const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0] * out_scale, v[1] * out_scale), hi = __floats2bfloat162_rn(v[2] * out_scale, v[3] * out_scale);
-        uint2 pk;
-        pk.x = *reinterpret_cast<const unsigned*>(&lo);
-        pk.y = *reinterpret_cast<const unsigned*>(&hi);
-        *reinterpret_cast<uint2*>(to) = pk;
+    const float scale = 1.0f / sqrtf(ss / (float)WIDTH + eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        float v[4] = {y[i].x * scale * ga[i].x, y[i].y * scale * ga[i].y, y[i].z * scale * ga[i].z, y[i].w * scale * ga[i].w};
+        if (gate != nullptr && gate_kind != 0) {
+            v[0] *= gate_act(gv[i].x, gate_kind); v[1] *= gate_act(gv[i].y, gate_kind);
+            v[2] *= gate_act(gv[i].z, gate_kind); v[3] *= gate_act(gv[i].w, gate_kind);
+        }
+        T* to = out + (size_t)t * ld_out + c0 + i * 4 * LPP;
+        if constexpr (sizeof(T) == 4) {
+            *reinterpret_cast<float4*>(to) = make_float4(v[0] * out_scale, v[1] * out_scale, v[2] * out_scale, v[3] * out_scale);
+        } else {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0] * out_scale, v[1] * out_scale), hi = __floats2bfloat162_rn(v[2] * out_scale, v[3] * out_scale);
+            uint2 pk;
+            pk.x = *reinterpret_cast<const unsigned*>(&lo);
+            pk.y = *reinterpret_cast<const unsigned*>(&hi);
+            *reinterpret_cast<uint2*>(to) = pk;
+        }
     }
 }
 
@@ -550,12 +560,13 @@ NIB_API int nib_gated_norm(const float* o, int ldo, const float* gate, int ldg, 
     const int width = n / groups, span = skip != nullptr ? n / n_coef : 1;
     const bool rows16 = (((uintptr_t)o | (uintptr_t)gate | (uintptr_t)gain | (uintptr_t)out) & 15) == 0 && ldo % 4 == 0 && ldg % 4 == 0
         && (ld_out * (dtype == NIB_F32 ? 4 : 2)) % 8 == 0 && (gain == nullptr || gain_len % 4 == 0);
-    if (norm && skip == nullptr && (gate == nullptr || !gate_first) && rows16 && (width == 16 || width == 32 || width == 64 || width == 128)
+    if (norm && skip == nullptr && (gate == nullptr || !gate_first) && rows16 && (width == 16 || width == 32 || width == 64 || width == 128 || width == 256)
         && (dtype == NIB_F32 || dtype == NIB_BF16)) {
-        const dim3 grid(ceil_div((long long)tokens * groups * (width / 4), 128));
-#define NIB_GV(T, LPP) NIB_CUDA(launch_pdl(gated_norm_vec_kernel<T, LPP>, grid, dim3(128), (size_t)0, stream, o, ldo, gate, ldg, gate_kind, gain, gain_len, eps, \
+        const int lanes = width >= 128 ? 32 : width / 4;
+        const dim3 grid(ceil_div((long long)tokens * groups * lanes, 128));
+#define NIB_GV(T, LPP, NV) NIB_CUDA(launch_pdl(gated_norm_vec_kernel<T, LPP, NV>, grid, dim3(128), (size_t)0, stream, o, ldo, gate, ldg, gate_kind, gain, gain_len, eps, \
                                            out_scale, (T*)out, ld_out, tokens, groups, floor_in, ldf, den_eps))
-#define NIB_GW(T) do { if (width == 16) NIB_GV(T, 4); else if (width == 32) NIB_GV(T, 8); else if (width == 64) NIB_GV(T, 16); else NIB_GV(T, 32); } while (0)
+#define NIB_GW(T) do { if (width == 16) NIB_GV(T, 4, 1); else if (width == 32) NIB_GV(T, 8, 1); else if (width == 64) NIB_GV(T, 16, 1); else if (width == 128) NIB_GV(T, 32, 1); else NIB_GV(T, 32, 2); } while (0)
         if (dtype == NIB_F32) NIB_GW(float); else NIB_GW(__nv_bfloat16);
 #undef NIB_GW
 #undef NIB_GV

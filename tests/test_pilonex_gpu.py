@@ -133,7 +133,7 @@ def test_gates_keep_a_running_maximum_across_steps(ops, heads, cap):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("m,heads,d", [(5, 3, 20), (3, 2, 300), (40, 1, 7), (9, 4, 64), (33, 2, 128), (7, 5, 16)])
+@pytest.mark.parametrize("m,heads,d", [(5, 3, 20), (3, 2, 300), (40, 1, 7), (9, 4, 64), (33, 2, 128), (7, 5, 16), (6, 3, 256), (5, 1, 32)])
 def test_norm_of_a_part_behind_its_divisor(ops, dtype, m, heads, d):
     """A part's number behind the channels divides it (its size, or the floor where that is larger, plus a small constant)."""
     o, gate = rnd(m, heads * (d + 1), seed=1), rnd(m, heads * d, seed=2)
