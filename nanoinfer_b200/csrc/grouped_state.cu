@@ -20,6 +20,9 @@
 //  * group_prepare: a warp per (group, head): unit keys and queries, decays, beta, the vectors W_t k_t, W_t q_t, W_(s,n] k_s,
 //    W_n, and the matrices A and D; parallel over the whole step.
 //    What the walk reads of a (group, head) lies in ONE block of the scratch.
+//  * state_step: steps in which no request brings more than GS_STEP_TOKENS tokens (a decode step): the rules as they stand, token by
+//    token, in one launch; a warp per GS_STEP_COLS value channels of a head of a request, every warp forming what it needs of q, k,
+//    the decays and beta by itself.
 //  * group_walk: a warp per one or two value channels of a head of a request, their key channels in the lanes' registers (two
 //    channels read a staged vector once: where the walk is bound by shared memory, not by its chain); the warps of a block
 //    share a group's block, which a warp of its own brings into shared memory (one bulk copy) several groups ahead. Per group: dot products with S_0 for the eight tokens, their sums over the lanes together (each
@@ -31,6 +34,7 @@
 using namespace nibp;
 
 constexpr int GS_T = 8;             // tokens per group
+constexpr int GS_STEP_TOKENS = 4, GS_STEP_COLS = 4;     // short steps: tokens per request at most, value channels per warp
 
 __device__ int g_group_walk_error = 0;      // 0, or (role << 16 | blockIdx.x) of the first wait that ran out (1 a walking warp, 2 the sending one)
 
@@ -53,6 +57,11 @@ __device__ __forceinline__ long long first_group(int row0, int req) { return row
 // exp(x) for x <= 0 or a little above: near zero 1 + expm1, so that a result near one is off by its own rounding alone (a decay
 // is raised to hundreds of powers along a sequence, which would multiply a bias of expf up).
 __device__ __forceinline__ float gs_decay_exp(float x) { return fabsf(x) < 0.5f ? 1.0f + expm1f(x) : expf(x); }
+
+// exp(-rate softplus(x))
+__device__ __forceinline__ float gs_step_decay(float x, float rate) {
+    return gs_decay_exp(-rate * (x > 0.f ? x + log1pf(expf(-x)) : log1pf(expf(x))));
+}
 
 // How z is read: GS_STEP per (head, key channel) logits of step sizes, decay = exp(-rate[h] * softplus(z + dt_bias));
 // GS_CHANNEL per (head, key channel) decays; GS_HEAD one decay per head.
@@ -126,11 +135,7 @@ group_prepare_kernel(const float* __restrict__ q, int ldq, const float* __restri
         for (int i = 0; i < CPL; ++i) {
             const int c = lane + 32 * i;
             float w = wv[t][i];
-            if (z_kind == GS_STEP && c < dk) {
-                const float x = w + bias[i];
-                const float step = x > 0.f ? x + log1pf(expf(-x)) : log1pf(expf(x));
-                w = gs_decay_exp(-r * step);
-            }
+            if (z_kind == GS_STEP && c < dk) w = gs_step_decay(w + bias[i], r);
             const float ku = kv[t][i] * ik, qu = qv[t][i] * iq;
             pre[i] *= w;
 #pragma unroll
@@ -410,6 +415,92 @@ group_walk_kernel(const float* __restrict__ work, const float* __restrict__ v, i
             if (j0 + n < cols && channel(i) < dk) head_state[(long long)(j0 + n) * dk + channel(i)] = S[n][i];
 }
 
+template <int CPL, bool DELTA>
+__global__ void __launch_bounds__(128)
+state_step_kernel(const float* __restrict__ q, int ldq, const float* __restrict__ k, int ldk, const float* __restrict__ v, int ldv,
+                  const float* __restrict__ z, int ldz, int z_kind, const float* __restrict__ dt_bias, const float* __restrict__ rate,
+                  const float* __restrict__ b, int ldb, const float* __restrict__ k_scale, float* __restrict__ state, long long state_ld,
+                  int state_off, const int* __restrict__ q_start, const int* __restrict__ slots, float* __restrict__ o, int ldo, int heads,
+                  int kq_heads, int dk, int dv, int ones, float q_scale, float unit_eps) {
+    constexpr int NC = GS_STEP_COLS;
+    pdl_launch_dependents();
+    pdl_wait();      // everything this kernel reads may come from the kernel before
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, req = blockIdx.z, h = blockIdx.y;
+    const int cols = dv + ones, j0 = (blockIdx.x * 4 + warp) * NC;
+    const int row0 = q_start[req], row1 = q_start[req + 1];
+    if (row0 >= row1 || j0 >= cols) return;     // a whole warp leaves together, and nothing below waits for the block
+    float* head_state = state + (long long)slots[req] * state_ld + state_off + (long long)h * cols * dk;
+    const int hq = h / (heads / kq_heads);
+    const float r = z_kind == GS_STEP ? rate[h] : 0.f;
+    float S[NC][CPL], bias[CPL];
+#pragma unroll
+    for (int i = 0; i < CPL; ++i) {
+        const int c = lane + 32 * i;
+        bias[i] = (z_kind == GS_STEP && c < dk) ? dt_bias[(size_t)h * dk + c] : 0.f;
+#pragma unroll
+        for (int n = 0; n < NC; ++n) S[n][i] = (c < dk && j0 + n < cols) ? head_state[(long long)(j0 + n) * dk + c] : 0.f;
+    }
+    for (int row = row0; row < row1; ++row) {
+        float kv[CPL], qv[CPL], w[CPL], val[NC];
+        const float wh = z_kind == GS_HEAD ? z[(size_t)row * ldz + h] : 1.f;
+        const float ks = k_scale != nullptr ? k_scale[(size_t)row * heads + h] : 1.f;
+        const float zb = DELTA ? b[(size_t)row * ldb + h] : 0.f;
+#pragma unroll
+        for (int i = 0; i < CPL; ++i) {
+            const int c = lane + 32 * i;
+            const bool in = c < dk;
+            kv[i] = in ? k[(size_t)row * ldk + (size_t)hq * dk + c] : 0.f;
+            qv[i] = in ? q[(size_t)row * ldq + (size_t)hq * dk + c] : 0.f;
+            w[i] = !in ? 1.f : (z_kind == GS_HEAD ? wh : z[(size_t)row * ldz + (size_t)h * dk + c]);
+        }
+#pragma unroll
+        for (int n = 0; n < NC; ++n)    // (a column of ones lies behind the others)
+            val[n] = j0 + n < dv ? v[(size_t)row * ldv + (size_t)h * dv + j0 + n] : 1.f;
+        float ik = ks, iq = q_scale;
+        if (unit_eps >= 0.f) {
+            float sk = 0.f, sq = 0.f;
+#pragma unroll
+            for (int i = 0; i < CPL; ++i) { sk = fmaf(kv[i], kv[i], sk); sq = fmaf(qv[i], qv[i], sq); }
+            ik = ks / sqrtf(warp_sum(sk) + unit_eps);
+            iq = q_scale / sqrtf(warp_sum(sq) + unit_eps);
+        }
+        float kq = 0.f, a[NC], out[NC];
+#pragma unroll
+        for (int n = 0; n < NC; ++n) a[n] = out[n] = 0.f;
+#pragma unroll
+        for (int i = 0; i < CPL; ++i) {
+            if (z_kind == GS_STEP && lane + 32 * i < dk) w[i] = gs_step_decay(w[i] + bias[i], r);
+            kv[i] *= ik;
+            qv[i] *= iq;
+            kq = fmaf(kv[i], qv[i], kq);
+#pragma unroll
+            for (int n = 0; n < NC; ++n) {
+                S[n][i] *= w[i];
+                if (DELTA) a[n] = fmaf(S[n][i], kv[i], a[n]);
+                out[n] = fmaf(S[n][i], qv[i], out[n]);
+            }
+        }
+        kq = warp_sum(kq);
+        const float beta = DELTA ? 1.0f / (1.0f + expf(-zb)) : 1.0f;
+#pragma unroll
+        for (int n = 0; n < NC; ++n) {
+            const float u = DELTA ? beta * (val[n] - warp_sum(a[n])) : val[n];
+            out[n] = fmaf(u, kq, warp_sum(out[n]));
+#pragma unroll
+            for (int i = 0; i < CPL; ++i) S[n][i] = fmaf(kv[i], u, S[n][i]);
+        }
+#pragma unroll
+        for (int n = 0; n < NC; ++n)
+            if (lane == n && j0 + n < cols)
+                o[(size_t)row * ldo + (j0 + n < dv ? (size_t)h * dv + j0 + n : (size_t)heads * dv + h)] = out[n];
+    }
+#pragma unroll
+    for (int n = 0; n < NC; ++n)
+#pragma unroll
+        for (int i = 0; i < CPL; ++i)
+            if (lane + 32 * i < dk && j0 + n < cols) head_state[(long long)(j0 + n) * dk + lane + 32 * i] = S[n][i];
+}
+
 namespace {
 
 template <int CPL, bool DELTA>
@@ -418,6 +509,13 @@ int launch_group(const float* q, int ldq, const float* k, int ldk, const float* 
                  const int* slots, float* o, int ldo, float* work, int n_req, int longest, int heads, int kq_heads, int dk, int dv, int ones,
                  float q_scale, float unit_eps, cudaStream_t stream) {
     using L = GsLayout<CPL, DELTA>;
+    if (longest <= GS_STEP_TOKENS) {
+        NIB_CUDA(launch_pdl(state_step_kernel<CPL, DELTA>, dim3(ceil_div(dv + ones, 4 * GS_STEP_COLS), heads, n_req), dim3(128), (size_t)0, stream, q, ldq,
+                            k, ldk, v, ldv, z, ldz, z_kind, dt_bias, rate, b, ldb, k_scale, state, state_ld, state_off, q_start, slots, o, ldo, heads,
+                            kq_heads, dk, dv, ones, q_scale, unit_eps));
+        NIB_LAUNCH_CHECK();
+        return 0;
+    }
     static bool configured = false;
     if (!configured) {
         NIB_CUDA(cudaFuncSetAttribute(group_walk_kernel<CPL, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, L::BYTES));
@@ -441,8 +539,9 @@ int launch_group(const float* q, int ldq, const float* k, int ldk, const float* 
 
 }  // namespace
 
-// Floats of scratch for a step of these sizes (delta: the rule with beta).
-NIB_API long long nib_grouped_state_scratch(long long tokens, int n_req, int heads, int dk, int delta) {
+// Floats of scratch for a step of these sizes (delta: the rule with beta); 0: a short step, which is one launch.
+NIB_API long long nib_grouped_state_scratch(long long tokens, int n_req, int longest, int heads, int dk, int delta) {
+    if (longest <= GS_STEP_TOKENS) return 0;
     const int c = dk <= 32 ? 1 : dk <= 64 ? 2 : dk <= 128 ? 4 : 8;
     const long long size = (delta ? 3 : 2) * GS_T * 32LL * c + 32LL * c + (delta ? 2 : 1) * GS_T * GS_T;
     return (tokens / GS_T + n_req) * heads * size;
@@ -467,7 +566,7 @@ NIB_API int nib_grouped_state_scan(const float* q, int ldq, const float* k, int 
                                    float unit_eps, cudaStream_t stream) {
     NIB_REQUIRE(heads > 0 && heads <= 65535 && kq_heads > 0 && heads % kq_heads == 0, "grouped_state_scan: %d heads do not share %d key heads", heads, kq_heads);
     NIB_REQUIRE(dk > 0 && dk <= 256 && dv > 0 && (ones == 0 || ones == 1), "grouped_state_scan: key size %d is outside 1..256", dk);
-    NIB_REQUIRE(z_kind >= GS_STEP && z_kind <= GS_HEAD && (z_kind != GS_STEP || (rate != nullptr && dt_bias != nullptr)) && scratch != nullptr
+    NIB_REQUIRE(z_kind >= GS_STEP && z_kind <= GS_HEAD && (z_kind != GS_STEP || (rate != nullptr && dt_bias != nullptr)) && (scratch != nullptr || longest <= GS_STEP_TOKENS)
                 && ((uintptr_t)scratch & 15) == 0, "grouped_state_scan: bad arguments");
     if (n_req <= 0 || tokens <= 0) return 0;
     NIB_REQUIRE(longest > 0 && n_req <= 65535, "grouped_state_scan: bad batch");

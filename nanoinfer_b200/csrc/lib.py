@@ -1040,7 +1040,7 @@ class Kernels:
             c_longlong(state.stride(0)), c_int(state_off), _ptr(ctx.q_start), _ptr(ctx.state_slots), _ptr(decay32), _ptr(write32), _ptr(floor32),
             c_int(ctx.host.num_requests), c_int(max(ctx.host.q_lens)), c_int(heads), self._stream()), "memory_gates")
 
-    # ---- walks over matrix states, eight tokens at a time (grouped_state.cu) -----------------------------------
+    # ---- walks over matrix states: short steps token by token, longer ones eight tokens at a time (grouped_state.cu) ----------
     def grouped_state_scan(self, q32, k32, v32, z32, state, state_off, ctx, o32, heads, kq_heads, dk, dv, beta32=None, rate32=None,
                            dt_bias32=None, q_scale=1.0, unit_eps=None, k_scale32=None, ones=False):
         """Per request and head, over the step's tokens in order, from and into ``state[slot, state_off:]`` (laid out [head, value
@@ -1077,9 +1077,10 @@ class Kernels:
         if k_scale32 is not None and not k_scale32.is_contiguous():
             raise KernelError("grouped_state_scan: k_scale must be contiguous")
         self._state_row(state, state_off, heads * (dv + extra) * dk, "grouped_state_scan state")
-        floats = self._lib.nib_grouped_state_scratch(c_longlong(m), c_int(ctx.host.num_requests), c_int(heads), c_int(dk), c_int(0 if beta32 is None else 1))
-        scratch = torch.empty(floats, dtype=torch.float32, device=q32.device)
-        self.launches += 1
+        floats = self._lib.nib_grouped_state_scratch(c_longlong(m), c_int(ctx.host.num_requests), c_int(max(ctx.host.q_lens)), c_int(heads), c_int(dk),
+                                                     c_int(0 if beta32 is None else 1))
+        scratch = torch.empty(floats, dtype=torch.float32, device=q32.device) if floats else None
+        self.launches += 1 if floats else 0        # a step with scratch is two launches
         self._check(self._lib.nib_grouped_state_scan(
             _ptr(q32), c_int(q32.stride(0)), _ptr(k32), c_int(k32.stride(0)), _ptr(v32), c_int(v32.stride(0)), _ptr(z32), c_int(z32.stride(0)),
             c_int(kind), _ptr(dt_bias32), _ptr(rate32), _ptr(beta32), c_int(0 if beta32 is None else beta32.stride(0)), _ptr(k_scale32), _ptr(state),

@@ -214,6 +214,36 @@ def test_walk_against_plain_and_cut_anywhere(ops, heads, kq, dk, dv, kind):
     ops.check_device_errors()
 
 
+@pytest.mark.parametrize("heads,kq,dk,dv", [(4, 2, 64, 64), (2, 2, 20, 33), (3, 1, 129, 6), (1, 1, 1, 1)])
+@pytest.mark.parametrize("kind", ["delta", "delta_decays", "channel", "head"])
+def test_short_steps_go_on_where_long_ones_stopped(ops, heads, kq, dk, dv, kind):
+    """A portion of 30 tokens, then steps of one to four tokens (one launch each), then one of 12, beside a request that is at
+    another place; slots that no request owns stay as they are."""
+    off = 3
+    const = walk_constants(heads, dk, kind)
+    size = heads * (dv + (1 if const.get("ones") else 0)) * dk
+    cuts = [30, 1, 1, 4, 1, 3, 2, 1, 12, 1]
+    n = sum(cuts)
+    g = walk_inputs(2 * n, heads, kq, dk, dv, 5, kind)
+    state = rnd(4, off + size + 1, seed=4, scale=0.3)
+    rstate = state.cpu().clone()
+    ctx, _, _ = batch([n, n], [0, 0], slots=[3, 1])
+    ref = run_walk(REF, g, list(range(2 * n)), rstate, off, to_cpu(ctx), heads, kq, dk, dv, const, "cpu")
+    got, pos, launches = ([], []), 0, []
+    for c in cuts:
+        ctx, _, _ = batch([c, c], [0, 0], slots=[3, 1])
+        before = ops.launches
+        out = run_walk(ops, g, list(range(pos, pos + c)) + list(range(n + pos, n + pos + c)), state, off, ctx, heads, kq, dk, dv, const)
+        launches.append(ops.launches - before)
+        got[0].append(out[:c])
+        got[1].append(out[c:])
+        pos += c
+    assert launches == [1 if c <= 4 else 2 for c in cuts]
+    assert_close(torch.cat(got[0] + got[1]), ref, torch.float32, "outputs")
+    assert_close(state, rstate, torch.float32, "states")
+    ops.check_device_errors()
+
+
 @pytest.mark.parametrize("kind,heads,kq,dk,dv", [("delta", 4, 2, 64, 48), ("head", 3, 3, 64, 70), ("delta", 2, 2, 128, 128), ("channel", 1, 1, 40, 8)])
 def test_unequal_requests_a_long_prompt_and_states_that_go_on(ops, kind, heads, kq, dk, dv):
     q_lens, slots, off = [700, 3, 1, 8, 64], [2, 0, 1, 4, 3], 7
