@@ -142,6 +142,7 @@ class GroupSpec:
     window: int                      # 0: every key is kept; w: only the last w keys are ever read
     entries: Tuple[int, ...]         # schedule entries that own a cache in this group
     tensors: Tuple = ()              # the PagedTensor descriptions of the group's entries
+    keep_first: int = 0              # with a window: the first so many positions of a request keep their pages
 
 
 class RequestCache:
@@ -152,7 +153,7 @@ class RequestCache:
         self.slot = slot
         self.length = 0                                   # positions committed
         self.tables: List[List[int]] = [[] for _ in range(num_groups)]
-        self.first_live: List[int] = [0] * num_groups     # first logical page still held
+        self.first_live: List[int] = [0] * num_groups     # first logical page still held (behind those of kept first positions)
         self.version = 0                                  # counts the changes of the block tables
         self.closed = False
 
@@ -253,7 +254,8 @@ class CacheManager:
         for g in self._window_groups:
             first = self._first_needed_page(g, rc.length)
             table = rc.tables[g]
-            for lp in range(rc.first_live[g], min(first, len(table))):
+            kept = -(-self.groups[g].keep_first // self.page_size)
+            for lp in range(max(rc.first_live[g], kept), min(first, len(table))):
                 if table[lp] >= 0:
                     self.pools[g].free(table[lp])
                     table[lp] = -1

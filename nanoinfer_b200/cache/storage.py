@@ -18,8 +18,8 @@ from .pages import CacheManager, GroupSpec
 
 
 def plan_groups(needs: Sequence[Tuple[Optional[CacheNeed], Optional[StateNeed], Optional[int]]]):
-    """Cache groups from the per-entry needs: entries that keep the same tensors with the same window
-    share a group. Returns (groups, group index of each entry or -1)."""
+    """Cache groups from the per-entry needs: entries that keep the same tensors with the same window (and kept first
+    positions) share a group. Returns (groups, group index of each entry or -1)."""
     keys: list = []
     members: List[List[int]] = []
     entry_group = []
@@ -38,7 +38,7 @@ def plan_groups(needs: Sequence[Tuple[Optional[CacheNeed], Optional[StateNeed], 
     for i, (need, _state, reads) in enumerate(needs):
         if reads is not None:
             entry_group[i] = entry_group[reads]
-    groups = [GroupSpec(k[1], tuple(m), k[0]) for k, m in zip(keys, members)]
+    groups = [GroupSpec(k[1], tuple(m), k[0], k[2]) for k, m in zip(keys, members)]
     return groups, entry_group
 
 

@@ -49,7 +49,7 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
 template <int HD, int NT>
 __device__ __forceinline__ void softmax_block(float (&s)[NT][4], unsigned (&p)[NT / 2][4], float (&o)[HD / 8][4],
                                               float (&m_run)[2], float (&l_run)[2], float scale2, int key_base,
-                                              const int (&vis_lo)[2], const int (&vis_hi)[2], int lane) {
+                                              const int (&vis_lo)[2], const int (&vis_hi)[2], int lane, int keep_first = 0) {
     const int t = lane & 3;
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
@@ -58,7 +58,7 @@ __device__ __forceinline__ void softmax_block(float (&s)[NT][4], unsigned (&p)[N
         for (int e = 0; e < 4; ++e) {
             const int r = e >> 1;
             const int key = key_base + n * 8 + 2 * t + (e & 1);
-            const bool vis = key >= vis_lo[r] && key <= vis_hi[r];
+            const bool vis = (key >= vis_lo[r] || key < keep_first) && key <= vis_hi[r];
             s[n][e] = vis ? s[n][e] * scale2 : -INFINITY;
             mx[r] = fmaxf(mx[r], s[n][e]);
         }

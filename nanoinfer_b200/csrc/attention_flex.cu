@@ -17,7 +17,9 @@
 //    slope[head] * (p - j). Keys are taken in blocks of 32 that start at absolute multiples of 32 with a running
 //    maximum and sum, so a position's result does not depend on how the request was cut into steps, nor on what else
 //    is in the batch. With `sinks` the softmax's denominator holds exp(sinks[head]) once more: a term without key and
-//    value, neither scaled nor capped. The output (dv wide per head) is multiplied by out_scale and written as float or T.
+//    value, neither scaled nor capped. With `keep_first` n the first n positions of a request are seen however far back they
+//    are. The output (dv wide per head) is multiplied by out_scale, with `gate` also by sigmoid of one number per (token, head),
+//    and written as float or T.
 #include "common.cuh"
 
 constexpr int FX_MAX_D = 256;
@@ -162,11 +164,12 @@ attention_prepare_kernel(const float* __restrict__ qkv, int ld, T* __restrict__ 
 
 // ---- the same for bfloat16 storage, eight elements a thread --------------------------------------------------------------
 // A block per token; a work item is eight consecutive elements of a head (two 16-byte loads of floats, one 16-byte store of
-// bfloat16), or, inside the rotated part of a q or k head, the eight elements at c and their mates at c + rot/2 together,
-// so that an angle's sine and cosine are formed once a pair. Takes: no norm, the norm over the whole projection, or the norm of
+// bfloat16), or, inside the rotated part of a q or k head, the eight elements at c and their mates at c + rot/2 together
+// (pairs (2i, 2i + 1): the eight elements are four pairs), so that an angle's sine and cosine are formed once a pair. Takes: no norm, the norm over the whole projection, or the norm of
 // every head where a head is 16, 32, 64 or 128 wide (the sums of squares of all heads first, a quarter of a head's width in lanes
 // each), pairs
-// (i, i + rot/2) with rot a multiple of 16, head sizes in multiples of 8, values of their own (blended or not). The token's
+// (i, i + rot/2) with rot a multiple of 16 or pairs (2i, 2i + 1) with rot a multiple of 8, head sizes in multiples of 8, values of their
+// own (blended or not) or the keys as projected. The token's
 // page and slot are looked up once. Same arithmetic per element as the kernel above.
 __device__ __forceinline__ void load8(const float* p, float (&x)[8]) {
     const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
@@ -188,7 +191,7 @@ attention_prepare_vec_kernel(const float* __restrict__ qkv, int ld, __nv_bfloat1
                              const int* __restrict__ positions, const int* __restrict__ req_index, const int* __restrict__ block_table,
                              int bt_stride, int page_size, __nv_bfloat16* __restrict__ k_pages, __nv_bfloat16* __restrict__ v_pages, int num_pages,
                              int heads, int kv_heads, int dk, int dv, int writes, const float* __restrict__ v_first, int ld_first,
-                             const float* __restrict__ vmix, int per_head_norm) {
+                             const float* __restrict__ vmix, int per_head_norm, int flags) {
     extern __shared__ float head_norm[];        // 1 / rms of every q, then every k head (norm of every head only)
     pdl_launch_dependents();
     pdl_wait();      // everything this kernel reads may come from the kernel before
@@ -231,8 +234,10 @@ attention_prepare_vec_kernel(const float* __restrict__ qkv, int ld, __nv_bfloat1
         const int page = block_table[(size_t)req_index[t] * bt_stride + pos / page_size];
         if (page >= 0 && page < num_pages) slot = (long long)page * kv_heads * page_size + (pos % page_size);   // else: a padding row of a replayed step
     }
-    const int half = rot >> 1;
-    const int per_head = half / 8 + (dk - rot) / 8;             // work items of a q or k head
+    const bool interleaved = (flags & FXP_INTERLEAVED) != 0;
+    const int half = rot >> 1, n_rot = interleaved ? rot / 8 : half / 8;
+    const int per_head = n_rot + (dk - rot) / 8;                // work items of a q or k head
+    const int v_at = (flags & FXP_VALUES_ARE_KEYS) ? nq : nq + nk;      // where a token's values stand in its row
     const int items_qk = (heads + kv_heads) * per_head, items_v = kv_heads * (dv / 8);
     const float lam = v_first != nullptr ? vmix[0] : 0.f;
     for (int it = tid; it < items_qk + items_v; it += 128) {
@@ -240,7 +245,7 @@ attention_prepare_vec_kernel(const float* __restrict__ qkv, int ld, __nv_bfloat1
             if (slot < 0) continue;
             const int c = (it - items_qk) * 8, head = c / dv, off = c - head * dv;
             float x[8];
-            load8(row + nq + nk + c, x);
+            load8(row + v_at + c, x);
             if (v_first != nullptr) {
                 float f[8];
                 load8(v_first + (size_t)t * ld_first + c, f);
@@ -260,7 +265,28 @@ attention_prepare_vec_kernel(const float* __restrict__ qkv, int ld, __nv_bfloat1
         const int gain_at = per_head_norm ? 0 : head * dk;      // a head's gain is shared by the heads
         __nv_bfloat16* dst = is_q ? q_out + (size_t)t * nq + (size_t)head * dk
                                   : k_pages + ((size_t)slot + (size_t)head * page_size) * dk;
-        if (w < half / 8) {                                     // eight rotated pairs: elements c.. and c + rot/2..
+        if (interleaved && w < n_rot) {                         // four rotated pairs side by side
+            const int c = w * 8;
+            float a[8];
+            load8(src + c, a);
+            if (gain != nullptr) {
+                float ga[8];
+                load8(gain + gain_at + c, ga);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) a[e] = a[e] * norm * ga[e];
+            }
+            const float4 fr = *reinterpret_cast<const float4*>(freq + c / 2);
+            const float f4[4] = {fr.x, fr.y, fr.z, fr.w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                float sn, cs;
+                sincosf((float)pos * f4[e], &sn, &cs);
+                const float u = a[2 * e], v = a[2 * e + 1];
+                a[2 * e] = u * cs - v * sn;
+                a[2 * e + 1] = v * cs + u * sn;
+            }
+            store8(dst + c, a);
+        } else if (w < n_rot) {                                 // eight rotated pairs: elements c.. and c + rot/2..
             const int c = w * 8;
             float a[8], b[8];
             load8(src + c, a);
@@ -285,7 +311,7 @@ attention_prepare_vec_kernel(const float* __restrict__ qkv, int ld, __nv_bfloat1
             store8(dst + c, a);
             store8(dst + c + half, b);
         } else {                                                // eight elements that are not rotated
-            const int c = rot + (w - half / 8) * 8;
+            const int c = rot + (w - n_rot) * 8;
             float a[8];
             load8(src + c, a);
             if (gain != nullptr) {
@@ -319,11 +345,11 @@ NIB_API int nib_attention_prepare(const float* qkv, int ld, void* q_out, const f
         && (q_gain == nullptr || ((uintptr_t)q_gain % 16 == 0 && (uintptr_t)k_gain % 16 == 0)) && (rot == 0 || (uintptr_t)freq % 16 == 0)
         && (v_first == nullptr || ((uintptr_t)v_first % 16 == 0 && ld_first % 4 == 0));
     const bool head_norm = q_gain != nullptr && !(flags & FXP_NORM_WHOLE) && (dk == 16 || dk == 32 || dk == 64 || dk == 128);
-    if (dtype == NIB_BF16 && tokens >= 256 && aligned16 && dk % 8 == 0 && dv % 8 == 0 && rot % 16 == 0 && (flags & ~FXP_NORM_WHOLE) == 0
+    if (dtype == NIB_BF16 && tokens >= 256 && aligned16 && dk % 8 == 0 && dv % 8 == 0 && rot % ((flags & FXP_INTERLEAVED) ? 8 : 16) == 0 && (flags & FXP_UNIT_NORM_AFTER) == 0
         && (q_gain == nullptr || (flags & FXP_NORM_WHOLE) || (head_norm && (heads + kv_heads) <= 8192))) {
         NIB_CUDA(launch_pdl(attention_prepare_vec_kernel, dim3(tokens), dim3(128), head_norm ? (size_t)(heads + kv_heads) * 4 : (size_t)0, stream, qkv, ld, (__nv_bfloat16*)q_out, q_gain, k_gain, eps, freq,
                             rot, positions, req_index, block_table, bt_stride, page_size, (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, num_pages, heads,
-                            kv_heads, dk, dv, writes, v_first, ld_first, vmix, head_norm ? 1 : 0));
+                            kv_heads, dk, dv, writes, v_first, ld_first, vmix, head_norm ? 1 : 0, flags));
         NIB_LAUNCH_CHECK();
         return 0;
     }
@@ -379,7 +405,7 @@ attention_flex_kernel(const T* __restrict__ q, int q_stride, TO* __restrict__ ou
                       const int* __restrict__ req_index, const int* __restrict__ block_table, int bt_stride, int page_size,
                       const T* __restrict__ k_pages, const T* __restrict__ v_pages, int num_pages, int m_tokens, int heads,
                       int kv_heads, int dk, int dv, float scale, float softcap, const float* __restrict__ slopes, int window,
-                      int chunk, float out_scale, const float* __restrict__ sinks) {
+                      int chunk, float out_scale, const float* __restrict__ sinks, int keep_first, const float* __restrict__ gate, int ld_gate) {
     __shared__ __align__(16) float q_s[FX_WARPS][FX_MAX_D];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long w = (long long)blockIdx.x * FX_WARPS + warp;
@@ -402,9 +428,11 @@ attention_flex_kernel(const T* __restrict__ q, int q_stride, TO* __restrict__ ou
 #pragma unroll
     for (int i = 0; i < FX_MAX_D / 32; ++i) acc[i] = 0.f;
 
-    for (int kb = (lo / 32) * 32; kb <= pos; kb += 32) {
+    const int lo_block = (lo / 32) * 32;
+    for (int kb = keep_first > 0 ? 0 : lo_block; kb <= pos; kb += 32) {
+        if (kb >= keep_first && kb < lo_block) kb = lo_block;      // between the kept tokens and the window
         const int j = kb + lane;
-        const bool valid = (j >= lo) && (j <= pos);
+        const bool valid = (j >= lo || j < keep_first) && (j <= pos);
         float s = -INFINITY;
         long long slot = -1;  // row of this lane's key in the pages: (page * kv_heads + kvh) * page_size + offset
         if (valid) {
@@ -443,7 +471,8 @@ attention_flex_kernel(const T* __restrict__ q, int q_stride, TO* __restrict__ ou
         corr_sink = (m_run == -INFINITY) ? 0.f : expf(m_run - m_new);
         l_run = l_run * corr_sink + expf(sk - m_new);
     }
-    const float inv = l_run > 0.f ? out_scale * corr_sink / l_run : 0.f;
+    float inv = l_run > 0.f ? out_scale * corr_sink / l_run : 0.f;
+    if (gate != nullptr) inv *= 1.0f / (1.0f + expf(-gate[(size_t)token * ld_gate + head]));
 #pragma unroll
     for (int i = 0; i < FX_MAX_D / 32; ++i) {
         const int d = lane + 32 * i;
@@ -457,16 +486,16 @@ NIB_API int nib_attention_flex(const void* q, int q_stride, void* out, int out_f
                                const int* block_table, int bt_stride, int page_size, const void* k_pages, const void* v_pages,
                                int num_pages, int m_tokens, int heads, int kv_heads, int dk, int dv, float scale, float softcap,
                                const float* slopes, int window, int chunk, float out_scale, const float* sinks, int dtype,
-                               cudaStream_t stream) {
+                               int keep_first, const float* gate, int ld_gate, cudaStream_t stream) {
     NIB_REQUIRE(m_tokens >= 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0, "attention: bad head counts %d / %d", heads, kv_heads);
     NIB_REQUIRE(dk > 0 && dk <= FX_MAX_D && dv > 0 && dv <= FX_MAX_D, "attention: head sizes %d / %d are outside 1..%d", dk, dv, FX_MAX_D);
-    NIB_REQUIRE(page_size > 0 && num_pages > 0 && window >= 0 && chunk >= 0 && softcap >= 0.f, "attention: bad page_size/num_pages/window/chunk/cap");
+    NIB_REQUIRE(page_size > 0 && num_pages > 0 && window >= 0 && chunk >= 0 && softcap >= 0.f && keep_first >= 0, "attention: bad page_size/num_pages/window/chunk/cap");
     if (m_tokens == 0) return 0;
     const int blocks = ceil_div((long long)m_tokens * heads, FX_WARPS);
 #define NIB_FX_LAUNCH(T, TO)                                                                                                       \
     attention_flex_kernel<T, TO><<<blocks, FX_WARPS * 32, 0, stream>>>((const T*)q, q_stride, (TO*)out, positions, req_index, block_table, \
         bt_stride, page_size, (const T*)k_pages, (const T*)v_pages, num_pages, m_tokens, heads, kv_heads, dk, dv, scale, softcap, slopes,  \
-        window, chunk, out_scale, sinks)
+        window, chunk, out_scale, sinks, keep_first, gate, ld_gate)
     if (dtype == NIB_F32) NIB_FX_LAUNCH(float, float);
     else if (dtype == NIB_BF16 && out_f32) NIB_FX_LAUNCH(__nv_bfloat16, float);
     else if (dtype == NIB_BF16) NIB_FX_LAUNCH(__nv_bfloat16, __nv_bfloat16);

@@ -10,7 +10,8 @@
 // attention_common.cuh. Key tiles start at absolute multiples of 64, so a position's result does not depend on what else
 // is in the batch; it depends on the cut only through which rows share a tile, i.e. by rounding. With `sinks` the
 // denominator of a row of head h holds exp(sinks[h]) once more (no key, no value): it enters where a row is normalized,
-// here or, with split keys, in the merge.
+// here or, with split keys, in the merge; so does `gate`, a factor sigmoid(gate[token, head]). With `keep_first` n the first n
+// positions of a request are seen however far back they are: their key tiles come ahead of the window's.
 #include "attention_common.cuh"
 
 namespace {
@@ -34,16 +35,16 @@ template <int D> struct FxTile {
 };
 
 // Rows key0..key0+63 of one kv head of a paged tensor whose rows hold `width` <= D elements; rows outside [lo, hi] or
-// without a page, and the columns from `width` on, are zero.
+// without a page, and the columns from `width` on, are zero; the first `keep` positions count as inside.
 template <int D>
 __device__ __forceinline__ void fx_load_tile(unsigned char* tile, const __nv_bfloat16* __restrict__ pages, int width,
                                              const int* __restrict__ bt, int page_size, int num_pages, int kv_heads, int kvh,
-                                             int key0, int lo, int hi, int tid) {
+                                             int key0, int lo, int hi, int keep, int tid) {
     constexpr int CPR = FxTile<D>::CPR;
     for (int i = tid; i < FB_N * CPR; i += FWARPS * 32) {
         const int r = i / CPR, c = i - r * CPR;
         const int j = key0 + r;
-        bool valid = (j >= lo) && (j <= hi) && (c * 8 < width);
+        bool valid = (j >= lo || j < keep) && (j <= hi) && (c * 8 < width);
         size_t off = 0;
         if (valid) {
             const int lp = j / page_size;
@@ -103,7 +104,7 @@ attention_flex_mma_kernel(const __nv_bfloat16* __restrict__ q_in, int q_stride, 
                           const __nv_bfloat16* __restrict__ k_pages, const __nv_bfloat16* __restrict__ v_pages, int num_pages,
                           int heads, int kv_heads, int dk, int dv, float scale, float softcap, const float* __restrict__ slopes,
                           int window, int chunk, float out_scale, int splits, float* __restrict__ part_o, float* __restrict__ part_ml,
-                          const float* __restrict__ sinks) {
+                          const float* __restrict__ sinks, int keep_first, const float* __restrict__ gate, int ld_gate) {
     extern __shared__ __align__(16) unsigned char smem[];
     const int req = blockIdx.y, kvh = blockIdx.z;
     const int n_rep = heads / kv_heads;
@@ -137,7 +138,7 @@ attention_flex_mma_kernel(const __nv_bfloat16* __restrict__ q_in, int q_stride, 
     int vis_lo[2], vis_hi[2];
     float slope2[2], sink2[2];
     const __nv_bfloat16* q_ptr[2];
-    long long out_off[2];
+    long long out_off[2], gate_off[2];
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
         const int row = row0 + warp * 16 + g + 8 * r;
@@ -150,7 +151,9 @@ attention_flex_mma_kernel(const __nv_bfloat16* __restrict__ q_in, int q_stride, 
             sink2[r] = sinks != nullptr ? sinks[head] * LOG2E : -INFINITY;
             q_ptr[r] = q_in + (size_t)(row_begin + ti) * q_stride + (size_t)head * dk;
             out_off[r] = ((long long)(row_begin + ti) * heads + head) * dv;
+            gate_off[r] = (long long)(row_begin + ti) * ld_gate + head;
         } else {
+            gate_off[r] = 0;
             vis_hi[r] = -1; vis_lo[r] = 0; slope2[r] = 0.f; sink2[r] = -INFINITY; q_ptr[r] = nullptr; out_off[r] = -1;
         }
     }
@@ -158,7 +161,10 @@ attention_flex_mma_kernel(const __nv_bfloat16* __restrict__ q_in, int q_stride, 
     const int last_row = min(rows_total, row0 + FWARPS * 16) - 1;
     const int hi_cta = pos0 + last_row / n_rep;
     const int lo_cta = first_visible(pos0 + row0 / n_rep);
-    int t_begin = lo_cta / FB_N, t_end = hi_cta / FB_N;
+    // tiles in turn: those that hold kept tokens and lie before the window's first, then the window's
+    const int t_first = lo_cta / FB_N, n_kept = min((keep_first + FB_N - 1) / FB_N, t_first);
+    auto tile_at = [&](int i) { return i < n_kept ? i : t_first + (i - n_kept); };
+    int t_begin = 0, t_end = n_kept + hi_cta / FB_N - t_first;
     if (splits > 1) {       // this CTA's share of the tiles; it may be empty
         const int per = (t_end - t_begin + splits) / splits;
         t_begin += split * per;
@@ -193,16 +199,17 @@ attention_flex_mma_kernel(const __nv_bfloat16* __restrict__ q_in, int q_stride, 
     unsigned char* v_buf[2] = {smem + 2 * FxTile<DKP>::BYTES, smem + 2 * FxTile<DKP>::BYTES + FxTile<DVP>::BYTES};
 
     if (t_begin <= t_end) {
-        fx_load_tile<DKP>(k_buf[0], k_pages, dk, bt, page_size, num_pages, kv_heads, kvh, t_begin * FB_N, lo_cta, hi_cta, tid);
-        fx_load_tile<DVP>(v_buf[0], v_pages, dv, bt, page_size, num_pages, kv_heads, kvh, t_begin * FB_N, lo_cta, hi_cta, tid);
+        fx_load_tile<DKP>(k_buf[0], k_pages, dk, bt, page_size, num_pages, kv_heads, kvh, tile_at(t_begin) * FB_N, lo_cta, hi_cta, keep_first, tid);
+        fx_load_tile<DVP>(v_buf[0], v_pages, dv, bt, page_size, num_pages, kv_heads, kvh, tile_at(t_begin) * FB_N, lo_cta, hi_cta, keep_first, tid);
     }
     fx_commit();
 
-    for (int tile = t_begin; tile <= t_end; ++tile) {
-        const int cur = (tile - t_begin) & 1;
-        if (tile < t_end) {
-            fx_load_tile<DKP>(k_buf[cur ^ 1], k_pages, dk, bt, page_size, num_pages, kv_heads, kvh, (tile + 1) * FB_N, lo_cta, hi_cta, tid);
-            fx_load_tile<DVP>(v_buf[cur ^ 1], v_pages, dv, bt, page_size, num_pages, kv_heads, kvh, (tile + 1) * FB_N, lo_cta, hi_cta, tid);
+    for (int turn = t_begin; turn <= t_end; ++turn) {
+        const int cur = (turn - t_begin) & 1, tile = tile_at(turn);
+        if (turn < t_end) {
+            const int next = tile_at(turn + 1) * FB_N;
+            fx_load_tile<DKP>(k_buf[cur ^ 1], k_pages, dk, bt, page_size, num_pages, kv_heads, kvh, next, lo_cta, hi_cta, keep_first, tid);
+            fx_load_tile<DVP>(v_buf[cur ^ 1], v_pages, dv, bt, page_size, num_pages, kv_heads, kvh, next, lo_cta, hi_cta, keep_first, tid);
         }
         fx_commit();
         fx_wait<1>();
@@ -230,7 +237,7 @@ attention_flex_mma_kernel(const __nv_bfloat16* __restrict__ q_in, int q_stride, 
             }
         }
         unsigned p[FB_N / 16][4];
-        softmax_block<DVP, FB_N / 8>(s, p, o, m_run, l_run, 1.0f, tile * FB_N, vis_lo, vis_hi, lane);
+        softmax_block<DVP, FB_N / 8>(s, p, o, m_run, l_run, 1.0f, tile * FB_N, vis_lo, vis_hi, lane, keep_first);
         fx_pv<DVP>(o, p, v_buf[cur], lane);
         __syncthreads();    // the tile may be overwritten by the load issued in the next iteration
     }
@@ -259,7 +266,8 @@ attention_flex_mma_kernel(const __nv_bfloat16* __restrict__ q_in, int q_stride, 
             corr = (m_run[r] == -INFINITY) ? 0.f : exp2f(m_run[r] - m_new);
             l_run[r] = l_run[r] * corr + exp2f(sink2[r] - m_new);
         }
-        const float inv = l_run[r] > 0.f ? out_scale * corr / l_run[r] : 0.f;
+        float inv = l_run[r] > 0.f ? out_scale * corr / l_run[r] : 0.f;
+        if (gate != nullptr) inv *= 1.0f / (1.0f + expf(-gate[gate_off[r]]));
         TO* orow = out + out_off[r];
 #pragma unroll
         for (int d = 0; d < DVP / 8; ++d)
@@ -271,7 +279,7 @@ attention_flex_mma_kernel(const __nv_bfloat16* __restrict__ q_in, int q_stride, 
 template <typename TO>
 __global__ void __launch_bounds__(128)
 attention_flex_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, TO* __restrict__ out, int splits, int dv,
-                            float out_scale, const float* __restrict__ sinks, int heads) {
+                            float out_scale, const float* __restrict__ sinks, int heads, const float* __restrict__ gate, int ld_gate) {
     pdl_wait();
     const size_t row = blockIdx.x;      // token * heads + head
     const float sink2 = sinks != nullptr ? sinks[row % heads] * LOG2E : -INFINITY;
@@ -282,7 +290,8 @@ attention_flex_merge_kernel(const float* __restrict__ part_o, const float* __res
         const float ms = part_ml[(row * splits + s) * 2];
         if (ms != -INFINITY) l += part_ml[(row * splits + s) * 2 + 1] * exp2f(ms - m);
     }
-    const float inv = l > 0.f ? out_scale / l : 0.f;
+    float inv = l > 0.f ? out_scale / l : 0.f;
+    if (gate != nullptr) inv *= 1.0f / (1.0f + expf(-gate[(row / heads) * ld_gate + row % heads]));
     for (int d = threadIdx.x; d < dv; d += 128) {
         float acc = 0.f;
         for (int s = 0; s < splits; ++s) {
@@ -297,7 +306,7 @@ template <int DKP, int DVP, typename TO>
 int fx_launch(const void* q, int q_stride, void* out, const int* q_start, const int* ctx_lens, const int* block_table, int bt_stride,
               int page_size, const void* k_pages, const void* v_pages, int num_pages, int n_req, int max_q_len, int heads, int kv_heads,
               int dk, int dv, float scale, float softcap, const float* slopes, int window, int chunk, float out_scale, int splits,
-              float* part_o, float* part_ml, int m_tokens, const float* sinks, cudaStream_t stream) {
+              float* part_o, float* part_ml, int m_tokens, const float* sinks, int keep_first, const float* gate, int ld_gate, cudaStream_t stream) {
     static bool configured = false;
     const int smem = 2 * FxTile<DKP>::BYTES + 2 * FxTile<DVP>::BYTES;
     if (!configured) {
@@ -309,10 +318,10 @@ int fx_launch(const void* q, int q_stride, void* out, const int* q_start, const 
     NIB_CUDA(launch_pdl(attention_flex_mma_kernel<DKP, DVP, TO>, grid, dim3(FWARPS * 32), (size_t)smem, stream, (const __nv_bfloat16*)q, q_stride,
                         (TO*)out, q_start, ctx_lens, block_table, bt_stride, page_size, (const __nv_bfloat16*)k_pages,
                         (const __nv_bfloat16*)v_pages, num_pages, heads, kv_heads, dk, dv, scale, softcap, slopes, window, chunk, out_scale,
-                        splits, part_o, part_ml, sinks));
+                        splits, part_o, part_ml, sinks, keep_first, gate, ld_gate));
     if (splits > 1)
         NIB_CUDA(launch_pdl(attention_flex_merge_kernel<TO>, dim3(m_tokens * heads), dim3(128), (size_t)0, stream, (const float*)part_o,
-                            (const float*)part_ml, (TO*)out, splits, dv, out_scale, sinks, heads));
+                            (const float*)part_ml, (TO*)out, splits, dv, out_scale, sinks, heads, gate, ld_gate));
     return 0;
 }
 
@@ -331,9 +340,10 @@ NIB_API int nib_attention_flex_mma(const void* q, int q_stride, void* out, int o
                                    const int* block_table, int bt_stride, int page_size, const void* k_pages, const void* v_pages,
                                    int num_pages, int n_req, int max_q_len, int heads, int kv_heads, int dk, int dv, float scale,
                                    float softcap, const float* slopes, int window, int chunk, float out_scale, int splits, float* part_o,
-                                   float* part_ml, int m_tokens, const float* sinks, cudaStream_t stream) {
+                                   float* part_ml, int m_tokens, const float* sinks, int keep_first, const float* gate, int ld_gate,
+                                   cudaStream_t stream) {
     NIB_REQUIRE(nib_attention_flex_mma_supported(heads, kv_heads, dk, dv, q_stride) == 1, "attention (tensor cores): head sizes %d / %d or head counts %d / %d are not taken", dk, dv, heads, kv_heads);
-    NIB_REQUIRE(n_req >= 0 && max_q_len > 0 && page_size > 0 && num_pages > 0 && window >= 0 && chunk >= 0 && softcap >= 0.f, "attention (tensor cores): bad sizes");
+    NIB_REQUIRE(n_req >= 0 && max_q_len > 0 && page_size > 0 && num_pages > 0 && window >= 0 && chunk >= 0 && softcap >= 0.f && keep_first >= 0, "attention (tensor cores): bad sizes");
     NIB_REQUIRE(splits <= 1 || (max_q_len * (heads / kv_heads) <= 64 && part_o != nullptr && part_ml != nullptr),
                 "attention (tensor cores): keys are split over CTAs only when a request's rows fit one tile, and with scratch");
     if (n_req == 0) return 0;
@@ -341,11 +351,11 @@ NIB_API int nib_attention_flex_mma(const void* q, int q_stride, void* out, int o
     do {                                                                                                                                    \
         const int rc = out_f32 ? fx_launch<DKP, DVP, float>(q, q_stride, out, q_start, ctx_lens, block_table, bt_stride, page_size, k_pages, \
                                                             v_pages, num_pages, n_req, max_q_len, heads, kv_heads, dk, dv, scale, softcap,   \
-                                                            slopes, window, chunk, out_scale, splits, part_o, part_ml, m_tokens, sinks, stream) \
+                                                            slopes, window, chunk, out_scale, splits, part_o, part_ml, m_tokens, sinks, keep_first, gate, ld_gate, stream) \
                                    : fx_launch<DKP, DVP, __nv_bfloat16>(q, q_stride, out, q_start, ctx_lens, block_table, bt_stride,         \
                                                                         page_size, k_pages, v_pages, num_pages, n_req, max_q_len, heads,     \
                                                                         kv_heads, dk, dv, scale, softcap, slopes, window, chunk, out_scale,  \
-                                                                        splits, part_o, part_ml, m_tokens, sinks, stream);                   \
+                                                                        splits, part_o, part_ml, m_tokens, sinks, keep_first, gate, ld_gate, stream);                   \
         if (rc != 0) return rc;                                                                                                             \
     } while (0)
     if (dk <= 64 && dv <= 64) NIB_FXM(64, 64);

@@ -23,8 +23,10 @@
 // A second instance of the kernel (FLEX) takes the options that other designs put on the scores: a soft cap
 // c tanh(s / c) (monotone, so the row's maximum is still the cap of the largest raw score; applied to every score in
 // 32-bit with the fast exponential and division before the exponent of the softmax), a chunked mask (a position sees its
-// own block of `chunk` positions, counted from the request's start), and a sink per head (exp(sink) once more in the
-// denominator, added where the row is divided by its sum). The instance without options is compiled without any of it.
+// own block of `chunk` positions, counted from the request's start), a sink per head (exp(sink) once more in the
+// denominator, added where the row is divided by its sum), kept first tokens (the first `keep_first` positions are seen however far
+// back they are: their key blocks come ahead of the window's), and a gate per (token, head) (a factor sigmoid(gate) where the row is
+// divided by its sum). The instance without options is compiled without any of it.
 //
 // Formula as in attention_generic.cu (cpp/src/ops.cpp:206-270); the reference's prefill attention is a
 // SIMT kernel with 32-key shared-memory slabs (cpp/src/cuda/cuda_backend.cu:489-575).
@@ -94,7 +96,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                             const int* __restrict__ q_start, const int* __restrict__ ctx_lens,
                             const int* __restrict__ block_table, int bt_stride, int page_size, int num_pages,
                             int heads, int kv_heads, float scale, int window, unsigned long long* trace, int trace_cap,
-                            float softcap, int chunk, const float* __restrict__ sinks, float out_scale) {
+                            float softcap, int chunk, const float* __restrict__ sinks, float out_scale, int keep_first,
+                            const float* __restrict__ gate, int ld_gate) {
     using C = Cfg<HD>;
     constexpr int KEYS = C::KEYS, STAGES = C::STAGES;
     extern __shared__ unsigned char smem_raw[];
@@ -130,7 +133,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const int hi_cta = pos0 + n_tok - 1;
     int lo_cta = window > 0 ? max(0, pos0 - window + 1) : 0;
     if (FLEX && chunk > 0) lo_cta = max(lo_cta, (pos0 / chunk) * chunk);      // (the first visible key never decreases with the position)
-    const int b_begin = lo_cta / KEYS, n_blk = hi_cta / KEYS - b_begin + 1;
+    const int b_begin = lo_cta / KEYS;
+    const int n_kept = FLEX ? min((keep_first + KEYS - 1) / KEYS, b_begin) : 0;      // key blocks with kept tokens before the window's first
+    const int n_blk = n_kept + hi_cta / KEYS - b_begin + 1;
+    auto block_at = [&](int j) { return FLEX && j < n_kept ? j : b_begin + j - n_kept; };
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int* bt = block_table + (size_t)req * bt_stride;
 
@@ -177,8 +183,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         // asked for while block j is being sent for and is looked at only a block later: the look-up's latency (more
         // than half a microsecond) must not stand between two blocks' copies.
         auto entry_of = [&](int j) -> int {
-            const int key = (b_begin + j) * KEYS + lane * page_size;
-            if (lane >= pages_per_block || key > hi_cta || key + page_size <= lo_cta) return -1;
+            const int key = block_at(j) * KEYS + lane * page_size;
+            if (lane >= pages_per_block || key > hi_cta || (key + page_size <= lo_cta && !(FLEX && key < keep_first))) return -1;
             return __ldg(bt + key / page_size);
         };
         int entry_next = entry_of(0);
@@ -306,7 +312,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             ok = __all_sync(0xffffffffu, ok);
             if (!ok) break;
             tc_fence_after();
-            const int key0 = (b_begin + j) * KEYS;
+            const int key0 = block_at(j) * KEYS;
             // the same branch for the whole warp: a warp that took both would do the work twice
             const bool all_visible = __all_sync(0xffffffffu, key0 >= lo && key0 + KEYS - 1 <= hi);
             // this thread's scores of the block: all loads are issued, then waited for once (a load from tensor memory
@@ -334,7 +340,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
                     for (int i = 0; i < 32; ++i) {
                         const int key = key0 + half * HK + c * 32 + i;
-                        if (!(key >= lo && key <= hi)) raw[c][i] = 0xff800000u;      // -inf: its probability will be 0
+                        if (!((key >= lo || (FLEX && key < keep_first)) && key <= hi)) raw[c][i] = 0xff800000u;      // -inf: its probability will be 0
                         mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(raw[c][i]));
                     }
                 }
@@ -424,7 +430,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             tc_fence_after();
             float l_all = xch[4 * 128 + row] + xch[5 * 128 + row];
             if (FLEX && sinks != nullptr && m_cur != -INFINITY) l_all += ex2(__ldg(sinks + head) * LOG2E - m_cur);   // the sink: no key, no value
-            const float inv = l_all > 0.f ? out_scale / l_all : 0.f;
+            float inv = l_all > 0.f ? out_scale / l_all : 0.f;
+            if (FLEX && gate != nullptr) inv *= 1.0f / (1.0f + expf(-gate[(size_t)(row_begin + tok0 + ti) * ld_gate + head]));
             __nv_bfloat16* orow = out + ((size_t)(row_begin + tok0 + ti) * heads + head) * HD + half * (HD / 2);
 #pragma unroll
             for (int c = 0; c < HD / 64; ++c) {
@@ -475,7 +482,7 @@ template <int HD, bool FLEX>
 int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, void* out, const int* q_start,
            const int* ctx_lens, const int* block_table, int bt_stride, int page_size, int num_pages, int n_req,
            int max_q_len, int heads, int kv_heads, float scale, int window, float softcap, int chunk, const float* sinks,
-           float out_scale, cudaStream_t stream) {
+           float out_scale, int keep_first, const float* gate, int ld_gate, cudaStream_t stream) {
     static bool configured = false;
     if (!configured) {
         NIB_CUDA(cudaFuncSetAttribute(attention_prefill_tc_kernel<HD, FLEX>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg<HD>::SMEM));
@@ -485,7 +492,7 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, 
     dim3 grid(ceil_div(max_q_len, tpt), n_req, kv_heads);
     NIB_CUDA(launch_pdl(attention_prefill_tc_kernel<HD, FLEX>, grid, dim3(THREADS), (size_t)Cfg<HD>::SMEM, stream, mq, mk, mv,
                         (__nv_bfloat16*)out, q_start, ctx_lens, block_table, bt_stride, page_size, num_pages, heads,
-                        kv_heads, scale, window, nib_trace_buffer(), nib_trace_capacity(), softcap, chunk, sinks, out_scale));
+                        kv_heads, scale, window, nib_trace_buffer(), nib_trace_capacity(), softcap, chunk, sinks, out_scale, keep_first, gate, ld_gate));
     return 0;
 }
 
@@ -511,15 +518,17 @@ NIB_API int nib_attention_tc_error() {
 }
 
 // Same arguments as nib_attention_prefill_mma plus the number of rows of qkv (m_tokens, for the map's extent), and the
-// options: softcap (0 = none), chunk (0 = none), sinks [heads] (null = none), a factor on the output (32-bit, before it is rounded).
+// options: softcap (0 = none), chunk (0 = none), sinks [heads] (null = none), a factor on the output (32-bit, before it is rounded),
+// keep_first (0 = none), gate [tokens, heads] with rows of ld_gate floats (null = none).
 NIB_API int nib_attention_prefill_tc(const void* qkv, int q_stride, void* out, const int* q_start, const int* ctx_lens,
                                      const int* block_table, int bt_stride, int page_size, const void* k_pages,
                                      const void* v_pages, int num_pages, int n_req, int max_q_len, int m_tokens,
                                      int heads, int kv_heads, int head_dim, float scale, int window, float softcap, int chunk,
-                                     const float* sinks, float out_scale, cudaStream_t stream) {
+                                     const float* sinks, float out_scale, int keep_first, const float* gate, int ld_gate,
+                                     cudaStream_t stream) {
     NIB_REQUIRE(nib_attention_prefill_tc_supported(heads, kv_heads, head_dim, page_size, q_stride),
                 "attention (tcgen05): head_dim %d, %d/%d heads, page size %d are not supported", head_dim, heads, kv_heads, page_size);
-    NIB_REQUIRE(n_req >= 0 && max_q_len > 0 && num_pages > 0 && window >= 0 && m_tokens > 0 && chunk >= 0 && softcap >= 0.f && scale > 0.f,
+    NIB_REQUIRE(n_req >= 0 && max_q_len > 0 && num_pages > 0 && window >= 0 && m_tokens > 0 && chunk >= 0 && softcap >= 0.f && scale > 0.f && keep_first >= 0,
                 "attention (tcgen05): bad sizes");
     NIB_REQUIRE((((uintptr_t)qkv | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)out) & 15) == 0, "attention (tcgen05): bases must be 16-byte aligned");
     NIB_REQUIRE(n_req <= 65535 && kv_heads <= 65535, "attention (tcgen05): too many requests or kv heads for one launch");
@@ -533,8 +542,8 @@ NIB_API int nib_attention_prefill_tc(const void* qkv, int q_stride, void* out, c
     if (make_map3(&mk, k_pages, head_dim, page_size, planes, head_dim, (long long)page_size * head_dim, page_size, 1)) return 1;
     if (make_map3(&mv, v_pages, head_dim, page_size, planes, head_dim, (long long)page_size * head_dim, page_size, 1)) return 1;
 #define NIB_TC_ATTN(HD, FLEX) launch<HD, FLEX>(mq, mk, mv, out, q_start, ctx_lens, block_table, bt_stride, page_size, num_pages, n_req, max_q_len, \
-                                               heads, kv_heads, scale, window, softcap, chunk, sinks, out_scale, stream)
-    const bool flex = softcap > 0.f || chunk > 0 || sinks != nullptr;
+                                               heads, kv_heads, scale, window, softcap, chunk, sinks, out_scale, keep_first, gate, ld_gate, stream)
+    const bool flex = softcap > 0.f || chunk > 0 || sinks != nullptr || (keep_first > 0 && window > 0) || gate != nullptr;
     if (head_dim == 64) return flex ? NIB_TC_ATTN(64, true) : NIB_TC_ATTN(64, false);
     return flex ? NIB_TC_ATTN(128, true) : NIB_TC_ATTN(128, false);
 #undef NIB_TC_ATTN

@@ -57,9 +57,10 @@ __device__ __forceinline__ float warp_max(float v) {
 }
 
 // Epilogues of the matrix products (the `epi` argument): STORE in the storage type, ADD into floats, F32 floats, SWIGLU
-// silu(gate) * up from two accumulators, QKV see the products; GLU the gated form with constants (NibGlu).
-enum NibEpi : int { EPI_STORE = 0, EPI_ADD = 1, EPI_F32 = 2, EPI_SWIGLU = 3, EPI_QKV = 4, EPI_GLU = 5 };
-__host__ __device__ constexpr bool epi_dual(int epi) { return epi == EPI_SWIGLU || epi == EPI_GLU; }     // two accumulators
+// silu(gate) * up from two accumulators, QKV see the products; GLU the gated form with constants (NibGlu); GEGLU
+// gelu(gate) * up with the tanh form of gelu.
+enum NibEpi : int { EPI_STORE = 0, EPI_ADD = 1, EPI_F32 = 2, EPI_SWIGLU = 3, EPI_QKV = 4, EPI_GLU = 5, EPI_GEGLU = 6 };
+__host__ __device__ constexpr bool epi_dual(int epi) { return epi == EPI_SWIGLU || epi == EPI_GLU || epi == EPI_GEGLU; }     // two accumulators
 
 // The gated product with constants: g = min(gate, limit), u = clamp(up, -limit, limit), g * sigmoid(alpha * g) * (u + shift).
 struct NibGlu { float alpha, limit, shift; };
@@ -74,6 +75,13 @@ __device__ __forceinline__ float nib_glu_fast(const NibGlu& p, float g, float u)
     u = fminf(fmaxf(u, -p.limit), p.limit);
     return __fdividef(g, 1.0f + __expf(-p.alpha * g)) * (u + p.shift);
 }
+
+// gelu(g) * u, gelu(g) = g (1 + tanh(y)) / 2 with y = sqrt(2/pi) (g + 0.044715 g^3). As (1 + tanh(y)) / 2 = 1 / (1 + e^(-2y)) it
+// costs one exponential and one division; 2 sqrt(2/pi) = 1.595769122.
+__device__ __forceinline__ float nib_gelu_twice_y(float g) { return 1.5957691216057308f * fmaf(0.044715f * g * g, g, g); }
+__device__ __forceinline__ float nib_geglu_exact(float g, float u) { return g / (1.0f + expf(-nib_gelu_twice_y(g))) * u; }
+// the fast exponential and division (2 ulp), for results that are rounded to bfloat16
+__device__ __forceinline__ float nib_geglu_fast(float g, float u) { return __fdividef(g, 1.0f + __expf(-nib_gelu_twice_y(g))) * u; }
 
 static inline int ceil_div(long long a, long long b) { return (int)((a + b - 1) / b); }
 

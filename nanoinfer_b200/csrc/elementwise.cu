@@ -179,6 +179,140 @@ NIB_API int nib_rmsnorm(const float* x, const float* gain, const int* rows, void
     return 0;
 }
 
+// ---------------------------------------------------------------------------------- LayerNorm
+// (x - mean) / sqrt(variance + eps) * gain + bias per row, the variance as the mean of the squared deviations (a second pass over
+// the row, which no cancellation can spoil). A block per row; fixed order of additions.
+template <typename T, int THREADS>
+__global__ void __launch_bounds__(THREADS)
+layernorm_kernel(const float* __restrict__ x, const float* __restrict__ gain, const float* __restrict__ bias, const int* __restrict__ rows,
+                 T* __restrict__ out, int hidden, float eps) {
+    __shared__ float part[2][THREADS / 32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int r = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const float* xr = x + (size_t)(rows ? rows[r] : r) * hidden;
+    auto block_sum = [&](float v, int slot) {
+        v = warp_sum(v);
+        if (lane == 0) part[slot][warp] = v;
+        __syncthreads();
+        return warp_sum(lane < THREADS / 32 ? part[slot][lane] : 0.f);
+    };
+    float sum = 0.f;
+    for (int c = threadIdx.x; c < hidden; c += THREADS) sum += xr[c];
+    const float mean = block_sum(sum, 0) / (float)hidden;
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < hidden; c += THREADS) {
+        const float d = xr[c] - mean;
+        ss = fmaf(d, d, ss);
+    }
+    const float scale = 1.0f / sqrtf(block_sum(ss, 1) / (float)hidden + eps);
+    T* o = out + (size_t)r * hidden;
+    for (int c = threadIdx.x; c < hidden; c += THREADS) Elem<T>::store(o + c, fmaf((xr[c] - mean) * scale, gain[c], bias[c]));
+}
+
+// A warp per row, the row in registers between the sums (widths that are multiples of 4 up to 128 * NV): read once, 16 bytes a
+// load. WARPS > 1: that many warps share a row (a step of few rows would otherwise leave a warp alone with NV loads and its sums).
+template <typename T, int NV, int WARPS>
+__global__ void __launch_bounds__(256)
+layernorm_rows_kernel(const float* __restrict__ x, const float* __restrict__ gain, const float* __restrict__ bias, const int* __restrict__ rows,
+                      T* __restrict__ out, int n_rows, int hidden, float eps) {
+    __shared__ float part[2][WARPS];
+    pdl_launch_dependents();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int r = WARPS > 1 ? blockIdx.x : blockIdx.x * (blockDim.x >> 5) + warp;
+    const int first = WARPS > 1 ? warp * 32 + lane : lane;
+    constexpr int STEP = 32 * WARPS;
+    const int n4 = hidden >> 2;
+    float4 g[NV], b[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {       // weights: fetched before the wait
+        const int c = first + STEP * i;
+        g[i] = c < n4 ? __ldg(reinterpret_cast<const float4*>(gain) + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        b[i] = c < n4 ? __ldg(reinterpret_cast<const float4*>(bias) + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    pdl_wait();
+    if (r >= n_rows) return;
+    auto row_sum = [&](float v, int slot) {
+        v = warp_sum(v);
+        if constexpr (WARPS > 1) {
+            if (lane == 0) part[slot][warp] = v;
+            __syncthreads();
+            v = 0.f;
+#pragma unroll
+            for (int w = 0; w < WARPS; ++w) v += part[slot][w];
+        }
+        return v;
+    };
+    const float4* xr = reinterpret_cast<const float4*>(x + (size_t)(rows ? rows[r] : r) * hidden);
+    float4 v[NV];
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = first + STEP * i;
+        v[i] = c < n4 ? xr[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) sum += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+    const float mean = row_sum(sum, 0) / (float)hidden;
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        if (first + STEP * i >= n4) continue;
+        v[i].x -= mean; v[i].y -= mean; v[i].z -= mean; v[i].w -= mean;
+        ss = fmaf(v[i].x, v[i].x, ss); ss = fmaf(v[i].y, v[i].y, ss);
+        ss = fmaf(v[i].z, v[i].z, ss); ss = fmaf(v[i].w, v[i].w, ss);
+    }
+    const float scale = 1.0f / sqrtf(row_sum(ss, 1) / (float)hidden + eps);
+    T* o = out + (size_t)r * hidden;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = first + STEP * i;
+        if (c >= n4) continue;
+        const float y0 = fmaf(v[i].x * scale, g[i].x, b[i].x), y1 = fmaf(v[i].y * scale, g[i].y, b[i].y);
+        const float y2 = fmaf(v[i].z * scale, g[i].z, b[i].z), y3 = fmaf(v[i].w * scale, g[i].w, b[i].w);
+        if constexpr (sizeof(T) == 4) {
+            reinterpret_cast<float4*>(o)[c] = make_float4(y0, y1, y2, y3);
+        } else {
+            __nv_bfloat162 lo = __floats2bfloat162_rn(y0, y1), hi = __floats2bfloat162_rn(y2, y3);
+            uint2 pk;
+            pk.x = *reinterpret_cast<unsigned*>(&lo);
+            pk.y = *reinterpret_cast<unsigned*>(&hi);
+            reinterpret_cast<uint2*>(o)[c] = pk;
+        }
+    }
+}
+
+template <typename T>
+int launch_layernorm(const float* x, const float* gain, const float* bias, const int* rows, T* out, int n_rows, int hidden, float eps,
+                     cudaStream_t stream) {
+    const bool vec = hidden % 4 == 0 && hidden <= 4096 && (((uintptr_t)x | (uintptr_t)gain | (uintptr_t)bias | (uintptr_t)out) & 15) == 0;
+    if (!vec) {
+        NIB_CUDA(launch_pdl(layernorm_kernel<T, 256>, dim3(n_rows), dim3(256), (size_t)0, stream, x, gain, bias, rows, out, hidden, eps));
+        return 0;
+    }
+#define NIB_LN(NV, WARPS, GRID, THREADS) \
+    NIB_CUDA(launch_pdl(layernorm_rows_kernel<T, NV, WARPS>, dim3(GRID), dim3(THREADS), (size_t)0, stream, x, gain, bias, rows, out, n_rows, hidden, eps))
+    // which form runs depends on the width alone, so that a row's result does not depend on what else is in the batch
+    if (hidden <= 128 * 4) NIB_LN(4, 1, ceil_div(n_rows, 4), 128);
+    else if (hidden <= 128 * 8) NIB_LN(2, 4, n_rows, 128);
+    else if (hidden <= 128 * 16) NIB_LN(4, 4, n_rows, 128);
+    else NIB_LN(4, 8, n_rows, 256);
+#undef NIB_LN
+    return 0;
+}
+
+NIB_API int nib_layernorm(const float* x, const float* gain, const float* bias, const int* rows, void* out, int n_rows, int hidden, float eps,
+                          int dtype, cudaStream_t stream) {
+    NIB_REQUIRE(n_rows >= 0 && hidden > 0, "layernorm: bad sizes rows=%d hidden=%d", n_rows, hidden);
+    NIB_REQUIRE(dtype == NIB_F32 || dtype == NIB_BF16, "layernorm: unknown dtype %d", dtype);
+    if (n_rows == 0) return 0;
+    const int rc = dtype == NIB_F32 ? launch_layernorm<float>(x, gain, bias, rows, (float*)out, n_rows, hidden, eps, stream)
+                                    : launch_layernorm<__nv_bfloat16>(x, gain, bias, rows, (__nv_bfloat16*)out, n_rows, hidden, eps, stream);
+    if (rc) return rc;
+    NIB_LAUNCH_CHECK();
+    return 0;
+}
+
 // ---------------------------------------------------------------------------------- rotation + page write
 // qkv row layout: [heads | kv_heads | kv_heads] x head_dim. Queries and keys are rotated in place
 // (pairs d, d + rot/2 for d < rot/2; elements >= rot are left as they are); rotated keys and the

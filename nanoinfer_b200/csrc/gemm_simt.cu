@@ -8,7 +8,8 @@
 //
 // Epilogues: STORE (T out = acc + bias), ADD (float out += acc + bias: the residual sum),
 // F32 (float out = acc + bias: logits), SWIGLU (two accumulators, W rows n and n + N:
-// T out = silu(gate) * up, silu(g) = g / (1 + exp(-g)), cpp/src/ops.cpp:86-93), GLU (the same with limits and constants).
+// T out = silu(gate) * up, silu(g) = g / (1 + exp(-g)), cpp/src/ops.cpp:86-93), GLU (the same with limits and constants),
+// GEGLU (gelu(gate) * up).
 #include "common.cuh"
 
 template <typename T, int EPI>
@@ -100,7 +101,7 @@ gemm_simt_kernel(const T* __restrict__ A, const T* __restrict__ W, const float* 
                 ((float*)out)[o] = v;
             } else {
                 const float g = v, u = acc2[DUAL ? i : 0][DUAL ? j : 0];
-                Elem<T>::store((T*)out + o, EPI == EPI_GLU ? nib_glu_exact(glu, g, u) : g / (1.0f + expf(-g)) * u);
+                Elem<T>::store((T*)out + o, EPI == EPI_GLU ? nib_glu_exact(glu, g, u) : EPI == EPI_GEGLU ? nib_geglu_exact(g, u) : g / (1.0f + expf(-g)) * u);
             }
         }
     }
@@ -117,6 +118,7 @@ static int launch_simt(const void* A, const void* W, const float* bias, void* ou
         case EPI_F32: gemm_simt_kernel<T, EPI_F32><<<grid, block, 0, stream>>>((const T*)A, (const T*)W, bias, out, M, N, K, lda, ldo, glu); break;
         case EPI_SWIGLU: gemm_simt_kernel<T, EPI_SWIGLU><<<grid, block, 0, stream>>>((const T*)A, (const T*)W, bias, out, M, N, K, lda, ldo, glu); break;
         case EPI_GLU: gemm_simt_kernel<T, EPI_GLU><<<grid, block, 0, stream>>>((const T*)A, (const T*)W, bias, out, M, N, K, lda, ldo, glu); break;
+        case EPI_GEGLU: gemm_simt_kernel<T, EPI_GEGLU><<<grid, block, 0, stream>>>((const T*)A, (const T*)W, bias, out, M, N, K, lda, ldo, glu); break;
         default: nib_set_error("gemm: unknown epilogue %d", epi); return 1;
     }
     NIB_LAUNCH_CHECK();
@@ -124,7 +126,7 @@ static int launch_simt(const void* A, const void* W, const float* bias, void* ou
 }
 
 // A [M, K] with row stride lda; W [N, K] (SWIGLU: [2N, K], gate rows then up rows); out [M, N] with
-// row stride ldo. epi: 0 store, 1 add into float, 2 store float, 3 swiglu, 5 the gated form with the constants glu.
+// row stride ldo. epi: 0 store, 1 add into float, 2 store float, 3 swiglu, 5 the gated form with the constants glu, 6 geglu.
 NIB_API int nib_gemm_simt(const void* A, const void* W, const float* bias, void* out, int M, int N, int K,
                           int lda, int ldo, int epi, int dtype, const NibGlu* glu, cudaStream_t stream) {
     NIB_REQUIRE(M >= 0 && N > 0 && K > 0 && lda >= K && ldo >= N, "gemm: bad sizes M=%d N=%d K=%d lda=%d ldo=%d", M, N, K, lda, ldo);

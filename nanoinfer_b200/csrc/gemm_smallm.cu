@@ -382,6 +382,7 @@ gemm_smallm_kernel(const void* __restrict__ A, const __nv_bfloat16* __restrict__
             else if (EPI == EPI_F32) ((float*)out)[o] = x;
             else if (EPI == EPI_SWIGLU) ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(__fdividef(x, 1.0f + __expf(-x)) * (v[ACCS - 1][e] * scale2[e & 1]));
             else if (EPI == EPI_GLU) ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(nib_glu_fast(glu, x, v[ACCS - 1][e] * scale2[e & 1]));
+            else if (EPI == EPI_GEGLU) ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(nib_geglu_fast(x, v[ACCS - 1][e] * scale2[e & 1]));
         }
     };
 
@@ -443,6 +444,7 @@ int launch_epi(int epi, const Args& a, cudaStream_t stream) {
         case EPI_F32: return launch_one<NT, KSPLIT, EPI_F32, NORM>(a, stream);
         case EPI_SWIGLU: return launch_one<NT, KSPLIT, EPI_SWIGLU, NORM>(a, stream);
         case EPI_GLU: return launch_one<NT, KSPLIT, EPI_GLU, NORM>(a, stream);
+        case EPI_GEGLU: return launch_one<NT, KSPLIT, EPI_GEGLU, NORM>(a, stream);
         case EPI_QKV:
             if constexpr (KSPLIT > 1) return launch_one<NT, KSPLIT, EPI_QKV, NORM>(a, stream);
             break;

@@ -95,6 +95,10 @@ __device__ __forceinline__ void emit_row16(void* __restrict__ out, const float (
 #pragma unroll
         for (int j = 0; j < 16; ++j) x[j] = nib_glu_fast(glu, x[j], u[j]);
     }
+    if (EPI == EPI_GEGLU) {
+#pragma unroll
+        for (int j = 0; j < 16; ++j) x[j] = nib_geglu_fast(x[j], u[j]);
+    }
     if (vec_ok && first + 16 <= n_out) {
         if (EPI == EPI_STORE || epi_dual(EPI)) {
             uint4 p0, p1;
@@ -216,6 +220,7 @@ __device__ __forceinline__ void emit16(void* __restrict__ out, const float (&v)[
             if (EPI == EPI_STORE) ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(x);
             else if (EPI == EPI_F32) ((float*)out)[o] = x;
             else if (EPI == EPI_GLU) ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(nib_glu_fast(glu, x, u[j]));
+            else if (EPI == EPI_GEGLU) ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(nib_geglu_fast(x, u[j]));
             else ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(__fdividef(x, 1.0f + __expf(-x)) * u[j]);
         }
     }
@@ -804,6 +809,9 @@ int launch_tc_epi(int epi, const CUtensorMap& mw, const CUtensorMap& ma, const f
         case EPI_GLU:
             if constexpr (TOK <= 128) return launch_tc<TOK, EPI_GLU>(mw, ma, bias, out, tokens, n_out, k, ldo, sk, stream, 0, QkvRows{}, glu);
             break;
+        case EPI_GEGLU:
+            if constexpr (TOK <= 128) return launch_tc<TOK, EPI_GEGLU>(mw, ma, bias, out, tokens, n_out, k, ldo, sk, stream);
+            break;
     }
     nib_set_error("gemm (tensor cores): unknown epilogue %d", epi);
     return 1;
@@ -841,6 +849,7 @@ int launch_pair_epi(int epi, const CUtensorMap& mm, const CUtensorMap& mn, const
         case EPI_F32: return launch_pair<NT, EPI_F32>(mm, mn, bias, out, tokens, n_out, k, ldo, vec_ok, splits, stream);
         case EPI_SWIGLU: return launch_pair<NT, EPI_SWIGLU>(mm, mn, bias, out, tokens, n_out, k, ldo, vec_ok, splits, stream);
         case EPI_GLU: return launch_pair<NT, EPI_GLU>(mm, mn, bias, out, tokens, n_out, k, ldo, vec_ok, splits, stream, glu);
+        case EPI_GEGLU: return launch_pair<NT, EPI_GEGLU>(mm, mn, bias, out, tokens, n_out, k, ldo, vec_ok, splits, stream);
     }
     nib_set_error("gemm (tensor cores, two SMs per tile): unknown epilogue %d", epi);
     return 1;
@@ -865,7 +874,7 @@ NIB_API int nib_gemm_tc_error() {
 }
 
 // A [tokens, K] bfloat16 with row stride lda; W [N, K] (SWIGLU: [2N, K]); out [tokens, N] with row
-// stride ldo. epi: 0 store bf16, 1 add into float, 2 store float, 3 swiglu, 5 the gated form with the constants glu. tok_tile: 0 = chosen here.
+// stride ldo. epi: 0 store bf16, 1 add into float, 2 store float, 3 swiglu, 5 the gated form with the constants glu, 6 geglu. tok_tile: 0 = chosen here.
 // splits: work items per output tile along K; 0 = chosen here (more than one only when the tiles alone
 // leave SMs idle and the scratch holds the partial sums), 1 = none. scratch/counters: a float buffer and
 // a zeroed int buffer that the kernels of one stream share (the counters are left zeroed).
@@ -1017,7 +1026,7 @@ NIB_API int nib_gemm_tc_pair(const void* A, const void* W, const float* bias, vo
     NIB_REQUIRE(!epi_dual(epi) || bias == nullptr, "gemm (two SMs per tile): the gated epilogues take no bias");
     NIB_REQUIRE(epi != EPI_GLU || glu != nullptr, "gemm (two SMs per tile): the gated epilogue needs its constants");
     const NibGlu constants = glu != nullptr ? *glu : NibGlu{};
-    NIB_REQUIRE((epi >= EPI_STORE && epi <= EPI_SWIGLU) || epi == EPI_GLU, "gemm (two SMs per tile): unknown epilogue %d", epi);
+    NIB_REQUIRE((epi >= EPI_STORE && epi <= EPI_SWIGLU) || epi == EPI_GLU || epi == EPI_GEGLU, "gemm (two SMs per tile): unknown epilogue %d", epi);
     NIB_REQUIRE(((uintptr_t)bias & 15) == 0, "gemm (two SMs per tile): the bias must be 16-byte aligned");
     if (tokens == 0) return 0;
     if (n_tile == 0) n_tile = 256;      // measured: the instruction of 128 columns runs at about half the rate, whatever the grid

@@ -22,8 +22,8 @@ class KernelError(RuntimeError):
 
 
 _DT = {torch.float32: 0, torch.bfloat16: 1}
-_EPI = {"store": 0, "add": 1, "f32": 2, "swiglu": 3, "glu": 5}
-_DUAL = (3, 5)          # the gated epilogues: two accumulators, gate rows and up rows
+_EPI = {"store": 0, "add": 1, "f32": 2, "swiglu": 3, "glu": 5, "geglu": 6}
+_DUAL = (3, 5, 6)       # the gated epilogues: two accumulators, gate rows and up rows
 _LAYOUT = {"interleaved": 0, "half": 1}     # which elements of a rotated vector make a pair
 
 
@@ -132,9 +132,10 @@ class Kernels:
                      "nib_linear_state_scan", "nib_conv_tokens", "nib_conv_tail", "nib_conv_step", "nib_token_shift", "nib_decay_map", "nib_step_sizes",
                      "nib_attention_prepare", "nib_attention_flex", "nib_attention_flex_mma", "nib_attention_flex_mma_supported",
                      "nib_rmsnorm_add", "nib_moe_route", "nib_moe_max_tiles", "nib_moe_group", "nib_moe_gemm_simt", "nib_moe_combine",
-                     "nib_moe_tc_supported", "nib_moe_tc_error", "nib_moe_gather_rows", "nib_moe_gemm_tc", "nib_moe_step", "nib_moe_step_supported", "nib_moe_identity", "nib_stream_mix", "nib_grouped_state_scan", "nib_grouped_state_error", "nib_pdl_skip_next", "nib_memory_gates"):
+                     "nib_moe_tc_supported", "nib_moe_tc_error", "nib_moe_gather_rows", "nib_moe_gemm_tc", "nib_moe_step", "nib_moe_step_supported", "nib_moe_identity", "nib_stream_mix", "nib_grouped_state_scan", "nib_grouped_state_error", "nib_pdl_skip_next", "nib_memory_gates", "nib_layernorm",
+                     "nib_decay_state_scan", "nib_decay_state_chunks_supported"):
             getattr(self._lib, name).restype = c_int
-        self._lib.nib_grouped_state_scratch.restype = c_longlong
+        self._lib.nib_grouped_state_scratch.restype = self._lib.nib_decay_state_scratch.restype = c_longlong
 
     # ---- plumbing ---------------------------------------------------------------------------
     def _check(self, rc: int, what: str) -> None:
@@ -246,6 +247,19 @@ class Kernels:
         self._check(self._lib.nib_rmsnorm(_ptr(x32), _ptr(gain32), _ptr(rows), _ptr(out), c_int(n), c_int(hidden),
                                           c_float(eps), c_int(_DT[out.dtype]), c_int(1 if self._norm_before_small_m else 0),
                                           self._stream()), "rmsnorm")
+
+    def layernorm(self, x32, gain32, bias32, eps, out, rows=None):
+        """out = (x32 - mean) / sqrt(variance + eps) * gain32 + bias32 row by row (of the rows that ``rows`` names)."""
+        _need(x32, torch.float32, "layernorm x"); _need(gain32, torch.float32, "layernorm gain"); _need(bias32, torch.float32, "layernorm bias")
+        _need(out, None, "layernorm out")
+        if rows is not None:
+            _need(rows, torch.int32, "layernorm rows")
+        n, hidden = out.shape
+        if x32.shape[1] != hidden or gain32.numel() != hidden or bias32.numel() != hidden or (rows is None and x32.shape[0] != n) \
+                or (rows is not None and rows.numel() != n):
+            raise KernelError("layernorm: shapes do not fit")
+        self._check(self._lib.nib_layernorm(_ptr(x32), _ptr(gain32), _ptr(bias32), _ptr(rows), _ptr(out), c_int(n), c_int(hidden), c_float(eps),
+                                            c_int(_DT[out.dtype]), self._stream()), "layernorm")
 
     def with_options(self, options: Optional[KernelOptions] = None, **changes) -> "Kernels":
         """Another instance on the same library and the same scratch memory (so: for use on the same stream) whose
@@ -393,8 +407,8 @@ class Kernels:
         """The error word of the tensor-core GEMM's bounded waits (0 = none); synchronises and clears it."""
         return self._lib.nib_gemm_tc_error()
 
-    def linear_swiglu(self, a, w_gate_up, out, glu=None):
-        """out[M,I] = silu(a . w[:I]^T) * (a . w[I:]^T). With ``glu`` = (alpha, limit, shift): g = min(gate, limit),
+    def linear_swiglu(self, a, w_gate_up, out, glu=None, act="silu"):
+        """out[M,I] = silu(a . w[:I]^T) * (a . w[I:]^T), with ``act`` 'gelu_tanh' gelu (its tanh form) in place of silu. With ``glu`` = (alpha, limit, shift): g = min(gate, limit),
         u = clamp(up, -limit, limit), g * sigmoid(alpha g) * (u + shift)."""
         if not isinstance(a, LazyNorm):
             _need(a, None, "swiglu a")
@@ -403,7 +417,10 @@ class Kernels:
         inter = w_gate_up.shape[0] // 2
         if w_gate_up.shape[0] != 2 * inter or w_gate_up.shape[1] != k or tuple(out.shape) != (m, inter):
             raise KernelError("linear_swiglu: shapes do not fit")
-        self._gemm(a, w_gate_up, None, out, m, inter, k, _EPI["swiglu" if glu is None else "glu"], _glu(glu))
+        if act not in ("silu", "gelu_tanh") or (glu is not None and act != "silu"):
+            raise KernelError(f"linear_swiglu: no gated form with '{act}'" + (" and constants" if glu is not None else ""))
+        epi = "geglu" if act == "gelu_tanh" else ("swiglu" if glu is None else "glu")
+        self._gemm(a, w_gate_up, None, out, m, inter, k, _EPI[epi], _glu(glu))
 
     def qkv_project(self, a, w_qkv, bias32, qkv, heads, kv_heads, head_dim, positions, req_index, rotary,
                     block_table, page_size, k_pages, v_pages, writes):
@@ -572,7 +589,7 @@ class Kernels:
                     _ptr(qkv), c_int(qkv.stride(0)), _ptr(out), q_start, lens, table, c_int(bt_stride), c_int(page_size),
                     _ptr(k_pages), _ptr(v_pages), c_int(num_pages), c_int(n_req - n_dec), c_int(max(q_lens[n_dec:])),
                     c_int(m), c_int(heads), c_int(kv_heads), c_int(head_dim), c_float(scale), c_int(window), c_float(0.0), c_int(0), None,
-                    c_float(1.0), self._stream()), "attention prefill (tcgen05)")
+                    c_float(1.0), c_int(0), None, c_int(0), self._stream()), "attention prefill (tcgen05)")
             else:
                 self._check(self._lib.nib_attention_prefill_mma(
                     _ptr(qkv), c_int(qkv.stride(0)), _ptr(out), q_start, lens, table, c_int(bt_stride), c_int(page_size),
@@ -683,12 +700,12 @@ class Kernels:
                                                       self._stream()), "depth_mix + rmsnorm (two gains)")
 
     def unary(self, in32, out, kind):
-        """out = f(in32) element by element with a change of storage type; kind: 'tanh' | 'copy' | 'sigmoid'."""
+        """out = f(in32) element by element with a change of storage type; kind: 'tanh' | 'copy' | 'sigmoid' | 'silu'."""
         self._rows(in32, torch.float32, "unary in"); self._rows(out, None, "unary out")
         if in32.shape != out.shape:
             raise KernelError("unary: shapes differ")
         self._check(self._lib.nib_unary(_ptr(in32), c_int(in32.stride(0)), _ptr(out), c_int(out.stride(0)), c_int(in32.shape[0]),
-                                        c_int(in32.shape[1]), c_int({"tanh": 0, "copy": 1, "sigmoid": 2}[kind]),
+                                        c_int(in32.shape[1]), c_int({"tanh": 0, "copy": 1, "sigmoid": 2, "silu": 3}[kind]),
                                         c_int(_DT[out.dtype]), self._stream()), "unary")
 
     def head_norm_gate(self, o32, gate32, gain32, eps, heads, d, out):
@@ -1020,6 +1037,82 @@ class Kernels:
             c_int(heads), c_int(kq_heads), c_int(dk), c_int(dv), c_float(q_scale), c_int(n_seg), c_int(seg_len if n_seg > 1 else 0), _ptr(scratch),
             self._stream()), "linear_state_scan")
 
+    # ---- matrix states with one decay per head: short steps token by token, prompts in chunks (decay_state.cu) --------------------
+    STEP_TOKENS = 16        # what a request may bring at most to a step that is taken token by token
+
+    def decay_state_scan(self, q32, k32, v32, state, state_off, ctx, o32, heads, kq_heads, dk, dv, act="none", decay32=None, raw32=None,
+                         dt_bias32=None, a_log32=None, exact=False):
+        """Per request and head, over the step's tokens in order, from and into ``state[slot, state_off:]`` (laid out [head, value
+        channel, key channel]): S <- d S + f k v^T, o = S^T q. q32, k32: [tokens, kq_heads * dk] (head h reads head h // (heads /
+        kq_heads)); v32, o32: [tokens, heads * dv]; ``act`` 'silu': q, k and v pass silu first. Fixed decays: ``decay32`` [2, heads], the
+        decays and their logarithms to the base 2, f = 1. Step sizes: f = softplus(raw32 + dt_bias32), d = exp(-exp(a_log32) f) with raw32
+        [tokens, heads] (f is also the factor on v).
+
+        A step in which no request brings more than STEP_TOKENS tokens goes token by token in 32-bit (one launch). Longer ones are taken
+        in chunks of 64 tokens on the tensor cores, where q, k and v enter as bfloat16 and everything else is 32-bit (three launches);
+        leading requests of one token go token by token beside them. ``exact`` (or sizes that the chunks do not take): the 32-bit walk
+        of ``linear_state_scan`` in place of the chunks."""
+        m = q32.shape[0]
+        for t, what, width in ((q32, "q", kq_heads * dk), (k32, "k", kq_heads * dk), (v32, "v", heads * dv), (o32, "o", heads * dv)):
+            self._rows(t, torch.float32, f"decay_state_scan {what}")
+            if tuple(t.shape) != (m, width):
+                raise KernelError(f"decay_state_scan: {what} does not fit")
+        if (decay32 is None) == (raw32 is None) or act not in ("none", "silu"):
+            raise KernelError("decay_state_scan: either fixed decays or step sizes; act is 'none' or 'silu'")
+        if raw32 is not None:
+            self._rows(raw32, torch.float32, "decay_state_scan raw")
+            _need(dt_bias32, torch.float32, "decay_state_scan bias"); _need(a_log32, torch.float32, "decay_state_scan a_log")
+            if tuple(raw32.shape) != (m, heads) or dt_bias32.numel() != heads or a_log32.numel() != heads:
+                raise KernelError("decay_state_scan: step sizes are [tokens, heads], their bias and rates [heads]")
+        else:
+            _need(decay32, torch.float32, "decay_state_scan decay")
+            if tuple(decay32.shape) != (2, heads):
+                raise KernelError("decay_state_scan: fixed decays are [2, heads]: the decays and their logarithms")
+        self._state_row(state, state_off, heads * dv * dk, "decay_state_scan state")
+        q_lens = ctx.host.q_lens
+        n_req, longest = len(q_lens), max(q_lens)
+        short = longest <= self.STEP_TOKENS
+        if not short and (exact or self._lib.nib_decay_state_chunks_supported(c_int(dk), c_int(dv)) != 1):
+            self._decay_state_exact(q32, k32, v32, state, state_off, ctx, o32, heads, kq_heads, dk, dv, act, decay32, raw32, dt_bias32, a_log32)
+            return
+        n_step = n_req if short else next((i for i, n in enumerate(q_lens) if n != 1), n_req)
+
+        def scan(first, count, tokens, most, scratch, what):
+            self._check(self._lib.nib_decay_state_scan(
+                _ptr(q32), c_int(q32.stride(0)), _ptr(k32), c_int(k32.stride(0)), _ptr(v32), c_int(v32.stride(0)), _ptr(raw32),
+                c_int(0 if raw32 is None else raw32.stride(0)), _ptr(dt_bias32), _ptr(a_log32), _ptr(None if decay32 is None else decay32[0]),
+                _ptr(None if decay32 is None else decay32[1]), c_int(1 if act == "silu" else 0), _ptr(state), c_longlong(state.stride(0)),
+                c_int(state_off), c_void_p(ctx.q_start.data_ptr() + 4 * first), c_void_p(ctx.state_slots.data_ptr() + 4 * first), _ptr(o32),
+                c_int(o32.stride(0)), c_int(tokens), c_int(count), c_int(most), c_int(heads), c_int(kq_heads), c_int(dk), c_int(dv), _ptr(scratch),
+                self._stream()), what)
+
+        if n_step:
+            scan(0, n_step, sum(q_lens[:n_step]), longest if short else 1, None, "decay_state_scan (short step)")
+        if n_step < n_req:
+            tokens, count = sum(q_lens[n_step:]), n_req - n_step
+            floats = self._lib.nib_decay_state_scratch(c_longlong(tokens), c_int(count), c_int(heads), c_int(dk), c_int(dv))
+            scratch = torch.empty(floats, dtype=torch.float32, device=q32.device)
+            self.launches += 2
+            scan(n_step, count, tokens, longest, scratch, "decay_state_scan (chunks)")
+
+    def _decay_state_exact(self, q32, k32, v32, state, state_off, ctx, o32, heads, kq_heads, dk, dv, act, decay32, raw32, dt_bias32, a_log32):
+        """The same in 32-bit whatever the length, from the unfused operations."""
+        m, dev = q32.shape[0], q32.device
+        if act == "silu":
+            q32, k32, v32 = (self._unary_new(t, "silu") for t in (q32, k32, v32))
+        step = None
+        if raw32 is not None:
+            step, decay = torch.empty((2, m, heads), dtype=torch.float32, device=dev).unbind(0)
+            self.step_sizes(raw32, dt_bias32, a_log32, step, decay)
+        else:
+            decay = decay32[:1].expand(m, heads)        # every row the same one
+        self.linear_state_scan(q32, k32, v32, decay, state, state_off, ctx, o32, heads, kq_heads, dk, dv, v_scale32=step)
+
+    def _unary_new(self, t32, kind):
+        out = torch.empty(t32.shape, dtype=torch.float32, device=t32.device)
+        self.unary(t32, out, kind)
+        return out
+
     def memory_gates(self, zi32, zf32, bi32, bf32, cap, state, state_off, ctx, decay32, write32, floor32):
         """Gates of a stabilized matrix memory, per (token, head): i = cap * tanh((zi32 + bi32) / cap), f = log sigmoid(cap *
         tanh((zf32 + bf32) / cap)), m_t = max(f + m_(t-1), i) from ``state[slot, state_off + head]`` (which becomes the last
@@ -1214,12 +1307,14 @@ class Kernels:
             _ptr(vmix32 if v_first32 is not None else None), self._stream()), "attention_prepare")
 
     def attention_flex(self, q, out, heads, kv_heads, dim, vdim, scale, softcap, slopes32, window, chunk, out_scale, ctx,
-                       block_table, page_size, k_pages, v_pages, sinks32=None):
+                       block_table, page_size, k_pages, v_pages, sinks32=None, keep_first=0, gate32=None):
         """Softmax attention of every token of the step over its request's cached keys: j <= own position, within
         ``window`` (0 = none) and within the own block of ``chunk`` positions (0 = none); score = (q . k) * scale, capped
         by ``softcap`` * tanh(. / softcap) (0 = none), minus slopes32[head] * distance (None = none). ``out``
         [tokens, heads * vdim] in float or the storage type, times ``out_scale``. With ``sinks32`` [heads] the softmax's
-        denominator holds exp(sinks32[head]) once more (no key, no value, neither scaled nor capped)."""
+        denominator holds exp(sinks32[head]) once more (no key, no value, neither scaled nor capped). The first ``keep_first``
+        positions of a request are seen whatever the window and the block are. With ``gate32`` [tokens, heads] (rows of any stride) head
+        h's output is multiplied by sigmoid(gate32[:, h])."""
         _need(q, None, "attention q"); _need(out, None, "attention out")
         _need(k_pages, q.dtype, "k_pages"); _need(v_pages, q.dtype, "v_pages"); _need(block_table, torch.int32, "block_table", contiguous=False)
         m = q.shape[0]
@@ -1236,8 +1331,17 @@ class Kernels:
             _need(sinks32, torch.float32, "attention sinks")
             if sinks32.numel() != heads:
                 raise KernelError("attention_flex: one sink per head")
+        ld_gate = 0
+        if gate32 is not None:
+            self._rows(gate32, torch.float32, "attention gate")
+            if tuple(gate32.shape) != (m, heads):
+                raise KernelError("attention_flex: one gate per (token, head)")
+            ld_gate = gate32.stride(0)
+        if keep_first < 0:
+            raise KernelError("attention_flex: a negative number of kept positions")
+        more = (c_int(keep_first), _ptr(gate32), c_int(ld_gate))
         n_rep = heads // max(1, kv_heads)
-        if q.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and dim == vdim and slopes32 is None \
+        if q.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and dim == vdim and slopes32 is None and scale > 0 \
                 and max(ctx.host.q_lens) * n_rep > 64 and not self.options.force_general_attention and not self.options.force_mma_prefill \
                 and self._lib.nib_attention_prefill_tc_supported(c_int(heads), c_int(kv_heads), c_int(dim), c_int(page_size), c_int(q.stride(0))) == 1:
             # prompt portions with heads of 64 or 128 (keys and values alike): the tcgen05 kernel's instance with options
@@ -1245,7 +1349,7 @@ class Kernels:
                 _ptr(q), c_int(q.stride(0)), _ptr(out), _ptr(ctx.q_start), _ptr(ctx.ctx_lens), _ptr(block_table), c_int(block_table.stride(0)),
                 c_int(page_size), _ptr(k_pages), _ptr(v_pages), c_int(k_pages.shape[0]), c_int(ctx.host.num_requests), c_int(max(ctx.host.q_lens)),
                 c_int(m), c_int(heads), c_int(kv_heads), c_int(dim), c_float(scale), c_int(window), c_float(softcap), c_int(chunk), _ptr(sinks32),
-                c_float(out_scale), self._stream()), "attention (options, tcgen05)")
+                c_float(out_scale), *more, self._stream()), "attention (options, tcgen05)")
             return
         if q.dtype == torch.bfloat16 and not self.options.force_general_attention and page_size > 0 \
                 and self._lib.nib_attention_flex_mma_supported(c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim), c_int(q.stride(0))) == 1:
@@ -1256,7 +1360,7 @@ class Kernels:
                 # tile after tile; two tiles per CTA are both in flight at once
                 keys = max(ctx.host.ctx_lens)
                 for bound in (window, chunk):
-                    keys = min(keys, bound) if bound > 0 else keys
+                    keys = min(keys, bound + keep_first) if bound > 0 else keys
                 most = max(1, (4 * max(1, self.sm_count)) // max(1, ctx.host.num_requests * kv_heads))
                 splits = self.options.fixed_decode_splits or max(1, min(-(-(keys // 64 + 1) // 2), most, 32))
                 if splits > 1:
@@ -1268,13 +1372,13 @@ class Kernels:
                 _ptr(block_table), c_int(block_table.stride(0)), c_int(page_size), _ptr(k_pages), _ptr(v_pages), c_int(k_pages.shape[0]),
                 c_int(ctx.host.num_requests), c_int(max(ctx.host.q_lens)), c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim), c_float(scale),
                 c_float(softcap), _ptr(slopes32), c_int(window), c_int(chunk), c_float(out_scale), c_int(splits), _ptr(part_o), _ptr(part_ml),
-                c_int(m), _ptr(sinks32), self._stream()), "attention (options, tensor cores)")
+                c_int(m), _ptr(sinks32), *more, self._stream()), "attention (options, tensor cores)")
             return
         self._check(self._lib.nib_attention_flex(
             _ptr(q), c_int(q.stride(0)), _ptr(out), c_int(1 if out.dtype == torch.float32 else 0), _ptr(ctx.positions), _ptr(ctx.req_index),
             _ptr(block_table), c_int(block_table.stride(0)), c_int(page_size), _ptr(k_pages), _ptr(v_pages), c_int(k_pages.shape[0]), c_int(m),
             c_int(heads), c_int(kv_heads), c_int(dim), c_int(vdim), c_float(scale), c_float(softcap), _ptr(slopes32), c_int(window), c_int(chunk),
-            c_float(out_scale), _ptr(sinks32), c_int(_DT[q.dtype]), self._stream()), "attention (options)")
+            c_float(out_scale), _ptr(sinks32), c_int(_DT[q.dtype]), *more, self._stream()), "attention (options)")
 
     # ---- recurrent mixers (recurrent.cu) -------------------------------------------------------------
     def delta_rule_scan(self, r32, k32, v32, a_logit32, w_logit32, state, ctx, o32, heads, d):

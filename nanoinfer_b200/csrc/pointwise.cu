@@ -105,7 +105,7 @@ NIB_API int nib_depth_mix(float* hist, float* x, const float* coef, int n, long 
 }
 
 // ---------------------------------------------------------------------------------- unary function + cast
-// out[t, c] = f(in[t, c]) for c < width; kind 0: tanh, 1: identity, 2: sigmoid.
+// out[t, c] = f(in[t, c]) for c < width; kind 0: tanh, 1: identity, 2: sigmoid, 3: silu.
 template <typename T>
 __global__ void unary_kernel(const float* __restrict__ in, int ld_in, T* __restrict__ out, int ld_out, int rows, int width, int kind) {
     pdl_launch_dependents();
@@ -116,12 +116,13 @@ __global__ void unary_kernel(const float* __restrict__ in, int ld_in, T* __restr
     float v = in[(size_t)t * ld_in + c];
     if (kind == 0) v = tanhf(v);
     else if (kind == 2) v = 1.0f / (1.0f + expf(-v));
+    else if (kind == 3) v = v / (1.0f + expf(-v));
     Elem<T>::store(out + (size_t)t * ld_out + c, v);
 }
 
 NIB_API int nib_unary(const float* in, int ld_in, void* out, int ld_out, int rows, int width, int kind, int dtype,
                       cudaStream_t stream) {
-    NIB_REQUIRE(rows >= 0 && width > 0 && kind >= 0 && kind <= 2, "unary: bad arguments");
+    NIB_REQUIRE(rows >= 0 && width > 0 && kind >= 0 && kind <= 3, "unary: bad arguments");
     if (rows == 0) return 0;
     const int blocks = ceil_div((long long)rows * width, 256);
     if (dtype == NIB_F32) NIB_CUDA(launch_pdl(unary_kernel<float>, dim3(blocks), dim3(256), (size_t)(0), stream, in, ld_in, (float*)out, ld_out, rows, width, kind));

@@ -59,9 +59,11 @@ class PagedTensor:
 class CacheNeed:
     """What a mixer keeps per token: any number of paged tensors (keys and values; keys alone; one latent; keys and
     values of different widths), all addressed through one block table. ``window`` 0 = every position is kept,
-    ``w`` = only the last ``w`` positions are ever read, so pages behind them are given back."""
+    ``w`` = only the last ``w`` positions are ever read, so pages behind them are given back; with ``keep_first`` n the
+    first n positions of a request are read as well and keep their pages."""
     tensors: Tuple[PagedTensor, ...]
     window: int = 0
+    keep_first: int = 0
 
     @staticmethod
     def keys_and_values(kv_heads: int, head_dim: int, window: int = 0) -> "CacheNeed":
@@ -70,7 +72,7 @@ class CacheNeed:
 
     def group_key(self):
         """Entries with equal keys share a cache group (one block table per request)."""
-        return (self.tensors, self.window)
+        return (self.tensors, self.window, self.keep_first if self.window else 0)
 
 
 @dataclass(frozen=True)

@@ -1,6 +1,7 @@
 """SwiGLU feed-forward: ``down( silu(gate(h)) * up(h) )``, no biases, added to the residual stream. With constants
 (``glu`` = (alpha, limit, shift)): ``g = min(gate(h), limit)``, ``u = clamp(up(h), -limit, limit)``,
-``down( g sigmoid(alpha g) (u + shift) )``.
+``down( g sigmoid(alpha g) (u + shift) )``. With ``act`` "gelu_tanh": ``down( gelu(gate(h)) * up(h) )`` with the tanh form
+``gelu(z) = z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))) / 2``.
 
 ``silu(g) = g / (1 + exp(-g))`` in 32-bit. Reference: cpp/src/model.cpp:217-223,
 cpp/src/ops.cpp:86-100, nanoinfer/layers.py:243-258.
@@ -17,19 +18,21 @@ from .spec import PartSpec, TensorSpec
 
 
 class SwiGLU(FeedForward):
-    """params: ``hidden``, ``intermediate``, optionally ``glu`` (alpha, limit, shift). tensors: ``gate_w up_w [intermediate, hidden]``,
-    ``down_w [hidden, intermediate]``."""
+    """params: ``hidden``, ``intermediate``, optionally ``glu`` (alpha, limit, shift) or ``act``. tensors: ``gate_w up_w [intermediate,
+    hidden]``, ``down_w [hidden, intermediate]``."""
 
     graph_safe = True   # launches do not depend on which requests are in the batch
     accepts_lazy_norm = True   # its first projection can apply the norm while reading its input
 
     @staticmethod
     def spec(prefix: str, hidden: int, intermediate: int,
-             names=("gate_proj.weight", "up_proj.weight", "down_proj.weight"), glu=None) -> PartSpec:
+             names=("gate_proj.weight", "up_proj.weight", "down_proj.weight"), glu=None, act: str = "silu") -> PartSpec:
         """``names``: what the gate, up and down matrices are called behind ``prefix``."""
         params = {"hidden": hidden, "intermediate": intermediate}
         if glu is not None:
             params["glu"] = tuple(float(x) for x in glu)
+        if act != "silu":
+            params["act"] = str(act)
         return PartSpec("swiglu", params, {
             "gate_w": TensorSpec(f"{prefix}.{names[0]}", (intermediate, hidden)),
             "up_w": TensorSpec(f"{prefix}.{names[1]}", (intermediate, hidden)),
@@ -40,14 +43,18 @@ class SwiGLU(FeedForward):
         super().__init__(spec, tensors, rt)
         self.hidden = int(spec.params["hidden"])
         self.intermediate = int(spec.params["intermediate"])
-        self.glu = spec.params.get("glu")
+        self.glu, self.act = spec.params.get("glu"), str(spec.params.get("act", "silu"))
+        if self.act not in ("silu", "gelu_tanh") or (self.act != "silu" and self.glu is not None):
+            raise ValueError(f"unknown activation '{self.act}', or one that takes no constants")
         # One fused operand: rows [gate | up].
         self.w_gate_up = rt.matrix(torch.cat([tensors["gate_w"], tensors["up_w"]], dim=0))
         self.w_down = rt.matrix(tensors["down_w"])
 
     def forward(self, h: torch.Tensor, residual32: torch.Tensor, ctx: StepContext) -> None:
         act = torch.empty((h.shape[0], self.intermediate), dtype=self.rt.dtype, device=h.device)
-        if self.glu is None:
+        if self.act != "silu":
+            self.ops.linear_swiglu(h, self.w_gate_up, act, act=self.act)
+        elif self.glu is None:
             self.ops.linear_swiglu(h, self.w_gate_up, act)
         else:
             self.ops.linear_swiglu(h, self.w_gate_up, act, self.glu)

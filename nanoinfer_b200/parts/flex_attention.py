@@ -1,6 +1,6 @@
 """Softmax attention over the paged cache with the options that decoder designs combine: keys and values of
 different widths, a short causal convolution on q, k and v, a per-head RMS norm of q and k, rotation of part of a head,
-a bias by distance, a soft cap on the scores, a window or a chunked mask, a sigmoid gate on the output.
+a bias by distance, a soft cap on the scores, a window (with kept first tokens) or a chunked mask, a sigmoid gate on the output.
 
 With ``q = W_q h + b_q`` (likewise k, v), in this order:
 
@@ -21,10 +21,11 @@ With ``q = W_q h + b_q`` (likewise k, v), in this order:
   rotation (``vdim`` = ``dim``);
 * ``score = (q . k) * scale``; with ``softcap`` c: ``c tanh(score / c)``; with ``slope_span`` s: head h of H loses
   ``2^(-s (h + 1) / H) * (i - j)`` at distance i - j;
-* position i sees j <= i; with ``window`` w only j > i - w; with ``chunk`` c only ``floor(j / c) == floor(i / c)``,
-  counted from the request's position 0;
+* position i sees j <= i; with ``window`` w only j > i - w, and with ``keep_first`` n also j < n (at its true distance); with
+  ``chunk`` c only ``floor(j / c) == floor(i / c)``, counted from the request's position 0;
 * softmax in 32-bit; with ``sink`` the denominator holds ``exp(sink_h)`` once more, a learned number per head without
-  key or value, neither scaled nor capped; weighted sum of v (``vdim`` wide), times ``sigmoid(W_g h)`` with ``out_gate``, then
+  key or value, neither scaled nor capped; weighted sum of v (``vdim`` wide), times ``sigmoid(W_g h)`` with ``out_gate`` (a number
+  per output channel; with ``out_gate`` "head" one per head, inside the attention's kernel), then
   ``out_scale * (W_o . + b_o)`` is added to the residual stream.
 
 What is cached per position is the key after convolution, norm and rotation, and the value after convolution.
@@ -55,8 +56,8 @@ def rotary_frequencies(dims: int, base: float, factor: float = 1.0, scaling=None
 
 class FlexAttention(ProjectedMixer):
     """params: ``hidden heads kv_heads dim vdim scale eps`` and the options ``bias`` (q, k, v), ``out_bias``, ``conv``
-    (taps), ``qk_norm``, ``rot`` ((dims, base) or None), ``softcap``, ``slope_span``, ``window``, ``chunk``,
-    ``out_gate``, ``out_scale``, ``rot_layout``, ``rot_factor``, ``rot_scaling``, ``unit_norm_after_rot``, ``values_from_keys``, ``sink``,
+    (taps), ``qk_norm``, ``rot`` ((dims, base) or None), ``softcap``, ``slope_span``, ``window``, ``keep_first``, ``chunk``,
+    ``out_gate`` (False, True or "head"), ``out_scale``, ``rot_layout``, ``rot_factor``, ``rot_scaling``, ``unit_norm_after_rot``, ``values_from_keys``, ``sink``,
     ``v_mix`` (None, "first" or "blend"), ``joint_input`` (the input product is made by a pair for both of its halves). tensors: ``q k o``, ``v`` unless the values are the keys, and, by option,
     ``q_b k_b v_b o_b q_conv k_conv v_conv q_norm k_norm g sink vmix``."""
 
@@ -66,9 +67,9 @@ class FlexAttention(ProjectedMixer):
     @staticmethod
     def spec(prefix: str, hidden: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, eps: float, *,
              bias: bool = False, out_bias: bool = False, conv: int = 0, qk_norm: bool = False, rot=None,
-             softcap: float = 0.0, slope_span: float = 0.0, window: int = 0, chunk: int = 0, out_gate: bool = False,
+             softcap: float = 0.0, slope_span: float = 0.0, window: int = 0, chunk: int = 0, out_gate=False,
              out_scale: float = 1.0, rot_layout: str = "half", rot_factor: float = 1.0, rot_scaling=None, unit_norm_after_rot: bool = False,
-             values_from_keys: bool = False, sink: bool = False, v_mix=None) -> PartSpec:
+             values_from_keys: bool = False, sink: bool = False, v_mix=None, keep_first: int = 0) -> PartSpec:
         """``qk_norm``: False, True (per head, a gain of the head's size) or "whole"."""
         nq, nk, nv = heads * dim, kv_heads * dim, kv_heads * vdim
         t = {"q": TensorSpec(f"{prefix}.q", (nq, hidden)), "k": TensorSpec(f"{prefix}.k", (nk, hidden)),
@@ -93,14 +94,15 @@ class FlexAttention(ProjectedMixer):
         if v_mix == "blend":
             t["vmix"] = TensorSpec(f"{prefix}.vmix", (), "mix01")
         if out_gate:
-            t["g"] = TensorSpec(f"{prefix}.g", (heads * vdim, hidden))
+            t["g"] = TensorSpec(f"{prefix}.g", (heads if out_gate == "head" else heads * vdim, hidden))
         params = {"hidden": hidden, "heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": float(scale),
                   "eps": float(eps), "bias": bias, "out_bias": out_bias, "conv": int(conv), "qk_norm": qk_norm,
                   "rot": None if rot is None else (int(rot[0]), float(rot[1])), "softcap": float(softcap),
                   "slope_span": float(slope_span), "window": int(window), "chunk": int(chunk), "out_gate": out_gate,
                   "out_scale": float(out_scale), "rot_layout": str(rot_layout), "rot_factor": float(rot_factor),
                   "unit_norm_after_rot": bool(unit_norm_after_rot), "values_from_keys": bool(values_from_keys),
-                  "sink": bool(sink), "v_mix": v_mix, "rot_scaling": dict(rot_scaling) if rot_scaling else None}
+                  "sink": bool(sink), "v_mix": v_mix, "rot_scaling": dict(rot_scaling) if rot_scaling else None,
+                  "keep_first": int(keep_first)}
         return PartSpec("flex_attention", params, t)
 
     def __init__(self, spec: PartSpec, tensors: Dict[str, torch.Tensor], rt: Runtime):
@@ -113,6 +115,9 @@ class FlexAttention(ProjectedMixer):
         self.scale, self.eps, self.out_scale = float(p["scale"]), float(p["eps"]), float(p.get("out_scale", 1.0))
         self.taps, self.softcap = int(p.get("conv", 0)), float(p.get("softcap", 0.0))
         self.window, self.chunk = int(p.get("window", 0)), int(p.get("chunk", 0))
+        self.keep_first = int(p.get("keep_first", 0))
+        if self.keep_first and not self.window:
+            raise ValueError("kept first tokens belong to a window")
         self.nq, self.nk, self.nv = self.heads * self.dim, self.kv_heads * self.dim, self.kv_heads * self.vdim
         self.values_from_keys = bool(p.get("values_from_keys"))
         if self.values_from_keys and (self.vdim != self.dim or self.taps):
@@ -124,8 +129,8 @@ class FlexAttention(ProjectedMixer):
         if self.rot_layout not in ("half", "interleaved"):
             raise ValueError(f"unknown layout of rotated pairs '{self.rot_layout}'")
         self.n_qkv = self.nq + self.nk + self.nv
-        self.out_gate = bool(p.get("out_gate"))
-        self.n_gate = self.heads * self.vdim if self.out_gate else 0
+        self.out_gate, self.head_gate = bool(p.get("out_gate")), p.get("out_gate") == "head"
+        self.n_gate = (self.heads if self.head_gate else self.heads * self.vdim) if self.out_gate else 0
         # One product for everything that reads h: rows [q | k | v | gate]; the gate has no bias.
         named = ("q", "k") if self.values_from_keys else ("q", "k", "v")
         rows = [tensors[n] for n in named] + ([tensors["g"]] if self.out_gate else [])
@@ -162,7 +167,7 @@ class FlexAttention(ProjectedMixer):
         # a chunk never looks further back than its own size, so pages behind it can go like a window's
         keep = self.window if self.window else self.chunk
         # (values that are the projected keys are still cached beside the keys: the cached key is normed and rotated)
-        return CacheNeed((PagedTensor("k", self.kv_heads, self.dim), PagedTensor("v", self.kv_heads, self.vdim)), keep)
+        return CacheNeed((PagedTensor("k", self.kv_heads, self.dim), PagedTensor("v", self.kv_heads, self.vdim)), keep, self.keep_first)
 
     def state_need(self) -> Optional[StateNeed]:
         return StateNeed(((self.taps - 1) * self.n_qkv,), torch.float32) if self.taps > 1 else None
@@ -187,14 +192,15 @@ class FlexAttention(ProjectedMixer):
                               self.freq, self.rot_dims, ctx, cache.block_table, cache.page_size, cache.pages["k"], cache.pages["v"],
                               cache.writes, layout=self.rot_layout, unit_norm_after=self.unit_norm_after,
                               values_are_keys=self.values_from_keys, norm_whole=self.norm_whole, v_first32=v_first, vmix32=self.vmix)
-        gated = self.out_gate
+        gated = self.out_gate and not self.head_gate
         attn = torch.empty((m, self.heads * self.vdim), dtype=torch.float32 if gated else self.rt.dtype, device=dev)
         ops.attention_flex(q, attn, self.heads, self.kv_heads, self.dim, self.vdim, self.scale, self.softcap, self.slopes,
                            self.window, self.chunk, 1.0 if gated else self.out_scale, ctx, cache.block_table, cache.page_size,
-                           cache.pages["k"], cache.pages["v"], sinks32=self.sinks)
+                           cache.pages["k"], cache.pages["v"], sinks32=self.sinks, keep_first=self.keep_first,
+                           gate32=p32[:, self.n_qkv:self.n_qkv + self.heads] if self.head_gate else None)
         if gated:
             a = torch.empty((m, self.heads * self.vdim), dtype=self.rt.dtype, device=dev)
-            ops.gated_norm(attn, a, gate32=p32[:, self.n_qkv:], gate_kind="sigmoid", out_scale=self.out_scale)
+            ops.gated_norm(attn, a, gate32=p32[:, self.n_qkv:self.n_qkv + self.n_gate], gate_kind="sigmoid", out_scale=self.out_scale)
             attn = a
         return attn
 

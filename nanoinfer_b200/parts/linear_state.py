@@ -4,7 +4,7 @@
 
 read either after the update (``o_t = S_t^T q_t``) or before it with a bonus for the current token
 (``o_t = (S_(t-1) + diag(u) k_t v_t^T)^T q_t``). A kernel of the library walks each of them (``ops.linear_state_scan``, token
-by token; ``ops.grouped_state_scan``, eight tokens at a time); the classes differ in where q, k, v and the decay come from and in what happens to o:
+by token; ``ops.grouped_state_scan``, eight tokens at a time; ``ops.decay_state_scan``, one decay per head, long steps in chunks); the classes differ in where q, k, v and the decay come from and in what happens to o:
 
 * ``GatedLinearAttention``: ``q = W_q h / sqrt(dim)``, ``k = W_k h``, ``v = W_v h``, decay per key channel
   ``sigmoid(W_a2 W_a1 h + b)^(1/tau)``; o is RMS-normed per head (gain of ``vdim``, shared by the heads), times
@@ -17,6 +17,8 @@ by token; ``ops.grouped_state_scan``, eight tokens at a time); the classes diffe
   last inputs are kept in the state); ``dt = softplus(dt + dt_bias)``; per head the decay is the scalar
   ``exp(-exp(A_log) dt)``, ``k = B`` and ``q = C`` of the head's group, ``v = dt x``; ``y = o + D x``, times ``silu(z)``,
   RMS-normed in ``norm_groups`` equal parts, times a gain, then ``W_o``.
+* ``LightningAttention``: ``q = silu(W_q h)``, ``k = silu(W_k h)``, ``v = silu(W_v h)``, a fixed decay per head; o of all heads is
+  RMS-normed together, times a gain, times ``sigmoid(W_g h)``, then ``W_o``.
 * ``StabilizedMatrixMemory``: ``q = W_q h / sqrt(dim)``, ``k = W_k h``, ``v = W_v h``; per head a log input gate
   ``i = cap tanh((W_i h + b_i) / cap)`` and a log forget gate ``f = log sigmoid(cap tanh((W_f h + b_f) / cap))``; with a running
   maximum ``m_t = max(f + m_(t-1), i)`` (zero at a request's start) the decay is the scalar ``exp(f + m_(t-1) - m_t)`` and
@@ -34,7 +36,7 @@ from typing import Dict
 import torch
 
 from ..registry import register_part
-from .base import LayerCache, Mixer, Runtime, StateNeed, StepContext, as_tensor
+from .base import LayerCache, Mixer, ProjectedMixer, Runtime, StateNeed, StepContext, as_tensor
 from .spec import PartSpec, TensorSpec
 
 
@@ -204,17 +206,60 @@ class Mamba2Mixer(Mixer):
         xbc_in = p32[:, inner:2 * inner + 2 * gn]
         xbc = torch.empty((m, inner + 2 * gn), dtype=torch.float32, device=dev)
         ops.conv_step(xbc_in, self.conv_w, self.conv_b, "silu", cache.state, 0, ctx, xbc, self.taps)
-        dt = torch.empty((m, self.heads), dtype=torch.float32, device=dev)
-        decay = torch.empty((m, self.heads), dtype=torch.float32, device=dev)
-        ops.step_sizes(p32[:, 2 * inner + 2 * gn:], self.dt_bias, self.a_log, dt, decay)
         o32 = torch.empty((m, inner), dtype=torch.float32, device=dev)
         x = xbc[:, :inner]
-        ops.linear_state_scan(xbc[:, inner + gn:], xbc[:, inner:inner + gn], x, decay, cache.state, self.conv_state, ctx, o32,
-                              self.heads, self.groups, self.n, self.vdim, v_scale32=dt)
+        ops.decay_state_scan(xbc[:, inner + gn:], xbc[:, inner:inner + gn], x, cache.state, self.conv_state, ctx, o32, self.heads, self.groups,
+                             self.n, self.vdim, raw32=p32[:, 2 * inner + 2 * gn:], dt_bias32=self.dt_bias, a_log32=self.a_log,
+                             exact=self.rt.dtype == torch.float32)
         gated = torch.empty((m, inner), dtype=self.rt.dtype, device=dev)
         ops.gated_norm(o32, gated, groups=self.norm_groups, eps=self.eps, gain32=self.gain, gate32=p32[:, :inner], gate_kind="silu",
                        gate_first=True, skip32=x, skip_coef32=self.skip, out_scale=self.out_scale)
         ops.linear(gated, self.w_o, None, residual32, "add")
+
+
+class LightningAttention(ProjectedMixer):
+    """params: ``hidden heads dim vdim decay`` (one number per head) ``eps out_scale``. tensors: ``q k [heads*dim, hidden]``, ``v g
+    [heads*vdim, hidden]``, ``norm [heads*vdim]``, ``o [hidden, heads*vdim]``."""
+
+    graph_safe = True   # launches do not depend on which requests are in the batch
+
+    @staticmethod
+    def spec(prefix: str, hidden: int, heads: int, dim: int, vdim: int, decay, eps: float, out_scale: float = 1.0) -> PartSpec:
+        nk, nv = heads * dim, heads * vdim
+        t = {"q": TensorSpec(f"{prefix}.q", (nk, hidden)), "k": TensorSpec(f"{prefix}.k", (nk, hidden)),
+             "v": TensorSpec(f"{prefix}.v", (nv, hidden)), "g": TensorSpec(f"{prefix}.g", (nv, hidden)),
+             "norm": TensorSpec(f"{prefix}.norm", (nv,), "gain"), "o": TensorSpec(f"{prefix}.o", (hidden, nv))}
+        return PartSpec("lightning_attention", {"hidden": hidden, "heads": heads, "dim": dim, "vdim": vdim, "decay": tuple(float(x) for x in decay),
+                                                "eps": float(eps), "out_scale": float(out_scale)}, t)
+
+    def __init__(self, spec: PartSpec, tensors: Dict[str, torch.Tensor], rt: Runtime):
+        super().__init__(spec, tensors, rt)
+        p = spec.params
+        self.heads, self.dim, self.vdim = int(p["heads"]), int(p["dim"]), int(p["vdim"])
+        self.eps, self.out_scale = float(p["eps"]), float(p.get("out_scale", 1.0))
+        self.nk, self.nv = self.heads * self.dim, self.heads * self.vdim
+        d = torch.tensor(p["decay"], dtype=torch.float64)
+        if d.numel() != self.heads or not bool(((d >= 0) & (d <= 1)).all()):
+            raise ValueError("one decay between 0 and 1 per head")
+        self.decay = rt.vector32(torch.stack([d, torch.log2(d)]))       # the decays and their logarithms, each rounded once
+        # One product for everything that reads h: rows [q | k | v | g].
+        self.take_input(torch.cat([tensors[x] for x in ("q", "k", "v", "g")], dim=0), None, bool(p.get("joint_input")))
+        self.gain = rt.vector32(tensors["norm"])
+        self.w_o = rt.matrix(tensors["o"])
+
+    def state_need(self) -> StateNeed:
+        # S as [head, value channel, key channel]
+        return StateNeed((self.heads * self.vdim * self.dim,), torch.float32)
+
+    def mix(self, p32: torch.Tensor, ctx: StepContext, cache: LayerCache) -> torch.Tensor:
+        m, dev, ops, nk, nv = p32.shape[0], p32.device, self.ops, self.nk, self.nv
+        o32 = torch.empty((m, nv), dtype=torch.float32, device=dev)
+        ops.decay_state_scan(p32[:, :nk], p32[:, nk:2 * nk], p32[:, 2 * nk:2 * nk + nv], cache.state, 0, ctx, o32, self.heads, self.heads,
+                             self.dim, self.vdim, act="silu", decay32=self.decay, exact=self.rt.dtype == torch.float32)
+        gated = torch.empty((m, nv), dtype=self.rt.dtype, device=dev)
+        ops.gated_norm(o32, gated, groups=1, eps=self.eps, gain32=self.gain, gate32=p32[:, 2 * nk + nv:2 * (nk + nv)], gate_kind="sigmoid",
+                       out_scale=self.out_scale)
+        return gated
 
 
 class StabilizedMatrixMemory(Mixer):
@@ -274,6 +319,7 @@ class StabilizedMatrixMemory(Mixer):
 
 
 register_part("gated_linear_attention", GatedLinearAttention)
+register_part("lightning_attention", LightningAttention)
 register_part("matrix_memory", StabilizedMatrixMemory)
 register_part("time_mix", ShiftedTimeMix)
 register_part("mamba2", Mamba2Mixer)

@@ -1,4 +1,5 @@
-"""RMSNorm: ``x * 1/sqrt(mean(x^2) + eps) * gain``, computed in 32-bit.
+"""RMSNorm: ``x * 1/sqrt(mean(x^2) + eps) * gain``, computed in 32-bit. LayerNorm: ``(x - mean) / sqrt(variance + eps) * gain +
+bias``, likewise.
 
 Reference: cpp/src/ops.cpp:272-292 (eps inside the root, added to the mean; gain last) and
 nanoinfer/layers.py:21-38.
@@ -70,5 +71,29 @@ class RMSNorm(Norm):
         return a, b
 
 
+class LayerNorm(Norm):
+    """``(x - mean(x)) / sqrt(mean((x - mean(x))^2) + eps) * gain + bias`` in 32-bit. params: ``size``, ``eps``. tensors:
+    ``gain [size]``, ``bias [size]``."""
+
+    graph_safe = True   # launches do not depend on which requests are in the batch
+
+    @staticmethod
+    def spec(size: int, eps: float, gain_name: str, bias_name: str) -> PartSpec:
+        return PartSpec("layernorm", {"size": size, "eps": eps},
+                        {"gain": TensorSpec(gain_name, (size,), "gain"), "bias": TensorSpec(bias_name, (size,), "bias")})
+
+    def __init__(self, spec: PartSpec, tensors: Dict[str, torch.Tensor], rt: Runtime):
+        super().__init__(spec, tensors, rt)
+        self.size, self.eps = int(spec.params["size"]), float(spec.params["eps"])
+        self.gain, self.bias = rt.vector32(tensors["gain"]), rt.vector32(tensors["bias"])
+
+    def forward(self, x32: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        n = x32.shape[0] if rows is None else rows.shape[0]
+        out = torch.empty((n, self.size), dtype=self.rt.dtype, device=x32.device)
+        self.ops.layernorm(x32, self.gain, self.bias, self.eps, out, rows)
+        return out
+
+
 register_part("rmsnorm", RMSNorm)
+register_part("layernorm", LayerNorm)
 

@@ -103,3 +103,4 @@ def _ensure_builtin() -> None:
     from .models import darotar as _darotar  # noqa: F401  registers Darotar
     from .models import dusilorn as _dusilorn  # noqa: F401  registers Dusilorn
     from .models import pilonex as _pilonex  # noqa: F401  registers Pilonex
+    from .models import vagulorn as _vagulorn  # noqa: F401  registers Vagulorn

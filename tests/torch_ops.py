@@ -22,6 +22,11 @@ class TorchOps:
         y = x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * gain32.double()
         out.copy_(y.to(out.dtype))
 
+    def layernorm(self, x32, gain32, bias32, eps, out, rows=None):
+        x = x32.double() if rows is None else x32[rows.long()].double()
+        d = x - x.mean(-1, keepdim=True)
+        out.copy_((d / torch.sqrt(d.pow(2).mean(-1, keepdim=True) + eps) * gain32.double() + bias32.double()).to(out.dtype))
+
     def linear(self, a, w, bias32, out, mode):
         a = as_tensor(a)
         y = a.double() @ w.double().t()
@@ -43,11 +48,14 @@ class TorchOps:
         g, u = torch.clamp(g, max=limit), torch.clamp(u, -limit, limit)
         return g / (1.0 + torch.exp(-alpha * g)) * (u + shift)
 
-    def linear_swiglu(self, a, w_gate_up, out, glu=None):
+    def linear_swiglu(self, a, w_gate_up, out, glu=None, act="silu"):
         a = as_tensor(a)
         inter = w_gate_up.shape[0] // 2
         g = a.double() @ w_gate_up[:inter].double().t()
         u = a.double() @ w_gate_up[inter:].double().t()
+        if act == "gelu_tanh":
+            out.copy_((torch.nn.functional.gelu(g, approximate="tanh") * u).to(out.dtype))
+            return
         out.copy_(self._glu(g, u, glu).to(out.dtype))
 
     def qkv_project(self, a, w_qkv, bias32, qkv, heads, kv_heads, head_dim, positions, req_index, rotary,
@@ -127,7 +135,7 @@ class TorchOps:
 
     def unary(self, in32, out, kind):
         x = in32.double()
-        out.copy_({"tanh": torch.tanh, "copy": lambda v: v, "sigmoid": torch.sigmoid}[kind](x).to(out.dtype))
+        out.copy_({"tanh": torch.tanh, "copy": lambda v: v, "sigmoid": torch.sigmoid, "silu": lambda v: v * torch.sigmoid(v)}[kind](x).to(out.dtype))
 
     def head_norm_gate(self, o32, gate32, gain32, eps, heads, d, out):
         m = o32.shape[0]
@@ -188,7 +196,7 @@ class TorchOps:
         v_pages[page[ok], :, (pos % page_size)[ok], :] = v[ok].to(v_pages.dtype)
 
     def attention_flex(self, q, out, heads, kv_heads, dim, vdim, scale, softcap, slopes32, window, chunk, out_scale, ctx,
-                       block_table, page_size, k_pages, v_pages, sinks32=None):
+                       block_table, page_size, k_pages, v_pages, sinks32=None, keep_first=0, gate32=None):
         m = q.shape[0]
         qh = q.double().view(m, heads, dim)
         rep = heads // kv_heads
@@ -198,7 +206,7 @@ class TorchOps:
             lo = max(0, pos - window + 1) if window else 0
             if chunk:
                 lo = max(lo, (pos // chunk) * chunk)
-            js = torch.arange(lo, pos + 1)
+            js = torch.cat([torch.arange(0, min(keep_first, lo)), torch.arange(lo, pos + 1)])
             pages = block_table[r, js // page_size].long()
             if (pages < 0).any():
                 continue        # a padding row
@@ -215,6 +223,8 @@ class TorchOps:
                 else:
                     w = torch.softmax(s, 0)
                 res[t, h] = w @ v[:, h // rep]
+        if gate32 is not None:
+            res = res * torch.sigmoid(gate32.double())[:, :, None]
         out.copy_((res.view(m, heads * vdim) * out_scale).to(out.dtype))
 
     # ---- gate, norm in groups, skip (pointwise.cu) ---------------------------------------------------
@@ -322,6 +332,28 @@ class TorchOps:
                     o = torch.einsum("hkv,hk->hv", s, q)
                 o32[t] = o.reshape(-1).to(torch.float32)
             flat.copy_(s.transpose(1, 2).reshape(-1).to(torch.float32))
+            start += q_len
+
+    def decay_state_scan(self, q32, k32, v32, state, state_off, ctx, o32, heads, kq_heads, dk, dv, act="none", decay32=None, raw32=None,
+                         dt_bias32=None, a_log32=None, exact=False):
+        m, rep = q32.shape[0], heads // kq_heads
+        f = (lambda z: z * torch.sigmoid(z)) if act == "silu" else (lambda z: z)
+        q, k = (f(x.double()).reshape(m, kq_heads, dk).repeat_interleave(rep, 1) for x in (q32, k32))
+        v = f(v32.double()).reshape(m, heads, dv)
+        if raw32 is not None:
+            step = torch.nn.functional.softplus(raw32.double() + dt_bias32.double(), threshold=1e9)
+            d = torch.exp(-torch.exp(a_log32.double()) * step)
+            v = v * step[:, :, None]
+        else:
+            d = decay32[0].double().expand(m, heads)
+        start = 0
+        for q_len, slot in zip(ctx.host.q_lens, ctx.host.slots):
+            flat = state[slot, state_off:state_off + heads * dv * dk]
+            s = flat.double().view(heads, dv, dk).clone()
+            for t in range(start, start + q_len):
+                s = d[t][:, None, None] * s + v[t][:, :, None] * k[t][:, None, :]
+                o32[t] = torch.einsum("hvk,hk->hv", s, q[t]).reshape(-1).to(torch.float32)
+            flat.copy_(s.reshape(-1).to(torch.float32))
             start += q_len
 
     def memory_gates(self, zi32, zf32, bi32, bf32, cap, state, state_off, ctx, decay32, write32, floor32):
