@@ -618,9 +618,32 @@ def pilonex_configs(size: dict):
     return pil, design_configs(dict(DESIGN_SIZES["1k"], **{k: size[k] for k in ("width", "heads", "head_dim", "ff_swiglu", "vocab", "layers")}))[1]
 
 
+# A Vagulorn stack at the same widths, layer for layer like the Vafozen stack: softmax attention whose values are its keys (a sliding
+# window beside four kept tokens, a gate per head) beside lightning attention, a state-space mixer, chunked attention, a state-space
+# mixer, twice; gelu-gated feed-forwards of the Qwen2 decoder's size; the softmax mixers have the Qwen2 decoder's head counts and head
+# size. Its closest existing model is Vafozen (parallel blocks with one norm, a pair of mixers, the same state-space mixer).
+VAGULORN_SIZES = {name: dict({k: v for k, v in size.items() if k != "decay_rank"}, window=1024, keep_first=4)
+                  for name, size in VAFOZEN_SIZES.items()}
+
+
+def vagulorn_configs(size: dict):
+    w, h, d, n = size["width"], size["heads"], size["head_dim"], size["side_heads"]
+    ff = {"kind": "dense", "ff": size["ff_swiglu"]}
+    half = {"heads": h, "kv_heads": 2, "dim": d, "vdim": d, "scale": d ** -0.5}
+    pair = {"left": dict(half, mask={"size": size["window"], "keep_first": size["keep_first"]}, rot={"dims": size["rot"], "base": 500000.0}),
+            "right": {"heads": n, "dim": d, "vdim": d, "decay": [1.0 - 2.0 ** -(3 + 2 * i) for i in range(n)]}, "left_scale": 1.0, "right_scale": 0.75}
+    chunked = dict(half, mask={"size": size["chunk"]}, rot={"dims": size["rot"], "base": 50000.0})
+    ssm = {"heads": size["ssm_heads"], "vdim": 2 * w // size["ssm_heads"], "state": size["ssm_state"], "groups": 2, "norm_groups": 2, "conv": 4}
+    kinds = [{"type": "parallel", "mixer": pair, "mlp": ff}, {"type": "mamba2", "mixer": ssm, "mlp": ff}, {"type": "attention", "mixer": chunked, "mlp": ff}]
+    layers = [kinds[(0, 1, 2, 1)[i % 4]] for i in range(size["layers"])]
+    vag = {"architecture": "Vagulorn", "vocab": size["vocab"], "width": w, "norm": {"eps": 1e-5}, "embedding": {"scale": 8.0}, "layers": layers}
+    return (vag,) + vafozen_configs(dict(size, decay_rank=64))
+
+
 def run_design(args) -> dict:
-    """Prefill and decode throughput of a design (Nezalorn, Vafozen, Darotar, Dusilorn, Pilonex) beside the Qwen2 decoder at equal size (random
-    weights, bfloat16, device-timed with CUDA events), and where one eager step's time goes, launch kind by launch kind."""
+    """Prefill and decode throughput of a design (Nezalorn, Vafozen, Darotar, Dusilorn, Pilonex, Vagulorn) beside the Qwen2 decoder at equal
+    size (Vagulorn: beside Vafozen as well; random weights, bfloat16, device-timed with CUDA events), and where one eager step's time goes,
+    launch kind by launch kind."""
     import numpy as np
     import torch
     from nanoinfer_b200 import load_model
@@ -633,14 +656,15 @@ def run_design(args) -> dict:
     design = args.design
     sizes, configs = {"nezalorn": (DESIGN_SIZES, design_configs), "vafozen": (VAFOZEN_SIZES, vafozen_configs),
                       "darotar": (DAROTAR_SIZES, darotar_configs), "dusilorn": (DUSILORN_SIZES, dusilorn_configs),
-                      "pilonex": (PILONEX_SIZES, pilonex_configs)}[design]
+                      "pilonex": (PILONEX_SIZES, pilonex_configs), "vagulorn": (VAGULORN_SIZES, vagulorn_configs)}[design]
+    beside = ("vafozen", "qwen2") if design == "vagulorn" else ("qwen2",)
     out = {"impl": "ours", "design": design, "dtype": "bf16", "data": "synthetic: seeded random weights and random token ids",
            "peaks": {"hbm_gbs": pk["hbm_gbs"], "bf16_tflops": pk["bf16_tflops"], "source": pk["source"]},
            "config": {"prefill_tokens": t_pre, "decode_batch": batch, "decode_context": ctx, "page_size": 16}, "sizes": {}}
     for name in (args.design_sizes.split(",") if args.design_sizes else sorted(sizes)):
         size = sizes[name]
         row = {}
-        for label, cfg_json in zip((design, "qwen2"), configs(size)):
+        for label, cfg_json in zip((design,) + beside, configs(size)):
             rng = np.random.default_rng(0)
             tmp = tempfile.mkdtemp(prefix="nanoinfer_b200_design_")
             try:
@@ -725,8 +749,10 @@ def run_design(args) -> dict:
                 row[label]["launch_kinds_us"] = kinds
             del model, engine, ops
             torch.cuda.empty_cache()
-        row["ratio_prefill"] = round(row[design]["prefill_tok_s"] / row["qwen2"]["prefill_tok_s"], 3)
-        row["ratio_decode"] = round(row[design]["decode_tok_s"] / row["qwen2"]["decode_tok_s"], 3)
+        for other in beside:        # the keys without a name are the ratios to the dense decoder
+            name_of = "" if other == "qwen2" else f"_{other}"
+            row["ratio_prefill" + name_of] = round(row[design]["prefill_tok_s"] / row[other]["prefill_tok_s"], 3)
+            row["ratio_decode" + name_of] = round(row[design]["decode_tok_s"] / row[other]["decode_tok_s"], 3)
         out["sizes"][name] = dict(row, size=size)
     return out
 
@@ -865,7 +891,7 @@ def main() -> int:
                     help="add a 'kernels' block: where the time of a decode step and of a prompt portion goes, kernel kind by "
                          "kind, with bytes or FLOPs and the fraction of the measured peak")
     ap.add_argument("--shape", default="0.5b", choices=sorted(SHAPES), help="layer sizes: the family's 0.5B (default), 1.5B or 7B")
-    ap.add_argument("--design", default=None, choices=["nezalorn", "vafozen", "darotar", "dusilorn", "pilonex"],
+    ap.add_argument("--design", default=None, choices=["nezalorn", "vafozen", "darotar", "dusilorn", "pilonex", "vagulorn"],
                     help="instead of the headline workload: prefill and decode throughput of this design beside the Qwen2 "
                          "decoder at equal size (--design-sizes, --prefill-tokens, --batch, --context up to 2048, --breakdown)")
     ap.add_argument("--design-sizes", default="", help="comma-separated names of DESIGN_SIZES (default: all)")

@@ -16,10 +16,9 @@
 // Only differences c_t - c_s <= 0 are exponentiated, never quotients of products, so a decay of zero is a zero; the sums are formed in
 // 64-bit and kept as two floats, so a strong decay early in a chunk does not cost the later differences their digits.
 // The products run on the tensor cores (mma.sync m16n8k16, bfloat16 operands, 32-bit sums). q, k and v are outputs of
-// projections and convolutions and enter as bfloat16; what is 32-bit by the design (states, decays, step sizes, and everything they
-// multiply) is split into a bfloat16 and a bfloat16 of the remainder, two products each: 16 bits and more of it take part.
-#include <type_traits>
-
+// projections and convolutions and enter as bfloat16 (they may be stored so, T, or as floats); what is 32-bit by the design (states,
+// decays, step sizes, and everything they multiply) is split into a bfloat16 and a bfloat16 of the remainder, two products each: 16
+// bits and more of it take part. Blocks take 64 value channels of a head; tiles come by cp.async where rows are aligned.
 #include "attention_common.cuh"
 
 namespace {
@@ -29,22 +28,58 @@ constexpr int DS_THREADS = 128;
 constexpr float NO_DECAY_LEFT = -1e30f; // log2 of a decay of zero
 
 struct DsIn {
-    const float *q, *k, *v;             // rows of ldq, ldk, ldv floats
+    const void *q, *k, *v;              // rows of ldq, ldk, ldv elements of type T
     const float *raw, *bias, *a_log;    // step sizes: raw [tokens] rows of ld_raw floats (null: fixed decays), bias and a_log [heads]
     const float *decay, *log2_decay;    // fixed decays and their logarithms [heads]
     const int *q_start, *slots;
     int ldq, ldk, ldv, ld_raw, heads, kq_heads, dk, dv, silu, vec;
+    template <typename T> __device__ __forceinline__ const T* q_at(size_t row, int head) const { return (const T*)q + row * ldq + (size_t)head * dk; }
+    template <typename T> __device__ __forceinline__ const T* k_at(size_t row, int head) const { return (const T*)k + row * ldk + (size_t)head * dk; }
+    template <typename T> __device__ __forceinline__ const T* v_at(size_t row, int head) const { return (const T*)v + row * ldv + (size_t)head * dv; }
 };
 
 __device__ __forceinline__ float ds_silu(float x) { return x / (1.0f + expf(-x)); }
 __device__ __forceinline__ float softplus(float x) { return x > 0.f ? x + log1pf(expf(-x)) : log1pf(expf(x)); }
+__device__ __forceinline__ float bf16_of(float x) { return __bfloat162float(__float2bfloat16_rn(x)); }
+
+// elements c .. c + 3 of a row of `width` elements as floats, zeros beyond its end; vec: the width is a multiple of four and the
+// row starts on a boundary of four elements
+__device__ __forceinline__ float4 row4(const float* p, int c, int width, bool vec) {
+    float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (vec) {
+        if (c < width) x = *reinterpret_cast<const float4*>(p + c);
+    } else {
+        if (c < width) x.x = p[c];
+        if (c + 1 < width) x.y = p[c + 1];
+        if (c + 2 < width) x.z = p[c + 2];
+        if (c + 3 < width) x.w = p[c + 3];
+    }
+    return x;
+}
+__device__ __forceinline__ float4 row4(const __nv_bfloat16* p, int c, int width, bool vec) {
+    float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (vec) {
+        if (c < width) {
+            const uint2 raw = *reinterpret_cast<const uint2*>(p + c);
+            const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+            x = make_float4(a.x, a.y, b.x, b.y);
+        }
+    } else {
+        if (c < width) x.x = __bfloat162float(p[c]);
+        if (c + 1 < width) x.y = __bfloat162float(p[c + 1]);
+        if (c + 2 < width) x.z = __bfloat162float(p[c + 2]);
+        if (c + 3 < width) x.w = __bfloat162float(p[c + 3]);
+    }
+    return x;
+}
+__device__ __forceinline__ void silu4(float4& x) { x.x = ds_silu(x.x); x.y = ds_silu(x.y); x.z = ds_silu(x.z); x.w = ds_silu(x.w); }
 
 // ---------------------------------------------------------------------------------- short steps
 // grid: (parts of the value channels, heads, requests). LANES lanes share R value channels; lane l holds the key channels
 // (l + LANES i) * 4 .. + 3.
 constexpr int R = 4;
 
-template <int LANES, int NV>
+template <typename T, int LANES, int NV>
 __global__ void __launch_bounds__(DS_THREADS)
 decay_step_kernel(const DsIn in, float* __restrict__ state, long long state_ld, int state_off, float* __restrict__ o, int ldo) {
     pdl_launch_dependents();
@@ -79,22 +114,12 @@ decay_step_kernel(const DsIn in, float* __restrict__ state, long long state_ld, 
 #pragma unroll
         for (int i = 0; i < NV; ++i) {
             const int c = (lane + LANES * i) * 4;
-            const float* pq = in.q + (size_t)t * in.ldq + (size_t)hq * dk + c;
-            const float* pk = in.k + (size_t)t * in.ldk + (size_t)hq * dk + c;
-            float4 a = make_float4(0.f, 0.f, 0.f, 0.f), b = a;
-            if (in.vec) {
-                if (c < dk) { a = *reinterpret_cast<const float4*>(pq); b = *reinterpret_cast<const float4*>(pk); }
-            } else {
-                if (c < dk) { a.x = pq[0]; b.x = pk[0]; }
-                if (c + 1 < dk) { a.y = pq[1]; b.y = pk[1]; }
-                if (c + 2 < dk) { a.z = pq[2]; b.z = pk[2]; }
-                if (c + 3 < dk) { a.w = pq[3]; b.w = pk[3]; }
-            }
+            const float4 a = row4(in.q_at<T>(t, hq), c, dk, in.vec != 0), b = row4(in.k_at<T>(t, hq), c, dk, in.vec != 0);
             qv[i][0] = a.x; qv[i][1] = a.y; qv[i][2] = a.z; qv[i][3] = a.w;
             kv[i][0] = b.x; kv[i][1] = b.y; kv[i][2] = b.z; kv[i][3] = b.w;
         }
 #pragma unroll
-        for (int r = 0; r < R; ++r) vv[r] = j0 + r < dv ? in.v[(size_t)t * in.ldv + (size_t)h * dv + j0 + r] : 0.f;
+        for (int r = 0; r < R; ++r) vv[r] = j0 + r < dv ? Elem<T>::load(in.v_at<T>(t, h) + j0 + r) : 0.f;
         float d = d_fixed, f = 1.0f;
         if (!fixed) {
             f = softplus(in.raw[(size_t)t * in.ld_raw + h] + bias);
@@ -148,11 +173,13 @@ decay_step_kernel(const DsIn in, float* __restrict__ state, long long state_ld, 
 }
 
 // ---------------------------------------------------------------------------------- chunks
-// A chunk's tile in shared memory: CH (or DP, for a state) rows of DP bfloat16, 16 bytes of padding each.
+// A chunk's tile in shared memory: CH rows of DP bfloat16, 16 bytes of padding each; a state's tile has as many rows, its value
+// channels.
 template <int DP> struct Tile {
     static constexpr int ROW = DP + 8;
     static constexpr int ELEMS = CH * ROW;
 };
+constexpr int DV = CH;                  // value channels of a block
 
 struct ChunkAt { int row, n, slot; };       // first flat row, tokens, index among the step's chunks
 
@@ -203,213 +230,250 @@ __device__ __forceinline__ void chunk_decays(const DsIn& in, const ChunkAt& at, 
     }
 }
 
-__device__ __forceinline__ float bf16_of(float x) { return __bfloat162float(__float2bfloat16_rn(x)); }
-
-// four floats of a row (zeros beyond its width or where the row does not exist)
-__device__ __forceinline__ float4 row4(const float* p, int c, int width, bool exists, bool vec) {
-    float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (!exists) return x;
-    if (vec) {
-        if (c < width) x = *reinterpret_cast<const float4*>(p + c);
-    } else {
-        if (c < width) x.x = p[c];
-        if (c + 1 < width) x.y = p[c + 1];
-        if (c + 2 < width) x.z = p[c + 2];
-        if (c + 3 < width) x.w = p[c + 3];
-    }
-    return x;
-}
-__device__ __forceinline__ void silu4(float4& x) { x.x = ds_silu(x.x); x.y = ds_silu(x.y); x.z = ds_silu(x.z); x.w = ds_silu(x.w); }
 __device__ __forceinline__ void put4(__nv_bfloat16* p, const float4& x) {
     *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(x.x, x.y), pack_bf16(x.z, x.w));
 }
 __device__ __forceinline__ float4 rest4(const float4& x) { return make_float4(x.x - bf16_of(x.x), x.y - bf16_of(x.y), x.z - bf16_of(x.z), x.w - bf16_of(x.w)); }
 
-// rows at.row .. of `src` (width floats from column 0 of a row) into a tile
-template <int DP>
-__device__ __forceinline__ void load_rows(__nv_bfloat16* tile, const float* __restrict__ src, int ld, const ChunkAt& at, int width, bool silu, bool vec) {
-#pragma unroll 4
+__device__ __forceinline__ void ds_cp_async_16(void* smem, const void* gmem, bool valid) {
+    const unsigned d = (unsigned)__cvta_generic_to_shared(smem);
+    const int n = valid ? 16 : 0;       // 0 source bytes: the destination is zero-filled
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(d), "l"(gmem), "r"(n));
+}
+__device__ __forceinline__ void ds_commit() { asm volatile("cp.async.commit_group;\n" ::); }
+template <int N> __device__ __forceinline__ void ds_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N)); }
+
+// n rows of `src` (row stride ld, `width` elements from its column 0 on) into a tile; rows and columns that do not exist are zeros.
+// vec: rows of T start on 16-byte boundaries and the width fills whole 16-byte groups.
+template <typename T, int DP>
+__device__ __forceinline__ void load_rows(__nv_bfloat16* tile, const T* __restrict__ src, int ld, int n, int width, bool silu, bool vec) {
+    if (sizeof(T) == 2 && vec && !silu) {
+        for (int i = threadIdx.x; i < CH * (DP / 8); i += DS_THREADS) {
+            const int r = i / (DP / 8), c = (i % (DP / 8)) * 8;
+            const bool ok = r < n && c < width;
+            ds_cp_async_16(tile + r * Tile<DP>::ROW + c, ok ? src + (size_t)r * ld + c : src, ok);
+        }
+        return;
+    }
+#pragma unroll 8
     for (int i = threadIdx.x; i < CH * (DP / 4); i += DS_THREADS) {
         const int r = i / (DP / 4), c = (i % (DP / 4)) * 4;
-        float4 x = row4(src + (size_t)(at.row + r) * ld, c, width, r < at.n, vec);
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (r < n) x = row4(src + (size_t)r * ld, c, width, vec);
         if (silu) silu4(x);
         put4(tile + r * Tile<DP>::ROW + c, x);
     }
 }
 
-// What a chunk adds to a zero state: local[chunk, head, value channel, key channel], and the chunk's whole decay.
-// grid: (chunks, heads, requests). A warp owns DVP / 4 value channels: rows of the product (weighted v)^T . k over the chunk's tokens.
-template <int DKP, int DVP>
+// Where a block stands: a chunk of a request, a head, 64 of its value channels. grid: (chunks, heads x blocks of value channels,
+// requests).
+struct Block { ChunkAt at; int h, hq, v0, nv; };
+__device__ __forceinline__ Block block_of(const DsIn& in) {
+    const int per_head = (in.dv + DV - 1) / DV, h = blockIdx.y / per_head, v0 = (blockIdx.y % per_head) * DV;
+    return {chunk_at(in.q_start, blockIdx.z, blockIdx.x), h, h / (in.heads / in.kq_heads), v0, min(DV, in.dv - v0)};
+}
+
+// What a chunk adds to a zero state: local[chunk, head, value channel, key channel], and the chunk's whole decay. A warp owns 16
+// value channels: rows of the product (weighted v)^T . k over the chunk's tokens; the weights go on v in registers, in 32-bit.
+template <typename T, int DKP>
 __global__ void __launch_bounds__(DS_THREADS)
 chunk_state_kernel(const DsIn in, float* __restrict__ local, float* __restrict__ decays) {
     extern __shared__ __align__(16) unsigned char smem[];
     __shared__ float hi_s[CH], lo_s[CH], f_s[CH];
     pdl_launch_dependents();
     pdl_wait();
-    const int h = blockIdx.y, req = blockIdx.z, hq = h / (in.heads / in.kq_heads);
-    const ChunkAt at = chunk_at(in.q_start, req, blockIdx.x);
+    const Block b = block_of(in);
+    const ChunkAt& at = b.at;
     if (at.n == 0) return;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, mat = lane >> 3, rr = lane & 7, g = lane >> 2, t = lane & 3;
+    constexpr int RK = Tile<DKP>::ROW, RV = Tile<DV>::ROW;
     __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(smem);
-    __nv_bfloat16* vh_s = k_s + Tile<DKP>::ELEMS;
-    __nv_bfloat16* vl_s = vh_s + Tile<DVP>::ELEMS;
-    if (warp == 0) chunk_decays(in, at, h, hi_s, lo_s, f_s);
-    load_rows<DKP>(k_s, in.k + (size_t)hq * in.dk, in.ldk, at, in.dk, in.silu != 0, in.vec != 0);
+    __nv_bfloat16* v_s = k_s + Tile<DKP>::ELEMS;
+    load_rows<T, DKP>(k_s, in.k_at<T>(at.row, b.hq), in.ldk, at.n, in.dk, in.silu != 0, in.vec != 0);
+    load_rows<T, DV>(v_s, in.v_at<T>(at.row, b.h) + b.v0, in.ldv, at.n, b.nv, in.silu != 0, in.vec != 0);
+    ds_commit();
+    if (warp == 0) chunk_decays(in, at, b.h, hi_s, lo_s, f_s);
+    ds_wait<0>();
     __syncthreads();
     const float end_hi = hi_s[CH - 1], end_lo = lo_s[CH - 1];
-#pragma unroll 4
-    for (int i = threadIdx.x; i < CH * (DVP / 4); i += DS_THREADS) {
-        const int r = i / (DVP / 4), c = (i % (DVP / 4)) * 4;
-        float4 x = row4(in.v + (size_t)(at.row + r) * in.ldv + (size_t)h * in.dv, c, in.dv, r < at.n, in.vec != 0);
-        if (in.silu) silu4(x);
-        const float w = exp2f((end_hi - hi_s[r]) + (end_lo - lo_s[r])) * f_s[r];
-        x.x *= w; x.y *= w; x.z *= w; x.w *= w;
-        put4(vh_s + r * Tile<DVP>::ROW + c, x);
-        put4(vl_s + r * Tile<DVP>::ROW + c, rest4(x));
-    }
-    __syncthreads();
-    constexpr int MT = DVP / 64;        // tiles of 16 value channels a warp
-    const int mat = lane >> 3, rr = lane & 7;
-    float acc[MT][DKP / 8][4];
+    float acc[DKP / 8][4];
 #pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int n = 0; n < DKP / 8; ++n) acc[m][n][0] = acc[m][n][1] = acc[m][n][2] = acc[m][n][3] = 0.f;
+    for (int n = 0; n < DKP / 8; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
 #pragma unroll
     for (int kb = 0; kb < CH / 16; ++kb) {
-        unsigned a_hi[MT][4], a_lo[MT][4];
+        unsigned a[4], a_hi[4], a_lo[4];       // A: value channel x token, out of [token][value channel]
+        ldmatrix_x4_trans(a, v_s + (kb * 16 + (mat >> 1) * 8 + rr) * RV + warp * 16 + (mat & 1) * 8);
 #pragma unroll
-        for (int m = 0; m < MT; ++m) {      // A: value channel x token, out of [token][value channel]
-            const int at_s = (kb * 16 + (mat >> 1) * 8 + rr) * Tile<DVP>::ROW + (warp * MT + m) * 16 + (mat & 1) * 8;
-            ldmatrix_x4_trans(a_hi[m], vh_s + at_s);
-            ldmatrix_x4_trans(a_lo[m], vl_s + at_s);
+        for (int half = 0; half < 2; ++half) {      // the thread's tokens: 2t, 2t + 1 of eight
+            const int s0 = kb * 16 + half * 8 + 2 * t;
+            const float w0 = exp2f((end_hi - hi_s[s0]) + (end_lo - lo_s[s0])) * f_s[s0];
+            const float w1 = exp2f((end_hi - hi_s[s0 + 1]) + (end_lo - lo_s[s0 + 1])) * f_s[s0 + 1];
+#pragma unroll
+            for (int r = 0; r < 2; ++r) {
+                const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a[2 * half + r]));
+                const float x = v.x * w0, y = v.y * w1;
+                a_hi[2 * half + r] = pack_bf16(x, y);
+                a_lo[2 * half + r] = pack_bf16(x - bf16_of(x), y - bf16_of(y));
+            }
         }
 #pragma unroll
         for (int np = 0; np < DKP / 16; ++np) {     // B: token x key channel
-            unsigned b[4];
-            ldmatrix_x4_trans(b, k_s + (kb * 16 + (mat & 1) * 8 + rr) * Tile<DKP>::ROW + np * 16 + (mat >> 1) * 8);
+            unsigned bk[4];
+            ldmatrix_x4_trans(bk, k_s + (kb * 16 + (mat & 1) * 8 + rr) * RK + np * 16 + (mat >> 1) * 8);
+            mma_bf16(acc[2 * np], a_hi, bk[0], bk[1]);
+            mma_bf16(acc[2 * np + 1], a_hi, bk[2], bk[3]);
+            mma_bf16(acc[2 * np], a_lo, bk[0], bk[1]);
+            mma_bf16(acc[2 * np + 1], a_lo, bk[2], bk[3]);
+        }
+    }
+    float* out = local + (((size_t)at.slot * in.heads + b.h) * in.dv + b.v0) * in.dk;
+    const bool pairs = in.dk % 2 == 0;
 #pragma unroll
-            for (int m = 0; m < MT; ++m) {
-                mma_bf16(acc[m][2 * np], a_hi[m], b[0], b[1]);
-                mma_bf16(acc[m][2 * np + 1], a_hi[m], b[2], b[3]);
-                mma_bf16(acc[m][2 * np], a_lo[m], b[0], b[1]);
-                mma_bf16(acc[m][2 * np + 1], a_lo[m], b[2], b[3]);
+    for (int r = 0; r < 2; ++r) {
+        const int j = warp * 16 + g + 8 * r;
+        if (j >= b.nv) continue;
+#pragma unroll
+        for (int n = 0; n < DKP / 8; ++n) {
+            const int c = n * 8 + 2 * t;
+            float* p = out + (size_t)j * in.dk + c;
+            if (pairs) {
+                if (c < in.dk) *reinterpret_cast<float2*>(p) = make_float2(acc[n][2 * r], acc[n][2 * r + 1]);
+            } else {
+                if (c < in.dk) p[0] = acc[n][2 * r];
+                if (c + 1 < in.dk) p[1] = acc[n][2 * r + 1];
             }
         }
     }
-    const int g = lane >> 2, t = lane & 3;
-    float* out = local + ((size_t)at.slot * in.heads + h) * in.dv * in.dk;
-#pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int r = 0; r < 2; ++r) {
-            const int j = (warp * MT + m) * 16 + g + 8 * r;
-            if (j >= in.dv) continue;
-#pragma unroll
-            for (int n = 0; n < DKP / 8; ++n) {
-                const int c = n * 8 + 2 * t;
-                float* p = out + (size_t)j * in.dk + c;
-                if (in.vec) {
-                    if (c < in.dk) *reinterpret_cast<float2*>(p) = make_float2(acc[m][n][2 * r], acc[m][n][2 * r + 1]);
-                } else {
-                    if (c < in.dk) p[0] = acc[m][n][2 * r];
-                    if (c + 1 < in.dk) p[1] = acc[m][n][2 * r + 1];
-                }
-            }
-        }
-    if (threadIdx.x == 0) decays[(size_t)at.slot * in.heads + h] = exp2f(end_hi + end_lo);
+    if (threadIdx.x == 0 && b.v0 == 0) decays[(size_t)at.slot * in.heads + b.h] = exp2f(end_hi + end_lo);
 }
 
 // local[chunk] (what the chunk adds) becomes the chunk's entry state; the slot's state moves past the request's last chunk. A thread
-// per four (VEC) or one state elements of a request; the chunks' loads run ahead of the chain.
-template <bool VEC>
-__global__ void __launch_bounds__(256)
+// per eight (SPLIT) or one state elements of a request; the chunks' loads run ahead of the chain. SPLIT: the entry states are written
+// as the products read them, eight elements' bfloat16 and then the bfloat16 of their remainders where the eight floats were.
+template <bool SPLIT>
+__global__ void __launch_bounds__(128)
 chunk_chain_kernel(float* __restrict__ state, long long state_ld, int state_off, const int* __restrict__ q_start, const int* __restrict__ slots,
                    float* __restrict__ local, const float* __restrict__ decays, int heads, int per_head) {
-    constexpr int N = VEC ? 4 : 1, AHEAD = 8;
-    using V = typename std::conditional<VEC, float4, float>::type;
+    constexpr int N = SPLIT ? 8 : 1, AHEAD = 8;
     pdl_launch_dependents();
     pdl_wait();
     const int req = blockIdx.y;
-    const long long e = ((long long)blockIdx.x * 256 + threadIdx.x) * N, elems = (long long)heads * per_head;
+    const long long e = ((long long)blockIdx.x * 128 + threadIdx.x) * N, elems = (long long)heads * per_head;
     const int len = q_start[req + 1] - q_start[req], chunks = (len + CH - 1) / CH;
     if (e >= elems || chunks == 0) return;
     const int h = (int)(e / per_head), slot0 = (q_start[req] - q_start[0]) / CH + req;
     float* st = state + (long long)slots[req] * state_ld + state_off + e;
     float* at = local + (size_t)slot0 * elems + e;
     const float* dec = decays + (size_t)slot0 * heads + h;
-    __align__(16) float S[N];
-    *reinterpret_cast<V*>(S) = *reinterpret_cast<const V*>(st);
+    auto load = [](const float* p, float (&x)[N]) {
+        if constexpr (SPLIT) {
+            const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+            x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w; x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
+        } else {
+            x[0] = *p;
+        }
+    };
+    float S[N];
+    if constexpr (SPLIT) {      // (a state may start at any column)
+#pragma unroll
+        for (int n = 0; n < N; ++n) S[n] = st[n];
+    } else {
+        S[0] = *st;
+    }
     for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
-        __align__(16) float x[AHEAD][N];
-        float d[AHEAD];
+        float x[AHEAD][N], d[AHEAD];
 #pragma unroll
         for (int i = 0; i < AHEAD; ++i)
             if (c0 + i < chunks) {
-                *reinterpret_cast<V*>(x[i]) = *reinterpret_cast<const V*>(at + (size_t)(c0 + i) * elems);
+                load(at + (size_t)(c0 + i) * elems, x[i]);
                 d[i] = dec[(size_t)(c0 + i) * heads];
             }
 #pragma unroll
         for (int i = 0; i < AHEAD; ++i)
             if (c0 + i < chunks) {
-                *reinterpret_cast<V*>(at + (size_t)(c0 + i) * elems) = *reinterpret_cast<const V*>(S);
+                float* to = at + (size_t)(c0 + i) * elems;
+                if constexpr (SPLIT) {
+                    unsigned hi[4], lo[4];
+#pragma unroll
+                    for (int n = 0; n < 4; ++n) {
+                        hi[n] = pack_bf16(S[2 * n], S[2 * n + 1]);
+                        lo[n] = pack_bf16(S[2 * n] - bf16_of(S[2 * n]), S[2 * n + 1] - bf16_of(S[2 * n + 1]));
+                    }
+                    reinterpret_cast<uint4*>(to)[0] = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+                    reinterpret_cast<uint4*>(to)[1] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+                } else {
+                    *to = S[0];
+                }
 #pragma unroll
                 for (int n = 0; n < N; ++n) S[n] = fmaf(d[i], S[n], x[i][n]);
             }
     }
-    *reinterpret_cast<V*>(st) = *reinterpret_cast<const V*>(S);
+#pragma unroll
+    for (int n = 0; n < N; ++n) st[n] = S[n];
 }
 
-// The outputs of a chunk from its entry state. grid: (chunks, heads, requests); a warp owns 16 tokens.
-template <int DKP, int DVP>
+// The outputs of a chunk from its entry state. A warp owns 16 tokens.
+template <typename T, int DKP>
 __global__ void __launch_bounds__(DS_THREADS)
-chunk_output_kernel(const DsIn in, const float* __restrict__ entry, float* __restrict__ o, int ldo) {
+chunk_output_kernel(const DsIn in, const float* __restrict__ entry, int split, float* __restrict__ o, int ldo) {
     extern __shared__ __align__(16) unsigned char smem[];
     __shared__ float hi_s[CH], lo_s[CH], f_s[CH];
     pdl_launch_dependents();
     pdl_wait();
-    const int h = blockIdx.y, req = blockIdx.z, hq = h / (in.heads / in.kq_heads);
-    const ChunkAt at = chunk_at(in.q_start, req, blockIdx.x);
+    const Block b = block_of(in);
+    const ChunkAt& at = b.at;
     if (at.n == 0) return;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, mat = lane >> 3, rr = lane & 7, g = lane >> 2, t4 = lane & 3;
-    constexpr int RK = Tile<DKP>::ROW, RV = Tile<DVP>::ROW;
+    constexpr int RK = Tile<DKP>::ROW, RV = Tile<DV>::ROW;
     __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem);
-    __nv_bfloat16* k_s = q_s + Tile<DKP>::ELEMS;
+    __nv_bfloat16* sh_s = q_s + Tile<DKP>::ELEMS;           // the entry state, [value channel][key channel], and its remainder
+    __nv_bfloat16* sl_s = sh_s + Tile<DKP>::ELEMS;
+    __nv_bfloat16* k_s = sl_s + Tile<DKP>::ELEMS;
     __nv_bfloat16* v_s = k_s + Tile<DKP>::ELEMS;
-    __nv_bfloat16* sh_s = v_s + Tile<DVP>::ELEMS;           // the entry state, [value channel][key channel], and its remainder
-    __nv_bfloat16* sl_s = sh_s + DVP * RK;
     const bool vec = in.vec != 0, silu = in.silu != 0;
-    const float* from = entry + ((size_t)at.slot * in.heads + h) * in.dv * in.dk;
-#pragma unroll 4
-    for (int i = threadIdx.x; i < DVP * (DKP / 4); i += DS_THREADS) {
-        const int r = i / (DKP / 4), c = (i % (DKP / 4)) * 4;
-        const float4 x = row4(from + (size_t)r * in.dk, c, in.dk, r < in.dv, vec);
-        put4(sh_s + r * RK + c, x);
-        put4(sl_s + r * RK + c, rest4(x));
+    const float* from = entry + (((size_t)at.slot * in.heads + b.h) * in.dv + b.v0) * in.dk;
+    load_rows<T, DKP>(q_s, in.q_at<T>(at.row, b.hq), in.ldq, at.n, in.dk, silu, vec);
+    if (split) {
+        for (int i = threadIdx.x; i < DV * (DKP / 8); i += DS_THREADS) {
+            const int r = i / (DKP / 8), c = (i % (DKP / 8)) * 8;
+            const bool ok = r < b.nv && c < in.dk;
+            const float* p = ok ? from + (size_t)r * in.dk + c : from;
+            ds_cp_async_16(sh_s + r * RK + c, p, ok);
+            ds_cp_async_16(sl_s + r * RK + c, p + (ok ? 4 : 0), ok);
+        }
+    } else {
+        for (int i = threadIdx.x; i < DV * (DKP / 4); i += DS_THREADS) {
+            const int r = i / (DKP / 4), c = (i % (DKP / 4)) * 4;
+            float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (r < b.nv) x = row4(from + (size_t)r * in.dk, c, in.dk, false);
+            put4(sh_s + r * RK + c, x);
+            put4(sl_s + r * RK + c, rest4(x));
+        }
     }
-    load_rows<DKP>(q_s, in.q + (size_t)hq * in.dk, in.ldq, at, in.dk, silu, vec);
-    load_rows<DKP>(k_s, in.k + (size_t)hq * in.dk, in.ldk, at, in.dk, silu, vec);
-    load_rows<DVP>(v_s, in.v + (size_t)h * in.dv, in.ldv, at, in.dv, silu, vec);
-    if (warp == 0) chunk_decays(in, at, h, hi_s, lo_s, f_s);
+    ds_commit();
+    load_rows<T, DKP>(k_s, in.k_at<T>(at.row, b.hq), in.ldk, at.n, in.dk, silu, vec);
+    load_rows<T, DV>(v_s, in.v_at<T>(at.row, b.h) + b.v0, in.ldv, at.n, b.nv, silu, vec);
+    ds_commit();
+    if (warp == 0) chunk_decays(in, at, b.h, hi_s, lo_s, f_s);
+    ds_wait<1>();
     __syncthreads();
-    if (warp * 16 >= at.n) return;
     unsigned q[DKP / 16][4];
 #pragma unroll
     for (int kk = 0; kk < DKP / 16; ++kk) ldmatrix_x4(q[kk], q_s + (warp * 16 + (mat & 1) * 8 + rr) * RK + kk * 16 + (mat >> 1) * 8);
-    float acc[DVP / 8][4];
+    float acc[DV / 8][4];
 #pragma unroll
-    for (int n = 0; n < DVP / 8; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
+    for (int n = 0; n < DV / 8; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
     // q . S_in
 #pragma unroll
     for (int kk = 0; kk < DKP / 16; ++kk)
 #pragma unroll
-        for (int np = 0; np < DVP / 16; ++np) {
+        for (int np = 0; np < DV / 16; ++np) {
             const int at_s = (np * 16 + (mat >> 1) * 8 + rr) * RK + kk * 16 + (mat & 1) * 8;
-            unsigned b[4], bl[4];
-            ldmatrix_x4(b, sh_s + at_s);
+            unsigned bh[4], bl[4];
+            ldmatrix_x4(bh, sh_s + at_s);
             ldmatrix_x4(bl, sl_s + at_s);
-            mma_bf16(acc[2 * np], q[kk], b[0], b[1]);
-            mma_bf16(acc[2 * np + 1], q[kk], b[2], b[3]);
+            mma_bf16(acc[2 * np], q[kk], bh[0], bh[1]);
+            mma_bf16(acc[2 * np + 1], q[kk], bh[2], bh[3]);
             mma_bf16(acc[2 * np], q[kk], bl[0], bl[1]);
             mma_bf16(acc[2 * np + 1], q[kk], bl[2], bl[3]);
         }
@@ -420,17 +484,20 @@ chunk_output_kernel(const DsIn in, const float* __restrict__ entry, float* __res
         t_lo[r] = lo_s[warp * 16 + g + 8 * r];
         const float w = exp2f(t_hi[r] + t_lo[r]);
 #pragma unroll
-        for (int n = 0; n < DVP / 8; ++n) { acc[n][2 * r] *= w; acc[n][2 * r + 1] *= w; }
+        for (int n = 0; n < DV / 8; ++n) { acc[n][2 * r] *= w; acc[n][2 * r + 1] *= w; }
     }
+    ds_wait<0>();
+    __syncthreads();
+    if (warp * 16 >= at.n) return;
     // the chunk's own tokens, 16 keys at a time up to the warp's last token
     for (int kb = 0; kb <= warp; ++kb) {
         float s[2][4] = {};
 #pragma unroll
         for (int kk = 0; kk < DKP / 16; ++kk) {
-            unsigned b[4];
-            ldmatrix_x4(b, k_s + (kb * 16 + (mat >> 1) * 8 + rr) * RK + kk * 16 + (mat & 1) * 8);
-            mma_bf16(s[0], q[kk], b[0], b[1]);
-            mma_bf16(s[1], q[kk], b[2], b[3]);
+            unsigned bk[4];
+            ldmatrix_x4(bk, k_s + (kb * 16 + (mat >> 1) * 8 + rr) * RK + kk * 16 + (mat & 1) * 8);
+            mma_bf16(s[0], q[kk], bk[0], bk[1]);
+            mma_bf16(s[1], q[kk], bk[2], bk[3]);
         }
         unsigned p_hi[4], p_lo[4];
 #pragma unroll
@@ -448,13 +515,13 @@ chunk_output_kernel(const DsIn in, const float* __restrict__ entry, float* __res
                 p_lo[2 * n + r] = pack_bf16(x[0] - bf16_of(x[0]), x[1] - bf16_of(x[1]));
             }
 #pragma unroll
-        for (int np = 0; np < DVP / 16; ++np) {
-            unsigned b[4];
-            ldmatrix_x4_trans(b, v_s + (kb * 16 + (mat & 1) * 8 + rr) * RV + np * 16 + (mat >> 1) * 8);
-            mma_bf16(acc[2 * np], p_hi, b[0], b[1]);
-            mma_bf16(acc[2 * np + 1], p_hi, b[2], b[3]);
-            mma_bf16(acc[2 * np], p_lo, b[0], b[1]);
-            mma_bf16(acc[2 * np + 1], p_lo, b[2], b[3]);
+        for (int np = 0; np < DV / 16; ++np) {
+            unsigned bv[4];
+            ldmatrix_x4_trans(bv, v_s + (kb * 16 + (mat & 1) * 8 + rr) * RV + np * 16 + (mat >> 1) * 8);
+            mma_bf16(acc[2 * np], p_hi, bv[0], bv[1]);
+            mma_bf16(acc[2 * np + 1], p_hi, bv[2], bv[3]);
+            mma_bf16(acc[2 * np], p_lo, bv[0], bv[1]);
+            mma_bf16(acc[2 * np + 1], p_lo, bv[2], bv[3]);
         }
     }
     const bool pairs = in.dv % 2 == 0 && ldo % 2 == 0 && ((uintptr_t)o & 7) == 0;
@@ -462,53 +529,72 @@ chunk_output_kernel(const DsIn in, const float* __restrict__ entry, float* __res
     for (int r = 0; r < 2; ++r) {
         const int tok = warp * 16 + g + 8 * r;
         if (tok >= at.n) continue;
-        float* row = o + (size_t)(at.row + tok) * ldo + (size_t)h * in.dv;
+        float* row = o + (size_t)(at.row + tok) * ldo + (size_t)b.h * in.dv + b.v0;
 #pragma unroll
-        for (int n = 0; n < DVP / 8; ++n) {
+        for (int n = 0; n < DV / 8; ++n) {
             const int c = n * 8 + 2 * t4;
             if (pairs) {
-                if (c < in.dv) *reinterpret_cast<float2*>(row + c) = make_float2(acc[n][2 * r], acc[n][2 * r + 1]);
+                if (c < b.nv) *reinterpret_cast<float2*>(row + c) = make_float2(acc[n][2 * r], acc[n][2 * r + 1]);
             } else {
-                if (c < in.dv) row[c] = acc[n][2 * r];
-                if (c + 1 < in.dv) row[c + 1] = acc[n][2 * r + 1];
+                if (c < b.nv) row[c] = acc[n][2 * r];
+                if (c + 1 < b.nv) row[c + 1] = acc[n][2 * r + 1];
             }
         }
     }
 }
 
-template <int DKP, int DVP>
+template <typename T, int DKP>
 int launch_chunks(const DsIn& in, float* state, long long state_ld, int state_off, float* o, int ldo, int n_req, int max_len, float* local,
                   float* decays, cudaStream_t stream) {
-    constexpr int SMEM_STATE = (Tile<DKP>::ELEMS + 2 * Tile<DVP>::ELEMS) * 2;
-    constexpr int SMEM_OUT = (2 * Tile<DKP>::ELEMS + Tile<DVP>::ELEMS + 2 * DVP * Tile<DKP>::ROW) * 2;
+    constexpr int SMEM_STATE = (Tile<DKP>::ELEMS + Tile<DV>::ELEMS) * 2, SMEM_OUT = (4 * Tile<DKP>::ELEMS + Tile<DV>::ELEMS) * 2;
     static bool configured = false;
     if (!configured) {
-        NIB_CUDA(cudaFuncSetAttribute(chunk_state_kernel<DKP, DVP>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_STATE));
-        NIB_CUDA(cudaFuncSetAttribute(chunk_output_kernel<DKP, DVP>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_OUT));
+        NIB_CUDA(cudaFuncSetAttribute(chunk_state_kernel<T, DKP>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_STATE));
+        NIB_CUDA(cudaFuncSetAttribute(chunk_output_kernel<T, DKP>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_OUT));
         configured = true;
     }
-    const dim3 grid(ceil_div(max_len, CH), in.heads, n_req);
-    NIB_CUDA(launch_pdl(chunk_state_kernel<DKP, DVP>, grid, dim3(DS_THREADS), (size_t)SMEM_STATE, stream, in, local, decays));
+    const dim3 grid(ceil_div(max_len, CH), in.heads * ceil_div(in.dv, DV), n_req);
+    NIB_CUDA(launch_pdl(chunk_state_kernel<T, DKP>, grid, dim3(DS_THREADS), (size_t)SMEM_STATE, stream, in, local, decays));
     const int per_head = in.dv * in.dk;
     const long long elems = (long long)in.heads * per_head;
-    const bool vec = per_head % 4 == 0 && state_off % 4 == 0 && state_ld % 4 == 0 && ((uintptr_t)state & 15) == 0 && ((uintptr_t)local & 15) == 0;
-    if (vec)
-        NIB_CUDA(launch_pdl(chunk_chain_kernel<true>, dim3(ceil_div(elems, 1024), n_req), dim3(256), (size_t)0, stream, state, state_ld, state_off,
+    const int split = in.dk % 8 == 0 && ((uintptr_t)local & 15) == 0 ? 1 : 0;
+    if (split)
+        NIB_CUDA(launch_pdl(chunk_chain_kernel<true>, dim3(ceil_div(elems, 1024), n_req), dim3(128), (size_t)0, stream, state, state_ld, state_off,
                             in.q_start, in.slots, local, (const float*)decays, in.heads, per_head));
     else
-        NIB_CUDA(launch_pdl(chunk_chain_kernel<false>, dim3(ceil_div(elems, 256), n_req), dim3(256), (size_t)0, stream, state, state_ld, state_off,
+        NIB_CUDA(launch_pdl(chunk_chain_kernel<false>, dim3(ceil_div(elems, 128), n_req), dim3(128), (size_t)0, stream, state, state_ld, state_off,
                             in.q_start, in.slots, local, (const float*)decays, in.heads, per_head));
-    NIB_CUDA(launch_pdl(chunk_output_kernel<DKP, DVP>, grid, dim3(DS_THREADS), (size_t)SMEM_OUT, stream, in, (const float*)local, o, ldo));
+    NIB_CUDA(launch_pdl(chunk_output_kernel<T, DKP>, grid, dim3(DS_THREADS), (size_t)SMEM_OUT, stream, in, (const float*)local, split, o, ldo));
     NIB_LAUNCH_CHECK();
     return 0;
 }
 
-template <int LANES, int NV>
+template <typename T, int LANES, int NV>
 int launch_step(const DsIn& in, float* state, long long state_ld, int state_off, float* o, int ldo, int n_req, cudaStream_t stream) {
     const dim3 grid(ceil_div(in.dv, (DS_THREADS / LANES) * R), in.heads, n_req);
-    NIB_CUDA(launch_pdl(decay_step_kernel<LANES, NV>, grid, dim3(DS_THREADS), (size_t)0, stream, in, state, state_ld, state_off, o, ldo));
+    NIB_CUDA(launch_pdl(decay_step_kernel<T, LANES, NV>, grid, dim3(DS_THREADS), (size_t)0, stream, in, state, state_ld, state_off, o, ldo));
     NIB_LAUNCH_CHECK();
     return 0;
+}
+
+template <typename T>
+int scan(DsIn in, float* state, long long state_ld, int state_off, float* o, int ldo, int tokens, int n_req, int max_len, float* scratch,
+         cudaStream_t stream) {
+    const int dk = in.dk, dv = in.dv;
+    if (scratch == nullptr) {       // four elements a load
+        auto aligned = [](const void* p, long long ld) { return ((uintptr_t)p & (4 * sizeof(T) - 1)) == 0 && ld % 4 == 0; };
+        in.vec = dk % 4 == 0 && aligned(in.q, in.ldq) && aligned(in.k, in.ldk) && ((uintptr_t)state & 15) == 0 && state_ld % 4 == 0 && state_off % 4 == 0;
+        if (dk <= 32) return launch_step<T, 8, 1>(in, state, state_ld, state_off, o, ldo, n_req, stream);
+        if (dk <= 64) return launch_step<T, 16, 1>(in, state, state_ld, state_off, o, ldo, n_req, stream);
+        if (dk <= 128) return launch_step<T, 32, 1>(in, state, state_ld, state_off, o, ldo, n_req, stream);
+        return launch_step<T, 32, 2>(in, state, state_ld, state_off, o, ldo, n_req, stream);
+    }
+    constexpr int G = 16 / sizeof(T);       // 16 bytes a load
+    auto aligned = [](const void* p, long long ld) { return ((uintptr_t)p & 15) == 0 && ld % G == 0; };
+    in.vec = dk % G == 0 && dv % G == 0 && aligned(in.q, in.ldq) && aligned(in.k, in.ldk) && aligned(in.v, in.ldv);
+    float* decays = scratch + ((long long)tokens / CH + n_req) * in.heads * dv * dk;
+    if (dk <= 64) return launch_chunks<T, 64>(in, state, state_ld, state_off, o, ldo, n_req, max_len, scratch, decays, stream);
+    return launch_chunks<T, 128>(in, state, state_ld, state_off, o, ldo, n_req, max_len, scratch, decays, stream);
 }
 
 }  // namespace
@@ -519,35 +605,23 @@ NIB_API long long nib_decay_state_scratch(long long tokens, int n_req, int heads
     return slots * heads * ((long long)dv * dk) + slots * heads;
 }
 
-NIB_API int nib_decay_state_chunks_supported(int dk, int dv) { return dk > 0 && dv > 0 && dk <= 128 && dv <= 128 ? 1 : 0; }
+NIB_API int nib_decay_state_chunks_supported(int dk, int dv) { return dk > 0 && dv > 0 && dk <= 128 ? 1 : 0; }
 
-// q_start [n_req + 1] and slots [n_req] of the requests taken here (rows are counted from the step's first one). scratch null: token
-// by token; else in chunks, with nib_decay_state_scratch floats for the requests' tokens.
-NIB_API int nib_decay_state_scan(const float* q, int ldq, const float* k, int ldk, const float* v, int ldv, const float* raw, int ld_raw,
+// q, k and v of `dtype`. q_start [n_req + 1] and slots [n_req] of the requests taken here (rows are counted from the step's first one).
+// scratch null: token by token; else in chunks, with nib_decay_state_scratch floats for the requests' tokens.
+NIB_API int nib_decay_state_scan(const void* q, int ldq, const void* k, int ldk, const void* v, int ldv, const float* raw, int ld_raw,
                                  const float* bias, const float* a_log, const float* decay, const float* log2_decay, int silu, float* state,
                                  long long state_ld, int state_off, const int* q_start, const int* slots, float* o, int ldo, int tokens, int n_req,
-                                 int max_len, int heads, int kq_heads, int dk, int dv, float* scratch, cudaStream_t stream) {
+                                 int max_len, int heads, int kq_heads, int dk, int dv, int dtype, float* scratch, cudaStream_t stream) {
     NIB_REQUIRE(heads > 0 && kq_heads > 0 && heads % kq_heads == 0, "decay_state_scan: %d heads do not share %d key heads", heads, kq_heads);
     NIB_REQUIRE(dk > 0 && dk <= 256 && dv > 0, "decay_state_scan: key size %d is outside 1..256", dk);
     NIB_REQUIRE(raw != nullptr ? (bias != nullptr && a_log != nullptr) : (decay != nullptr && log2_decay != nullptr),
                 "decay_state_scan: step sizes need bias and a_log, fixed decays their logarithms");
-    NIB_REQUIRE(n_req >= 0 && n_req <= 65535 && heads <= 65535 && max_len >= 0, "decay_state_scan: bad counts");
+    NIB_REQUIRE(n_req >= 0 && n_req <= 65535 && (long long)heads * ceil_div(dv, DV) <= 65535 && max_len >= 0, "decay_state_scan: bad counts");
+    NIB_REQUIRE(scratch == nullptr || nib_decay_state_chunks_supported(dk, dv) == 1, "decay_state_scan: chunks take keys up to 128, not %d", dk);
     if (n_req == 0 || max_len == 0) return 0;
-    auto aligned = [](const void* p, long long ld) { return ((uintptr_t)p & 15) == 0 && ld % 4 == 0; };
-    DsIn in{q, k, v, raw, bias, a_log, decay, log2_decay, q_start, slots, ldq, ldk, ldv, ld_raw, heads, kq_heads, dk, dv, silu, 0};
-    const bool qk_vec = dk % 4 == 0 && aligned(q, ldq) && aligned(k, ldk);
-    if (scratch == nullptr) {
-        in.vec = qk_vec && aligned(state, state_ld) && state_off % 4 == 0 ? 1 : 0;
-        if (dk <= 32) return launch_step<8, 1>(in, state, state_ld, state_off, o, ldo, n_req, stream);
-        if (dk <= 64) return launch_step<16, 1>(in, state, state_ld, state_off, o, ldo, n_req, stream);
-        if (dk <= 128) return launch_step<32, 1>(in, state, state_ld, state_off, o, ldo, n_req, stream);
-        return launch_step<32, 2>(in, state, state_ld, state_off, o, ldo, n_req, stream);
-    }
-    NIB_REQUIRE(nib_decay_state_chunks_supported(dk, dv) == 1, "decay_state_scan: chunks take sizes up to 128, not %d / %d", dk, dv);
-    in.vec = qk_vec && dv % 4 == 0 && aligned(v, ldv) && ((uintptr_t)scratch & 15) == 0 ? 1 : 0;
-    float* decays = scratch + ((long long)tokens / CH + n_req) * heads * dv * dk;
-    if (dk <= 64 && dv <= 64) return launch_chunks<64, 64>(in, state, state_ld, state_off, o, ldo, n_req, max_len, scratch, decays, stream);
-    if (dk <= 64) return launch_chunks<64, 128>(in, state, state_ld, state_off, o, ldo, n_req, max_len, scratch, decays, stream);
-    if (dv <= 64) return launch_chunks<128, 64>(in, state, state_ld, state_off, o, ldo, n_req, max_len, scratch, decays, stream);
-    return launch_chunks<128, 128>(in, state, state_ld, state_off, o, ldo, n_req, max_len, scratch, decays, stream);
+    const DsIn in{q, k, v, raw, bias, a_log, decay, log2_decay, q_start, slots, ldq, ldk, ldv, ld_raw, heads, kq_heads, dk, dv, silu, 0};
+    if (dtype == NIB_F32) return scan<float>(in, state, state_ld, state_off, o, ldo, tokens, n_req, max_len, scratch, stream);
+    NIB_REQUIRE(dtype == NIB_BF16, "decay_state_scan: unknown dtype %d", dtype);
+    return scan<__nv_bfloat16>(in, state, state_ld, state_off, o, ldo, tokens, n_req, max_len, scratch, stream);
 }

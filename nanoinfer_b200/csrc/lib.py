@@ -943,7 +943,7 @@ class Kernels:
         """Row by row: y = o32 (+ skip_coef32[head of c] * skip32); times act(gate32) if ``gate_first``; with ``groups`` > 0
         divided by the root mean square of each of ``groups`` equal parts (``eps`` inside the root); times ``gain32`` (a gain
         per channel, or one of a part's size shared by the parts); times act(gate32) if not ``gate_first``; times
-        ``out_scale``. gate_kind: 'none' | 'sigmoid' | 'silu'. ``skip_coef32`` holds one coefficient per head. With ``floor32``
+        ``out_scale``. The skip may be bfloat16. gate_kind: 'none' | 'sigmoid' | 'silu'. ``skip_coef32`` holds one coefficient per head. With ``floor32``
         [tokens, groups] the rows of o32 hold ``groups`` more numbers d behind the channels, a divisor per part:
         y = o32 / (max(|d|, floor32) + den_eps) comes first."""
         self._rows(o32, torch.float32, "gated_norm o"); self._rows(out, None, "gated_norm out")
@@ -959,7 +959,7 @@ class Kernels:
             raise KernelError("gated_norm: a gate needs its kind, a skip its coefficients")
         for t, what in ((gate32, "gate"), (skip32, "skip")):
             if t is not None:
-                self._rows(t, torch.float32, f"gated_norm {what}")
+                self._rows(t, torch.float32 if what == "gate" else None, f"gated_norm {what}")
                 if tuple(t.shape) != (m, n):
                     raise KernelError(f"gated_norm: {what} does not fit")
         for t, what in ((gain32, "gain"), (skip_coef32, "skip coefficients")):
@@ -975,7 +975,8 @@ class Kernels:
             c_int(1 if gate_first else 0), _ptr(gain32), c_int(0 if gain32 is None else gain32.numel()), _ptr(skip32),
             c_int(0 if skip32 is None else skip32.stride(0)), _ptr(skip_coef32), c_int(0 if skip_coef32 is None else skip_coef32.numel()),
             c_int(groups), c_int(norm), c_float(eps), c_float(out_scale), _ptr(out), c_int(out.stride(0)), c_int(m), c_int(n),
-            c_int(_DT[out.dtype]), _ptr(floor32), c_int(0 if floor32 is None else floor32.stride(0)), c_float(den_eps), self._stream()), "gated_norm")
+            c_int(_DT[out.dtype]), _ptr(floor32), c_int(0 if floor32 is None else floor32.stride(0)), c_float(den_eps),
+            c_int(0 if skip32 is None else _DT[skip32.dtype]), self._stream()), "gated_norm")
 
     # ---- matrix states that decay (linear_state.cu) -------------------------------------------------------
     @staticmethod
@@ -1040,11 +1041,11 @@ class Kernels:
     # ---- matrix states with one decay per head: short steps token by token, prompts in chunks (decay_state.cu) --------------------
     STEP_TOKENS = 16        # what a request may bring at most to a step that is taken token by token
 
-    def decay_state_scan(self, q32, k32, v32, state, state_off, ctx, o32, heads, kq_heads, dk, dv, act="none", decay32=None, raw32=None,
+    def decay_state_scan(self, q, k, v, state, state_off, ctx, o32, heads, kq_heads, dk, dv, act="none", decay32=None, raw32=None,
                          dt_bias32=None, a_log32=None, exact=False):
         """Per request and head, over the step's tokens in order, from and into ``state[slot, state_off:]`` (laid out [head, value
-        channel, key channel]): S <- d S + f k v^T, o = S^T q. q32, k32: [tokens, kq_heads * dk] (head h reads head h // (heads /
-        kq_heads)); v32, o32: [tokens, heads * dv]; ``act`` 'silu': q, k and v pass silu first. Fixed decays: ``decay32`` [2, heads], the
+        channel, key channel]): S <- d S + f k v^T, o = S^T q. q, k: [tokens, kq_heads * dk] (head h reads head h // (heads /
+        kq_heads)); v, o32: [tokens, heads * dv]; q, k and v are floats or bfloat16; ``act`` 'silu': q, k and v pass silu first. Fixed decays: ``decay32`` [2, heads], the
         decays and their logarithms to the base 2, f = 1. Step sizes: f = softplus(raw32 + dt_bias32), d = exp(-exp(a_log32) f) with raw32
         [tokens, heads] (f is also the factor on v).
 
@@ -1052,9 +1053,9 @@ class Kernels:
         in chunks of 64 tokens on the tensor cores, where q, k and v enter as bfloat16 and everything else is 32-bit (three launches);
         leading requests of one token go token by token beside them. ``exact`` (or sizes that the chunks do not take): the 32-bit walk
         of ``linear_state_scan`` in place of the chunks."""
-        m = q32.shape[0]
-        for t, what, width in ((q32, "q", kq_heads * dk), (k32, "k", kq_heads * dk), (v32, "v", heads * dv), (o32, "o", heads * dv)):
-            self._rows(t, torch.float32, f"decay_state_scan {what}")
+        m = q.shape[0]
+        for t, what, width in ((q, "q", kq_heads * dk), (k, "k", kq_heads * dk), (v, "v", heads * dv), (o32, "o", heads * dv)):
+            self._rows(t, torch.float32 if what == "o" else q.dtype, f"decay_state_scan {what}")
             if tuple(t.shape) != (m, width):
                 raise KernelError(f"decay_state_scan: {what} does not fit")
         if (decay32 is None) == (raw32 is None) or act not in ("none", "silu"):
@@ -1073,40 +1074,41 @@ class Kernels:
         n_req, longest = len(q_lens), max(q_lens)
         short = longest <= self.STEP_TOKENS
         if not short and (exact or self._lib.nib_decay_state_chunks_supported(c_int(dk), c_int(dv)) != 1):
-            self._decay_state_exact(q32, k32, v32, state, state_off, ctx, o32, heads, kq_heads, dk, dv, act, decay32, raw32, dt_bias32, a_log32)
+            self._decay_state_exact(q, k, v, state, state_off, ctx, o32, heads, kq_heads, dk, dv, act, decay32, raw32, dt_bias32, a_log32)
             return
         n_step = n_req if short else next((i for i, n in enumerate(q_lens) if n != 1), n_req)
 
         def scan(first, count, tokens, most, scratch, what):
             self._check(self._lib.nib_decay_state_scan(
-                _ptr(q32), c_int(q32.stride(0)), _ptr(k32), c_int(k32.stride(0)), _ptr(v32), c_int(v32.stride(0)), _ptr(raw32),
+                _ptr(q), c_int(q.stride(0)), _ptr(k), c_int(k.stride(0)), _ptr(v), c_int(v.stride(0)), _ptr(raw32),
                 c_int(0 if raw32 is None else raw32.stride(0)), _ptr(dt_bias32), _ptr(a_log32), _ptr(None if decay32 is None else decay32[0]),
                 _ptr(None if decay32 is None else decay32[1]), c_int(1 if act == "silu" else 0), _ptr(state), c_longlong(state.stride(0)),
                 c_int(state_off), c_void_p(ctx.q_start.data_ptr() + 4 * first), c_void_p(ctx.state_slots.data_ptr() + 4 * first), _ptr(o32),
-                c_int(o32.stride(0)), c_int(tokens), c_int(count), c_int(most), c_int(heads), c_int(kq_heads), c_int(dk), c_int(dv), _ptr(scratch),
-                self._stream()), what)
+                c_int(o32.stride(0)), c_int(tokens), c_int(count), c_int(most), c_int(heads), c_int(kq_heads), c_int(dk), c_int(dv),
+                c_int(_DT[q.dtype]), _ptr(scratch), self._stream()), what)
 
         if n_step:
             scan(0, n_step, sum(q_lens[:n_step]), longest if short else 1, None, "decay_state_scan (short step)")
         if n_step < n_req:
             tokens, count = sum(q_lens[n_step:]), n_req - n_step
             floats = self._lib.nib_decay_state_scratch(c_longlong(tokens), c_int(count), c_int(heads), c_int(dk), c_int(dv))
-            scratch = torch.empty(floats, dtype=torch.float32, device=q32.device)
+            scratch = torch.empty(floats, dtype=torch.float32, device=q.device)
             self.launches += 2
             scan(n_step, count, tokens, longest, scratch, "decay_state_scan (chunks)")
 
-    def _decay_state_exact(self, q32, k32, v32, state, state_off, ctx, o32, heads, kq_heads, dk, dv, act, decay32, raw32, dt_bias32, a_log32):
+    def _decay_state_exact(self, q, k, v, state, state_off, ctx, o32, heads, kq_heads, dk, dv, act, decay32, raw32, dt_bias32, a_log32):
         """The same in 32-bit whatever the length, from the unfused operations."""
-        m, dev = q32.shape[0], q32.device
+        m, dev = q.shape[0], q.device
+        q, k, v = (t.float() for t in (q, k, v))        # (nothing to do for floats)
         if act == "silu":
-            q32, k32, v32 = (self._unary_new(t, "silu") for t in (q32, k32, v32))
+            q, k, v = (self._unary_new(t, "silu") for t in (q, k, v))
         step = None
         if raw32 is not None:
             step, decay = torch.empty((2, m, heads), dtype=torch.float32, device=dev).unbind(0)
             self.step_sizes(raw32, dt_bias32, a_log32, step, decay)
         else:
             decay = decay32[:1].expand(m, heads)        # every row the same one
-        self.linear_state_scan(q32, k32, v32, decay, state, state_off, ctx, o32, heads, kq_heads, dk, dv, v_scale32=step)
+        self.linear_state_scan(q, k, v, decay, state, state_off, ctx, o32, heads, kq_heads, dk, dv, v_scale32=step)
 
     def _unary_new(self, t32, kind):
         out = torch.empty(t32.shape, dtype=torch.float32, device=t32.device)
@@ -1182,9 +1184,9 @@ class Kernels:
             c_float(q_scale), c_float(-1.0 if unit_eps is None else unit_eps), self._stream()), "grouped_state_scan")
 
     def conv_tokens(self, x32, w32, bias32, act, state, state_off, ctx, out32, taps):
-        """out32[t, c] = act(bias32[c] + sum_j w32[c, j] * x32[t - (taps-1-j), c]) within each request; inputs before the
+        """out32[t, c] (floats or bfloat16) = act(bias32[c] + sum_j w32[c, j] * x32[t - (taps-1-j), c]) within each request; inputs before the
         step's first token come from ``state[slot, state_off + i * width + c]`` (i = 0 oldest). act: 'none' | 'silu'."""
-        self._rows(x32, torch.float32, "conv_tokens x"); self._rows(out32, torch.float32, "conv_tokens out"); _need(w32, torch.float32, "conv_tokens w")
+        self._rows(x32, torch.float32, "conv_tokens x"); self._rows(out32, None, "conv_tokens out"); _need(w32, torch.float32, "conv_tokens w")
         m, width = x32.shape
         if tuple(w32.shape) != (width, taps) or tuple(out32.shape) != (m, width) or (bias32 is not None and bias32.numel() != width):
             raise KernelError("conv_tokens: shapes do not fit")
@@ -1195,7 +1197,7 @@ class Kernels:
         self._check(self._lib.nib_conv_tokens(
             _ptr(x32), c_int(x32.stride(0)), _ptr(w32), _ptr(bias32), c_int({"none": 0, "silu": 1}[act]), _ptr(state if taps > 1 else None),
             c_longlong(state.stride(0) if taps > 1 else 0), c_int(state_off), _ptr(ctx.q_start), _ptr(ctx.req_index), _ptr(ctx.state_slots),
-            _ptr(out32), c_int(out32.stride(0)), c_int(m), c_int(width), c_int(taps), self._stream()), "conv_tokens")
+            _ptr(out32), c_int(out32.stride(0)), c_int(m), c_int(width), c_int(taps), c_int(_DT[out32.dtype]), self._stream()), "conv_tokens")
 
     def conv_tail(self, x32, state, state_off, ctx, taps):
         """The state's history rows become each request's last taps-1 rows of x32 (older rows move up when the step brought
@@ -1214,7 +1216,7 @@ class Kernels:
             if taps > 1:
                 self.conv_tail(x32, state, state_off, ctx, taps)
             return
-        self._rows(x32, torch.float32, "conv_step x"); self._rows(out32, torch.float32, "conv_step out"); _need(w32, torch.float32, "conv_step w")
+        self._rows(x32, torch.float32, "conv_step x"); self._rows(out32, None, "conv_step out"); _need(w32, torch.float32, "conv_step w")
         m, width = x32.shape
         if tuple(w32.shape) != (width, taps) or tuple(out32.shape) != (m, width) or (bias32 is not None and bias32.numel() != width):
             raise KernelError("conv_step: shapes do not fit")
@@ -1225,7 +1227,7 @@ class Kernels:
         self._check(self._lib.nib_conv_step(
             _ptr(x32), c_int(x32.stride(0)), _ptr(w32), _ptr(bias32), c_int({"none": 0, "silu": 1}[act]), _ptr(state if taps > 1 else None),
             c_longlong(state.stride(0) if taps > 1 else 0), c_int(state_off), _ptr(ctx.q_start), _ptr(ctx.state_slots), _ptr(out32),
-            c_int(out32.stride(0)), c_int(ctx.host.num_requests), c_int(width), c_int(taps), self._stream()), "conv_step")
+            c_int(out32.stride(0)), c_int(ctx.host.num_requests), c_int(width), c_int(taps), c_int(_DT[out32.dtype]), self._stream()), "conv_step")
 
     def token_shift(self, h, mu32, state, state_off, ctx, mixes):
         """mixes[s, t] = h[t] + (h[t-1] - h[t]) * mu32[s]; the token before a request's first one in the step is

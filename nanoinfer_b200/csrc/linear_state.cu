@@ -322,11 +322,12 @@ NIB_API int nib_linear_state_scan(const float* q, int ldq, const float* k, int l
 // ---------------------------------------------------------------------------------- short causal convolution
 // y[t, c] = act(bias[c] + sum_j w[c, j] * u[t - (taps-1-j), c]) within each request; inputs before the step's first token
 // come from the state's history rows (state[slot, off + i * width + c], i = 0 oldest .. taps-2), zeros at a request's
-// start. One thread per (token, channel), taps added in ascending order. act: 0 none, 1 silu.
+// start. One thread per (token, channel), taps added in ascending order. act: 0 none, 1 silu. The result is written as T.
+template <typename T>
 __global__ void __launch_bounds__(256)
 conv_tokens_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ w, const float* __restrict__ bias, int act,
                    const float* __restrict__ state, long long state_ld, int state_off, const int* __restrict__ q_start,
-                   const int* __restrict__ req_index, const int* __restrict__ slots, float* __restrict__ y, int ldy,
+                   const int* __restrict__ req_index, const int* __restrict__ slots, T* __restrict__ y, int ldy,
                    int tokens, int width, int taps) {
     pdl_launch_dependents();
     pdl_wait();      // everything this kernel reads may come from the kernel before
@@ -343,7 +344,7 @@ conv_tokens_kernel(const float* __restrict__ x, int ldx, const float* __restrict
         acc = fmaf(w[(size_t)c * taps + j], u, acc);
     }
     if (act == 1) acc = acc / (1.0f + expf(-acc));
-    y[(size_t)t * ldy + c] = acc;
+    Elem<T>::store(y + (size_t)t * ldy + c, acc);
 }
 
 // The same, four channels and eight consecutive tokens a thread: the inputs of a token's window slide through registers, so
@@ -351,11 +352,11 @@ conv_tokens_kernel(const float* __restrict__ x, int ldx, const float* __restrict
 // bias).
 constexpr int CONV_VEC_TAPS = 8, CONV_VEC_TOKENS = 8;
 
-template <int TAPS>
+template <typename T, int TAPS>
 __global__ void __launch_bounds__(128)
 conv_tokens_vec_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ w, const float* __restrict__ bias, int act,
                        const float* __restrict__ state, long long state_ld, int state_off, const int* __restrict__ q_start,
-                       const int* __restrict__ req_index, const int* __restrict__ slots, float* __restrict__ y, int ldy,
+                       const int* __restrict__ req_index, const int* __restrict__ slots, T* __restrict__ y, int ldy,
                        int tokens, int width) {
     pdl_launch_dependents();
     const int c = (blockIdx.y * 128 + threadIdx.x) * 4, t0 = blockIdx.x * CONV_VEC_TOKENS, t1 = min(tokens, t0 + CONV_VEC_TOKENS);
@@ -396,7 +397,13 @@ conv_tokens_vec_kernel(const float* __restrict__ x, int ldx, const float* __rest
 #pragma unroll
             for (int e = 0; e < 4; ++e) acc[e] = acc[e] / (1.0f + expf(-acc[e]));
         }
-        *reinterpret_cast<float4*>(y + (size_t)t * ldy + c) = make_float4(acc[0], acc[1], acc[2], acc[3]);
+        T* to = y + (size_t)t * ldy + c;
+        if constexpr (sizeof(T) == 4) {
+            *reinterpret_cast<float4*>(to) = make_float4(acc[0], acc[1], acc[2], acc[3]);
+        } else {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(acc[0], acc[1]), hi = __floats2bfloat162_rn(acc[2], acc[3]);
+            *reinterpret_cast<uint2*>(to) = make_uint2(*reinterpret_cast<const unsigned*>(&lo), *reinterpret_cast<const unsigned*>(&hi));
+        }
 #pragma unroll
         for (int j = 0; j < TAPS - 2; ++j) win[j] = win[j + 1];
         if (TAPS > 1) win[TAPS > 1 ? TAPS - 2 : 0] = u;
@@ -421,25 +428,34 @@ conv_tail_kernel(const float* __restrict__ x, int ldx, float* __restrict__ state
     }
 }
 
-NIB_API int nib_conv_tokens(const float* x, int ldx, const float* w, const float* bias, int act, const float* state, long long state_ld,
-                            int state_off, const int* q_start, const int* req_index, const int* slots, float* y, int ldy, int tokens,
-                            int width, int taps, cudaStream_t stream) {
-    NIB_REQUIRE(tokens >= 0 && width > 0 && taps >= 1 && (taps == 1 || state != nullptr), "conv_tokens: bad sizes or no state for %d taps", taps);
-    if (tokens == 0) return 0;
-    if (taps <= CONV_VEC_TAPS && width % 4 == 0 && ldx % 4 == 0 && ldy % 4 == 0 && (((uintptr_t)x | (uintptr_t)y) & 15) == 0) {
+template <typename T>
+static int launch_conv_tokens(const float* x, int ldx, const float* w, const float* bias, int act, const float* state, long long state_ld,
+                              int state_off, const int* q_start, const int* req_index, const int* slots, T* y, int ldy, int tokens, int width,
+                              int taps, cudaStream_t stream) {
+    if (taps <= CONV_VEC_TAPS && width % 4 == 0 && ldx % 4 == 0 && ldy % 4 == 0 && ((uintptr_t)x & 15) == 0 && ((uintptr_t)y & (4 * sizeof(T) - 1)) == 0) {
         const dim3 grid(ceil_div(tokens, CONV_VEC_TOKENS), ceil_div(width, 512));
 #define NIB_CV(TAPS) \
-    case TAPS: NIB_CUDA(launch_pdl(conv_tokens_vec_kernel<TAPS>, grid, dim3(128), (size_t)0, stream, x, ldx, w, bias, act, state, state_ld, state_off, \
+    case TAPS: NIB_CUDA(launch_pdl(conv_tokens_vec_kernel<T, TAPS>, grid, dim3(128), (size_t)0, stream, x, ldx, w, bias, act, state, state_ld, state_off, \
                                    q_start, req_index, slots, y, ldy, tokens, width)); break;
         switch (taps) { NIB_CV(1) NIB_CV(2) NIB_CV(3) NIB_CV(4) NIB_CV(5) NIB_CV(6) NIB_CV(7) NIB_CV(8) }
 #undef NIB_CV
         NIB_LAUNCH_CHECK();
         return 0;
     }
-    NIB_CUDA(launch_pdl(conv_tokens_kernel, dim3(ceil_div((long long)tokens * width, 256)), dim3(256), (size_t)0, stream, x, ldx, w, bias, act,
+    NIB_CUDA(launch_pdl(conv_tokens_kernel<T>, dim3(ceil_div((long long)tokens * width, 256)), dim3(256), (size_t)0, stream, x, ldx, w, bias, act,
                         state, state_ld, state_off, q_start, req_index, slots, y, ldy, tokens, width, taps));
     NIB_LAUNCH_CHECK();
     return 0;
+}
+
+NIB_API int nib_conv_tokens(const float* x, int ldx, const float* w, const float* bias, int act, const float* state, long long state_ld,
+                            int state_off, const int* q_start, const int* req_index, const int* slots, void* y, int ldy, int tokens,
+                            int width, int taps, int dtype, cudaStream_t stream) {
+    NIB_REQUIRE(tokens >= 0 && width > 0 && taps >= 1 && (taps == 1 || state != nullptr), "conv_tokens: bad sizes or no state for %d taps", taps);
+    NIB_REQUIRE(dtype == NIB_F32 || dtype == NIB_BF16, "conv_tokens: unknown dtype %d", dtype);
+    if (tokens == 0) return 0;
+    return dtype == NIB_F32 ? launch_conv_tokens(x, ldx, w, bias, act, state, state_ld, state_off, q_start, req_index, slots, (float*)y, ldy, tokens, width, taps, stream)
+                            : launch_conv_tokens(x, ldx, w, bias, act, state, state_ld, state_off, q_start, req_index, slots, (__nv_bfloat16*)y, ldy, tokens, width, taps, stream);
 }
 
 NIB_API int nib_conv_tail(const float* x, int ldx, float* state, long long state_ld, int state_off, const int* q_start, const int* slots,
@@ -457,10 +473,11 @@ NIB_API int nib_conv_tail(const float* x, int ldx, float* state, long long state
 // conv_tokens_kernel (taps added in ascending order from the bias).
 constexpr int CONV_STEP_MAX_TAPS = 16;
 
+template <typename T>
 __global__ void __launch_bounds__(256)
 conv_step_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ w, const float* __restrict__ bias, int act,
                  float* __restrict__ state, long long state_ld, int state_off, const int* __restrict__ q_start,
-                 const int* __restrict__ slots, float* __restrict__ y, int ldy, int n_req, int width, int taps) {
+                 const int* __restrict__ slots, T* __restrict__ y, int ldy, int n_req, int width, int taps) {
     pdl_launch_dependents();
     pdl_wait();      // everything this kernel reads may come from the kernel before
     const long long e = (long long)blockIdx.x * 256 + threadIdx.x;
@@ -485,7 +502,7 @@ conv_step_kernel(const float* __restrict__ x, int ldx, const float* __restrict__
         for (int j = 0; j < CONV_STEP_MAX_TAPS; ++j)
             if (j == taps - 1) acc = fmaf(wt[j], u, acc);
         if (act == 1) acc = acc / (1.0f + expf(-acc));
-        y[(size_t)(first + i) * ldy + c] = acc;
+        Elem<T>::store(y + (size_t)(first + i) * ldy + c, acc);
 #pragma unroll
         for (int j = 0; j < CONV_STEP_MAX_TAPS - 1; ++j) {
             if (j < taps - 2) win[j] = win[j + 1 < CONV_STEP_MAX_TAPS - 1 ? j + 1 : j];
@@ -498,13 +515,19 @@ conv_step_kernel(const float* __restrict__ x, int ldx, const float* __restrict__
 }
 
 NIB_API int nib_conv_step(const float* x, int ldx, const float* w, const float* bias, int act, float* state, long long state_ld,
-                          int state_off, const int* q_start, const int* slots, float* y, int ldy, int n_req, int width, int taps,
-                          cudaStream_t stream) {
+                          int state_off, const int* q_start, const int* slots, void* y, int ldy, int n_req, int width, int taps,
+                          int dtype, cudaStream_t stream) {
     NIB_REQUIRE(n_req >= 0 && width > 0 && taps >= 1 && taps <= CONV_STEP_MAX_TAPS && (taps == 1 || state != nullptr),
                 "conv_step: bad sizes, more than %d taps, or no state", CONV_STEP_MAX_TAPS);
+    NIB_REQUIRE(dtype == NIB_F32 || dtype == NIB_BF16, "conv_step: unknown dtype %d", dtype);
     if (n_req == 0) return 0;
-    NIB_CUDA(launch_pdl(conv_step_kernel, dim3(ceil_div((long long)n_req * width, 256)), dim3(256), (size_t)0, stream, x, ldx, w, bias, act,
-                        state, state_ld, state_off, q_start, slots, y, ldy, n_req, width, taps));
+    const dim3 grid(ceil_div((long long)n_req * width, 256));
+    if (dtype == NIB_F32)
+        NIB_CUDA(launch_pdl(conv_step_kernel<float>, grid, dim3(256), (size_t)0, stream, x, ldx, w, bias, act, state, state_ld, state_off, q_start,
+                            slots, (float*)y, ldy, n_req, width, taps));
+    else
+        NIB_CUDA(launch_pdl(conv_step_kernel<__nv_bfloat16>, grid, dim3(256), (size_t)0, stream, x, ldx, w, bias, act, state, state_ld, state_off,
+                            q_start, slots, (__nv_bfloat16*)y, ldy, n_req, width, taps));
     NIB_LAUNCH_CHECK();
     return 0;
 }

@@ -406,16 +406,17 @@ NIB_API int nib_depth_mix_norm_pair(float* hist, float* x, const float* coef, in
 //     y = y * gain[c % gain_len]                        gain_len = n (a gain per channel) or a part's size (shared)
 //     y = y * act(gate)                                 if not gate_first
 //     out = y * out_scale
-// act: 1 sigmoid, 2 silu, 0 none. With norm the part is read twice (sum of squares, then the result).
+// act: 1 sigmoid, 2 silu, 0 none. With norm the part is read twice (sum of squares, then the result). The skip's rows are floats
+// or, TS, bfloat16.
 __device__ __forceinline__ float gate_act(float g, int kind) {
     const float s = 1.0f / (1.0f + expf(-g));
     return kind == 1 ? s : g * s;
 }
 
-template <typename T>
+template <typename T, typename TS>
 __global__ void __launch_bounds__(128)
 gated_norm_kernel(const float* __restrict__ o, int ldo, const float* __restrict__ gate, int ldg, int gate_kind, int gate_first,
-                  const float* __restrict__ gain, int gain_len, const float* __restrict__ skip, int lds,
+                  const float* __restrict__ gain, int gain_len, const TS* __restrict__ skip, int lds,
                   const float* __restrict__ coef, int coef_span, int norm, float eps, float out_scale,
                   T* __restrict__ out, int ld_out, int tokens, int groups, int width, const float* __restrict__ floor_in, int ldf, float den_eps) {
     pdl_launch_dependents();
@@ -427,7 +428,7 @@ gated_norm_kernel(const float* __restrict__ o, int ldo, const float* __restrict_
     const float* orow = o + (size_t)t * ldo;
     const float den = floor_in != nullptr ? fmaxf(fabsf(orow[groups * width + part_i]), floor_in[(size_t)t * ldf + part_i]) + den_eps : 1.0f;
     const float* grow = gate != nullptr ? gate + (size_t)t * ldg : nullptr;
-    const float* srow = skip != nullptr ? skip + (size_t)t * lds : nullptr;
+    const TS* srow = skip != nullptr ? skip + (size_t)t * lds : nullptr;
     const bool early = grow != nullptr && gate_kind != 0 && gate_first != 0;
     const bool late = grow != nullptr && gate_kind != 0 && gate_first == 0;
     float scale = 1.0f;
@@ -436,7 +437,7 @@ gated_norm_kernel(const float* __restrict__ o, int ldo, const float* __restrict_
         for (int j = lane; j < width; j += 32) {
             const int c = c0 + j;
             float y = floor_in != nullptr ? orow[c] / den : orow[c];
-            if (srow != nullptr) y = fmaf(coef[c / coef_span], srow[c], y);
+            if (srow != nullptr) y = fmaf(coef[c / coef_span], Elem<TS>::load(srow + c), y);
             if (early) y *= gate_act(grow[c], gate_kind);
             ss = fmaf(y, y, ss);
         }
@@ -446,7 +447,7 @@ gated_norm_kernel(const float* __restrict__ o, int ldo, const float* __restrict_
     for (int j = lane; j < width; j += 32) {
         const int c = c0 + j;
         float y = floor_in != nullptr ? orow[c] / den : orow[c];
-        if (srow != nullptr) y = fmaf(coef[c / coef_span], srow[c], y);
+        if (srow != nullptr) y = fmaf(coef[c / coef_span], Elem<TS>::load(srow + c), y);
         if (early) y *= gate_act(grow[c], gate_kind);
         y *= scale;
         if (gain != nullptr) y *= gain[c % gain_len];
@@ -457,10 +458,10 @@ gated_norm_kernel(const float* __restrict__ o, int ldo, const float* __restrict_
 
 // The same for wide parts (a state-space mixer's norm over thousands of channels): a block of 256 threads per
 // (token, part), so that the few rows of a decode step are not walked by one warp each.
-template <typename T>
+template <typename T, typename TS>
 __global__ void __launch_bounds__(256)
 gated_norm_block_kernel(const float* __restrict__ o, int ldo, const float* __restrict__ gate, int ldg, int gate_kind, int gate_first,
-                        const float* __restrict__ gain, int gain_len, const float* __restrict__ skip, int lds,
+                        const float* __restrict__ gain, int gain_len, const TS* __restrict__ skip, int lds,
                         const float* __restrict__ coef, int coef_span, int norm, float eps, float out_scale,
                         T* __restrict__ out, int ld_out, int tokens, int groups, int width, const float* __restrict__ floor_in, int ldf, float den_eps) {
     pdl_launch_dependents();
@@ -470,7 +471,7 @@ gated_norm_block_kernel(const float* __restrict__ o, int ldo, const float* __res
     const float* orow = o + (size_t)t * ldo;
     const float den = floor_in != nullptr ? fmaxf(fabsf(orow[groups * width + part_i]), floor_in[(size_t)t * ldf + part_i]) + den_eps : 1.0f;
     const float* grow = gate != nullptr ? gate + (size_t)t * ldg : nullptr;
-    const float* srow = skip != nullptr ? skip + (size_t)t * lds : nullptr;
+    const TS* srow = skip != nullptr ? skip + (size_t)t * lds : nullptr;
     const bool early = grow != nullptr && gate_kind != 0 && gate_first != 0;
     const bool late = grow != nullptr && gate_kind != 0 && gate_first == 0;
     float scale = 1.0f;
@@ -479,7 +480,7 @@ gated_norm_block_kernel(const float* __restrict__ o, int ldo, const float* __res
         for (int j = threadIdx.x; j < width; j += 256) {
             const int c = c0 + j;
             float y = floor_in != nullptr ? orow[c] / den : orow[c];
-            if (srow != nullptr) y = fmaf(coef[c / coef_span], srow[c], y);
+            if (srow != nullptr) y = fmaf(coef[c / coef_span], Elem<TS>::load(srow + c), y);
             if (early) y *= gate_act(grow[c], gate_kind);
             ss = fmaf(y, y, ss);
         }
@@ -488,7 +489,7 @@ gated_norm_block_kernel(const float* __restrict__ o, int ldo, const float* __res
     for (int j = threadIdx.x; j < width; j += 256) {
         const int c = c0 + j;
         float y = floor_in != nullptr ? orow[c] / den : orow[c];
-        if (srow != nullptr) y = fmaf(coef[c / coef_span], srow[c], y);
+        if (srow != nullptr) y = fmaf(coef[c / coef_span], Elem<TS>::load(srow + c), y);
         if (early) y *= gate_act(grow[c], gate_kind);
         y *= scale;
         if (gain != nullptr) y *= gain[c % gain_len];
@@ -550,9 +551,112 @@ gated_norm_vec_kernel(const float* __restrict__ o, int ldo, const float* __restr
     }
 }
 
+// The same for wide parts in rows of whole 16-byte groups, without a divisor: a block per (token, part), NV times four channels a
+// thread, held in registers between the sum of squares and the result (every row is read once).
+__device__ __forceinline__ float4 four_of(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 four_of(const __nv_bfloat16* p) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+
+template <typename T, typename TS, int THREADS, int NV>
+__global__ void __launch_bounds__(THREADS)
+gated_norm_wide_kernel(const float* __restrict__ o, int ldo, const float* __restrict__ gate, int ldg, int gate_kind, int gate_first,
+                       const float* __restrict__ gain, int gain_len, const TS* __restrict__ skip, int lds, const float* __restrict__ coef, int coef_span,
+                       int norm, float eps, float out_scale, T* __restrict__ out, int ld_out, int groups, int width) {
+    __shared__ float part[THREADS / 32];
+    pdl_launch_dependents();
+    const int t = blockIdx.x / groups, c0 = (blockIdx.x % groups) * width, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    float4 ga[NV];
+    float cf[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {      // weights: fetched before the wait
+        const int j = (threadIdx.x + THREADS * i) * 4;
+        ga[i] = gain != nullptr && j < width ? __ldg(reinterpret_cast<const float4*>(gain + (c0 + j) % gain_len)) : make_float4(1.f, 1.f, 1.f, 1.f);
+        cf[i] = skip != nullptr && j < width ? __ldg(coef + (c0 + j) / coef_span) : 0.f;
+    }
+    pdl_wait();
+    float4 y[NV], gv[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int j = (threadIdx.x + THREADS * i) * 4;
+        y[i] = gv[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (j >= width) continue;
+        y[i] = four_of(o + (size_t)t * ldo + c0 + j);
+        if (gate != nullptr) gv[i] = four_of(gate + (size_t)t * ldg + c0 + j);
+        if (skip != nullptr) {
+            const float4 x = four_of(skip + (size_t)t * lds + c0 + j);
+            y[i].x = fmaf(cf[i], x.x, y[i].x); y[i].y = fmaf(cf[i], x.y, y[i].y); y[i].z = fmaf(cf[i], x.z, y[i].z); y[i].w = fmaf(cf[i], x.w, y[i].w);
+        }
+    }
+    const bool gated = gate != nullptr && gate_kind != 0;
+    if (gated) {
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            gv[i] = make_float4(gate_act(gv[i].x, gate_kind), gate_act(gv[i].y, gate_kind), gate_act(gv[i].z, gate_kind), gate_act(gv[i].w, gate_kind));
+            if (gate_first) { y[i].x *= gv[i].x; y[i].y *= gv[i].y; y[i].z *= gv[i].z; y[i].w *= gv[i].w; }
+        }
+    }
+    float scale = out_scale;
+    if (norm) {
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) ss = fmaf(y[i].x, y[i].x, fmaf(y[i].y, y[i].y, fmaf(y[i].z, y[i].z, fmaf(y[i].w, y[i].w, ss))));
+        ss = warp_sum(ss);
+        if (lane == 0) part[warp] = ss;
+        __syncthreads();
+        ss = 0.f;
+#pragma unroll
+        for (int w = 0; w < THREADS / 32; ++w) ss += part[w];
+        scale = out_scale / sqrtf(ss / (float)width + eps);
+    }
+    const bool late = gated && !gate_first;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int j = (threadIdx.x + THREADS * i) * 4;
+        if (j >= width) continue;
+        float v[4] = {y[i].x * scale * ga[i].x, y[i].y * scale * ga[i].y, y[i].z * scale * ga[i].z, y[i].w * scale * ga[i].w};
+        if (late) { v[0] *= gv[i].x; v[1] *= gv[i].y; v[2] *= gv[i].z; v[3] *= gv[i].w; }
+        T* to = out + (size_t)t * ld_out + c0 + j;
+        if constexpr (sizeof(T) == 4) {
+            *reinterpret_cast<float4*>(to) = make_float4(v[0], v[1], v[2], v[3]);
+        } else {
+            const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+            *reinterpret_cast<uint2*>(to) = make_uint2(*reinterpret_cast<const unsigned*>(&lo), *reinterpret_cast<const unsigned*>(&hi));
+        }
+    }
+}
+
+template <typename T, typename TS>
+static int launch_gated_norm(const float* o, int ldo, const float* gate, int ldg, int gate_kind, int gate_first, const float* gain, int gain_len,
+                             const TS* skip, int lds, const float* coef, int span, int groups, int norm, float eps, float out_scale, T* out, int ld_out,
+                             int tokens, int width, const float* floor_in, int ldf, float den_eps, cudaStream_t stream) {
+    auto on = [](const void* p, long long ld, size_t elem) { return ((uintptr_t)p & (4 * elem - 1)) == 0 && ld % 4 == 0; };
+    if (width > 256 && width <= 4096 && width % 4 == 0 && floor_in == nullptr && on(o, ldo, 4) && on(gate, ldg, 4) && on(skip, lds, sizeof(TS)) && on(out, ld_out, sizeof(T))
+        && on(gain, gain_len, 4) && (skip == nullptr || span % 4 == 0)) {
+#define NIB_GN(THREADS, NV) NIB_CUDA(launch_pdl(gated_norm_wide_kernel<T, TS, THREADS, NV>, dim3(tokens * groups), dim3(THREADS), (size_t)0, stream, o, ldo, gate, ldg, \
+                                                gate_kind, gate_first, gain, gain_len, skip, lds, coef, span, norm, eps, out_scale, out, ld_out, groups, width))
+        if (width <= 512) NIB_GN(128, 1);
+        else if (width <= 1024) NIB_GN(256, 1);
+        else if (width <= 2048) NIB_GN(256, 2);
+        else NIB_GN(256, 4);
+#undef NIB_GN
+    } else if (width > 256) {
+        NIB_CUDA(launch_pdl(gated_norm_block_kernel<T, TS>, dim3(tokens * groups), dim3(256), (size_t)(0), stream, o, ldo, gate, ldg, gate_kind, gate_first, gain,
+                            gain_len, skip, lds, coef, span, norm, eps, out_scale, out, ld_out, tokens, groups, width, floor_in, ldf, den_eps));
+    } else {
+        NIB_CUDA(launch_pdl(gated_norm_kernel<T, TS>, dim3(ceil_div((long long)tokens * groups, 4)), dim3(128), (size_t)(0), stream, o, ldo, gate, ldg, gate_kind,
+                            gate_first, gain, gain_len, skip, lds, coef, span, norm, eps, out_scale, out, ld_out, tokens, groups, width, floor_in, ldf, den_eps));
+    }
+    NIB_LAUNCH_CHECK();
+    return 0;
+}
+
 NIB_API int nib_gated_norm(const float* o, int ldo, const float* gate, int ldg, int gate_kind, int gate_first, const float* gain,
-                           int gain_len, const float* skip, int lds, const float* coef, int n_coef, int groups, int norm, float eps,
-                           float out_scale, void* out, int ld_out, int tokens, int n, int dtype, const float* floor_in, int ldf, float den_eps, cudaStream_t stream) {
+                           int gain_len, const void* skip, int lds, const float* coef, int n_coef, int groups, int norm, float eps,
+                           float out_scale, void* out, int ld_out, int tokens, int n, int dtype, const float* floor_in, int ldf, float den_eps, int skip_dtype,
+                           cudaStream_t stream) {
     NIB_REQUIRE(tokens >= 0 && n > 0 && groups > 0 && n % groups == 0, "gated_norm: %d channels do not split into %d parts", n, groups);
     NIB_REQUIRE(gain == nullptr || (gain_len > 0 && n % gain_len == 0), "gated_norm: a gain of %d does not tile %d channels", gain_len, n);
     NIB_REQUIRE(skip == nullptr || (coef != nullptr && n_coef > 0 && n % n_coef == 0), "gated_norm: bad skip coefficients");
@@ -574,20 +678,12 @@ NIB_API int nib_gated_norm(const float* o, int ldo, const float* gate, int ldg, 
         NIB_LAUNCH_CHECK();
         return 0;
     }
-    if (width > 256) {
-        const dim3 grid(tokens * groups);
-        if (dtype == NIB_F32) NIB_CUDA(launch_pdl(gated_norm_block_kernel<float>, grid, dim3(256), (size_t)(0), stream, o, ldo, gate, ldg, gate_kind, gate_first, gain, gain_len, skip, lds, coef, span, norm, eps, out_scale, (float*)out, ld_out, tokens, groups, width, floor_in, ldf, den_eps));
-        else if (dtype == NIB_BF16) NIB_CUDA(launch_pdl(gated_norm_block_kernel<__nv_bfloat16>, grid, dim3(256), (size_t)(0), stream, o, ldo, gate, ldg, gate_kind, gate_first, gain, gain_len, skip, lds, coef, span, norm, eps, out_scale, (__nv_bfloat16*)out, ld_out, tokens, groups, width, floor_in, ldf, den_eps));
-        else NIB_REQUIRE(false, "gated_norm: unknown dtype %d", dtype);
-        NIB_LAUNCH_CHECK();
-        return 0;
-    }
-    const int blocks = ceil_div((long long)tokens * groups, 4);
-    if (dtype == NIB_F32) NIB_CUDA(launch_pdl(gated_norm_kernel<float>, dim3(blocks), dim3(128), (size_t)(0), stream, o, ldo, gate, ldg, gate_kind, gate_first, gain, gain_len, skip, lds, coef, span, norm, eps, out_scale, (float*)out, ld_out, tokens, groups, width, floor_in, ldf, den_eps));
-    else if (dtype == NIB_BF16) NIB_CUDA(launch_pdl(gated_norm_kernel<__nv_bfloat16>, dim3(blocks), dim3(128), (size_t)(0), stream, o, ldo, gate, ldg, gate_kind, gate_first, gain, gain_len, skip, lds, coef, span, norm, eps, out_scale, (__nv_bfloat16*)out, ld_out, tokens, groups, width, floor_in, ldf, den_eps));
-    else NIB_REQUIRE(false, "gated_norm: unknown dtype %d", dtype);
-    NIB_LAUNCH_CHECK();
-    return 0;
+    NIB_REQUIRE((dtype == NIB_F32 || dtype == NIB_BF16) && (skip_dtype == NIB_F32 || skip_dtype == NIB_BF16), "gated_norm: unknown dtype %d / %d", dtype, skip_dtype);
+#define NIB_GN(T, TS) launch_gated_norm<T, TS>(o, ldo, gate, ldg, gate_kind, gate_first, gain, gain_len, (const TS*)skip, lds, coef, span, groups, norm, eps, out_scale, \
+                                               (T*)out, ld_out, tokens, width, floor_in, ldf, den_eps, stream)
+    if (dtype == NIB_F32) return skip_dtype == NIB_F32 ? NIB_GN(float, float) : NIB_GN(float, __nv_bfloat16);
+    return skip_dtype == NIB_F32 ? NIB_GN(__nv_bfloat16, float) : NIB_GN(__nv_bfloat16, __nv_bfloat16);
+#undef NIB_GN
 }
 
 // ---------------------------------------------------------------------------------- norm of a branch's output, added

@@ -26,7 +26,8 @@ by token; ``ops.grouped_state_scan``, eight tokens at a time; ``ops.decay_state_
   (of ones); ``o`` is divided by ``max(|n . q|, exp(-m_t)) + 1e-6``, then by its root mean square per head, times a gain of all
   heads' size, times ``sigmoid(W_g h)``, then ``W_o``.
 
-Everything that enters the walk is 32-bit: the projections leave the matrix kernels as floats. Each adds
+What enters the walk is 32-bit: the projections leave the matrix kernels as floats (``Mamba2Mixer`` keeps its convolution's outputs in
+the storage type). Each adds
 ``out_scale`` times its result to the residual stream.
 """
 from __future__ import annotations
@@ -204,7 +205,7 @@ class Mamba2Mixer(Mixer):
         p32 = torch.empty((m, 2 * inner + 2 * gn + self.heads), dtype=torch.float32, device=dev)
         ops.linear(h, self.w_in, None, p32, "f32")
         xbc_in = p32[:, inner:2 * inner + 2 * gn]
-        xbc = torch.empty((m, inner + 2 * gn), dtype=torch.float32, device=dev)
+        xbc = torch.empty((m, inner + 2 * gn), dtype=self.rt.dtype, device=dev)
         ops.conv_step(xbc_in, self.conv_w, self.conv_b, "silu", cache.state, 0, ctx, xbc, self.taps)
         o32 = torch.empty((m, inner), dtype=torch.float32, device=dev)
         x = xbc[:, :inner]

@@ -161,7 +161,7 @@ def mamba2_mixer(h, w, p, m, eps):
     xbc = silu(short_conv(xbc, w[p + ".conv"], w[p + ".conv.b"]))
     x, b, c = torch.split(xbc, [inner, gn, gn], dim=1)
     x, b, c = x.reshape(t_len, heads, dv), b.reshape(t_len, groups, n), c.reshape(t_len, groups, n)
-    dt = torch.log1p(torch.exp(dt + w[p + ".dt_bias"]))
+    dt = torch.logaddexp(dt + w[p + ".dt_bias"], torch.zeros((), dtype=F))
     rep = heads // groups
     y = matrix_state(c.repeat_interleave(rep, 1), b.repeat_interleave(rep, 1), x * dt[:, :, None], torch.exp(-torch.exp(w[p + ".A_log"]) * dt))
     y = (y + w[p + ".D"][:, None] * x).reshape(t_len, inner) * silu(z)

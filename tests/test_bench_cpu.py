@@ -127,3 +127,23 @@ def test_the_sixth_designs_bench_sizes_are_configurations_the_registry_takes():
         assert kinds.count("parallel") == 4 and kinds.count("mlstm") == 2
         moe = pil["layers"][1]["mlp"]
         assert moe["router"]["top"] * moe["expert"]["ff"] == size["ff_swiglu"] == pil["layers"][0]["mlp"]["ff"]
+
+
+def test_the_seventh_designs_bench_sizes_are_configurations_the_registry_takes():
+    """``--design vagulorn``: all three models of a size are valid configurations of equal width, depth and vocabulary; the two designs
+    agree layer by layer in feed-forwards, head counts and state-space mixers."""
+    from nanoinfer_b200.registry import config_from_json_dict, plan_for
+    for size in bench.VAGULORN_SIZES.values():
+        vag, vaf, dense = bench.vagulorn_configs(size)
+        plans = [plan_for(config_from_json_dict(c)) for c in (vag, vaf, dense)]
+        assert [len(p.layers) for p in plans] == [size["layers"]] * 3
+        assert len({p.hidden_size for p in plans}) == len({p.vocab_size for p in plans}) == 1
+        kinds = [layer["type"] for layer in vag["layers"]]
+        assert (kinds.count("parallel"), kinds.count("mamba2"), kinds.count("attention")) == (2, 4, 2)
+        for a, b in zip(vag["layers"], vaf["layers"]):
+            assert a["mlp"] == b["mlp"]
+            if a["type"] == "mamba2":
+                assert a["mixer"] == b["mixer"]
+            else:
+                lt = a["mixer"].get("left", a["mixer"])
+                assert all(lt[k] == b["mixer"]["left"][k] for k in ("heads", "kv_heads", "dim", "vdim", "scale"))

@@ -334,14 +334,14 @@ class TorchOps:
             flat.copy_(s.transpose(1, 2).reshape(-1).to(torch.float32))
             start += q_len
 
-    def decay_state_scan(self, q32, k32, v32, state, state_off, ctx, o32, heads, kq_heads, dk, dv, act="none", decay32=None, raw32=None,
+    def decay_state_scan(self, q, k, v, state, state_off, ctx, o32, heads, kq_heads, dk, dv, act="none", decay32=None, raw32=None,
                          dt_bias32=None, a_log32=None, exact=False):
-        m, rep = q32.shape[0], heads // kq_heads
+        m, rep = q.shape[0], heads // kq_heads
         f = (lambda z: z * torch.sigmoid(z)) if act == "silu" else (lambda z: z)
-        q, k = (f(x.double()).reshape(m, kq_heads, dk).repeat_interleave(rep, 1) for x in (q32, k32))
-        v = f(v32.double()).reshape(m, heads, dv)
+        q, k = (f(x.double()).reshape(m, kq_heads, dk).repeat_interleave(rep, 1) for x in (q, k))
+        v = f(v.double()).reshape(m, heads, dv)
         if raw32 is not None:
-            step = torch.nn.functional.softplus(raw32.double() + dt_bias32.double(), threshold=1e9)
+            step = torch.logaddexp(raw32.double() + dt_bias32.double(), torch.zeros((), dtype=torch.float64))
             d = torch.exp(-torch.exp(a_log32.double()) * step)
             v = v * step[:, :, None]
         else:
