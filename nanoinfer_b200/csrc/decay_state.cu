@@ -18,7 +18,10 @@
 // The products run on the tensor cores (mma.sync m16n8k16, bfloat16 operands, 32-bit sums). q, k and v are outputs of
 // projections and convolutions and enter as bfloat16 (they may be stored so, T, or as floats); what is 32-bit by the design (states,
 // decays, step sizes, and everything they multiply) is split into a bfloat16 and a bfloat16 of the remainder, two products each: 16
-// bits and more of it take part. Blocks take 64 value channels of a head; tiles come by cp.async where rows are aligned.
+// bits and more of it take part. Blocks take 64 value channels of a head; tiles come by cp.async where rows are aligned. What passes
+// between the three kernels lies in the order of the products' fragments: a lane's eight numbers of a 16 x 16 piece of a state (value
+// channels g and g + 8, key channels 2t, 2t + 1, 2t + 8, 2t + 9 of it, g = lane / 4, t = lane % 4) are 32 consecutive bytes, which
+// chunk_state holds in its accumulators and chunk_output multiplies with as they come from memory.
 #include "attention_common.cuh"
 
 namespace {
@@ -173,13 +176,23 @@ decay_step_kernel(const DsIn in, float* __restrict__ state, long long state_ld, 
 }
 
 // ---------------------------------------------------------------------------------- chunks
-// A chunk's tile in shared memory: CH rows of DP bfloat16, 16 bytes of padding each; a state's tile has as many rows, its value
-// channels.
+// A chunk's tile in shared memory: CH rows of DP bfloat16, 16 bytes of padding each.
 template <int DP> struct Tile {
     static constexpr int ROW = DP + 8;
     static constexpr int ELEMS = CH * ROW;
 };
-constexpr int DV = CH;                  // value channels of a block
+constexpr int DV = 64;                  // value channels of a block
+constexpr int PIECE = 16 * 16;          // floats of a piece of a state
+__host__ __device__ constexpr int keys_padded(int dk) { return dk <= 64 ? 64 : 128; }
+// pieces of one head's state: [blocks of value channels][keys / 16][4]
+__host__ __device__ inline int pieces_of(int dk, int dv) { return (dv + DV - 1) / DV * (keys_padded(dk) / 16) * (DV / 16); }
+
+// powers of two; what is below 2^-126 is zero
+__device__ __forceinline__ float ds_exp2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 
 struct ChunkAt { int row, n, slot; };       // first flat row, tokens, index among the step's chunks
 
@@ -233,7 +246,6 @@ __device__ __forceinline__ void chunk_decays(const DsIn& in, const ChunkAt& at, 
 __device__ __forceinline__ void put4(__nv_bfloat16* p, const float4& x) {
     *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(x.x, x.y), pack_bf16(x.z, x.w));
 }
-__device__ __forceinline__ float4 rest4(const float4& x) { return make_float4(x.x - bf16_of(x.x), x.y - bf16_of(x.y), x.z - bf16_of(x.z), x.w - bf16_of(x.w)); }
 
 __device__ __forceinline__ void ds_cp_async_16(void* smem, const void* gmem, bool valid) {
     const unsigned d = (unsigned)__cvta_generic_to_shared(smem);
@@ -266,17 +278,18 @@ __device__ __forceinline__ void load_rows(__nv_bfloat16* tile, const T* __restri
 }
 
 // Where a block stands: a chunk of a request, a head, 64 of its value channels. grid: (chunks, heads x blocks of value channels,
-// requests).
-struct Block { ChunkAt at; int h, hq, v0, nv; };
+// requests). piece: the first of the block's pieces of the chunk's state.
+struct Block { ChunkAt at; int h, hq, v0, nv; size_t piece; };
 __device__ __forceinline__ Block block_of(const DsIn& in) {
     const int per_head = (in.dv + DV - 1) / DV, h = blockIdx.y / per_head, v0 = (blockIdx.y % per_head) * DV;
-    return {chunk_at(in.q_start, blockIdx.z, blockIdx.x), h, h / (in.heads / in.kq_heads), v0, min(DV, in.dv - v0)};
+    const ChunkAt at = chunk_at(in.q_start, blockIdx.z, blockIdx.x);
+    return {at, h, h / (in.heads / in.kq_heads), v0, min(DV, in.dv - v0), ((size_t)at.slot * in.heads + h) * pieces_of(in.dk, in.dv) + v0 / 16 * (keys_padded(in.dk) / 16)};
 }
 
-// What a chunk adds to a zero state: local[chunk, head, value channel, key channel], and the chunk's whole decay. A warp owns 16
+// What a chunk adds to a zero state: local[chunk, head, piece], and the chunk's whole decay. A warp owns 16
 // value channels: rows of the product (weighted v)^T . k over the chunk's tokens; the weights go on v in registers, in 32-bit.
 template <typename T, int DKP>
-__global__ void __launch_bounds__(DS_THREADS)
+__global__ void __launch_bounds__(DS_THREADS, 5)
 chunk_state_kernel(const DsIn in, float* __restrict__ local, float* __restrict__ decays) {
     extern __shared__ __align__(16) unsigned char smem[];
     __shared__ float hi_s[CH], lo_s[CH], f_s[CH];
@@ -306,8 +319,8 @@ chunk_state_kernel(const DsIn in, float* __restrict__ local, float* __restrict__
 #pragma unroll
         for (int half = 0; half < 2; ++half) {      // the thread's tokens: 2t, 2t + 1 of eight
             const int s0 = kb * 16 + half * 8 + 2 * t;
-            const float w0 = exp2f((end_hi - hi_s[s0]) + (end_lo - lo_s[s0])) * f_s[s0];
-            const float w1 = exp2f((end_hi - hi_s[s0 + 1]) + (end_lo - lo_s[s0 + 1])) * f_s[s0 + 1];
+            const float w0 = ds_exp2((end_hi - hi_s[s0]) + (end_lo - lo_s[s0])) * f_s[s0];
+            const float w1 = ds_exp2((end_hi - hi_s[s0 + 1]) + (end_lo - lo_s[s0 + 1])) * f_s[s0 + 1];
 #pragma unroll
             for (int r = 0; r < 2; ++r) {
                 const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a[2 * half + r]));
@@ -326,96 +339,80 @@ chunk_state_kernel(const DsIn in, float* __restrict__ local, float* __restrict__
             mma_bf16(acc[2 * np + 1], a_lo, bk[2], bk[3]);
         }
     }
-    float* out = local + (((size_t)at.slot * in.heads + b.h) * in.dv + b.v0) * in.dk;
-    const bool pairs = in.dk % 2 == 0;
+    float* out = local + (b.piece + warp) * PIECE + lane * 8;       // (zeros where the head has fewer channels)
 #pragma unroll
-    for (int r = 0; r < 2; ++r) {
-        const int j = warp * 16 + g + 8 * r;
-        if (j >= b.nv) continue;
-#pragma unroll
-        for (int n = 0; n < DKP / 8; ++n) {
-            const int c = n * 8 + 2 * t;
-            float* p = out + (size_t)j * in.dk + c;
-            if (pairs) {
-                if (c < in.dk) *reinterpret_cast<float2*>(p) = make_float2(acc[n][2 * r], acc[n][2 * r + 1]);
-            } else {
-                if (c < in.dk) p[0] = acc[n][2 * r];
-                if (c + 1 < in.dk) p[1] = acc[n][2 * r + 1];
-            }
-        }
+    for (int kk = 0; kk < DKP / 16; ++kk) {
+        float4* to = reinterpret_cast<float4*>(out + kk * 4 * PIECE);
+        to[0] = make_float4(acc[2 * kk][0], acc[2 * kk][1], acc[2 * kk + 1][0], acc[2 * kk + 1][1]);
+        to[1] = make_float4(acc[2 * kk][2], acc[2 * kk][3], acc[2 * kk + 1][2], acc[2 * kk + 1][3]);
     }
-    if (threadIdx.x == 0 && b.v0 == 0) decays[(size_t)at.slot * in.heads + b.h] = exp2f(end_hi + end_lo);
+    if (threadIdx.x == 0 && b.v0 == 0) decays[(size_t)at.slot * in.heads + b.h] = ds_exp2(end_hi + end_lo);
 }
 
 // local[chunk] (what the chunk adds) becomes the chunk's entry state; the slot's state moves past the request's last chunk. A thread
-// per eight (SPLIT) or one state elements of a request; the chunks' loads run ahead of the chain. SPLIT: the entry states are written
-// as the products read them, eight elements' bfloat16 and then the bfloat16 of their remainders where the eight floats were.
-template <bool SPLIT>
+// per lane of a piece; the chunks' loads run ahead of the chain. The entry states are written as the products read them: a lane's
+// eight bfloat16 and then the bfloat16 of their remainders where its eight floats were.
 __global__ void __launch_bounds__(128)
 chunk_chain_kernel(float* __restrict__ state, long long state_ld, int state_off, const int* __restrict__ q_start, const int* __restrict__ slots,
-                   float* __restrict__ local, const float* __restrict__ decays, int heads, int per_head) {
-    constexpr int N = SPLIT ? 8 : 1, AHEAD = 8;
+                   float* __restrict__ local, const float* __restrict__ decays, int heads, int dk, int dv) {
+    constexpr int AHEAD = 8;
     pdl_launch_dependents();
     pdl_wait();
-    const int req = blockIdx.y;
-    const long long e = ((long long)blockIdx.x * 128 + threadIdx.x) * N, elems = (long long)heads * per_head;
+    const int req = blockIdx.y, pieces = pieces_of(dk, dv), per_keys = keys_padded(dk) / 16;
+    const long long w = (long long)blockIdx.x * 4 + (threadIdx.x >> 5), all = (long long)heads * pieces;
     const int len = q_start[req + 1] - q_start[req], chunks = (len + CH - 1) / CH;
-    if (e >= elems || chunks == 0) return;
-    const int h = (int)(e / per_head), slot0 = (q_start[req] - q_start[0]) / CH + req;
-    float* st = state + (long long)slots[req] * state_ld + state_off + e;
-    float* at = local + (size_t)slot0 * elems + e;
+    if (w >= all || chunks == 0) return;
+    const int lane = threadIdx.x & 31, h = (int)(w / pieces), piece = (int)(w % pieces), slot0 = (q_start[req] - q_start[0]) / CH + req;
+    const int j0 = piece / (4 * per_keys) * DV + piece % 4 * 16 + (lane >> 2), c0 = piece / 4 % per_keys * 16 + 2 * (lane & 3);
+    float* st = state + (long long)slots[req] * state_ld + state_off + (long long)h * dv * dk;
+    float* at = local + ((size_t)slot0 * all + w) * PIECE + lane * 8;
+    const size_t step = (size_t)all * PIECE;
     const float* dec = decays + (size_t)slot0 * heads + h;
-    auto load = [](const float* p, float (&x)[N]) {
-        if constexpr (SPLIT) {
-            const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
-            x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w; x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
-        } else {
-            x[0] = *p;
-        }
-    };
-    float S[N];
-    if constexpr (SPLIT) {      // (a state may start at any column)
+    float S[8];
 #pragma unroll
-        for (int n = 0; n < N; ++n) S[n] = st[n];
-    } else {
-        S[0] = *st;
+    for (int n = 0; n < 8; ++n) {
+        const int j = j0 + (n & 4) * 2, c = c0 + (n & 2) * 4 + (n & 1);
+        S[n] = j < dv && c < dk ? st[(long long)j * dk + c] : 0.f;
     }
-    for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
-        float x[AHEAD][N], d[AHEAD];
+    for (int k0 = 0; k0 < chunks; k0 += AHEAD) {
+        float4 x[AHEAD][2];
+        float d[AHEAD];
 #pragma unroll
         for (int i = 0; i < AHEAD; ++i)
-            if (c0 + i < chunks) {
-                load(at + (size_t)(c0 + i) * elems, x[i]);
-                d[i] = dec[(size_t)(c0 + i) * heads];
+            if (k0 + i < chunks) {
+                const float4* from = reinterpret_cast<const float4*>(at + (size_t)(k0 + i) * step);
+                x[i][0] = from[0];
+                x[i][1] = from[1];
+                d[i] = dec[(size_t)(k0 + i) * heads];
             }
 #pragma unroll
         for (int i = 0; i < AHEAD; ++i)
-            if (c0 + i < chunks) {
-                float* to = at + (size_t)(c0 + i) * elems;
-                if constexpr (SPLIT) {
-                    unsigned hi[4], lo[4];
+            if (k0 + i < chunks) {
+                uint4* to = reinterpret_cast<uint4*>(at + (size_t)(k0 + i) * step);
+                unsigned hi[4], lo[4];
 #pragma unroll
-                    for (int n = 0; n < 4; ++n) {
-                        hi[n] = pack_bf16(S[2 * n], S[2 * n + 1]);
-                        lo[n] = pack_bf16(S[2 * n] - bf16_of(S[2 * n]), S[2 * n + 1] - bf16_of(S[2 * n + 1]));
-                    }
-                    reinterpret_cast<uint4*>(to)[0] = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-                    reinterpret_cast<uint4*>(to)[1] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
-                } else {
-                    *to = S[0];
+                for (int n = 0; n < 4; ++n) {
+                    hi[n] = pack_bf16(S[2 * n], S[2 * n + 1]);
+                    lo[n] = pack_bf16(S[2 * n] - bf16_of(S[2 * n]), S[2 * n + 1] - bf16_of(S[2 * n + 1]));
                 }
+                to[0] = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+                to[1] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+                const float add[8] = {x[i][0].x, x[i][0].y, x[i][0].z, x[i][0].w, x[i][1].x, x[i][1].y, x[i][1].z, x[i][1].w};
 #pragma unroll
-                for (int n = 0; n < N; ++n) S[n] = fmaf(d[i], S[n], x[i][n]);
+                for (int n = 0; n < 8; ++n) S[n] = fmaf(d[i], S[n], add[n]);
             }
     }
 #pragma unroll
-    for (int n = 0; n < N; ++n) st[n] = S[n];
+    for (int n = 0; n < 8; ++n) {
+        const int j = j0 + (n & 4) * 2, c = c0 + (n & 2) * 4 + (n & 1);
+        if (j < dv && c < dk) st[(long long)j * dk + c] = S[n];
+    }
 }
 
 // The outputs of a chunk from its entry state. A warp owns 16 tokens.
 template <typename T, int DKP>
-__global__ void __launch_bounds__(DS_THREADS)
-chunk_output_kernel(const DsIn in, const float* __restrict__ entry, int split, float* __restrict__ o, int ldo) {
+__global__ void __launch_bounds__(DS_THREADS, 5)
+chunk_output_kernel(const DsIn in, const float* __restrict__ entry, float* __restrict__ o, int ldo) {
     extern __shared__ __align__(16) unsigned char smem[];
     __shared__ float hi_s[CH], lo_s[CH], f_s[CH];
     pdl_launch_dependents();
@@ -426,30 +423,10 @@ chunk_output_kernel(const DsIn in, const float* __restrict__ entry, int split, f
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, mat = lane >> 3, rr = lane & 7, g = lane >> 2, t4 = lane & 3;
     constexpr int RK = Tile<DKP>::ROW, RV = Tile<DV>::ROW;
     __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem);
-    __nv_bfloat16* sh_s = q_s + Tile<DKP>::ELEMS;           // the entry state, [value channel][key channel], and its remainder
-    __nv_bfloat16* sl_s = sh_s + Tile<DKP>::ELEMS;
-    __nv_bfloat16* k_s = sl_s + Tile<DKP>::ELEMS;
+    __nv_bfloat16* k_s = q_s + Tile<DKP>::ELEMS;
     __nv_bfloat16* v_s = k_s + Tile<DKP>::ELEMS;
     const bool vec = in.vec != 0, silu = in.silu != 0;
-    const float* from = entry + (((size_t)at.slot * in.heads + b.h) * in.dv + b.v0) * in.dk;
     load_rows<T, DKP>(q_s, in.q_at<T>(at.row, b.hq), in.ldq, at.n, in.dk, silu, vec);
-    if (split) {
-        for (int i = threadIdx.x; i < DV * (DKP / 8); i += DS_THREADS) {
-            const int r = i / (DKP / 8), c = (i % (DKP / 8)) * 8;
-            const bool ok = r < b.nv && c < in.dk;
-            const float* p = ok ? from + (size_t)r * in.dk + c : from;
-            ds_cp_async_16(sh_s + r * RK + c, p, ok);
-            ds_cp_async_16(sl_s + r * RK + c, p + (ok ? 4 : 0), ok);
-        }
-    } else {
-        for (int i = threadIdx.x; i < DV * (DKP / 4); i += DS_THREADS) {
-            const int r = i / (DKP / 4), c = (i % (DKP / 4)) * 4;
-            float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (r < b.nv) x = row4(from + (size_t)r * in.dk, c, in.dk, false);
-            put4(sh_s + r * RK + c, x);
-            put4(sl_s + r * RK + c, rest4(x));
-        }
-    }
     ds_commit();
     load_rows<T, DKP>(k_s, in.k_at<T>(at.row, b.hq), in.ldk, at.n, in.dk, silu, vec);
     load_rows<T, DV>(v_s, in.v_at<T>(at.row, b.h) + b.v0, in.ldv, at.n, b.nv, silu, vec);
@@ -464,25 +441,24 @@ chunk_output_kernel(const DsIn in, const float* __restrict__ entry, int split, f
 #pragma unroll
     for (int n = 0; n < DV / 8; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
     // q . S_in
+    const uint4* state = reinterpret_cast<const uint4*>(entry + b.piece * PIECE + lane * 8);
 #pragma unroll
     for (int kk = 0; kk < DKP / 16; ++kk)
 #pragma unroll
         for (int np = 0; np < DV / 16; ++np) {
-            const int at_s = (np * 16 + (mat >> 1) * 8 + rr) * RK + kk * 16 + (mat & 1) * 8;
-            unsigned bh[4], bl[4];
-            ldmatrix_x4(bh, sh_s + at_s);
-            ldmatrix_x4(bl, sl_s + at_s);
-            mma_bf16(acc[2 * np], q[kk], bh[0], bh[1]);
-            mma_bf16(acc[2 * np + 1], q[kk], bh[2], bh[3]);
-            mma_bf16(acc[2 * np], q[kk], bl[0], bl[1]);
-            mma_bf16(acc[2 * np + 1], q[kk], bl[2], bl[3]);
+            const uint4* piece = state + (kk * 4 + np) * (PIECE / 4);       // the state's bfloat16, then its remainders
+            const uint4 bh = piece[0], bl = piece[1];
+            mma_bf16(acc[2 * np], q[kk], bh.x, bh.y);
+            mma_bf16(acc[2 * np + 1], q[kk], bh.z, bh.w);
+            mma_bf16(acc[2 * np], q[kk], bl.x, bl.y);
+            mma_bf16(acc[2 * np + 1], q[kk], bl.z, bl.w);
         }
     float t_hi[2], t_lo[2];
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
         t_hi[r] = hi_s[warp * 16 + g + 8 * r];
         t_lo[r] = lo_s[warp * 16 + g + 8 * r];
-        const float w = exp2f(t_hi[r] + t_lo[r]);
+        const float w = ds_exp2(t_hi[r] + t_lo[r]);
 #pragma unroll
         for (int n = 0; n < DV / 8; ++n) { acc[n][2 * r] *= w; acc[n][2 * r + 1] *= w; }
     }
@@ -508,7 +484,7 @@ chunk_output_kernel(const DsIn in, const float* __restrict__ entry, int split, f
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
                     const int key = kb * 16 + n * 8 + 2 * t4 + e, tok = warp * 16 + g + 8 * r;
-                    const float w = key <= tok ? exp2f((t_hi[r] - hi_s[key]) + (t_lo[r] - lo_s[key])) * f_s[key] : 0.f;
+                    const float w = key <= tok ? ds_exp2((t_hi[r] - hi_s[key]) + (t_lo[r] - lo_s[key])) * f_s[key] : 0.f;
                     x[e] = s[n][2 * r + e] * w;
                 }
                 p_hi[2 * n + r] = pack_bf16(x[0], x[1]);
@@ -546,7 +522,7 @@ chunk_output_kernel(const DsIn in, const float* __restrict__ entry, int split, f
 template <typename T, int DKP>
 int launch_chunks(const DsIn& in, float* state, long long state_ld, int state_off, float* o, int ldo, int n_req, int max_len, float* local,
                   float* decays, cudaStream_t stream) {
-    constexpr int SMEM_STATE = (Tile<DKP>::ELEMS + Tile<DV>::ELEMS) * 2, SMEM_OUT = (4 * Tile<DKP>::ELEMS + Tile<DV>::ELEMS) * 2;
+    constexpr int SMEM_STATE = (Tile<DKP>::ELEMS + Tile<DV>::ELEMS) * 2, SMEM_OUT = (2 * Tile<DKP>::ELEMS + Tile<DV>::ELEMS) * 2;
     static bool configured = false;
     if (!configured) {
         NIB_CUDA(cudaFuncSetAttribute(chunk_state_kernel<T, DKP>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_STATE));
@@ -555,16 +531,9 @@ int launch_chunks(const DsIn& in, float* state, long long state_ld, int state_of
     }
     const dim3 grid(ceil_div(max_len, CH), in.heads * ceil_div(in.dv, DV), n_req);
     NIB_CUDA(launch_pdl(chunk_state_kernel<T, DKP>, grid, dim3(DS_THREADS), (size_t)SMEM_STATE, stream, in, local, decays));
-    const int per_head = in.dv * in.dk;
-    const long long elems = (long long)in.heads * per_head;
-    const int split = in.dk % 8 == 0 && ((uintptr_t)local & 15) == 0 ? 1 : 0;
-    if (split)
-        NIB_CUDA(launch_pdl(chunk_chain_kernel<true>, dim3(ceil_div(elems, 1024), n_req), dim3(128), (size_t)0, stream, state, state_ld, state_off,
-                            in.q_start, in.slots, local, (const float*)decays, in.heads, per_head));
-    else
-        NIB_CUDA(launch_pdl(chunk_chain_kernel<false>, dim3(ceil_div(elems, 128), n_req), dim3(128), (size_t)0, stream, state, state_ld, state_off,
-                            in.q_start, in.slots, local, (const float*)decays, in.heads, per_head));
-    NIB_CUDA(launch_pdl(chunk_output_kernel<T, DKP>, grid, dim3(DS_THREADS), (size_t)SMEM_OUT, stream, in, (const float*)local, split, o, ldo));
+    NIB_CUDA(launch_pdl(chunk_chain_kernel, dim3(ceil_div((long long)in.heads * pieces_of(in.dk, in.dv), 4), n_req), dim3(128), (size_t)0, stream, state,
+                        state_ld, state_off, in.q_start, in.slots, local, (const float*)decays, in.heads, in.dk, in.dv));
+    NIB_CUDA(launch_pdl(chunk_output_kernel<T, DKP>, grid, dim3(DS_THREADS), (size_t)SMEM_OUT, stream, in, (const float*)local, o, ldo));
     NIB_LAUNCH_CHECK();
     return 0;
 }
@@ -592,7 +561,7 @@ int scan(DsIn in, float* state, long long state_ld, int state_off, float* o, int
     constexpr int G = 16 / sizeof(T);       // 16 bytes a load
     auto aligned = [](const void* p, long long ld) { return ((uintptr_t)p & 15) == 0 && ld % G == 0; };
     in.vec = dk % G == 0 && dv % G == 0 && aligned(in.q, in.ldq) && aligned(in.k, in.ldk) && aligned(in.v, in.ldv);
-    float* decays = scratch + ((long long)tokens / CH + n_req) * in.heads * dv * dk;
+    float* decays = scratch + ((long long)tokens / CH + n_req) * in.heads * pieces_of(dk, dv) * PIECE;
     if (dk <= 64) return launch_chunks<T, 64>(in, state, state_ld, state_off, o, ldo, n_req, max_len, scratch, decays, stream);
     return launch_chunks<T, 128>(in, state, state_ld, state_off, o, ldo, n_req, max_len, scratch, decays, stream);
 }
@@ -602,7 +571,7 @@ int scan(DsIn in, float* state, long long state_ld, int state_off, float* o, int
 // Floats of scratch for a step of `tokens` tokens of n_req requests in chunks: entry states, then decays.
 NIB_API long long nib_decay_state_scratch(long long tokens, int n_req, int heads, int dk, int dv) {
     const long long slots = tokens / CH + n_req;
-    return slots * heads * ((long long)dv * dk) + slots * heads;
+    return slots * heads * pieces_of(dk, dv) * PIECE + slots * heads;
 }
 
 NIB_API int nib_decay_state_chunks_supported(int dk, int dv) { return dk > 0 && dv > 0 && dk <= 128 ? 1 : 0; }
@@ -618,6 +587,7 @@ NIB_API int nib_decay_state_scan(const void* q, int ldq, const void* k, int ldk,
     NIB_REQUIRE(raw != nullptr ? (bias != nullptr && a_log != nullptr) : (decay != nullptr && log2_decay != nullptr),
                 "decay_state_scan: step sizes need bias and a_log, fixed decays their logarithms");
     NIB_REQUIRE(n_req >= 0 && n_req <= 65535 && (long long)heads * ceil_div(dv, DV) <= 65535 && max_len >= 0, "decay_state_scan: bad counts");
+    NIB_REQUIRE(((uintptr_t)scratch & 15) == 0, "decay_state_scan: scratch must start on a 16-byte boundary");
     NIB_REQUIRE(scratch == nullptr || nib_decay_state_chunks_supported(dk, dv) == 1, "decay_state_scan: chunks take keys up to 128, not %d", dk);
     if (n_req == 0 || max_len == 0) return 0;
     const DsIn in{q, k, v, raw, bias, a_log, decay, log2_decay, q_start, slots, ldq, ldk, ldv, ld_raw, heads, kq_heads, dk, dv, silu, 0};
