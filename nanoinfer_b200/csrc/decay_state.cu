@@ -18,7 +18,8 @@
 // The products run on the tensor cores (mma.sync m16n8k16, bfloat16 operands, 32-bit sums). q, k and v are outputs of
 // projections and convolutions and enter as bfloat16 (they may be stored so, T, or as floats); what is 32-bit by the design (states,
 // decays, step sizes, and everything they multiply) is split into a bfloat16 and a bfloat16 of the remainder, two products each: 16
-// bits and more of it take part. Blocks take 64 value channels of a head; tiles come by cp.async where rows are aligned. What passes
+// bits and more of it take part. A block takes units, 64 value channels of a head each: two that share q and k where such pairs
+// exist, else one; tiles come by cp.async where rows are aligned. What passes
 // between the three kernels lies in the order of the products' fragments: a lane's eight numbers of a 16 x 16 piece of a state (value
 // channels g and g + 8, key channels 2t, 2t + 1, 2t + 8, 2t + 9 of it, g = lane / 4, t = lane % 4) are 32 consecutive bytes, which
 // chunk_state holds in its accumulators and chunk_output multiplies with as they come from memory.
@@ -75,7 +76,9 @@ __device__ __forceinline__ float4 row4(const __nv_bfloat16* p, int c, int width,
     }
     return x;
 }
-__device__ __forceinline__ void silu4(float4& x) { x.x = ds_silu(x.x); x.y = ds_silu(x.y); x.z = ds_silu(x.z); x.w = ds_silu(x.w); }
+// with the fast exponential and division (2 ulp), for results that are rounded to bfloat16
+__device__ __forceinline__ float silu_fast(float x) { return __fdividef(x, 1.0f + __expf(-x)); }
+__device__ __forceinline__ void silu4(float4& x) { x = make_float4(silu_fast(x.x), silu_fast(x.y), silu_fast(x.z), silu_fast(x.w)); }
 
 // ---------------------------------------------------------------------------------- short steps
 // grid: (parts of the value channels, heads, requests). LANES lanes share R value channels; lane l holds the key channels
@@ -181,10 +184,10 @@ template <int DP> struct Tile {
     static constexpr int ROW = DP + 8;
     static constexpr int ELEMS = CH * ROW;
 };
-constexpr int DV = 64;                  // value channels of a block
+constexpr int DV = 64;                  // value channels of a unit
 constexpr int PIECE = 16 * 16;          // floats of a piece of a state
 __host__ __device__ constexpr int keys_padded(int dk) { return dk <= 64 ? 64 : 128; }
-// pieces of one head's state: [blocks of value channels][keys / 16][4]
+// pieces of one head's state: [units][keys / 16][4]
 __host__ __device__ inline int pieces_of(int dk, int dv) { return (dv + DV - 1) / DV * (keys_padded(dk) / 16) * (DV / 16); }
 
 // powers of two; what is below 2^-126 is zero
@@ -204,10 +207,10 @@ __device__ __forceinline__ ChunkAt chunk_at(const int* __restrict__ q_start, int
     return {row, max(0, min(CH, last - row)), (first - q_start[0]) / CH + req + c};
 }
 
-// Warp 0: per token of the chunk the sum of the decays' log2 (as two floats) and the factor on the value; tokens that do not
+// One warp: per token of the chunk the sum of the decays' log2 (as two floats) and the factor on the value; tokens that do not
 // exist do not decay.
 __device__ __forceinline__ void chunk_decays(const DsIn& in, const ChunkAt& at, int h, float* hi_s, float* lo_s, float* f_s) {
-    const int lane = threadIdx.x;
+    const int lane = threadIdx.x & 31;
     double sum[2];
     float f[2];
     const bool fixed = in.raw == nullptr;
@@ -277,76 +280,82 @@ __device__ __forceinline__ void load_rows(__nv_bfloat16* tile, const T* __restri
     }
 }
 
-// Where a block stands: a chunk of a request, a head, 64 of its value channels. grid: (chunks, heads x blocks of value channels,
-// requests). piece: the first of the block's pieces of the chunk's state.
-struct Block { ChunkAt at; int h, hq, v0, nv; size_t piece; };
-__device__ __forceinline__ Block block_of(const DsIn& in) {
-    const int per_head = (in.dv + DV - 1) / DV, h = blockIdx.y / per_head, v0 = (blockIdx.y % per_head) * DV;
-    const ChunkAt at = chunk_at(in.q_start, blockIdx.z, blockIdx.x);
-    return {at, h, h / (in.heads / in.kq_heads), v0, min(DV, in.dv - v0), ((size_t)at.slot * in.heads + h) * pieces_of(in.dk, in.dv) + v0 / 16 * (keys_padded(in.dk) / 16)};
+// Where a block stands: a chunk of a request and U units that share q and k. grid: (chunks, units / U, requests). piece: the first
+// of a unit's pieces of the chunk's state.
+struct Unit { int h, v0, nv; size_t piece; };
+__device__ __forceinline__ Unit unit_of(const DsIn& in, const ChunkAt& at, int u) {
+    const int per_head = (in.dv + DV - 1) / DV, h = u / per_head, v0 = (u % per_head) * DV;
+    return {h, v0, min(DV, in.dv - v0), ((size_t)at.slot * in.heads + h) * pieces_of(in.dk, in.dv) + v0 / 16 * (keys_padded(in.dk) / 16)};
 }
 
 // What a chunk adds to a zero state: local[chunk, head, piece], and the chunk's whole decay. A warp owns 16
 // value channels: rows of the product (weighted v)^T . k over the chunk's tokens; the weights go on v in registers, in 32-bit.
-template <typename T, int DKP>
+template <typename T, int DKP, int U>
 __global__ void __launch_bounds__(DS_THREADS, 5)
 chunk_state_kernel(const DsIn in, float* __restrict__ local, float* __restrict__ decays) {
     extern __shared__ __align__(16) unsigned char smem[];
-    __shared__ float hi_s[CH], lo_s[CH], f_s[CH];
+    __shared__ __align__(16) float hi_s[U][CH], lo_s[U][CH], f_s[U][CH];
     pdl_launch_dependents();
     pdl_wait();
-    const Block b = block_of(in);
-    const ChunkAt& at = b.at;
+    const ChunkAt at = chunk_at(in.q_start, blockIdx.z, blockIdx.x);
     if (at.n == 0) return;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, mat = lane >> 3, rr = lane & 7, g = lane >> 2, t = lane & 3;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, mat = lane >> 3, rr = lane & 7, t = lane & 3, u0 = blockIdx.y * U;
     constexpr int RK = Tile<DKP>::ROW, RV = Tile<DV>::ROW;
     __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(smem);
     __nv_bfloat16* v_s = k_s + Tile<DKP>::ELEMS;
-    load_rows<T, DKP>(k_s, in.k_at<T>(at.row, b.hq), in.ldk, at.n, in.dk, in.silu != 0, in.vec != 0);
-    load_rows<T, DV>(v_s, in.v_at<T>(at.row, b.h) + b.v0, in.ldv, at.n, b.nv, in.silu != 0, in.vec != 0);
+    load_rows<T, DKP>(k_s, in.k_at<T>(at.row, unit_of(in, at, u0).h / (in.heads / in.kq_heads)), in.ldk, at.n, in.dk, in.silu != 0, in.vec != 0);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+        const Unit b = unit_of(in, at, u0 + u);
+        load_rows<T, DV>(v_s + u * Tile<DV>::ELEMS, in.v_at<T>(at.row, b.h) + b.v0, in.ldv, at.n, b.nv, in.silu != 0, in.vec != 0);
+    }
     ds_commit();
-    if (warp == 0) chunk_decays(in, at, b.h, hi_s, lo_s, f_s);
+    if (warp < U) chunk_decays(in, at, unit_of(in, at, u0 + warp).h, hi_s[warp], lo_s[warp], f_s[warp]);
     ds_wait<0>();
     __syncthreads();
-    const float end_hi = hi_s[CH - 1], end_lo = lo_s[CH - 1];
-    float acc[DKP / 8][4];
+#pragma unroll 1
+    for (int u = 0; u < U; ++u) {
+        const Unit b = unit_of(in, at, u0 + u);
+        const float end_hi = hi_s[u][CH - 1], end_lo = lo_s[u][CH - 1];
+        float acc[DKP / 8][4];
 #pragma unroll
-    for (int n = 0; n < DKP / 8; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
+        for (int n = 0; n < DKP / 8; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
+#pragma unroll 1      // (unrolled, the kernel waits for its own instructions: they run once a block)
+        for (int kb = 0; kb < CH / 16; ++kb) {
+            unsigned a[4], a_hi[4], a_lo[4];       // A: value channel x token, out of [token][value channel]
+            ldmatrix_x4_trans(a, v_s + u * Tile<DV>::ELEMS + (kb * 16 + (mat >> 1) * 8 + rr) * RV + warp * 16 + (mat & 1) * 8);
 #pragma unroll
-    for (int kb = 0; kb < CH / 16; ++kb) {
-        unsigned a[4], a_hi[4], a_lo[4];       // A: value channel x token, out of [token][value channel]
-        ldmatrix_x4_trans(a, v_s + (kb * 16 + (mat >> 1) * 8 + rr) * RV + warp * 16 + (mat & 1) * 8);
+            for (int half = 0; half < 2; ++half) {      // the thread's tokens: 2t, 2t + 1 of eight
+                const int s0 = kb * 16 + half * 8 + 2 * t;
+                const float w0 = ds_exp2((end_hi - hi_s[u][s0]) + (end_lo - lo_s[u][s0])) * f_s[u][s0];
+                const float w1 = ds_exp2((end_hi - hi_s[u][s0 + 1]) + (end_lo - lo_s[u][s0 + 1])) * f_s[u][s0 + 1];
 #pragma unroll
-        for (int half = 0; half < 2; ++half) {      // the thread's tokens: 2t, 2t + 1 of eight
-            const int s0 = kb * 16 + half * 8 + 2 * t;
-            const float w0 = ds_exp2((end_hi - hi_s[s0]) + (end_lo - lo_s[s0])) * f_s[s0];
-            const float w1 = ds_exp2((end_hi - hi_s[s0 + 1]) + (end_lo - lo_s[s0 + 1])) * f_s[s0 + 1];
+                for (int r = 0; r < 2; ++r) {
+                    const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a[2 * half + r]));
+                    const float x = v.x * w0, y = v.y * w1;
+                    a_hi[2 * half + r] = pack_bf16(x, y);
+                    a_lo[2 * half + r] = pack_bf16(x - bf16_of(x), y - bf16_of(y));
+                }
+            }
 #pragma unroll
-            for (int r = 0; r < 2; ++r) {
-                const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a[2 * half + r]));
-                const float x = v.x * w0, y = v.y * w1;
-                a_hi[2 * half + r] = pack_bf16(x, y);
-                a_lo[2 * half + r] = pack_bf16(x - bf16_of(x), y - bf16_of(y));
+            for (int np = 0; np < DKP / 16; ++np) {     // B: token x key channel
+                unsigned bk[4];
+                ldmatrix_x4_trans(bk, k_s + (kb * 16 + (mat & 1) * 8 + rr) * RK + np * 16 + (mat >> 1) * 8);
+                mma_bf16(acc[2 * np], a_hi, bk[0], bk[1]);
+                mma_bf16(acc[2 * np + 1], a_hi, bk[2], bk[3]);
+                mma_bf16(acc[2 * np], a_lo, bk[0], bk[1]);
+                mma_bf16(acc[2 * np + 1], a_lo, bk[2], bk[3]);
             }
         }
+        float* out = local + (b.piece + warp) * PIECE + lane * 8;       // (zeros where the head has fewer channels)
 #pragma unroll
-        for (int np = 0; np < DKP / 16; ++np) {     // B: token x key channel
-            unsigned bk[4];
-            ldmatrix_x4_trans(bk, k_s + (kb * 16 + (mat & 1) * 8 + rr) * RK + np * 16 + (mat >> 1) * 8);
-            mma_bf16(acc[2 * np], a_hi, bk[0], bk[1]);
-            mma_bf16(acc[2 * np + 1], a_hi, bk[2], bk[3]);
-            mma_bf16(acc[2 * np], a_lo, bk[0], bk[1]);
-            mma_bf16(acc[2 * np + 1], a_lo, bk[2], bk[3]);
+        for (int kk = 0; kk < DKP / 16; ++kk) {
+            float4* to = reinterpret_cast<float4*>(out + kk * 4 * PIECE);
+            to[0] = make_float4(acc[2 * kk][0], acc[2 * kk][1], acc[2 * kk + 1][0], acc[2 * kk + 1][1]);
+            to[1] = make_float4(acc[2 * kk][2], acc[2 * kk][3], acc[2 * kk + 1][2], acc[2 * kk + 1][3]);
         }
+        if (threadIdx.x == 0 && b.v0 == 0) decays[(size_t)at.slot * in.heads + b.h] = ds_exp2(end_hi + end_lo);
     }
-    float* out = local + (b.piece + warp) * PIECE + lane * 8;       // (zeros where the head has fewer channels)
-#pragma unroll
-    for (int kk = 0; kk < DKP / 16; ++kk) {
-        float4* to = reinterpret_cast<float4*>(out + kk * 4 * PIECE);
-        to[0] = make_float4(acc[2 * kk][0], acc[2 * kk][1], acc[2 * kk + 1][0], acc[2 * kk + 1][1]);
-        to[1] = make_float4(acc[2 * kk][2], acc[2 * kk][3], acc[2 * kk + 1][2], acc[2 * kk + 1][3]);
-    }
-    if (threadIdx.x == 0 && b.v0 == 0) decays[(size_t)at.slot * in.heads + b.h] = ds_exp2(end_hi + end_lo);
 }
 
 // local[chunk] (what the chunk adds) becomes the chunk's entry state; the slot's state moves past the request's last chunk. A thread
@@ -409,131 +418,153 @@ chunk_chain_kernel(float* __restrict__ state, long long state_ld, int state_off,
     }
 }
 
-// The outputs of a chunk from its entry state. A warp owns 16 tokens.
-template <typename T, int DKP>
-__global__ void __launch_bounds__(DS_THREADS, 5)
+// The outputs of a chunk from its entry state. A warp owns 16 tokens; what q . k gives serves all of the block's units.
+template <typename T, int DKP, int U>
+__global__ void __launch_bounds__(DS_THREADS, U == 1 ? 5 : 4)
 chunk_output_kernel(const DsIn in, const float* __restrict__ entry, float* __restrict__ o, int ldo) {
     extern __shared__ __align__(16) unsigned char smem[];
-    __shared__ float hi_s[CH], lo_s[CH], f_s[CH];
+    __shared__ __align__(16) float hi_s[U][CH], lo_s[U][CH], f_s[U][CH];
     pdl_launch_dependents();
     pdl_wait();
-    const Block b = block_of(in);
-    const ChunkAt& at = b.at;
+    const ChunkAt at = chunk_at(in.q_start, blockIdx.z, blockIdx.x);
     if (at.n == 0) return;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, mat = lane >> 3, rr = lane & 7, g = lane >> 2, t4 = lane & 3;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, mat = lane >> 3, rr = lane & 7, g = lane >> 2, t4 = lane & 3, u0 = blockIdx.y * U;
     constexpr int RK = Tile<DKP>::ROW, RV = Tile<DV>::ROW;
     __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem);
     __nv_bfloat16* k_s = q_s + Tile<DKP>::ELEMS;
     __nv_bfloat16* v_s = k_s + Tile<DKP>::ELEMS;
     const bool vec = in.vec != 0, silu = in.silu != 0;
-    load_rows<T, DKP>(q_s, in.q_at<T>(at.row, b.hq), in.ldq, at.n, in.dk, silu, vec);
+    const int hq = unit_of(in, at, u0).h / (in.heads / in.kq_heads);
+    load_rows<T, DKP>(q_s, in.q_at<T>(at.row, hq), in.ldq, at.n, in.dk, silu, vec);
     ds_commit();
-    load_rows<T, DKP>(k_s, in.k_at<T>(at.row, b.hq), in.ldk, at.n, in.dk, silu, vec);
-    load_rows<T, DV>(v_s, in.v_at<T>(at.row, b.h) + b.v0, in.ldv, at.n, b.nv, silu, vec);
+    load_rows<T, DKP>(k_s, in.k_at<T>(at.row, hq), in.ldk, at.n, in.dk, silu, vec);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+        const Unit b = unit_of(in, at, u0 + u);
+        load_rows<T, DV>(v_s + u * Tile<DV>::ELEMS, in.v_at<T>(at.row, b.h) + b.v0, in.ldv, at.n, b.nv, silu, vec);
+    }
     ds_commit();
-    if (warp == 0) chunk_decays(in, at, b.h, hi_s, lo_s, f_s);
+    if (warp < U) chunk_decays(in, at, unit_of(in, at, u0 + warp).h, hi_s[warp], lo_s[warp], f_s[warp]);
     ds_wait<1>();
     __syncthreads();
-    unsigned q[DKP / 16][4];
+    Unit b[U];
 #pragma unroll
-    for (int kk = 0; kk < DKP / 16; ++kk) ldmatrix_x4(q[kk], q_s + (warp * 16 + (mat & 1) * 8 + rr) * RK + kk * 16 + (mat >> 1) * 8);
-    float acc[DV / 8][4];
+    for (int u = 0; u < U; ++u) b[u] = unit_of(in, at, u0 + u);
+    const __nv_bfloat16* q_w = q_s + (warp * 16 + (mat & 1) * 8 + rr) * RK + (mat >> 1) * 8;
+    float acc[U][DV / 8][4];
 #pragma unroll
-    for (int n = 0; n < DV / 8; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
-    // q . S_in
-    const uint4* state = reinterpret_cast<const uint4*>(entry + b.piece * PIECE + lane * 8);
+    for (int u = 0; u < U; ++u)
 #pragma unroll
-    for (int kk = 0; kk < DKP / 16; ++kk)
+        for (int n = 0; n < DV / 8; ++n) acc[u][n][0] = acc[u][n][1] = acc[u][n][2] = acc[u][n][3] = 0.f;
+    // q . S_in. (The loops over keys stay loops: unrolled, the kernel waits for its own instructions, which run once a block.)
+#pragma unroll 1
+    for (int kk = 0; kk < DKP / 16; ++kk) {
+        unsigned q[4];
+        ldmatrix_x4(q, q_w + kk * 16);
 #pragma unroll
-        for (int np = 0; np < DV / 16; ++np) {
-            const uint4* piece = state + (kk * 4 + np) * (PIECE / 4);       // the state's bfloat16, then its remainders
-            const uint4 bh = piece[0], bl = piece[1];
-            mma_bf16(acc[2 * np], q[kk], bh.x, bh.y);
-            mma_bf16(acc[2 * np + 1], q[kk], bh.z, bh.w);
-            mma_bf16(acc[2 * np], q[kk], bl.x, bl.y);
-            mma_bf16(acc[2 * np + 1], q[kk], bl.z, bl.w);
+        for (int u = 0; u < U; ++u) {
+            const uint4* piece = reinterpret_cast<const uint4*>(entry + (b[u].piece + kk * 4) * PIECE + lane * 8);      // the state's bfloat16, then its remainders
+#pragma unroll
+            for (int np = 0; np < DV / 16; ++np) {
+                const uint4 bh = piece[np * (PIECE / 4)], bl = piece[np * (PIECE / 4) + 1];
+                mma_bf16(acc[u][2 * np], q, bh.x, bh.y);
+                mma_bf16(acc[u][2 * np + 1], q, bh.z, bh.w);
+                mma_bf16(acc[u][2 * np], q, bl.x, bl.y);
+                mma_bf16(acc[u][2 * np + 1], q, bl.z, bl.w);
+            }
         }
-    float t_hi[2], t_lo[2];
-#pragma unroll
-    for (int r = 0; r < 2; ++r) {
-        t_hi[r] = hi_s[warp * 16 + g + 8 * r];
-        t_lo[r] = lo_s[warp * 16 + g + 8 * r];
-        const float w = ds_exp2(t_hi[r] + t_lo[r]);
-#pragma unroll
-        for (int n = 0; n < DV / 8; ++n) { acc[n][2 * r] *= w; acc[n][2 * r + 1] *= w; }
     }
+    float t_hi[U][2], t_lo[U][2];
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            t_hi[u][r] = hi_s[u][warp * 16 + g + 8 * r];
+            t_lo[u][r] = lo_s[u][warp * 16 + g + 8 * r];
+            const float w = ds_exp2(t_hi[u][r] + t_lo[u][r]);
+#pragma unroll
+            for (int n = 0; n < DV / 8; ++n) { acc[u][n][2 * r] *= w; acc[u][n][2 * r + 1] *= w; }
+        }
     ds_wait<0>();
     __syncthreads();
     if (warp * 16 >= at.n) return;
-    // the chunk's own tokens, 16 keys at a time up to the warp's last token
+    // the chunk's own tokens, 16 keys at a time up to the warp's last token; what q . k gives serves all units
+#pragma unroll 1
     for (int kb = 0; kb <= warp; ++kb) {
         float s[2][4] = {};
-#pragma unroll
+        const __nv_bfloat16* k_w = k_s + (kb * 16 + (mat >> 1) * 8 + rr) * RK + (mat & 1) * 8;
+#pragma unroll 2
         for (int kk = 0; kk < DKP / 16; ++kk) {
-            unsigned bk[4];
-            ldmatrix_x4(bk, k_s + (kb * 16 + (mat >> 1) * 8 + rr) * RK + kk * 16 + (mat & 1) * 8);
-            mma_bf16(s[0], q[kk], bk[0], bk[1]);
-            mma_bf16(s[1], q[kk], bk[2], bk[3]);
+            unsigned q[4], bk[4];
+            ldmatrix_x4(q, q_w + kk * 16);
+            ldmatrix_x4(bk, k_w + kk * 16);
+            mma_bf16(s[0], q, bk[0], bk[1]);
+            mma_bf16(s[1], q, bk[2], bk[3]);
         }
-        unsigned p_hi[4], p_lo[4];
 #pragma unroll
-        for (int n = 0; n < 2; ++n)
+        for (int u = 0; u < U; ++u) {
+            unsigned p_hi[4], p_lo[4];
 #pragma unroll
-            for (int r = 0; r < 2; ++r) {
-                float x[2];
+            for (int n = 0; n < 2; ++n) {
+                const int key = kb * 16 + n * 8 + 2 * t4;
+                const float2 k_hi = *reinterpret_cast<const float2*>(&hi_s[u][key]), k_lo = *reinterpret_cast<const float2*>(&lo_s[u][key]);
+                const float2 f = *reinterpret_cast<const float2*>(&f_s[u][key]);
 #pragma unroll
-                for (int e = 0; e < 2; ++e) {
-                    const int key = kb * 16 + n * 8 + 2 * t4 + e, tok = warp * 16 + g + 8 * r;
-                    const float w = key <= tok ? ds_exp2((t_hi[r] - hi_s[key]) + (t_lo[r] - lo_s[key])) * f_s[key] : 0.f;
-                    x[e] = s[n][2 * r + e] * w;
+                for (int r = 0; r < 2; ++r) {
+                    const int tok = warp * 16 + g + 8 * r;
+                    const float w0 = ds_exp2((t_hi[u][r] - k_hi.x) + (t_lo[u][r] - k_lo.x)) * f.x, w1 = ds_exp2((t_hi[u][r] - k_hi.y) + (t_lo[u][r] - k_lo.y)) * f.y;
+                    const float x0 = key <= tok ? s[n][2 * r] * w0 : 0.f, x1 = key + 1 <= tok ? s[n][2 * r + 1] * w1 : 0.f;
+                    p_hi[2 * n + r] = pack_bf16(x0, x1);
+                    p_lo[2 * n + r] = pack_bf16(x0 - bf16_of(x0), x1 - bf16_of(x1));
                 }
-                p_hi[2 * n + r] = pack_bf16(x[0], x[1]);
-                p_lo[2 * n + r] = pack_bf16(x[0] - bf16_of(x[0]), x[1] - bf16_of(x[1]));
             }
 #pragma unroll
-        for (int np = 0; np < DV / 16; ++np) {
-            unsigned bv[4];
-            ldmatrix_x4_trans(bv, v_s + (kb * 16 + (mat & 1) * 8 + rr) * RV + np * 16 + (mat >> 1) * 8);
-            mma_bf16(acc[2 * np], p_hi, bv[0], bv[1]);
-            mma_bf16(acc[2 * np + 1], p_hi, bv[2], bv[3]);
-            mma_bf16(acc[2 * np], p_lo, bv[0], bv[1]);
-            mma_bf16(acc[2 * np + 1], p_lo, bv[2], bv[3]);
+            for (int np = 0; np < DV / 16; ++np) {
+                unsigned bv[4];
+                ldmatrix_x4_trans(bv, v_s + u * Tile<DV>::ELEMS + (kb * 16 + (mat & 1) * 8 + rr) * RV + np * 16 + (mat >> 1) * 8);
+                mma_bf16(acc[u][2 * np], p_hi, bv[0], bv[1]);
+                mma_bf16(acc[u][2 * np + 1], p_hi, bv[2], bv[3]);
+                mma_bf16(acc[u][2 * np], p_lo, bv[0], bv[1]);
+                mma_bf16(acc[u][2 * np + 1], p_lo, bv[2], bv[3]);
+            }
         }
     }
     const bool pairs = in.dv % 2 == 0 && ldo % 2 == 0 && ((uintptr_t)o & 7) == 0;
 #pragma unroll
-    for (int r = 0; r < 2; ++r) {
-        const int tok = warp * 16 + g + 8 * r;
-        if (tok >= at.n) continue;
-        float* row = o + (size_t)(at.row + tok) * ldo + (size_t)b.h * in.dv + b.v0;
+    for (int u = 0; u < U; ++u)
 #pragma unroll
-        for (int n = 0; n < DV / 8; ++n) {
-            const int c = n * 8 + 2 * t4;
-            if (pairs) {
-                if (c < b.nv) *reinterpret_cast<float2*>(row + c) = make_float2(acc[n][2 * r], acc[n][2 * r + 1]);
-            } else {
-                if (c < b.nv) row[c] = acc[n][2 * r];
-                if (c + 1 < b.nv) row[c + 1] = acc[n][2 * r + 1];
+        for (int r = 0; r < 2; ++r) {
+            const int tok = warp * 16 + g + 8 * r;
+            if (tok >= at.n) continue;
+            float* row = o + (size_t)(at.row + tok) * ldo + (size_t)b[u].h * in.dv + b[u].v0;
+#pragma unroll
+            for (int n = 0; n < DV / 8; ++n) {
+                const int c = n * 8 + 2 * t4;
+                if (pairs) {
+                    if (c < b[u].nv) *reinterpret_cast<float2*>(row + c) = make_float2(acc[u][n][2 * r], acc[u][n][2 * r + 1]);
+                } else {
+                    if (c < b[u].nv) row[c] = acc[u][n][2 * r];
+                    if (c + 1 < b[u].nv) row[c + 1] = acc[u][n][2 * r + 1];
+                }
             }
         }
-    }
 }
 
-template <typename T, int DKP>
+template <typename T, int DKP, int U>
 int launch_chunks(const DsIn& in, float* state, long long state_ld, int state_off, float* o, int ldo, int n_req, int max_len, float* local,
                   float* decays, cudaStream_t stream) {
-    constexpr int SMEM_STATE = (Tile<DKP>::ELEMS + Tile<DV>::ELEMS) * 2, SMEM_OUT = (2 * Tile<DKP>::ELEMS + Tile<DV>::ELEMS) * 2;
+    constexpr int SMEM_STATE = (Tile<DKP>::ELEMS + U * Tile<DV>::ELEMS) * 2, SMEM_OUT = (2 * Tile<DKP>::ELEMS + U * Tile<DV>::ELEMS) * 2;
     static bool configured = false;
     if (!configured) {
-        NIB_CUDA(cudaFuncSetAttribute(chunk_state_kernel<T, DKP>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_STATE));
-        NIB_CUDA(cudaFuncSetAttribute(chunk_output_kernel<T, DKP>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_OUT));
+        NIB_CUDA(cudaFuncSetAttribute(chunk_state_kernel<T, DKP, U>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_STATE));
+        NIB_CUDA(cudaFuncSetAttribute(chunk_output_kernel<T, DKP, U>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_OUT));
         configured = true;
     }
-    const dim3 grid(ceil_div(max_len, CH), in.heads * ceil_div(in.dv, DV), n_req);
-    NIB_CUDA(launch_pdl(chunk_state_kernel<T, DKP>, grid, dim3(DS_THREADS), (size_t)SMEM_STATE, stream, in, local, decays));
+    const dim3 grid(ceil_div(max_len, CH), in.heads * ceil_div(in.dv, DV) / U, n_req);
+    NIB_CUDA(launch_pdl(chunk_state_kernel<T, DKP, U>, grid, dim3(DS_THREADS), (size_t)SMEM_STATE, stream, in, local, decays));
     NIB_CUDA(launch_pdl(chunk_chain_kernel, dim3(ceil_div((long long)in.heads * pieces_of(in.dk, in.dv), 4), n_req), dim3(128), (size_t)0, stream, state,
                         state_ld, state_off, in.q_start, in.slots, local, (const float*)decays, in.heads, in.dk, in.dv));
-    NIB_CUDA(launch_pdl(chunk_output_kernel<T, DKP>, grid, dim3(DS_THREADS), (size_t)SMEM_OUT, stream, in, (const float*)local, o, ldo));
+    NIB_CUDA(launch_pdl(chunk_output_kernel<T, DKP, U>, grid, dim3(DS_THREADS), (size_t)SMEM_OUT, stream, in, (const float*)local, o, ldo));
     NIB_LAUNCH_CHECK();
     return 0;
 }
@@ -562,8 +593,13 @@ int scan(DsIn in, float* state, long long state_ld, int state_off, float* o, int
     auto aligned = [](const void* p, long long ld) { return ((uintptr_t)p & 15) == 0 && ld % G == 0; };
     in.vec = dk % G == 0 && dv % G == 0 && aligned(in.q, in.ldq) && aligned(in.k, in.ldk) && aligned(in.v, in.ldv);
     float* decays = scratch + ((long long)tokens / CH + n_req) * in.heads * pieces_of(dk, dv) * PIECE;
-    if (dk <= 64) return launch_chunks<T, 64>(in, state, state_ld, state_off, o, ldo, n_req, max_len, scratch, decays, stream);
-    return launch_chunks<T, 128>(in, state, state_ld, state_off, o, ldo, n_req, max_len, scratch, decays, stream);
+    // pairs of units of heads with the same q and k, once their blocks fill the GPU
+    const int sharing = in.heads / in.kq_heads * ceil_div(dv, DV);
+    const bool two = sharing % 2 == 0 && (long long)in.heads * ceil_div(dv, DV) * ceil_div(tokens, CH) >= 4LL * 148;
+#define NIB_DS(DKP, U) launch_chunks<T, DKP, U>(in, state, state_ld, state_off, o, ldo, n_req, max_len, scratch, decays, stream)
+    if (dk <= 64) return two ? NIB_DS(64, 2) : NIB_DS(64, 1);
+    return two ? NIB_DS(128, 2) : NIB_DS(128, 1);
+#undef NIB_DS
 }
 
 }  // namespace

@@ -12,7 +12,7 @@ The feed-forward is absent or ``W_down (gelu(W_gate h) * (W_up h))`` with the ta
 ``embedding.scale``; the head is the embedding table without that factor.
 
 config.json: ``architecture``, ``vocab``, ``width``, ``norm.eps``, ``embedding.scale``, ``layers``: a list of ``{"type", "mixer": {...},
-"mlp": {"kind": "dense", "ff"} | null}``. ``mixer`` of ``attention``: ``heads kv_heads dim vdim scale mask.size rot.{dims, base}``; of
+"mlp": {"kind": "dense", "ff"} | null}``. ``mixer`` of ``attention``: ``heads kv_heads dim vdim scale mask.size rot.{dims, base}`` (``mask`` may be absent); of
 ``parallel``: ``left_scale right_scale``, ``left``: the same with ``mask.{size, keep_first}`` (``vdim`` = ``dim``), ``right``: ``heads dim vdim
 decay`` (a list, one per head); of ``mamba2``: ``heads vdim state groups norm_groups conv``.
 
@@ -73,10 +73,11 @@ def _check_softmax(m: Mapping[str, Any], where: str, values_are_keys: bool) -> N
     if dims % 2 or dims > dim:
         raise ConfigError(f"config.json: {where}.rot.dims must be even and at most dim")
     _num(rot, "base", where + ".rot")
-    mask = _obj(m, "mask", where)
-    _int(mask, "size", where + ".mask")
-    if mask.get("keep_first") is not None:
-        _int(mask, "keep_first", where + ".mask", least=0)
+    if m.get("mask") is not None:       # without one every earlier position is seen
+        mask = _obj(m, "mask", where)
+        _int(mask, "size", where + ".mask")
+        if mask.get("keep_first") is not None:
+            _int(mask, "keep_first", where + ".mask", least=0)
 
 
 def _check_lightning(m: Mapping[str, Any], where: str) -> None:
@@ -150,16 +151,23 @@ def _rot(m: Mapping[str, Any]):
     return int(m["rot"]["dims"]), float(m["rot"]["base"])
 
 
+def _mask(m: Mapping[str, Any]):
+    """(size, kept first tokens) of a mixer's mask; size 0 without one."""
+    mask = m.get("mask")
+    return (0, 0) if mask is None else (int(mask["size"]), int(mask.get("keep_first") or 0))
+
+
 def _mixer(prefix: str, hidden: int, kind: str, m: Mapping[str, Any], eps: float):
     if kind == "mamba2":
         return Mamba2Mixer.spec(prefix, hidden, int(m["heads"]), int(m["vdim"]), int(m["state"]), int(m["groups"]), int(m["norm_groups"]),
                                 int(m["conv"]), eps)
     if kind == "attention":
-        return FlexAttention.spec(prefix, hidden, *_softmax_dims(m), eps, qk_norm=True, rot=_rot(m), chunk=int(m["mask"]["size"]))
+        return FlexAttention.spec(prefix, hidden, *_softmax_dims(m), eps, qk_norm=True, rot=_rot(m), chunk=_mask(m)[0])
     left, right = m["left"], m["right"]
+    window, keep_first = _mask(left)
     return SideBySide.spec(
         FlexAttention.spec(f"{prefix}.left", hidden, *_softmax_dims(left), eps, qk_norm=True, rot=_rot(left), rot_layout="interleaved",
-                           values_from_keys=True, window=int(left["mask"]["size"]), keep_first=int(left["mask"].get("keep_first") or 0),
+                           values_from_keys=True, window=window, keep_first=keep_first,
                            out_gate="head", out_scale=float(m["left_scale"])),
         LightningAttention.spec(f"{prefix}.right", hidden, int(right["heads"]), int(right["dim"]), int(right.get("vdim", right["dim"])),
                                 right["decay"], eps, float(m["right_scale"])))

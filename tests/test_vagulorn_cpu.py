@@ -109,7 +109,7 @@ def test_config_refuses_what_it_cannot_run():
                lambda c: c["layers"][1]["mixer"]["right"].update(decay=[0.5, 0.5]),        # three heads
                lambda c: c["layers"][1]["mixer"]["right"].update(decay=[0.5, 1.5, 0.5]),
                lambda c: c["layers"][1]["mixer"].pop("right_scale"),
-               lambda c: c["layers"][2]["mixer"].pop("mask"),
+               lambda c: c["layers"][2]["mixer"].pop("rot"),
                lambda c: c["layers"][2]["mixer"]["rot"].update(dims=14),                   # wider than the head
                lambda c: c["layers"][0]["mixer"].update(norm_groups=5),
                lambda c: c["layers"][0].update(type="lstm"),
@@ -261,6 +261,16 @@ def test_every_constant_of_config_moves_the_result(tmp_path):
                               chunked(2, 2, 8, chunk, cdims, cbase, scale=cscale, ff=16), ssm(2, 4, 6, 2, 2, 3)], scale=emb, eps=eps)
     variants(tmp_path, [one(), one(scales=(0.5, 0.7)), one(scales=(1.0, -0.5)), one(window=5), one(keep=1), one(keep=None), one(decay=(0.5, 0.8)),
                         one(base=30.0), one(dims=8), one(scale=1.0), one(chunk=6), one(cdims=4), one(cbase=15.0), one(cscale=0.8), one(emb=0.5), one(eps=0.1)])
+
+
+def test_without_a_mask_every_earlier_position_is_seen(tmp_path):
+    wide = model(40, 24, [chunked(2, 1, 8, 1000, 4, 50.0, ff=16), pair(softmax(2, 1, 8, 1000, 8, 20.0), lightning(1, 4, 4), ff=16)])
+    bare = json.loads(json.dumps(wide))
+    bare["layers"][0]["mixer"].pop("mask")
+    bare["layers"][1]["mixer"]["left"].pop("mask")
+    ids = tokens(23, 40, 3)
+    ref = plain_logits(write_model(str(tmp_path / "wide"), wide, 4), ids)
+    close(run_cut(host_engine(write_model(str(tmp_path / "bare"), bare, 4)), "x", ids, [9, 1, 13]), ref)
 
 
 @pytest.mark.parametrize("groups,parts", [(1, 1), (2, 4), (4, 2)])

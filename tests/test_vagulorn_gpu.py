@@ -248,6 +248,21 @@ def test_unequal_requests_side_by_side(ops, kind, heads, kq, dk, dv, dtype):
         near(state, rstate, f"state {step}")
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("heads,kq,dk,dv", [(32, 2, 24, 40), (12, 6, 72, 68), (10, 10, 128, 130), (16, 1, 64, 64)])
+def test_many_heads_that_share_their_keys(ops, heads, kq, dk, dv, dtype):
+    """Enough heads and tokens that a block takes two units (heads of one group, or the value channels of one head), beside sizes
+    where it does not; a short request between two long ones."""
+    q_lens, slots = [1000, 30, 800], [1, 0, 2]
+    g, kw = state_inputs(sum(q_lens), heads, kq, dk, dv, "steps", seed=5, dtype=dtype)
+    ctx, _, _ = batch(q_lens, [0] * 3, slots=slots)
+    state = rnd(3, heads * dv * dk, seed=9, scale=0.3)
+    rstate = state.cpu().clone()
+    rows = list(range(sum(q_lens)))
+    near(run_scan(ops, g, kw, rows, state, 0, ctx, heads, kq, dk, dv), run_scan(REF, g, kw, rows, rstate, 0, to_cpu(ctx), heads, kq, dk, dv, "cpu"), "outputs")
+    near(state, rstate, "states")
+
+
 @pytest.mark.parametrize("n", [3, 16, 17, 200])
 def test_activations_stand_before_the_state(ops, n):
     heads, dk, dv = 3, 24, 20
