@@ -46,7 +46,8 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
 // Online-softmax update of one warp's 16 rows with a block of NT*8 score columns.
 // s holds raw dots; scale2 = scale * log2(e). vis_lo/vis_hi: visible key range of the thread's two
 // rows (row g -> [0], row g+8 -> [1]); key_base: key of column 0. Produces P as A fragments.
-template <int HD, int NT>
+// KEPT: keys below keep_first are visible as well.
+template <int HD, int NT, bool KEPT = false>
 __device__ __forceinline__ void softmax_block(float (&s)[NT][4], unsigned (&p)[NT / 2][4], float (&o)[HD / 8][4],
                                               float (&m_run)[2], float (&l_run)[2], float scale2, int key_base,
                                               const int (&vis_lo)[2], const int (&vis_hi)[2], int lane, int keep_first = 0) {
@@ -58,7 +59,7 @@ __device__ __forceinline__ void softmax_block(float (&s)[NT][4], unsigned (&p)[N
         for (int e = 0; e < 4; ++e) {
             const int r = e >> 1;
             const int key = key_base + n * 8 + 2 * t + (e & 1);
-            const bool vis = (key >= vis_lo[r] || key < keep_first) && key <= vis_hi[r];
+            const bool vis = (KEPT ? (key >= vis_lo[r] || key < keep_first) : key >= vis_lo[r]) && key <= vis_hi[r];
             s[n][e] = vis ? s[n][e] * scale2 : -INFINITY;
             mx[r] = fmaxf(mx[r], s[n][e]);
         }

@@ -237,7 +237,7 @@ attention_flex_mma_kernel(const __nv_bfloat16* __restrict__ q_in, int q_stride, 
             }
         }
         unsigned p[FB_N / 16][4];
-        softmax_block<DVP, FB_N / 8>(s, p, o, m_run, l_run, 1.0f, tile * FB_N, vis_lo, vis_hi, lane, keep_first);
+        softmax_block<DVP, FB_N / 8, true>(s, p, o, m_run, l_run, 1.0f, tile * FB_N, vis_lo, vis_hi, lane, keep_first);
         fx_pv<DVP>(o, p, v_buf[cur], lane);
         __syncthreads();    // the tile may be overwritten by the load issued in the next iteration
     }

@@ -44,7 +44,6 @@ struct DsIn {
 
 __device__ __forceinline__ float ds_silu(float x) { return x / (1.0f + expf(-x)); }
 __device__ __forceinline__ float softplus(float x) { return x > 0.f ? x + log1pf(expf(-x)) : log1pf(expf(x)); }
-__device__ __forceinline__ float bf16_of(float x) { return __bfloat162float(__float2bfloat16_rn(x)); }
 
 // elements c .. c + 3 of a row of `width` elements as floats, zeros beyond its end; vec: the width is a multiple of four and the
 // row starts on a boundary of four elements
@@ -207,12 +206,10 @@ __device__ __forceinline__ ChunkAt chunk_at(const int* __restrict__ q_start, int
     return {row, max(0, min(CH, last - row)), (first - q_start[0]) / CH + req + c};
 }
 
-// One warp: per token of the chunk the sum of the decays' log2 (as two floats) and the factor on the value; tokens that do not
-// exist do not decay.
-__device__ __forceinline__ void chunk_decays(const DsIn& in, const ChunkAt& at, int h, float* hi_s, float* lo_s, float* f_s) {
+// One warp: per token of the chunk (2 lane and 2 lane + 1 a lane) the sum of the decays' log2 up to it and the factor on its value;
+// tokens that do not exist do not decay.
+__device__ __forceinline__ void chunk_sums(const DsIn& in, const ChunkAt& at, int h, double (&sum)[2], float (&f)[2]) {
     const int lane = threadIdx.x & 31;
-    double sum[2];
-    float f[2];
     const bool fixed = in.raw == nullptr;
     const float rate2 = fixed ? 0.f : expf(in.a_log[h]) * LOG2E, bias = fixed ? 0.f : in.bias[h];
     const float fixed2 = fixed ? fmaxf(in.log2_decay[h], NO_DECAY_LEFT) : 0.f;
@@ -236,14 +233,29 @@ __device__ __forceinline__ void chunk_decays(const DsIn& in, const ChunkAt& at, 
     }
     double up = __shfl_up_sync(0xffffffffu, before, 1);
     if (lane == 0) up = 0.0;
+    sum[0] += up;
+    sum[1] += up;
+}
+
+// The sums as two floats each, so that differences of them keep their digits.
+__device__ __forceinline__ void chunk_decays(const DsIn& in, const ChunkAt& at, int h, float* hi_s, float* lo_s, float* f_s) {
+    const int lane = threadIdx.x & 31;
+    double sum[2];
+    float f[2];
+    chunk_sums(in, at, h, sum, f);
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
-        const double c = up + sum[e];
-        const float hi = (float)c;
+        const float hi = (float)sum[e];
         hi_s[2 * lane + e] = hi;
-        lo_s[2 * lane + e] = (float)(c - (double)hi);
+        lo_s[2 * lane + e] = (float)(sum[e] - (double)hi);
         f_s[2 * lane + e] = f[e];
     }
+}
+
+// x and y as bfloat16 and as the bfloat16 of what that leaves out
+__device__ __forceinline__ void split2(float x, float y, unsigned& hi, unsigned& lo) {
+    hi = pack_bf16(x, y);
+    lo = pack_bf16(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xffff0000u));
 }
 
 __device__ __forceinline__ void put4(__nv_bfloat16* p, const float4& x) {
@@ -294,7 +306,7 @@ template <typename T, int DKP, int U>
 __global__ void __launch_bounds__(DS_THREADS, 5)
 chunk_state_kernel(const DsIn in, float* __restrict__ local, float* __restrict__ decays) {
     extern __shared__ __align__(16) unsigned char smem[];
-    __shared__ __align__(16) float hi_s[U][CH], lo_s[U][CH], f_s[U][CH];
+    __shared__ __align__(16) float w_s[U][CH];      // what a token's value is multiplied with: its factor and the decays behind it
     pdl_launch_dependents();
     pdl_wait();
     const ChunkAt at = chunk_at(in.q_start, blockIdx.z, blockIdx.x);
@@ -310,13 +322,20 @@ chunk_state_kernel(const DsIn in, float* __restrict__ local, float* __restrict__
         load_rows<T, DV>(v_s + u * Tile<DV>::ELEMS, in.v_at<T>(at.row, b.h) + b.v0, in.ldv, at.n, b.nv, in.silu != 0, in.vec != 0);
     }
     ds_commit();
-    if (warp < U) chunk_decays(in, at, unit_of(in, at, u0 + warp).h, hi_s[warp], lo_s[warp], f_s[warp]);
+    if (warp < U) {
+        const Unit b = unit_of(in, at, u0 + warp);
+        double sum[2];
+        float f[2];
+        chunk_sums(in, at, b.h, sum, f);
+        const double end = __shfl_sync(0xffffffffu, sum[1], 31);
+        *reinterpret_cast<float2*>(&w_s[warp][2 * lane]) = make_float2(ds_exp2((float)(end - sum[0])) * f[0], ds_exp2((float)(end - sum[1])) * f[1]);
+        if (lane == 0 && b.v0 == 0) decays[(size_t)at.slot * in.heads + b.h] = ds_exp2((float)end);
+    }
     ds_wait<0>();
     __syncthreads();
 #pragma unroll 1
     for (int u = 0; u < U; ++u) {
         const Unit b = unit_of(in, at, u0 + u);
-        const float end_hi = hi_s[u][CH - 1], end_lo = lo_s[u][CH - 1];
         float acc[DKP / 8][4];
 #pragma unroll
         for (int n = 0; n < DKP / 8; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
@@ -326,15 +345,11 @@ chunk_state_kernel(const DsIn in, float* __restrict__ local, float* __restrict__
             ldmatrix_x4_trans(a, v_s + u * Tile<DV>::ELEMS + (kb * 16 + (mat >> 1) * 8 + rr) * RV + warp * 16 + (mat & 1) * 8);
 #pragma unroll
             for (int half = 0; half < 2; ++half) {      // the thread's tokens: 2t, 2t + 1 of eight
-                const int s0 = kb * 16 + half * 8 + 2 * t;
-                const float w0 = ds_exp2((end_hi - hi_s[u][s0]) + (end_lo - lo_s[u][s0])) * f_s[u][s0];
-                const float w1 = ds_exp2((end_hi - hi_s[u][s0 + 1]) + (end_lo - lo_s[u][s0 + 1])) * f_s[u][s0 + 1];
+                const float2 w = *reinterpret_cast<const float2*>(&w_s[u][kb * 16 + half * 8 + 2 * t]);
 #pragma unroll
                 for (int r = 0; r < 2; ++r) {
                     const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a[2 * half + r]));
-                    const float x = v.x * w0, y = v.y * w1;
-                    a_hi[2 * half + r] = pack_bf16(x, y);
-                    a_lo[2 * half + r] = pack_bf16(x - bf16_of(x), y - bf16_of(y));
+                    split2(v.x * w.x, v.y * w.y, a_hi[2 * half + r], a_lo[2 * half + r]);
                 }
             }
 #pragma unroll
@@ -354,7 +369,6 @@ chunk_state_kernel(const DsIn in, float* __restrict__ local, float* __restrict__
             to[0] = make_float4(acc[2 * kk][0], acc[2 * kk][1], acc[2 * kk + 1][0], acc[2 * kk + 1][1]);
             to[1] = make_float4(acc[2 * kk][2], acc[2 * kk][3], acc[2 * kk + 1][2], acc[2 * kk + 1][3]);
         }
-        if (threadIdx.x == 0 && b.v0 == 0) decays[(size_t)at.slot * in.heads + b.h] = ds_exp2(end_hi + end_lo);
     }
 }
 
@@ -400,10 +414,7 @@ chunk_chain_kernel(float* __restrict__ state, long long state_ld, int state_off,
                 uint4* to = reinterpret_cast<uint4*>(at + (size_t)(k0 + i) * step);
                 unsigned hi[4], lo[4];
 #pragma unroll
-                for (int n = 0; n < 4; ++n) {
-                    hi[n] = pack_bf16(S[2 * n], S[2 * n + 1]);
-                    lo[n] = pack_bf16(S[2 * n] - bf16_of(S[2 * n]), S[2 * n + 1] - bf16_of(S[2 * n + 1]));
-                }
+                for (int n = 0; n < 4; ++n) split2(S[2 * n], S[2 * n + 1], hi[n], lo[n]);
                 to[0] = make_uint4(hi[0], hi[1], hi[2], hi[3]);
                 to[1] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
                 const float add[8] = {x[i][0].x, x[i][0].y, x[i][0].z, x[i][0].w, x[i][1].x, x[i][1].y, x[i][1].z, x[i][1].w};
@@ -514,8 +525,7 @@ chunk_output_kernel(const DsIn in, const float* __restrict__ entry, float* __res
                     const int tok = warp * 16 + g + 8 * r;
                     const float w0 = ds_exp2((t_hi[u][r] - k_hi.x) + (t_lo[u][r] - k_lo.x)) * f.x, w1 = ds_exp2((t_hi[u][r] - k_hi.y) + (t_lo[u][r] - k_lo.y)) * f.y;
                     const float x0 = key <= tok ? s[n][2 * r] * w0 : 0.f, x1 = key + 1 <= tok ? s[n][2 * r + 1] * w1 : 0.f;
-                    p_hi[2 * n + r] = pack_bf16(x0, x1);
-                    p_lo[2 * n + r] = pack_bf16(x0 - bf16_of(x0), x1 - bf16_of(x1));
+                    split2(x0, x1, p_hi[2 * n + r], p_lo[2 * n + r]);
                 }
             }
 #pragma unroll
